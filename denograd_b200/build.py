@@ -10,7 +10,12 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OUT_DIR = os.path.join(HERE, "lib")
 LIB = os.path.join(OUT_DIR, "libjsgrad_cuda.so")
-SOURCES = ["device.cu", "elementwise.cu", "gemv.cu", "matvec_w8.cu", "gemm_small.cu", "gemm_tc.cu", "attention.cu", "attention_chunk.cu", "comm.cu", "sample.cu", "step.cu", "program.cu"]
+# The whole library is every source below.  A component is the part one model family needs on its own, linked as a
+# library of that name, so that a fresh checkout which serves one model does not compile the other families' kernels.
+CORE = ["device.cu", "comm.cu", "elementwise.cu", "sample.cu", "tensor_map.cu"]
+COMPONENTS = {"hybrid": CORE + ["dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu"]}
+SOURCES = CORE + ["gemv.cu", "matvec_w8.cu", "gemm_small.cu", "gemm_tc.cu", "attention.cu", "attention_chunk.cu", "step.cu", "program.cu",
+                  "dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu"]
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC,-fvisibility=hidden", "--expt-relaxed-constexpr"]
 
@@ -29,13 +34,23 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def _headers() -> list[str]:
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))] + [os.path.join(HERE, "..", "include", "jsgrad_cuda.h")]
+
+
+def fresh(component: str | None = None) -> bool:
+    """Whether the library (of a component, or the whole one) exists and is newer than everything it is made of."""
+    lib = os.path.join(OUT_DIR, f"libjsgrad_cuda_{component}.so") if component else LIB
+    return not _stale(lib, [os.path.join(CSRC, f) for f in (COMPONENTS[component] if component else SOURCES)] + _headers())
+
+
+def build(force: bool = False, verbose: bool = False, component: str | None = None) -> str:
     os.makedirs(OUT_DIR, exist_ok=True)
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    headers.append(os.path.join(HERE, "..", "include", "jsgrad_cuda.h"))
+    lib = os.path.join(OUT_DIR, f"libjsgrad_cuda_{component}.so") if component else LIB
+    headers = _headers()
     objs = []
     procs = []
-    for src in SOURCES:
+    for src in COMPONENTS[component] if component else SOURCES:
         s = os.path.join(CSRC, src)
         o = os.path.join(OUT_DIR, src.replace(".cu", ".o"))
         objs.append(o)
@@ -52,11 +67,13 @@ def build(force: bool = False, verbose: bool = False) -> str:
         failed |= p.returncode != 0
     if failed:
         raise RuntimeError("nvcc failed")
-    if force or procs or _stale(LIB, objs):
-        cmd = [nvcc(), *ARCH, "-shared", "-o", LIB, *objs, "-Xcompiler", "-fPIC", "-ldl"]
-        subprocess.run(cmd, check=True)
-    return LIB
+    if force or procs or _stale(lib, objs):
+        part = f"{lib}.{os.getpid()}"
+        subprocess.run([nvcc(), *ARCH, "-shared", "-o", part, *objs, "-Xcompiler", "-fPIC", "-ldl"], check=True)
+        os.replace(part, lib)
+    return lib
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="-v" in sys.argv))
+    names = [a for a in sys.argv[1:] if a in COMPONENTS]
+    print(build(force="--force" in sys.argv, verbose="-v" in sys.argv, component=names[0] if names else None))

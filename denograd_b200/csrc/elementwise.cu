@@ -4,6 +4,7 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "stream.cuh"
 #include "transcendental.cuh"
 
 // ------------------------------------------------------------------------------------------------ embedding
@@ -452,4 +453,26 @@ JG_API int jg_fill_normal_f16_2d(jg_dev* dev, uint64_t dst, uint64_t seed, uint6
   fill_normal_f16_2d_kernel<<<fill_blocks(dev, rows * cols), 256, 0, dev->stream>>>((__half*)dst, seed, rows, cols, full_cols,
                                                                                    row0, col0, std / 65536.0f);
   return jg_after_launch(dev, "fill_normal_f16_2d");
+}
+
+// The seeded normal fill in another element type, rows `ld` elements apart.
+template <typename T>
+__global__ void fill_normal_kernel(T* __restrict__ dst, unsigned long long seed, unsigned long long rows, unsigned long long cols,
+                                   unsigned long long ld, float c) {
+  const unsigned long long n = rows * cols;
+  for (unsigned long long i = blockIdx.x * (unsigned long long)blockDim.x + threadIdx.x; i < n;
+       i += (unsigned long long)gridDim.x * blockDim.x) {
+    const int S = (int)(synth_sum16(synth_word(seed, 3 * i)) + synth_sum16(synth_word(seed, 3 * i + 1)) + synth_sum16(synth_word(seed, 3 * i + 2)));
+    dst[i / cols * ld + i % cols] = from_f32<T>(__fmul_rn((float)(S - 393210), c));
+  }
+}
+
+JG_API int jg_fill_normal(jg_dev* dev, uint64_t dst, int32_t dtype, uint64_t seed, uint64_t rows, uint64_t cols, uint64_t ld, float std) {
+  JG_ENTER(dev);
+  JG_REQUIRE(rows > 0 && cols > 0 && ld >= cols && jg_aligned(dst, 4) && (dtype == JG_F32 || dtype == JG_BF16), "fill_normal: bad arguments");
+  jg_mark_fresh(dev, dst, rows * ld * (dtype == JG_F32 ? 4 : 2));
+  const int blocks = fill_blocks(dev, rows * cols);
+  if (dtype == JG_F32) fill_normal_kernel<float><<<blocks, 256, 0, dev->stream>>>((float*)dst, seed, rows, cols, ld, std / 65536.0f);
+  else fill_normal_kernel<bf16><<<blocks, 256, 0, dev->stream>>>((bf16*)dst, seed, rows, cols, ld, std / 65536.0f);
+  return jg_after_launch(dev, "fill_normal");
 }

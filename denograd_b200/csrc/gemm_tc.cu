@@ -23,11 +23,11 @@
 // Every mbarrier wait is bounded: a wait that does not complete sets an error word and the CTA winds down (cluster
 // barriers are still reached, tensor memory is released in every case); the host reports JG_ETIMEDOUT at the next
 // synchronisation.
-#include <cuda.h>
 #include <stdlib.h>
 #include <string.h>
 
 #include "common.cuh"
+#include "tcgen05.cuh"
 #include "transcendental.cuh"
 
 enum { TC_STORE = 0, TC_RESIDUAL = 1, TC_SWIGLU = 2, TC_PARTIAL = 4 };
@@ -36,11 +36,6 @@ constexpr int TC_BM = 128;  // weight rows per CTA (MMA M)
 constexpr int TC_BK = 64;   // k per stage: 64 halves = one 128-byte swizzle row
 // Threads of a CTA: warp 0 TMA, warp 1 MMA, then EPW epilogue warps for each 32-lane quarter of tensor memory.
 constexpr int tc_threads(int epw) { return 64 + 128 * epw; }
-// Polls of one mbarrier phase before a wait gives up.  A try_wait that fails returns after the hardware's own
-// suspend time (up to ~1 us), so the limit is of the order of seconds; every wait starts after the kernel's dependency
-// wait, i.e. it only ever measures this kernel's own TMA / MMA progress.
-constexpr uint32_t TC_SPIN_LIMIT = 1u << 24;
-
 struct TcArgs {
   __half* y;
   float* y32;
@@ -51,84 +46,6 @@ struct TcArgs {
   const __half* s0;  // int8 weights: per-output-row scales of the (first / second) matrix
   const __half* s1;
 };
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void mbar_init(uint64_t* bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
-}
-__device__ __forceinline__ void mbar_expect_tx(uint64_t* bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-// Bounded wait for the phase with the given parity; false = gave up.
-__device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity) {
-  const uint32_t addr = smem_u32(bar);
-  for (uint32_t i = 0; i < TC_SPIN_LIMIT; i++) {
-    uint32_t ok;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(ok)
-        : "r"(addr), "r"(parity)
-        : "memory");
-    if (ok) return true;
-  }
-  return false;
-}
-__device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, int c0, int c1, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-               ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1)
-               : "memory");
-}
-// K-major operand tile in 128-byte swizzled shared memory: rows of 128 bytes, 8-row groups 1024 bytes apart.
-__device__ __forceinline__ uint64_t umma_desc(const void* tile) {
-  const uint32_t lo = ((smem_u32(tile) & 0x3FFFFu) >> 4) | (1u << 16);  // start address, leading byte offset = 1 (unused)
-  const uint32_t hi = 64u | (1u << 14) | (2u << 29);                    // stride 1024 B, descriptor version 1, SWIZZLE_128B
-  return (uint64_t)lo | ((uint64_t)hi << 32);
-}
-__device__ __forceinline__ void umma_f16(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-      : "r"(taddr)
-      : "memory");
-}
-
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, float (&r)[16]) {
-  uint32_t u[16];
-  tmem_ld16(taddr, u);
-  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-  for (int j = 0; j < 16; j++) r[j] = __uint_as_float(u[j]);
-}
-// Cluster-wide barrier with release / acquire semantics (orders the distributed-shared-memory traffic around it).
-__device__ __forceinline__ void cluster_barrier() {
-  __syncwarp();
-  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-// Shared-memory address `local` as seen in the CTA of rank `rank` of this cluster.
-__device__ __forceinline__ uint32_t map_to_rank(uint32_t local, uint32_t rank) {
-  uint32_t remote;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
-  return remote;
-}
-__device__ __forceinline__ void st_cluster_f32(uint32_t addr, float v) {
-  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory");
-}
 
 template <int TN, int EPI, bool W8 = false, bool HALF = false>
 struct TcCfg {
@@ -549,68 +466,8 @@ __global__ void __launch_bounds__(Tc2Cfg<EPI>::THREADS) gemm_tc_pair_kernel(cons
 }
 
 // ------------------------------------------------------------------------------------------------ host side
-typedef CUresult (*encode_tiled_fn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                    const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-static encode_tiled_fn g_encode = nullptr;
-
-// `bytes` = element size: 2 for fp16 operands (128-byte swizzle, the layout the MMA descriptors name), 1 for int8
-// weight tiles, which land unswizzled (64-byte rows) for the converting warps
-static int make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, const char* what, int bytes = 2) {
-  if (!g_encode) {
-    void* fn = nullptr;
-    cudaDriverEntryPointQueryResult qres;
-    cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres);
-    if (e != cudaSuccess || fn == nullptr) {
-      jg_set_error("cuTensorMapEncodeTiled is not available from this driver");
-      return JG_ENOTSUP;
-    }
-    g_encode = (encode_tiled_fn)fn;
-  }
-  const cuuint64_t dims[2] = {cols, rows};           // innermost first
-  const cuuint64_t strides[1] = {cols * (cuuint64_t)bytes};  // bytes between rows
-  const cuuint32_t box[2] = {(cuuint32_t)TC_BK, box_rows};
-  const cuuint32_t estr[2] = {1, 1};
-  CUresult r = g_encode(m, bytes == 2 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_UINT8, 2, const_cast<void*>(base), dims,
-                        strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        bytes == 2 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (r != CUDA_SUCCESS) {
-    jg_set_error("tensor map for %s (%llu x %llu) rejected: CUresult %d", what, (unsigned long long)rows, (unsigned long long)cols, (int)r);
-    return JG_EINVAL;
-  }
-  return JG_OK;
-}
-
-// Encoded maps are kept per (base, rows, cols, box rows): a model's weights and workspaces keep their addresses, so a
-// step after the first finds all of its maps here instead of encoding three per launch.
-struct MapKey { const void* base; uint64_t rows, cols; uint32_t box_rows; int bytes; };
-struct MapSlot { MapKey k; CUtensorMap m; bool used; };
-constexpr int MAP_SLOTS = 1024;
-static MapSlot g_maps[MAP_SLOTS];
-
 static int cached_map(const CUtensorMap** out, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, const char* what, int bytes = 2) {
-  uint64_t h = (uint64_t)(uintptr_t)base * 0x9E3779B97F4A7C15ull ^ (rows * 0xBF58476D1CE4E5B9ull) ^ (cols << 20) ^ box_rows ^ ((uint64_t)bytes << 40);
-  h ^= h >> 29;
-  for (int probe = 0; probe < 8; probe++) {
-    MapSlot& s = g_maps[(h + probe) % MAP_SLOTS];
-    if (s.used && s.k.base == base && s.k.rows == rows && s.k.cols == cols && s.k.box_rows == box_rows && s.k.bytes == bytes) { *out = &s.m; return JG_OK; }
-    if (!s.used) {
-      int rc = make_map(&s.m, base, rows, cols, box_rows, what, bytes);
-      if (rc) return rc;
-      s.k = MapKey{base, rows, cols, box_rows, bytes};
-      s.used = true;
-      *out = &s.m;
-      return JG_OK;
-    }
-  }
-  MapSlot& s = g_maps[h % MAP_SLOTS];  // neighbourhood full: replace
-  int rc = make_map(&s.m, base, rows, cols, box_rows, what, bytes);
-  if (rc) { s.used = false; return rc; }
-  s.k = MapKey{base, rows, cols, box_rows, bytes};
-  s.used = true;
-  *out = &s.m;
-  return JG_OK;
+  return jg_tensor_map(out, base, rows, cols, cols, box_rows, what, bytes);
 }
 
 template <int TN, int EPI, bool W8 = false, bool HALF = false>

@@ -27,8 +27,11 @@ constexpr int SMP_MAX_CLUSTER = 8;
 constexpr int SMP_MAXK = 512;      // beyond 512 the reference's cumulative sum changes shape; nobody samples from more
 constexpr int SMP_MAX_BLOCKS = 2048;  // 256-element blocks of the k = 0 draw: vocabularies up to 524288
 
+__device__ __forceinline__ float logit_f32(__half v) { return __half2float(v); }
+__device__ __forceinline__ float logit_f32(float v) { return v; }
+
 struct SampleArgs {
-  const __half* logits;  // [B][V] fp16, widened to fp32 as Transformer.forward does (jsgrad/models/llama.ts:210)
+  const void* logits;    // [B][V] fp16, widened to fp32 as Transformer.forward does (jsgrad/models/llama.ts:210), or fp32
   const float* u;        // [B] uniform samples in [0, 1)
   int32_t* counter;      // [B][V] alpha counters, or null
   int32_t* tokens;       // [B]
@@ -47,6 +50,7 @@ struct SliceCursor {
   __device__ __forceinline__ void next() { if (++off == per) { off = 0; owner++; } }
 };
 
+template <typename LT>
 __global__ void __launch_bounds__(SMP_THREADS, 1) sample_kernel(const SampleArgs a) {
   extern __shared__ __align__(16) float tbuf[];  // this CTA's slice of y, then e, then t
   __shared__ float s_red[32];
@@ -74,7 +78,7 @@ __global__ void __launch_bounds__(SMP_THREADS, 1) sample_kernel(const SampleArgs
   // ---- y = (logit - penalty) * (1 / temperature), NaN -> -inf; maximum over the row
   float lmax = -INFINITY;
   for (int i = tid; i < nloc; i += SMP_THREADS) {
-    float x = __half2float(a.logits[(size_t)b * V + j0 + i]);
+    float x = logit_f32(reinterpret_cast<const LT*>(a.logits)[(size_t)b * V + j0 + i]);
     if (a.counter != nullptr) {
       const int c = a.counter[(size_t)b * V + j0 + i];
       const float pen = __fadd_rn(__fmul_rn((float)c, a.af), __fmul_rn(c >= 0 ? 1.0f : 0.0f, a.ap));
@@ -253,19 +257,20 @@ __global__ void __launch_bounds__(SMP_THREADS, 1) sample_kernel(const SampleArgs
 // per row (what Tensor.rand hands to multinomial); alpha_counter int32 [B][V] or 0.  temp must be >= 1e-6 (below
 // that `sample` is an argmax: jg_argmax).  The reference applies `sample` to one flattened row (jsgrad/models/llama.ts:
 // 132,212); rows here are independent.
-JG_API int jg_sample(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B,
-                     int32_t V, float temp, int32_t k, float p, float af, float ap) {
+template <typename LT>
+static int run_sample(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B,
+                      int32_t V, float temp, int32_t k, float p, float af, float ap) {
   JG_ENTER(dev);
   JG_REQUIRE(B > 0 && B <= 65535 && V > 0, "sample: bad shape B=%d V=%d", B, V);
   JG_REQUIRE(p >= 0.f && p <= 1.f, "sample: p must be between 0 and 1");
   JG_REQUIRE(k >= 0 && k <= V, "sample: k must be between 0 and numel");
   JG_REQUIRE(k <= SMP_MAXK, "sample: k=%d above %d is not implemented", k, SMP_MAXK);
   JG_REQUIRE(temp >= 1e-6f, "sample: temperature below 1e-6 selects argmax (jg_argmax)");
-  JG_REQUIRE(jg_aligned(tokens_out, 4) && jg_aligned(logits, 2) && jg_aligned(u, 4) && (alpha_counter == 0 || jg_aligned(alpha_counter, 4)),
+  JG_REQUIRE(jg_aligned(tokens_out, 4) && jg_aligned(logits, sizeof(LT)) && jg_aligned(u, 4) && (alpha_counter == 0 || jg_aligned(alpha_counter, 4)),
              "sample: null or misaligned pointer");
   JG_REQUIRE((V + 255) / 256 <= SMP_MAX_BLOCKS, "sample: a vocabulary of %d exceeds %d", V, SMP_MAX_BLOCKS * 256);
   SampleArgs a = {};
-  a.logits = (const __half*)logits; a.u = (const float*)u; a.tokens = (int32_t*)tokens_out;
+  a.logits = (const void*)logits; a.u = (const float*)u; a.tokens = (int32_t*)tokens_out;
   a.counter = (af != 0.f || ap != 0.f) ? (int32_t*)alpha_counter : nullptr;
   JG_REQUIRE(!(af != 0.f || ap != 0.f) || alpha_counter != 0, "sample: alpha penalties need the counter buffer");
   a.V = V; a.k = k; a.af = af; a.ap = ap;
@@ -287,8 +292,17 @@ JG_API int jg_sample(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t
   static size_t smem_set[8] = {0, 0, 0, 0, 0, 0, 0, 0};
   const int slot = dev->ordinal & 7;
   if (smem > 48 * 1024 - 40 * 1024 && smem > smem_set[slot]) {
-    JG_CUDA(cudaFuncSetAttribute(sample_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit));
+    JG_CUDA(cudaFuncSetAttribute(sample_kernel<LT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit));
     smem_set[slot] = limit;
   }
-  return jg_launch_cluster(dev, "sample", sample_kernel, dim3((unsigned)cs, (unsigned)B), dim3(SMP_THREADS), smem, cs, a);
+  return jg_launch_cluster(dev, "sample", sample_kernel<LT>, dim3((unsigned)cs, (unsigned)B), dim3(SMP_THREADS), smem, cs, a);
+}
+
+JG_API int jg_sample(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B,
+                     int32_t V, float temp, int32_t k, float p, float af, float ap) {
+  return run_sample<__half>(dev, tokens_out, logits, u, alpha_counter, B, V, temp, k, p, af, ap);
+}
+JG_API int jg_sample_f32(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B,
+                         int32_t V, float temp, int32_t k, float p, float af, float ap) {
+  return run_sample<float>(dev, tokens_out, logits, u, alpha_counter, B, V, temp, k, p, af, ap);
 }

@@ -25,8 +25,19 @@ import numpy as np
 
 from . import ffi
 
-_DTYPE_SIZE = {"float16": 2, "int8": 1, "uint8": 1, "int32": 4, "float32": 4, "uint64": 8}
-_NP = {"float16": np.float16, "int8": np.int8, "uint8": np.uint8, "int32": np.int32, "float32": np.float32, "uint64": np.uint64}
+_DTYPE_SIZE = {"float16": 2, "bfloat16": 2, "int8": 1, "uint8": 1, "int32": 4, "float32": 4, "uint64": 8}
+_NP = {"float16": np.float16, "int8": np.int8, "uint8": np.uint8, "int32": np.int32, "float32": np.float32, "uint64": np.uint64,
+       "bfloat16": np.uint16}  # numpy has no bfloat16: its bit patterns
+
+
+def to_bf16_bits(a: np.ndarray) -> np.ndarray:
+    """float32 values -> bfloat16 bit patterns (uint16), rounded to nearest even."""
+    b = np.ascontiguousarray(a, np.float32).view(np.uint32)
+    return ((b + np.uint32(0x7FFF) + ((b >> np.uint32(16)) & np.uint32(1))) >> np.uint32(16)).astype(np.uint16)
+
+
+def from_bf16_bits(b: np.ndarray) -> np.ndarray:
+    return (np.ascontiguousarray(b, np.uint16).astype(np.uint32) << np.uint32(16)).view(np.float32)
 
 
 class CUDAAllocator:
@@ -281,7 +292,8 @@ class Tensor:
         return Tensor(b, shape=(stop - start,) + tuple(self.shape[1:]))
 
     def assign(self, arr: np.ndarray) -> "Tensor":
-        self.buf.copyin(np.asarray(arr, dtype=_NP[self.dtype]).reshape(self.shape))
+        host = to_bf16_bits(arr) if self.dtype == "bfloat16" else np.asarray(arr, dtype=_NP[self.dtype])
+        self.buf.copyin(host.reshape(self.shape))
         return self
 
     def realize(self) -> "Tensor":
@@ -290,7 +302,7 @@ class Tensor:
     def numpy(self) -> np.ndarray:
         out = np.empty(self.shape, _NP[self.dtype])
         self.buf.copyout(out)
-        return out
+        return from_bf16_bits(out) if self.dtype == "bfloat16" else out
 
     def item(self):
         assert self.numel() == 1

@@ -39,6 +39,43 @@ class StepDesc(C.Structure):
                [("embed_rows", C.c_int64)]
 
 
+JG_F32, JG_BF16 = 0, 1
+DENSE_STORE, DENSE_GLU, DENSE_MINGRU, DENSE_LOGITS = 0, 1, 2, 3
+
+
+def _fields(spec: str) -> list:
+    """'i32 a b; u64 c' -> ctypes fields, one group of names per type."""
+    kinds = {"i32": C.c_int32, "u64": C.c_uint64, "f32": C.c_float}
+    return [(n, kinds[g.split()[0]]) for g in spec.split(";") for n in g.split()[1:]]
+
+
+class Batch(C.Structure):
+    _fields_ = _fields("i32 B Sc; u64 pos seq")
+
+
+class StreamDesc(C.Structure):
+    _fields_ = _fields("i32 width groups; f32 eps; i32 reserved; u64 x y w_add x_out w_norm rows")
+
+
+class DenseDesc(C.Structure):
+    _fields_ = _fields("i32 dtype epilogue N K ldx ldw ldy out_f32; f32 limit; i32 reserved; "
+                       "u64 x w0 w1 w2 b0 b1 b2 y key state") + [("stream", StreamDesc)]
+
+
+class MinGruDesc(C.Structure):
+    _fields_ = _fields("i32 dtype width ldp ldo; u64 proj state out")
+
+
+class DeltaDesc(C.Structure):
+    _fields_ = _fields("i32 dtype heads kv_heads dim vdim taps ldp ldo; f32 eps; i32 reserved; "
+                       "u64 proj conv_w a_log dt_bias norm_w state tail scratch out")
+
+
+class LatentDesc(C.Structure):
+    _fields_ = _fields("i32 dtype heads dim rot_dim vdim kv_rank window ldp ldo ldc ld_u page pages_per_slot n_slots rot_pairs rot_rows; "
+                       "f32 eps scale; u64 proj pool block_table rot norm_w sink ukv scratch out scratch_bytes")
+
+
 _vp, _i32, _i64, _u64, _f32, _f64, _sz = C.c_void_p, C.c_int32, C.c_int64, C.c_uint64, C.c_float, C.c_double, C.c_size_t
 _P = C.POINTER
 
@@ -104,6 +141,7 @@ SIGNATURES: dict[str, list] = {
     "jg_fill_uniform_i8": [_vp, _u64, _u64, _u64, _u64],
     "jg_fill_scale_f16": [_vp, _u64, _u64, _u64, _u64, _f32],
     "jg_fill_const_f16": [_vp, _u64, _u64, _f32],
+    "jg_fill_normal": [_vp, _u64, _i32, _u64, _u64, _u64, _u64, _f32],
     "jg_fill_normal_f16_2d": [_vp, _u64, _u64, _u64, _u64, _u64, _u64, _u64, _f32],
     "jg_fill_uniform_i8_2d": [_vp, _u64, _u64, _u64, _u64, _u64, _u64, _u64],
     "jg_comm_unique_id": [C.c_char_p, _vp],
@@ -128,10 +166,34 @@ SIGNATURES: dict[str, list] = {
     "jg_comm_group_end": [],
     "jg_linear_partial": [_vp, _u64, _u64, _u64, _u64, _i32, _i32, _i32],
     "jg_residual_add_f32": [_vp, _u64, _u64, _i64],
+    "jg_stream_embed": [_vp, _P(Batch), _u64, _u64, _u64, _i32, _i32, _i32, _i32],
+    "jg_stream_norm": [_vp, _P(Batch), _P(StreamDesc), _u64, _i32, _i32],
+    "jg_dense": [_vp, _P(Batch), _P(DenseDesc)],
+    "jg_mingru_scan": [_vp, _P(Batch), _P(MinGruDesc)],
+    "jg_delta_scratch_floats": [_P(DeltaDesc), _i32, _P(_u64)],
+    "jg_delta_rule": [_vp, _P(Batch), _P(DeltaDesc)],
+    "jg_latent_scratch_bytes": [_P(LatentDesc), _i32, _i32, _P(_u64)],
+    "jg_latent_attn": [_vp, _P(Batch), _P(LatentDesc)],
+    "jg_sample_f32": [_vp, _u64, _u64, _u64, _u64, _i32, _i32, _f32, _i32, _f32, _f32, _f32],
     "jg_norm_logits_argmax_shard": [_vp, _u64, _u64, _u64, _u64, _f32, _u64, _u64, _i32, _i32, _i32, _i32],
 }
 
 _lib: C.CDLL | None = None
+_partial = False
+
+
+def use_component(name: str) -> str:
+    """Bind the library of one model family (build.COMPONENTS) instead of the whole one, compiling what it needs first.
+    An up-to-date whole library is used as it is.  Must come before the first call into the library."""
+    global LIB_PATH, _partial
+    if _lib is not None or os.environ.get("JG_LIB"):
+        return LIB_PATH
+    from . import build
+    if build.fresh():
+        LIB_PATH, _partial = build.LIB, False
+    else:
+        LIB_PATH, _partial = build.build(component=name), True
+    return LIB_PATH
 
 
 def load() -> C.CDLL:
@@ -144,6 +206,8 @@ def load() -> C.CDLL:
                           "(there is no CPU fallback for the CUDA device)")
     lib = C.CDLL(LIB_PATH)
     for name, args in SIGNATURES.items():
+        if _partial and not hasattr(lib, name):  # another model family's kernel: calling it raises
+            continue
         fn = getattr(lib, name)  # AttributeError if the symbol is not exported
         fn.argtypes = args
         fn.restype = C.c_int

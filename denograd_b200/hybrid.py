@@ -1,0 +1,596 @@
+"""Decoders given as a list of layers, each with its own kind of mixer and an optional feed-forward.
+
+  stream x (fp32) = embedding rows
+  per layer   x <- x + norm_b(mixer(norm(x)));  with a feed-forward: x <- x + norm_b(ff(norm(x)))
+  logits      = head norm(x)
+
+Mixers (`MIXERS`): ``mingru`` (gated linear recurrence), ``latent_attention`` (low-rank keys and values, sliding window,
+sinks, YaRN rotary), ``delta`` (gated delta rule with short convolutions).  Feed-forwards (`FEED_FORWARDS`): ``dense`` (clamped
+gated unit with biases).  Norms divide groups of channels by their own root mean square.  A model's configuration gives
+every size; `ARCHITECTURES` (registry.py) maps a configuration to the model.
+
+How a step runs: each layer contributes library calls to a *plan* — descriptors of device addresses, made once per
+workspace — and a step walks the plan with the batch (sequences, tokens per sequence, positions, slots) as the only
+argument that changes.  With 1-2 rows the plan has no calls for norms and residual sums: the projection that follows takes
+the fp32 stream and does them in its prologue, and the minGRU recurrence is the epilogue of its projections.  A decode step
+is captured into a CUDA graph.
+"""
+from __future__ import annotations
+
+import ctypes as C
+import math
+
+import numpy as np
+
+from . import ffi
+from .cache import SlotStates
+from .decoder import Decoder, TinyJit
+from .device import CUDA, Tensor
+from .nn import _dev
+
+DTYPES = {"float32": ffi.JG_F32, "bfloat16": ffi.JG_BF16}
+
+
+def round_up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+# ------------------------------------------------------------------------------------------------ parameters
+class Param:
+    """Where one checkpoint tensor goes: `shape` values, rows of `cols` in device rows `ld` apart (zeros in between)."""
+
+    def __init__(self, tensor: Tensor, shape: tuple, ld: int | None = None):
+        self.tensor, self.shape, self.ld = tensor, tuple(shape), ld
+
+    def assign(self, arr: np.ndarray) -> None:
+        arr = np.asarray(arr, np.float32)
+        if self.ld is not None and self.ld != self.shape[-1]:
+            wide = np.zeros(self.shape[:-1] + (self.ld,), np.float32)
+            wide[..., :self.shape[-1]] = arr
+            arr = wide
+        self.tensor.assign(arr)
+
+
+class Matrix:
+    """Projection weights [N][ld] of the model's element type; `parts` names runs of rows after checkpoint tensors."""
+
+    def __init__(self, m: "HybridTransformer", params: dict, parts: list[tuple[str, int]], K: int):
+        self.N, self.K, self.ld = sum(n for _, n in parts), K, round_up(K, 8)
+        self.weight = Tensor.zeros((self.N, self.ld), m.dtype, m.dev)
+        self.row0, r = {}, 0
+        for name, n in parts:
+            params[name] = Param(self.weight.view_rows(r, r + n), (n, K), self.ld)
+            self.row0[name], r = r, r + n
+
+    @property
+    def ptr(self) -> int:
+        return self.weight.ptr
+
+    def rows_ptr(self, name: str) -> int:
+        return self.weight.ptr + self.row0[name] * self.ld * self.weight.nbytes // self.weight.numel()
+
+
+def vector(m: "HybridTransformer", params: dict, parts: list[tuple[str, tuple]], pad: int = 0) -> Tensor:
+    """fp32 parameters of consecutive checkpoint tensors (scalars per channel, taps, ...), `pad` zeros behind them."""
+    width = parts[0][1][1:]
+    n = sum(s[0] for _, s in parts)
+    t = Tensor.zeros((n + pad,) + width, "float32", m.dev)
+    r = 0
+    for name, s in parts:
+        params[name] = Param(t.view_rows(r, r + s[0]), s)
+        r += s[0]
+    return t
+
+
+# ------------------------------------------------------------------------------------------------ plans
+class Plan:
+    """The calls of one step on one workspace, and where the residual stream stands while it is being written.
+
+    A sublayer's output `y` is not added to the stream by the kernel that made it: the sum, the norm before it and the norm
+    after it happen together in whatever reads the stream next (`into`)."""
+
+    def __init__(self, model: "HybridTransformer", ws: "_Rows", fused: bool, single: bool):
+        self.model, self.ws, self.fused, self.single = model, ws, fused, single
+        self.calls: list[tuple] = []
+        self.cur = 0          # stream buffer that holds x
+        self.pending = None   # norm weight of a sum that is still to be made (ws.y)
+
+    def call(self, name: str, *args) -> None:
+        self.calls.append((name,) + args)
+
+    def stream(self, w_norm: Tensor | None, rows: int = 0, keep: bool = True) -> ffi.StreamDesc:
+        m, ws = self.model, self.ws
+        out = 0
+        src = ws.x[self.cur].ptr
+        y, w_add = (ws.y.ptr, self.pending.ptr) if self.pending is not None else (0, 0)
+        if self.pending is not None and keep:
+            if self.fused:
+                self.cur ^= 1
+            out = ws.x[self.cur].ptr
+            self.pending = None
+        return ffi.StreamDesc(m.width, m.groups, m.eps, 0, src, y, w_add, out, w_norm.ptr if w_norm is not None else 0, rows)
+
+    def dense(self, desc: ffi.DenseDesc, w_norm: Tensor) -> None:
+        """A projection of the normed stream."""
+        if self.fused:
+            desc.stream = self.stream(w_norm)
+        else:
+            self.call("jg_stream_norm", self.stream(w_norm), self.ws.h.ptr, self.model.ld_width, self.model.dt)
+            desc.x, desc.ldx = self.ws.h.ptr, self.model.ld_width
+        self.call("jg_dense", desc)
+
+    def project(self, w: Matrix, w_norm: Tensor, bias: int = 0) -> int:
+        """Normed stream -> ws.proj; returns the row stride."""
+        ld = round_up(w.N, 8)
+        self.dense(ffi.DenseDesc(self.model.dt, ffi.DENSE_STORE, w.N, w.K, 0, w.ld, ld, 0, 0.0, 0, 0, w.ptr, 0, 0, bias, 0, 0,
+                                 self.ws.proj.ptr), w_norm)
+        return ld
+
+    def output(self, w: Matrix, x: int, ldx: int, w_add: Tensor, bias: int = 0) -> None:
+        """The sublayer's last projection -> ws.y, to be normed with w_add and added to the stream."""
+        m = self.model
+        self.call("jg_dense", ffi.DenseDesc(m.dt, ffi.DENSE_STORE, w.N, w.K, ldx, w.ld, m.width, 1, 0.0, 0, x, w.ptr, 0, 0, bias, 0, 0,
+                                            self.ws.y.ptr))
+        self.pending = w_add
+
+    def finish_layer(self) -> None:
+        self.calls.append(None)  # a boundary for `HybridTransformer.layer_outputs`
+
+    def run(self, batch: ffi.Batch) -> None:
+        ref, h = C.byref(batch), self.model.dev.handle
+        for c in self.calls:
+            if c is not None:
+                ffi.call(c[0], h, ref, *c[1:])
+
+
+# ------------------------------------------------------------------------------------------------ mixers
+class MinGRU:
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        W = self.width = int(cfg["width"])
+        self.w = Matrix(m, params, [(name + "z", W), (name + "x", W), (name + "g", W)], m.width)
+        self.gate_ptrs = [self.w.rows_ptr(name + n) for n in "zxg"]
+        self.bias = vector(m, params, [(name + "z.b", (W,)), (name + "x.b", (W,))], pad=W)  # the output gate has none
+        self.o = Matrix(m, params, [(name + "o", m.width)], W)
+        self.state = m.states.per_slot((W,), "float32")
+        self.proj_ld, self.act_ld, self.scratch = round_up(3 * W, 8), round_up(W, 8), lambda B, Sc: 0
+
+    def plan(self, p: Plan, w_norm: Tensor, w_add: Tensor) -> None:
+        m, ws, W = p.model, p.ws, self.width
+        if p.fused and p.single:
+            b = self.bias.ptr
+            p.dense(ffi.DenseDesc(m.dt, ffi.DENSE_MINGRU, W, m.width, 0, self.w.ld, self.act_ld, 0, 0.0, 0, 0, *self.gate_ptrs, b, b + 4 * W, 0,
+                                  ws.act.ptr, 0, self.state.ptr), w_norm)
+        else:
+            ld = p.project(self.w, w_norm, self.bias.ptr)
+            p.call("jg_mingru_scan", ffi.MinGruDesc(m.dt, W, ld, self.act_ld, ws.proj.ptr, self.state.ptr, ws.act.ptr))
+        p.output(self.o, ws.act.ptr, self.act_ld, w_add)
+
+
+class GatedDelta:
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        H, G, d, v, taps = (int(cfg[k]) for k in ("heads", "kv_heads", "dim", "vdim", "conv"))
+        self.sizes = (H, G, d, v, taps)
+        qkv = [(name + "q", G * d), (name + "k", G * d), (name + "v", H * v)]
+        self.w = Matrix(m, params, qkv + [(name + "b", H), (name + "a", H), (name + "g", H * v)], m.width)
+        self.conv = vector(m, params, [(n + ".conv", (c, taps)) for n, c in qkv])
+        self.a_log, self.dt_bias = vector(m, params, [(name + "A_log", (H,))]), vector(m, params, [(name + "dt_bias", (H,))])
+        self.norm = vector(m, params, [(name + "norm", (v,))])
+        self.o = Matrix(m, params, [(name + "o", m.width)], H * v)
+        self.state = m.states.per_slot((H, v, round_up(d, 4)), "float32")
+        self.tail = m.states.per_slot((taps, 2 * G * d + H * v), m.dtype)
+        self.proj_ld, self.act_ld = round_up(self.w.N, 8), round_up(H * v, 8)
+
+    def desc(self, m: "HybridTransformer") -> ffi.DeltaDesc:
+        return ffi.DeltaDesc(m.dt, *self.sizes, self.proj_ld, self.act_ld, m.eps, 0, 0, self.conv.ptr, self.a_log.ptr, self.dt_bias.ptr,
+                             self.norm.ptr, self.state.ptr, self.tail.ptr)
+
+    def scratch(self, B: int, Sc: int) -> int:
+        H, G, d, v, taps = self.sizes
+        n = C.c_uint64(0)
+        ffi.call("jg_delta_scratch_floats", C.byref(ffi.DeltaDesc(0, H, G, d, v, taps)), B * Sc, C.byref(n))
+        return 4 * n.value
+
+    def plan(self, p: Plan, w_norm: Tensor, w_add: Tensor) -> None:
+        p.project(self.w, w_norm)
+        d = self.desc(p.model)
+        d.proj, d.scratch, d.out = p.ws.proj.ptr, p.ws.scratch.ptr, p.ws.act.ptr
+        p.call("jg_delta_rule", d)
+        p.output(self.o, p.ws.act.ptr, self.act_ld, w_add)
+
+
+def yarn_table(dims: int, base: float, scaling: dict | None, positions: int) -> np.ndarray:
+    """fp32 [positions][dims / 2][2]: cos and sin of position * frequency, both times YaRN's attention factor.  The
+    frequencies base^(-2i / dims) are divided by `factor` where their wavelength exceeds the original context, left alone where
+    it is short, and blended linearly in between (`slow` and `fast` are rotations over the original context)."""
+    i = np.arange(dims // 2, dtype=np.float64)
+    f = float(base) ** (-2.0 * i / dims)
+    gain = 1.0
+    if scaling:
+        def pair_of(turns: float) -> float:  # the pair that turns that often over the original context
+            return dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+
+        lo, hi = max(math.floor(pair_of(scaling["fast"])), 0), min(math.ceil(pair_of(scaling["slow"])), dims - 1)
+        blend = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+        f = f / scaling["factor"] * blend + f * (1.0 - blend)
+        gain = 0.1 * math.log(scaling["factor"]) + 1.0
+    a = np.arange(positions, dtype=np.float64)[:, None] * f
+    return (np.stack([np.cos(a), np.sin(a)], axis=-1) * gain).astype(np.float32)
+
+
+class LatentAttention:
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        H, d, rd, v, rank = (int(cfg[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+        self.H, self.dim, self.rd, self.vd, self.rank = H, d, rd, v, rank
+        self.scale = float(cfg["scale"])
+        self.window = int((cfg.get("mask") or {}).get("size") or 0)
+        rot = cfg["rot"]
+        self.pairs = int(rot["dims"]) // 2
+        if 2 * self.pairs > rd:
+            raise ValueError(f"rotary over {rot['dims']} of {rd} dimensions")
+        self.rot = m.shared_table(("yarn", rot["dims"], rot["base"], tuple(sorted((rot.get("scaling") or {}).items()))),
+                                  lambda: yarn_table(int(rot["dims"]), float(rot["base"]), rot.get("scaling"), m.max_context))
+        self.w = Matrix(m, params, [(name + "q", H * (d + rd)), (name + "dkv", rank + rd)], m.width)
+        self.norm = vector(m, params, [(name + "dkv.norm", (rank,))])
+        self.ukv = Matrix(m, params, [(name + "uk", H * d), (name + "uv", H * v)], rank)
+        self.sink = vector(m, params, [(name + "sink", (H,))])
+        self.o = Matrix(m, params, [(name + "o", m.width)], H * v)
+        self.ring = m.states.ring(round_up(rank + rd, 8), m.dtype, self.window)
+        self.eps, self.max_context, self.dt = m.eps, m.max_context, m.dt
+        self.proj_ld, self.act_ld = round_up(self.w.N, 8), round_up(H * v, 8)
+
+    def desc(self) -> ffi.LatentDesc:
+        r = self.ring
+        return ffi.LatentDesc(self.dt, self.H, self.dim, self.rd, self.vd, self.rank, self.window, self.proj_ld, self.act_ld, r.row, self.ukv.ld,
+                              r.page, r.pages_per_slot, r.table.shape[0], self.pairs, self.max_context, self.eps, self.scale, 0, r.pool.ptr,
+                              r.table.ptr, self.rot.ptr, self.norm.ptr, self.sink.ptr, self.ukv.ptr)
+
+    def scratch(self, B: int, Sc: int) -> int:
+        n = C.c_uint64(0)
+        ffi.call("jg_latent_scratch_bytes", C.byref(self.desc()), B, Sc, C.byref(n))
+        return n.value
+
+    def plan(self, p: Plan, w_norm: Tensor, w_add: Tensor) -> None:
+        p.project(self.w, w_norm)
+        d = self.desc()
+        d.proj, d.scratch, d.scratch_bytes, d.out = p.ws.proj.ptr, p.ws.scratch.ptr, p.ws.scratch.nbytes, p.ws.act.ptr
+        p.call("jg_latent_attn", d)
+        p.output(self.o, p.ws.act.ptr, self.act_ld, w_add)
+
+
+class DenseGLU:
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        f = int(cfg["ff"])
+        self.limit = float(cfg["limit"])
+        self.gate, self.up = Matrix(m, params, [(name + "gate", f)], m.width), Matrix(m, params, [(name + "up", f)], m.width)
+        self.down = Matrix(m, params, [(name + "down", m.width)], f)
+        self.gate_b, self.up_b = vector(m, params, [(name + "gate.b", (f,))]), vector(m, params, [(name + "up.b", (f,))])
+        self.down_b = vector(m, params, [(name + "down.b", (m.width,))])
+        self.ffn_ld = round_up(f, 8)
+
+    def plan(self, p: Plan, w_norm: Tensor, w_add: Tensor) -> None:
+        m, g = p.model, self.gate
+        p.dense(ffi.DenseDesc(m.dt, ffi.DENSE_GLU, g.N, g.K, 0, g.ld, self.ffn_ld, 0, self.limit, 0, 0, g.ptr, self.up.ptr, 0, self.gate_b.ptr,
+                              self.up_b.ptr, 0, p.ws.ffn.ptr), w_norm)
+        p.output(self.down, p.ws.ffn.ptr, self.ffn_ld, w_add, self.down_b.ptr)
+
+
+MIXERS = {"mingru": MinGRU, "latent_attention": LatentAttention, "delta": GatedDelta}
+FEED_FORWARDS = {"dense": DenseGLU}
+
+
+class Layer:
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        D = m.width
+        if cfg["type"] not in MIXERS:
+            raise ValueError(f"unknown mixer {cfg['type']!r} (known: {', '.join(MIXERS)})")
+        self.mixer = MIXERS[cfg["type"]](m, cfg["mixer"], name + "mix.", params)
+        self.norm1, self.norm1b = (vector(m, params, [(name + n, (D,))]) for n in ("norm1", "norm1b"))
+        self.mlp = None
+        if cfg.get("mlp"):
+            kind = cfg["mlp"].get("kind", "dense")
+            if kind not in FEED_FORWARDS:
+                raise ValueError(f"unknown feed-forward {kind!r} (known: {', '.join(FEED_FORWARDS)})")
+            self.mlp = FEED_FORWARDS[kind](m, cfg["mlp"], name + "mlp.", params)
+            self.norm2, self.norm2b = (vector(m, params, [(name + n, (D,))]) for n in ("norm2", "norm2b"))
+
+    def plan(self, p: Plan) -> None:
+        self.mixer.plan(p, self.norm1, self.norm1b)
+        if self.mlp is not None:
+            self.mlp.plan(p, self.norm2, self.norm2b)
+        p.finish_layer()
+
+
+# ------------------------------------------------------------------------------------------------ workspaces
+class _Rows:
+    """Activation buffers for up to `cap` rows of B sequences, and the plans that use them."""
+
+    def __init__(self, m: "HybridTransformer", B: int, cap: int):
+        dev, layers = m.dev, m.layers
+        self.B, self.cap = B, cap
+        self.tokens, self.next_tokens = Tensor.zeros((cap,), "int32", dev), Tensor.zeros((B,), "int32", dev)
+        self.pos, self.seq = Tensor.zeros((B,), "int32", dev), Tensor.zeros((B,), "int32", dev)
+        self.x = [Tensor.zeros((cap, m.width), "float32", dev) for _ in range(2 if cap <= 2 else 1)]
+        self.y = Tensor.zeros((cap, m.width), "float32", dev)
+        self.h = Tensor.zeros((cap, m.ld_width), m.dtype, dev)
+        self.proj = Tensor.zeros((cap, max(l.mixer.proj_ld for l in layers)), m.dtype, dev)
+        self.act = Tensor.zeros((cap, max(l.mixer.act_ld for l in layers)), m.dtype, dev)
+        ffn = max((l.mlp.ffn_ld for l in layers if l.mlp is not None), default=0)
+        self.ffn = Tensor.zeros((cap, ffn * (2 if m.dtype == "float32" else 1)), m.dtype, dev) if ffn else None
+        Sc = max(1, cap // B)
+        self.scratch = Tensor.empty((max(max(l.mixer.scratch(B, s) for l in layers for s in {1, Sc}), 16),), "uint8", dev)
+        self.batch = ffi.Batch(B, 1, self.pos.ptr, self.seq.ptr)
+        self.plans: dict[tuple, Plan] = {}
+        self.heads: dict[tuple, tuple] = {}
+        self.logits = None
+
+
+class _Step(_Rows):
+    """A decode step's workspace: one row per sequence, logits and picks of each, page-locked staging (cf. call_host)."""
+
+    def __init__(self, m: "HybridTransformer", B: int):
+        super().__init__(m, B, B)
+        self.logits = Tensor.zeros((B, m.vocab_size), "float32", m.dev)
+        self.key = Tensor.zeros((B,), "uint64", m.dev)
+        self._dev, self._pinned = m.dev, C.c_void_p()
+        ffi.call("jg_host_alloc", 3 * 4 * B, C.byref(self._pinned))
+        arr = np.ctypeslib.as_array((C.c_int32 * (3 * B)).from_address(self._pinned.value))
+        self.h_tokens, self.h_pos, self.h_next = arr[:B], arr[B:2 * B], arr[2 * B:]
+
+    def __del__(self):
+        try:
+            if self._pinned and self._dev.handle is not None:
+                ffi.call("jg_host_free", self._pinned)
+        except Exception:
+            pass
+
+
+class HybridTransformer(Decoder):
+    """A decoder over `config` (`width`, `vocab`, `norm`, `layers`).  dtype: 'bfloat16' or 'float32'."""
+
+    def __init__(self, config: dict, dtype: str = "bfloat16", max_context: int = 8192, max_batch: int = 1, jit: bool = True, device=None,
+                 page_size: int = 64, max_rows: int = 2048):
+        if dtype not in DTYPES:
+            raise ValueError(f"dtype {dtype!r}: expected one of {', '.join(DTYPES)}")
+        dev = _dev(device)
+        self.dev, self.dtype, self.dt = dev, dtype, DTYPES[dtype]
+        self.width, self.vocab_size = int(config["width"]), int(config["vocab"])
+        self.groups, self.eps = int(config["norm"].get("groups", 1)), float(config["norm"]["eps"])
+        if self.width % self.groups:
+            raise ValueError(f"width {self.width} does not divide into {self.groups} norm groups")
+        self.ld_width = round_up(self.width, 8)
+        self.max_context, self.max_batch, self.max_rows = max_context, max_batch, max(1, min(max_rows, max_context * max_batch))
+        self.states = SlotStates(dev, max_batch, max_context, self.max_rows, page_size)
+        self._tables: dict = {}
+        self.params: dict[str, Param] = {}
+        self.embed = Matrix(self, self.params, [("embed", self.vocab_size)], self.width)
+        self.layers = [Layer(self, c, f"l{i}.", self.params) for i, c in enumerate(config["layers"])]
+        self.norm = vector(self, self.params, [("final.norm", (self.width,))])
+        self.head = Matrix(self, self.params, [("head", self.vocab_size)], self.width)
+        self._steps: dict[int, _Step] = {}
+        self._chunks: dict[tuple[int, int], _Rows] = {}
+        self._row_slots: list[int] = []
+        self._slot_jit: TinyJit | None = None
+        self._slot_ws: _Step | None = None
+        self._out: dict[int, tuple[Tensor, Tensor, Tensor]] = {}
+        self._init_decoder(dev, jit)
+
+    def shared_table(self, key, make) -> Tensor:
+        if key not in self._tables:
+            self._tables[key] = Tensor(make(), device=self.dev)
+        return self._tables[key]
+
+    def load_state_dict(self, weights: dict[str, np.ndarray]) -> "HybridTransformer":
+        """Copy host arrays (exact values of the checkpoint) into the model by name: every tensor, and no other."""
+        missing, extra = sorted(set(self.params) - set(weights)), sorted(set(weights) - set(self.params))
+        if missing or extra:
+            raise KeyError(f"checkpoint does not fit the configuration: missing {missing[:4]}, unexpected {extra[:4]}")
+        for name, p in self.params.items():
+            if tuple(weights[name].shape) != p.shape:
+                raise ValueError(f"Shape mismatch in {name}: Expected shape {p.shape}, but found {tuple(weights[name].shape)} in the checkpoint.")
+            p.assign(weights[name])
+        return self
+
+    # ------------------------------------------------------------------------------------------ workspaces and plans
+    def _workspace(self, B: int) -> _Step:
+        if B > self.max_batch:
+            raise ValueError(f"batch {B} exceeds max_batch {self.max_batch}")
+        if B not in self._steps:
+            self._steps[B] = _Step(self, B)
+            self._steps[B].seq.assign(self._rows_of(B))
+        return self._steps[B]
+
+    def _rows_of(self, B: int) -> np.ndarray:
+        """Slots of batch rows 0 .. B - 1: taken on first use and kept."""
+        while len(self._row_slots) < B:
+            self._row_slots.append(self.states.acquire())
+        return np.array(self._row_slots[:B], np.int32)
+
+    def _chunk(self, B: int, rows: int) -> _Rows:
+        cap = 1
+        while cap < rows:
+            cap *= 2
+        cap = min(max(cap, B), max(self.max_rows, B))
+        cap = max(cap, rows)
+        if (B, cap) not in self._chunks:
+            self._chunks[(B, cap)] = _Rows(self, B, cap)
+        return self._chunks[(B, cap)]
+
+    def _plan(self, ws: _Rows, R: int, single: bool) -> Plan:
+        fused = R <= 2
+        key = (fused, single and fused)
+        if key not in ws.plans:
+            p = Plan(self, ws, *key)
+            if fused and len(ws.x) < 2:
+                ws.x.append(Tensor.zeros(ws.x[0].shape, "float32", self.dev))
+            p.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size)
+            for layer in self.layers:
+                layer.plan(p)
+            ws.plans[key] = p
+        return ws.plans[key]
+
+    def _run_layers(self, ws: _Rows, B: int, Sc: int) -> Plan:
+        ws.batch.B, ws.batch.Sc = B, Sc
+        p = self._plan(ws, B * Sc, Sc == 1)
+        p.run(ws.batch)
+        return p
+
+    def _run_head(self, p: Plan, n: int, rows: int, logits: Tensor, key: Tensor, picks: int) -> None:
+        """Final norm, logits and greedy picks of n rows of the stream: the first n, or those `rows` (device int32) names."""
+        ws, w = p.ws, self.head
+        hk = (n, rows, id(p))
+        if hk not in ws.heads:
+            st = p.stream(self.norm, rows, keep=False)
+            d = ffi.DenseDesc(self.dt, ffi.DENSE_LOGITS, w.N, w.K, 0, w.ld, self.vocab_size, 1, 0.0, 0, 0, w.ptr, 0, 0, 0, 0, 0, logits.ptr, key.ptr)
+            if n <= 2:
+                d.stream = st
+            else:
+                d.ldx = self.ld_width
+            ws.heads[hk] = (st, d, ffi.Batch(n, 1, ws.pos.ptr, ws.seq.ptr))
+        st, d, batch = ws.heads[hk]
+        d.y, d.key = logits.ptr, key.ptr
+        if n > 2:
+            h = self._head_rows(ws, n)
+            d.x = h
+            self.dev.call("jg_stream_norm", C.byref(batch), st, h, self.ld_width, self.dt)
+        self.dev.call("jg_dense", C.byref(batch), d)
+        self.dev.call("jg_argmax_finalize", picks, key.ptr, n)
+
+    def _head_rows(self, ws: _Rows, n: int) -> int:
+        if n <= ws.cap:
+            return ws.h.ptr
+        raise ValueError(f"{n} output rows from {ws.cap} rows")
+
+    def _step(self, ws: _Step, advance: bool = False) -> None:
+        """One token per row: reads ws.tokens / ws.pos / ws.seq, writes ws.logits and ws.next_tokens."""
+        p = self._run_layers(ws, ws.B, 1)
+        self._run_head(p, ws.B, 0, ws.logits, ws.key, ws.next_tokens.ptr)
+        if advance:
+            self.dev.call("jg_copy", ws.tokens.ptr, ws.next_tokens.ptr, 4 * ws.B)
+            self.dev.call("jg_pos_advance", ws.pos.ptr, ws.B)
+
+    # ------------------------------------------------------------------------------------------ decoder hooks
+    def _advance(self, B: int, start_pos: int, n: int) -> None:
+        for s in self._rows_of(B):
+            self.states.advance(int(s), start_pos, n)
+
+    def reusable_prefix(self, n: int) -> int:
+        """State cannot be wound back: what was fed last is reusable only when it is exactly those n tokens."""
+        return n if n and self._row_slots and self.states.length[self._row_slots[0]] == n else 0
+
+    def _feed_rows(self, toks: np.ndarray, start_pos: int, slots: np.ndarray, want: np.ndarray | None) -> list[np.ndarray]:
+        """Tokens [B, S] from start_pos on, in passes of up to max_rows rows.  `want` (B = 1): places whose logits are copied
+        out, a list of [n, vocab] per pass.  Without it the rows of the last position leave logits and picks in the batch's
+        step workspace."""
+        B, S = toks.shape
+        per = max(1, self.max_rows // B)
+        got = []
+        for s0 in range(0, S, per):
+            part = toks[:, s0:s0 + per]
+            Sc = part.shape[1]
+            ws = self._chunk(B, B * Sc)
+            buf = np.zeros((ws.cap,), np.int32)
+            buf[:B * Sc] = part.T.reshape(-1)
+            ws.tokens.assign(buf)
+            ws.pos.assign(np.full((B,), start_pos + s0, np.int32))
+            ws.seq.assign(slots)
+            p = self._run_layers(ws, B, Sc)
+            if want is None:
+                if s0 + Sc >= S:
+                    wsb = self._workspace(B)
+                    rows = self._row_list(ws, np.arange((Sc - 1) * B, Sc * B))
+                    self._run_head(p, B, rows, wsb.logits, wsb.key, wsb.next_tokens.ptr)
+                continue
+            places = want[(want >= s0) & (want < s0 + Sc)] - s0
+            if len(places):
+                n = len(places)
+                logits, key, picks = self._outputs(n)
+                self._run_head(p, n, self._row_list(ws, places), logits, key, picks.ptr)
+                got.append(logits.numpy()[:n])
+        return got
+
+    def _row_list(self, ws: _Rows, rows: np.ndarray) -> int:
+        if getattr(ws, "rows", None) is None:
+            ws.rows = Tensor.zeros((ws.cap,), "int32", self.dev)
+        buf = np.zeros((ws.cap,), np.int32)
+        buf[:len(rows)] = rows
+        ws.rows.assign(buf)
+        return ws.rows.ptr
+
+    def _outputs(self, n: int) -> tuple[Tensor, Tensor, Tensor]:
+        cap = 1
+        while cap < n:
+            cap *= 2
+        if cap not in self._out:
+            self._out[cap] = (Tensor.zeros((cap, self.vocab_size), "float32", self.dev), Tensor.zeros((cap,), "uint64", self.dev),
+                              Tensor.zeros((cap,), "int32", self.dev))
+        return self._out[cap]
+
+    def forward(self, tokens, start_pos: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 0.8,
+                alpha_f: float = 0.0, alpha_p: float = 0.0) -> Tensor:
+        """Tokens int32 [B, S] at positions start_pos ..; the pick after the last one, int32 [B]."""
+        toks = tokens.numpy() if isinstance(tokens, Tensor) else np.asarray(tokens, dtype=np.int32)
+        B, S = toks.shape
+        ws = self._workspace(B)
+        self._advance(B, start_pos, S)
+        self._feed_rows(toks, start_pos, self._rows_of(B), None)
+        return self._pick(ws, temperature, top_k, top_p, alpha_f, alpha_p)
+
+    # ------------------------------------------------------------------------------------------ requests with slots of their own
+    def acquire_slot(self) -> int:
+        return self.states.acquire()
+
+    def release_slot(self, slot: int) -> None:
+        self.states.release(slot)
+
+    def feed(self, slot: int, tokens, start_pos: int, want=()) -> np.ndarray:
+        toks = np.asarray(tokens, np.int32).reshape(1, -1)
+        want = np.asarray(list(want), np.int64)
+        S = toks.shape[1]
+        if S == 0:
+            return np.zeros((0, self.vocab_size), np.float32)
+        if len(want) and (want.min() < 0 or want.max() >= S):
+            raise ValueError(f"wanted places {want.tolist()} outside a portion of {S} tokens")
+        self.states.advance(slot, start_pos, S)
+        if S == 1 and self._jit_enabled:  # the captured decode step
+            if self._slot_ws is None:
+                self._slot_ws = _Step(self, 1)
+                self._slot_jit = TinyJit(lambda: self._step(self._slot_ws), self.dev)
+            ws = self._slot_ws
+            ws.tokens.assign(toks[0])
+            ws.pos.assign(np.array([start_pos], np.int32))
+            ws.seq.assign(np.array([slot], np.int32))
+            self._slot_jit.call()
+            return np.repeat(ws.logits.numpy(), len(want), axis=0)
+        uniq, back = np.unique(want, return_inverse=True)
+        got = self._feed_rows(toks, start_pos, np.array([slot], np.int32), uniq)
+        return np.concatenate(got)[back] if got else np.zeros((0, self.vocab_size), np.float32)
+
+    def layer_outputs(self, slot: int, tokens, start_pos: int = 0) -> np.ndarray:
+        """The residual stream after every layer, fp32 [layers, S, width] (inspection: one portion, up to max_rows tokens)."""
+        toks = np.asarray(tokens, np.int32).reshape(-1)
+        S = len(toks)
+        self.states.advance(slot, start_pos, S)
+        ws = self._chunk(1, S)
+        buf = np.zeros((ws.cap,), np.int32)
+        buf[:S] = toks
+        ws.tokens.assign(buf)
+        ws.pos.assign(np.array([start_pos], np.int32))
+        ws.seq.assign(np.array([slot], np.int32))
+        ws.batch.B, ws.batch.Sc = 1, S
+        out, peek = [], Plan(self, ws, S <= 2, S == 1)
+        if S <= 2 and len(ws.x) < 2:
+            ws.x.append(Tensor.zeros(ws.x[0].shape, "float32", self.dev))
+        peek.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size)
+        res = Tensor.zeros((ws.cap, self.width), "float32", self.dev)
+        for layer in self.layers:
+            layer.plan(peek)
+            st = peek.stream(None, keep=False)
+            st.x_out = res.ptr
+            peek.call("jg_stream_norm", st, 0, self.ld_width, self.dt)
+            peek.run(ws.batch)
+            peek.calls.clear()
+            out.append(res.numpy()[:S])
+        return np.stack(out)
+
+    def last_logits(self, B: int) -> np.ndarray:
+        return self._workspace(B).logits.numpy()

@@ -21,7 +21,8 @@ import os
 import numpy as np
 
 from . import ffi
-from .device import CUDA, CUDAGraph, Device, Tensor
+from .decoder import Decoder, TinyJit, sample  # noqa: F401
+from .device import CUDA, Tensor
 from .nn import Embedding, Linear, RMSNorm, _dev
 
 
@@ -215,38 +216,6 @@ class TransformerBlock:
     __call__ = call
 
 
-_alpha_counter: dict[tuple, Tensor] = {}  # the reference keeps one module-level counter (jsgrad/models/llama.ts:130)
-
-
-def sample(logits: Tensor, temp: float, k: int, p: float, af: float, ap: float, u: Tensor | None = None,
-           out: Tensor | None = None) -> Tensor:
-    """`sample` (jsgrad/models/llama.ts:131-185) per row of fp16 logits [rows, V]: argmax with the lowest index among
-    equals when temp < 1e-6, else alpha penalties, softmax(logits / temp), top-k, approximate top-p and the multinomial
-    draw in one kernel.  `u`: float32 [rows] uniform samples for the draw; by default they come from the restated
-    Tensor.rand stream (denograd_b200.rand, seeded by rand.manual_seed)."""
-    V = logits.shape[-1]
-    rows = logits.numel() // V
-    if p < 0 or p > 1:
-        raise ValueError("p must be between 0 and 1")
-    if k < 0 or k > V:
-        raise ValueError("k must be between 0 and numel")
-    out = out if out is not None else Tensor.empty((rows,), "int32", logits.dev)
-    if temp < 1e-6:
-        logits.dev.call("jg_argmax", out.ptr, logits.ptr, rows, V)
-        return out
-    if u is None:
-        from . import rand
-        u = Tensor(rand.rand(rows, logits.dev.device), device=logits.dev)
-    counter_ptr = 0
-    if af or ap:
-        key = (logits.dev.device, rows, V)
-        if key not in _alpha_counter:
-            _alpha_counter[key] = Tensor.zeros((rows, V), "int32", logits.dev)
-        counter_ptr = _alpha_counter[key].ptr
-    logits.dev.call("jg_sample", out.ptr, logits.ptr, u.ptr, counter_ptr, rows, V, float(temp), int(k), float(p), float(af), float(ap))
-    return out
-
-
 def _norm_first(rows: int, int8: bool, dim: int = 0) -> bool:
     """Whether RMSNorm runs as its own kernel ahead of a projection.  The matrix-vector kernels fuse the norm into
     their prologue; the tensor-core kernels take normalised rows: fp16 weights from 3 rows on; int8 weights beyond 1
@@ -344,35 +313,7 @@ class _StepPlan:
             pass
 
 
-class TinyJit:
-    """Call 0 runs eagerly, call 1 runs while being captured, later calls replay the capture
-    (jsgrad/engine/jit.ts:273-353).  The wrapped function must read its varying inputs from device memory."""
-
-    def __init__(self, fxn, dev: CUDA):
-        self.fxn, self.dev = fxn, dev
-        self.cnt = 0
-        self.graph: CUDAGraph | None = None
-
-    def reset(self) -> None:
-        self.cnt, self.graph = 0, None
-
-    def call(self, *args):
-        if self.cnt == 0:
-            self.fxn(*args)
-        elif self.cnt == 1:
-            g = CUDAGraph(self.dev)
-            with g:
-                self.fxn(*args)
-            self.graph = g
-            g.launch()  # a captured launch list has not run yet
-        else:
-            self.graph.launch()
-        self.cnt += 1
-
-    __call__ = call
-
-
-class Transformer:
+class Transformer(Decoder):
     def __init__(self, dim: int, hidden_dim: int, n_heads: int, n_layers: int, norm_eps: float, vocab_size: int,
                  linear=Linear, embedding=Embedding, n_kv_heads: int | None = None, rope_theta: float = 10000,
                  max_context: int = 1024, jit: bool = True, feed_forward=FeedForward, device=None, max_batch: int = 1,
@@ -422,9 +363,7 @@ class Transformer:
         for i, layer in enumerate(self.layers):
             layer.attention._kv, layer.attention._layer = self._kv, i
         self._ws: dict[int, _Workspace] = {}
-        self._jit_enabled = jit
-        self._forward_jit: dict[int, TinyJit] = {}
-        self._loop_graph: dict[int, CUDAGraph] = {}
+        self._init_decoder(dev, jit)
         self._step_plan = None  # None: not tried yet, False: this model keeps the launch-per-op step
 
     def new_cache(self) -> None:
@@ -542,15 +481,6 @@ class Transformer:
             self._step(ws)
         return self._pick(ws, temperature, top_k, top_p, alpha_f, alpha_p)
 
-    def _pick(self, ws: _Workspace, temperature: float, top_k: int, top_p: float, alpha_f: float, alpha_p: float) -> Tensor:
-        """The token of the last step: the greedy pick the logits kernel already made, or — temperature >= 1e-6 —
-        `sample` over the step's logits (jsgrad/models/llama.ts:212)."""
-        if temperature < 1e-6:
-            return ws.next_tokens
-        if self._tp is not None:
-            raise NotImplementedError("stochastic sampling over a vocabulary-sharded output layer: gather the logits first")
-        return sample(ws.logits, temperature, top_k, top_p, alpha_f, alpha_p, out=ws.next_tokens)
-
     def _max_chunk_rows(self) -> int:
         """Rows one projection call takes: 64 on the mma.sync kernel (int8 weights, or fp16 shapes off the tile grid),
         2048 when every projection of a block also fits the tcgen05 kernel (out features % 128, in features % 64)."""
@@ -633,93 +563,13 @@ class Transformer:
                 tp.all_reduce_max(wsb.key)
             dev.call("jg_argmax_finalize", wsb.next_tokens.ptr, wsb.key.ptr, B)
 
-    def call(self, tokens, start_pos: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 0.8,
-             alpha_f: float = 0.0, alpha_p: float = 0.0) -> Tensor:
-        """Transformer.call (jsgrad/models/llama.ts:214-220): single-token calls after position 0 go through the jit."""
-        toks = tokens.numpy() if isinstance(tokens, Tensor) else np.asarray(tokens, dtype=np.int32)
-        B, S = toks.shape
-        if S == 1 and self._jit_enabled and start_pos != 0:
-            if start_pos + 1 > self.max_context:
-                raise ValueError(f"start_pos {start_pos} + 1 exceeds max_context {self.max_context}")
-            ws = self._workspace(B)
-            ws.tokens.assign(toks[:, 0])
-            ws.pos.assign(np.full((B,), start_pos, np.int32))
-            if B not in self._forward_jit:
-                self._forward_jit[B] = TinyJit(lambda: self._step(ws), self.dev)
-            self._forward_jit[B].call()
-            return self._pick(ws, temperature, top_k, top_p, alpha_f, alpha_p)
-        return self.forward(toks, start_pos, temperature, top_k, top_p, alpha_f, alpha_p)
-
-    __call__ = call
-
-    def call_host(self, tokens: np.ndarray, start_pos: int) -> np.ndarray:
-        """`call(...)` followed by reading the ids back (`.item()` in the reference's loop), for one new token per
-        row after position 0, with the copies staged through page-locked memory: per step B*8 bytes go up (tokens and
-        positions), the captured step runs, B*4 bytes come back.  tokens: int32 [B, 1] -> int32 [B]."""
-        B = tokens.shape[0]
-        if start_pos == 0 or not self._jit_enabled:
-            return self.call(tokens, start_pos).numpy()
-        if start_pos + 1 > self.max_context:
-            raise ValueError(f"start_pos {start_pos} + 1 exceeds max_context {self.max_context}")
-        ws = self._workspace(B)
-        ws.h_tokens[:] = tokens.reshape(B)
-        ws.h_pos[:] = start_pos
-        dev = self.dev
-        dev.call("jg_copyin_async", ws.tokens.ptr, ws.h_tokens.ctypes.data, 4 * B)
-        dev.call("jg_copyin_async", ws.pos.ptr, ws.h_pos.ctypes.data, 4 * B)
-        if B not in self._forward_jit:
-            self._forward_jit[B] = TinyJit(lambda: self._step(ws), self.dev)
-        self._forward_jit[B].call()
-        dev.call("jg_copyout_async", ws.h_next.ctypes.data, ws.next_tokens.ptr, 4 * B)
-        dev.synchronize()
-        return ws.h_next.copy()
-
-    # ------------------------------------------------------------------------------------------ device-resident loop
-    def decode_loop(self, first_tokens, start_pos: int, n_steps: int, collect: bool = True,
-                    resume: bool = False) -> np.ndarray | None:
-        """Greedy-decode `n_steps` tokens per row with no host round trip between steps: the captured step feeds its
-        own output back on the device.  Returns the generated ids [B, n_steps] (read back after the last step), or
-        None when `collect` is false.  With `resume` the tokens and positions already on the device (left by the
-        previous loop) are continued and `first_tokens` only gives the batch size; nothing is copied or synchronised,
-        so a caller can time a run of steps with events."""
-        toks = np.asarray(first_tokens, dtype=np.int32).reshape(-1)
-        B = toks.shape[0]
-        if start_pos + n_steps > self.max_context:
-            raise ValueError(f"start_pos {start_pos} + {n_steps} steps exceeds max_context {self.max_context}")
-        ws = self._workspace(B)
-        if not resume:
-            ws.tokens.assign(toks)
-            ws.pos.assign(np.full((B,), start_pos, np.int32))
-        plan = self._single_kernel_step(B)
-        if plan is not None:
-            # the persistent kernel loops over the steps itself: one launch for the whole run, picks land in `hist`
-            if ws.hist is None or ws.hist.shape[0] < n_steps:
-                ws.hist = Tensor.empty((max(n_steps, 64), B), "int32", self.dev)
-            ffi.call("jg_step_run", plan.handle, ws.tokens.ptr, ws.pos.ptr, ws.h.ptr, ws.qkv.ptr, ws.attn.ptr, ws.ffn.ptr,
-                     ws.logits.ptr, ws.hist.ptr, B, n_steps, 1)
-            if not collect:
-                return None
-            out = ws.hist.numpy()[:n_steps].T.copy()
-            self.dev.call("jg_copy", ws.next_tokens.ptr, ws.hist.ptr + 4 * B * (n_steps - 1), 4 * B)
-            return out
-        if B not in self._loop_graph:
-            if resume:
-                raise ValueError("nothing to resume: run decode_loop once without `resume` first")
-            self._step(ws, advance=True)  # eager once (sizes smem attributes), then restore the inputs and capture
-            ws.tokens.assign(toks)
-            ws.pos.assign(np.full((B,), start_pos, np.int32))
-            g = CUDAGraph(self.dev)
-            with g:
-                self._step(ws, advance=True)
-            self._loop_graph[B] = g
-        g = self._loop_graph[B]
-        hist = Tensor.empty((n_steps, B), "int32", self.dev) if collect else None
-        for i in range(n_steps):
-            g.launch()
-            if collect:
-                self.dev.call("jg_copy", hist.ptr + 4 * B * i, ws.next_tokens.ptr, 4 * B)
-        return hist.numpy().T.copy() if collect else None
-
-    def last_logits(self, B: int) -> np.ndarray:
-        """fp16 logits of the last step widened to fp32 (`.float()` at jsgrad/models/llama.ts:210), [B, vocab]."""
-        return self._workspace(B).logits.numpy().astype(np.float32)
+    def _loop_launch(self, ws: _Workspace, n_steps: int) -> Tensor | None:
+        """The persistent kernel loops over the steps itself: one launch for the whole run, picks land in `hist`."""
+        plan = self._single_kernel_step(ws.B)
+        if plan is None:
+            return None
+        if ws.hist is None or ws.hist.shape[0] < n_steps:
+            ws.hist = Tensor.empty((max(n_steps, 64), ws.B), "int32", self.dev)
+        ffi.call("jg_step_run", plan.handle, ws.tokens.ptr, ws.pos.ptr, ws.h.ptr, ws.qkv.ptr, ws.attn.ptr, ws.ffn.ptr,
+                 ws.logits.ptr, ws.hist.ptr, ws.B, n_steps, 1)
+        return ws.hist

@@ -27,8 +27,9 @@ def bf16_to_f16(raw: np.ndarray) -> np.ndarray:
         return (raw.astype(np.uint32) << 16).view(np.float32).astype(np.float16)
 
 
-def safe_load(path: str) -> dict[str, np.ndarray]:
-    """Read every tensor of a .safetensors file (memory-mapped; BF16 tensors come back as float16)."""
+def safe_load(path: str, widen_bf16: bool = False) -> dict[str, np.ndarray]:
+    """Read every tensor of a .safetensors file (memory-mapped).  BF16 tensors come back as float16, or exactly, as
+    float32, with `widen_bf16`."""
     with open(path, "rb") as f:
         head = f.read(8)
         if len(head) != 8:
@@ -48,7 +49,8 @@ def safe_load(path: str) -> dict[str, np.ndarray]:
             raise ValueError(f"{path}: tensor {name} lies outside the file")
         raw, shape, tag = data[lo:hi], tuple(info["shape"]), info["dtype"]
         if tag == "BF16":
-            arr = bf16_to_f16(raw.view(np.uint16))
+            bits = raw.view(np.uint16)
+            arr = (bits.astype(np.uint32) << 16).view(np.float32) if widen_bf16 else bf16_to_f16(bits)
         elif tag in _SAFE_DTYPES:
             arr = raw.view(_SAFE_DTYPES[tag])
         else:
@@ -78,17 +80,17 @@ def safe_save(tensors: dict[str, np.ndarray], path: str, metadata: dict | None =
             f.write(v.tobytes())
 
 
-def load_checkpoint(path: str) -> dict[str, np.ndarray]:
+def load_checkpoint(path: str, widen_bf16: bool = False) -> dict[str, np.ndarray]:
     """One .safetensors file, or a sharded checkpoint through its *.index.json (weight_map: tensor name -> file name,
     files next to the index), as Llama3._load resolves them (jsgrad/models/llama3.ts:201-213)."""
     if path.endswith(".index.json"):
         with open(path) as f:
             weight_map = json.load(f)["weight_map"]
         base = os.path.dirname(path)
-        parts = {fn: safe_load(os.path.join(base, fn)) for fn in sorted(set(weight_map.values()))}
+        parts = {fn: safe_load(os.path.join(base, fn), widen_bf16) for fn in sorted(set(weight_map.values()))}
         return {k: parts[fn][k] for k, fn in weight_map.items()}
     if path.endswith(".safetensors"):
-        return safe_load(path)
+        return safe_load(path, widen_bf16)
     if path.endswith(".gguf"):
         from .gguf import gguf_load
         return gguf_load(np.memmap(path, dtype=np.uint8, mode="r"))[1]

@@ -85,3 +85,26 @@ def fill_model(model, base_seed: int = BASE_SEED) -> dict[str, Tensor]:
         fill_tensor(name, t, base_seed)
         done.add(t.ptr)
     return sd
+
+
+def fill_hybrid(model, base_seed: int = BASE_SEED) -> None:
+    """Fill a layer-list model (hybrid.HybridTransformer): matrices ~N(0, WEIGHT_STD) on the device, norm weights 1, the few
+    per-channel parameters (biases, taps, decays, sinks) from the same generator on the host."""
+    for name, p in model.params.items():
+        seed = name_seed(name, base_seed)
+        if p.ld is not None:
+            t = p.tensor
+            t.dev.call("jg_fill_normal", t.ptr, model.dt, seed, p.shape[0], p.shape[1], p.ld, WEIGHT_STD)
+            continue
+        n = int(np.prod(p.shape))
+        u = (_word(seed, np.arange(n, dtype=np.uint64)) >> np.uint64(40)).astype(np.float64) / 2.0 ** 24
+        leaf = name.rsplit(".", 1)[-1]
+        if "norm" in leaf:
+            v = np.ones(n)
+        elif leaf == "A_log":
+            v = np.log(0.02 + u)
+        elif leaf == "conv":
+            v = u - 0.25
+        else:
+            v = 0.2 * (u - 0.5)
+        p.assign(v.reshape(p.shape))

@@ -86,6 +86,16 @@ export const SYMBOLS = {
   jg_fill_uniform_i8: fn([ptr, u64, u64, u64, u64]),
   jg_fill_scale_f16: fn([ptr, u64, u64, u64, u64, f32]),
   jg_fill_const_f16: fn([ptr, u64, u64, f32]),
+  jg_fill_normal: fn([ptr, u64, i32, u64, u64, u64, u64, f32]),
+  jg_stream_embed: fn([ptr, buf, u64, u64, u64, i32, i32, i32, i32]),
+  jg_stream_norm: fn([ptr, buf, buf, u64, i32, i32]),
+  jg_dense: fn([ptr, buf, buf]),
+  jg_mingru_scan: fn([ptr, buf, buf]),
+  jg_delta_scratch_floats: fn([buf, i32, buf]),
+  jg_delta_rule: fn([ptr, buf, buf]),
+  jg_latent_scratch_bytes: fn([buf, i32, i32, buf]),
+  jg_latent_attn: fn([ptr, buf, buf]),
+  jg_sample_f32: fn([ptr, u64, u64, u64, u64, i32, i32, f32, i32, f32, f32, f32]),
   jg_fill_normal_f16_2d: fn([ptr, u64, u64, u64, u64, u64, u64, u64, f32]),
   jg_fill_uniform_i8_2d: fn([ptr, u64, u64, u64, u64, u64, u64, u64]),
   jg_comm_unique_id: fn([buf, buf]),

@@ -382,12 +382,101 @@ int jg_dequant_i8_f16(jg_dev* dev, uint64_t dst, uint64_t w, uint64_t scale, int
  * device serves NF4 weights (the packed form stays the resident one; the copy is a per-call scratch). */
 int jg_dequant_nf4_f16(jg_dev* dev, uint64_t dst, uint64_t w, uint64_t scale, int64_t n, int32_t block);
 
+/* ---- Models given as a list of layers (denograd_b200/hybrid.py): recurrent mixers and latent attention with a norm before
+ *      and after every sublayer.  They have no counterpart in the reference, whose one decoder is the Llama block above.
+ *      T = the element type of weights and activations, `dtype` below: bf16 for serving, float for everything in 32 bits.
+ *      Independent of T the residual stream, norms, attention scores and weights, gates and recurrent state are fp32, and
+ *      so are small parameters (norm weights, biases, convolution taps, sinks, decays).
+ *      Rows of a call: Sc consecutive tokens of each of B sequences, position-major (row = s * B + b); sequence b starts
+ *      at position pos[b] and owns slot seq[b] of every per-sequence store.  A sequence that starts at position 0 never
+ *      reads what its slot held before.  Weight matrices are [N][ldw] with ldw a multiple of 16 bytes and zeros between
+ *      K and ldw; activation rows carry finite values there. */
+#define JG_F32 0
+#define JG_BF16 1
+#define JG_DENSE_STORE 0   /* y = x W0^T + b0 */
+#define JG_DENSE_GLU 1     /* g = min(x W0^T + b0, limit), u = clamp(x W1^T + b1, +-limit); y = g sigmoid(1.702 g) (u + 1) */
+#define JG_DENSE_MINGRU 2  /* W0, W1, W2 = update gate, candidate, output gate: one token of jg_mingru_scan per row */
+#define JG_DENSE_LOGITS 3  /* y = x W0^T in fp32, and (value, lowest index) keys for jg_argmax_finalize */
+
+typedef struct {
+  int32_t B, Sc;
+  uint64_t pos, seq; /* device int32 [B] each */
+} jg_batch;
+
+/* x <- x + norm(y) * w_add (y = 0: nothing), stored to x_out (0: not); h = norm(x) * w_norm (0: nothing).  norm divides each
+ * of `groups` equal parts of a row by sqrt(mean(part^2) + eps).  rows (0 = identity): device int32 row numbers into x, y. */
+typedef struct {
+  int32_t width, groups;
+  float eps;
+  int32_t reserved;
+  uint64_t x, y, w_add, x_out, w_norm, rows;
+} jg_stream_desc;
+
+/* x = 0: the rows are h of `stream` (1-2 rows; x_out must be another buffer than x).  fp32 GLU of 3+ rows uses the rows M
+ * .. 2M of y as scratch. */
+typedef struct {
+  int32_t dtype, epilogue, N, K, ldx, ldw, ldy, out_f32;
+  float limit;
+  int32_t reserved;
+  uint64_t x, w0, w1, w2, b0, b1, b2, y, key, state;
+  jg_stream_desc stream;
+} jg_dense_desc;
+
+/* minGRU: z = sigmoid(zin), c = u >= 0 ? u + 1/2 : sigmoid(u); S <- (1 - z) S + z c; out = S silu(g), element by element.
+ * proj: T [R][ldp] = zin | u | g, `width` each (biases included); state: fp32 [slots][width]; out: T [R][ldo]. */
+typedef struct {
+  int32_t dtype, width, ldp, ldo;
+  uint64_t proj, state, out;
+} jg_mingru_desc;
+
+/* Gated delta rule.  proj: T [R][ldp] = q | k (kv_heads x dim each) | v (heads x vdim) | b | a (heads each) | g (heads x vdim).
+ * q, k, v: causal convolution of `taps` taps per channel, silu; q, k unit vectors per head, q / sqrt(dim).
+ * S <- exp(-exp(a_log) softplus(a + dt_bias)) S; u = sigmoid(b) (v - S^T k); S <- S + k u^T; o = S^T q;
+ * out = o / rms(o) * norm_w * silu(g).  state: fp32 [slots][heads][vdim][dim4] (S transposed, dim4 = dim rounded up to 4);
+ * tail: T [slots][taps][channels], the last inputs of the convolution, indexed by position modulo taps.
+ * scratch: fp32, jg_delta_scratch_floats(desc, R). */
+typedef struct {
+  int32_t dtype, heads, kv_heads, dim, vdim, taps, ldp, ldo;
+  float eps;
+  int32_t reserved;
+  uint64_t proj, conv_w, a_log, dt_bias, norm_w, state, tail, scratch, out;
+} jg_delta_desc;
+
+/* Latent attention.  proj: T [R][ldp] = q (heads x (dim | rot_dim)) | latent (kv_rank) | rotated key part (rot_dim).
+ * The cache keeps per position the normed latent and the rotated key part, T [n_pages][page][ldc]: positions
+ * [i * page, (i + 1) * page) of slot s live on page block_table[s][i % pages_per_slot], so that a window needs only as many
+ * pages as it and one call's tokens span.  rot: fp32 [rot_rows][rot_pairs][2] (cos, sin).  window = 0: every earlier
+ * position.  The denominator of the softmax also contains exp(sink[h]).  uk, uv: [heads * dim][ld_u], [heads * vdim][ld_u]
+ * contiguous (uv = uk + heads * dim rows).  scratch: jg_latent_scratch_bytes(desc, B, Sc) bytes. */
+typedef struct {
+  int32_t dtype, heads, dim, rot_dim, vdim, kv_rank, window, ldp, ldo, ldc, ld_u, page, pages_per_slot, n_slots, rot_pairs, rot_rows;
+  float eps, scale;
+  uint64_t proj, pool, block_table, rot, norm_w, sink, ukv, scratch, out;
+  uint64_t scratch_bytes;
+} jg_latent_desc;
+
+/* embedding rows (T [vocab][ld]) widened into the fp32 residual stream */
+int jg_stream_embed(jg_dev* dev, const jg_batch* batch, uint64_t out, uint64_t tokens, uint64_t table, int32_t dtype, int32_t dim,
+                    int32_t ld, int32_t vocab);
+int jg_stream_norm(jg_dev* dev, const jg_batch* batch, const jg_stream_desc* s, uint64_t h, int32_t ldh, int32_t dtype);
+int jg_dense(jg_dev* dev, const jg_batch* batch, const jg_dense_desc* d);
+int jg_mingru_scan(jg_dev* dev, const jg_batch* batch, const jg_mingru_desc* d);
+int jg_delta_scratch_floats(const jg_delta_desc* d, int32_t rows, uint64_t* out);
+int jg_delta_rule(jg_dev* dev, const jg_batch* batch, const jg_delta_desc* d);
+int jg_latent_scratch_bytes(const jg_latent_desc* d, int32_t B, int32_t Sc, uint64_t* out);
+int jg_latent_attn(jg_dev* dev, const jg_batch* batch, const jg_latent_desc* d);
+/* jg_sample over fp32 logits */
+int jg_sample_f32(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B, int32_t V,
+                  float temp, int32_t k, float p, float af, float ap);
+
 /* ---- Seeded synthetic tensors (stand-in for Tensor.randn/uniform, jsgrad/tensor.ts:796-843, which the
  *      workloads replace by fixed distributions).  Counter-based, so any sub-range can be generated. */
 int jg_fill_normal_f16(jg_dev* dev, uint64_t dst, uint64_t seed, uint64_t first, uint64_t n, float std);
 int jg_fill_uniform_i8(jg_dev* dev, uint64_t dst, uint64_t seed, uint64_t first, uint64_t n);
 int jg_fill_scale_f16(jg_dev* dev, uint64_t dst, uint64_t seed, uint64_t first, uint64_t n, float base);
 int jg_fill_const_f16(jg_dev* dev, uint64_t dst, uint64_t n, float value);
+/* the normal fill as T = bf16 or float, [rows][cols] with ld elements between rows (what lies between is left alone) */
+int jg_fill_normal(jg_dev* dev, uint64_t dst, int32_t dtype, uint64_t seed, uint64_t rows, uint64_t cols, uint64_t ld, float std);
 /* [rows][cols] window at (row0, col0) of a [*][full_cols] tensor: a shard gets the values the whole tensor would. */
 int jg_fill_normal_f16_2d(jg_dev* dev, uint64_t dst, uint64_t seed, uint64_t rows, uint64_t cols, uint64_t full_cols,
                           uint64_t row0, uint64_t col0, float std);

@@ -24,6 +24,9 @@ in the KV cache, greedy decoding.  One JSON line is printed by rank 0:
   cpu_baseline  the CPU restatement of the reference's CLANG path (oracle/), timed on this host's cores on a bounded
              sample: full-width 1-, 4- and 8-layer slices with 512 positions in the cache, extrapolated in depth.
 
+`--hybrid SIZE` runs another workload in place of the default one: a layer-list model (Matulorn) with the layer sizes of the
+Llama of that size, prefill and decode at several batch sizes, call by call, with the Llama at the same sizes beside it.
+
 `--impl reference` times that CPU restatement as the reference arm (the reference itself needs a JS runtime and
 clang, neither of which exists here).
 """
@@ -563,6 +566,207 @@ def run_gpu(args) -> None:
         rig.dist.destroy_process_group()
 
 
+# ------------------------------------------------------------------------------------------------ layer-list models
+def hybrid_config(size: str, layers: int = 0) -> dict:
+    """A Matulorn configuration with the layer sizes of the Llama of that size: same width, depth, feed-forward and
+    vocabulary; of every four layers one is latent attention, one minGRU and two are gated delta."""
+    p, _ = arch(size)
+    d, ff, L = p["dim"], p["hidden_dim"], layers or p["n_layers"]
+    H = d // 128
+    mixers = [{"type": "latent_attention", "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "mask": {"size": 4096},
+                                                     "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}},
+                                                     "scale": 192 ** -0.5}},
+              {"type": "delta", "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}},
+              {"type": "mingru", "mixer": {"width": d}},
+              {"type": "delta", "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}]
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    return {"architecture": "Matulorn", "width": d, "vocab": p["vocab_size"], "norm": {"eps": 1e-6, "groups": 4},
+            "layers": [dict(mixers[i % 4], mlp=mlp) for i in range(L)]}
+
+
+def hybrid_bytes(cfg: dict, B: int, T: float) -> float:
+    """Bytes one decode step has to move: every matrix once, recurrent state read and written, the cached window read."""
+    d, by = cfg["width"], 2.0 * cfg["vocab"] * cfg["width"]
+    for lc in cfg["layers"]:
+        m = lc["mixer"]
+        if lc["type"] == "mingru":
+            by += 2.0 * 4 * d * m["width"] + B * 8.0 * m["width"]
+        elif lc["type"] == "delta":
+            qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            by += 2.0 * d * (2 * qk + 3 * v + 2 * m["heads"]) + B * (8.0 * m["heads"] * m["dim"] * m["vdim"] + 2.0 * m["conv"] * (2 * qk + v))
+        else:
+            H, r = m["heads"], m["kv_rank"]
+            by += 2.0 * (d * (H * (m["dim"] + m["rot_dim"]) + r + m["rot_dim"]) + H * (m["dim"] + m["vdim"]) * r + d * H * m["vdim"])
+            by += B * 2.0 * min(T, m["mask"]["size"]) * (r + m["rot_dim"])
+        by += 2.0 * 3 * d * lc["mlp"]["ff"]
+    return by
+
+
+def hybrid_flops(cfg: dict, B: int, S: int) -> float:
+    """Flops of a prompt of S tokens from an empty state: projections on all rows, the head on the last ones, windowed causal
+    attention over expanded keys and values, 8 flops per state element and token of the delta rule."""
+    d, fl = cfg["width"], 2.0 * B * cfg["vocab"] * cfg["width"]
+    for lc in cfg["layers"]:
+        m = lc["mixer"]
+        if lc["type"] == "mingru":
+            w = 4.0 * d * m["width"]
+        elif lc["type"] == "delta":
+            qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            w = d * (2.0 * qk + 3 * v + 2 * m["heads"])
+            fl += 8.0 * B * S * m["heads"] * m["dim"] * m["vdim"]
+        else:
+            H, r, W = m["heads"], m["kv_rank"], m["mask"]["size"]
+            w = d * (H * (m["dim"] + m["rot_dim"]) + r + m["rot_dim"]) + H * (m["dim"] + m["vdim"]) * r + d * H * m["vdim"]
+            pairs = S * S / 2.0 if S <= W else W * W / 2.0 + (S - W) * float(W)
+            fl += 2.0 * B * H * pairs * (m["dim"] + m["rot_dim"] + m["vdim"])
+        fl += 2.0 * B * S * (w + 3.0 * d * lc["mlp"]["ff"])
+    return fl
+
+
+def record_calls(fn) -> list[tuple]:
+    """The library's kernel calls that fn makes (they run as well)."""
+    from denograd_b200 import ffi
+    calls, real = [], ffi.call
+
+    def call(name, *a):
+        real(name, *a)
+        if not name.startswith(("jg_copy", "jg_memset", "jg_alloc", "jg_free", "jg_device", "jg_timer", "jg_graph", "jg_host", "jg_launch")):
+            calls.append((name, a))
+    ffi.call = call
+    try:
+        fn()
+    finally:
+        ffi.call = real
+    return calls
+
+
+def call_work(name: str, a: tuple, R: int, T: float) -> tuple[str, float, float] | None:
+    """(label, bytes, flops) of one recorded projection or mixer call on R rows with T cached positions."""
+    from denograd_b200 import ffi
+    if name == "jg_dense":
+        d = a[2]
+        nw = {ffi.DENSE_GLU: 2, ffi.DENSE_MINGRU: 3}.get(d.epilogue, 1)
+        n = nw * d.N
+        kind = {ffi.DENSE_GLU: "gate/up + GLU", ffi.DENSE_MINGRU: "minGRU gates + recurrence", ffi.DENSE_LOGITS: "logits"}.get(d.epilogue, "projection")
+        return f"{kind} {n}x{d.K}" + (" (norms fused)" if d.x == 0 else ""), 2.0 * n * d.K + R * (2.0 * d.K + 2.0 * d.N), 2.0 * R * n * d.K
+    if name == "jg_latent_attn":
+        d = a[2]
+        span = min(T, d.window) if d.window else T
+        ukv = d.heads * (d.dim + d.vdim) * d.kv_rank
+        pairs = span if R == 1 or span < R else span  # decode: every row sees `span`
+        return "latent attention", 2.0 * ukv + 2.0 * span * (d.kv_rank + d.rot_dim) * (R if T > R else 1), 2.0 * R * ukv + 2.0 * d.heads * R * pairs * (d.dim + d.rot_dim + d.vdim) * (0.5 if T <= R else 1.0)
+    if name == "jg_delta_rule":
+        d = a[2]
+        st = d.heads * d.dim * d.vdim
+        return "delta rule", 8.0 * st + R * 2.0 * (d.ldp + d.ldo), 8.0 * R * st
+    if name == "jg_mingru_scan":
+        d = a[2]
+        return "minGRU scan", R * 2.0 * (d.ldp + d.ldo) + 8.0 * d.width, 0.0
+    if name in ("jg_norm_linear", "jg_linear", "jg_norm_swiglu", "jg_norm_logits_argmax_shard"):
+        M, N, K = {"jg_norm_linear": a[-3:], "jg_linear": a[-3:], "jg_norm_swiglu": a[-3:], "jg_norm_logits_argmax_shard": a[-4:-1]}[name]
+        n = 2 * N if name == "jg_norm_swiglu" else N
+        return f"{name[3:]} {n}x{K}", 2.0 * n * K + M * (2.0 * K + 2.0 * N), 2.0 * M * n * K
+    if name in ("jg_attn_decode_fused", "jg_attn_chunk", "jg_rope_kvwrite_rows", "jg_rmsnorm", "jg_stream_norm", "jg_stream_embed", "jg_embed"):
+        return name[3:], 0.0, 0.0
+    return None
+
+
+def time_calls(dev, calls: list[tuple], R: int, T: float, p: dict | None = None) -> list[dict]:
+    """Each kind of call on its own: all layers' calls of that kind back to back (their weights are far larger than L2
+    together), CUDA events, against the measured copy bandwidth and bf16 rate."""
+    from denograd_b200 import ffi
+    peaks, groups = measured_peaks(), {}
+    for name, a in calls:
+        w = call_work(name, a, R, T)
+        if w is None:
+            continue
+        label, by, fl = w
+        if p is not None and name in ("jg_attn_decode_fused", "jg_attn_chunk"):
+            hd, G = p["dim"] // p["n_heads"], p["n_kv_heads"]
+            by = 4.0 * T * G * hd * (R if name == "jg_attn_decode_fused" else 1)
+            fl = 4.0 * p["n_heads"] * hd * R * (T if name == "jg_attn_decode_fused" else T / 2.0)
+        g = groups.setdefault(label, {"calls": [], "bytes": by, "flops": fl})
+        g["calls"].append((name, a))
+    out = []
+    for label, g in groups.items():
+        reps = max(2, 48 // len(g["calls"]))
+        for n, a in g["calls"]:
+            ffi.call(n, *a)
+        dev.synchronize()
+        dev.timer_start()
+        for _ in range(reps):
+            for n, a in g["calls"]:
+                ffi.call(n, *a)
+        us = dev.timer_stop() / (reps * len(g["calls"])) * 1e6
+        t_min = max(g["bytes"] / (peaks["hbm_gbs"] * 1e3), g["flops"] / (peaks["tflops"] * 1e6))
+        out.append({"call": label, "per_step": len(g["calls"]), "us": round(us, 2), "roofline_us": round(t_min, 2), "frac": round(t_min / us, 3)})
+    return out
+
+
+def run_hybrid(args) -> None:
+    """Prefill and decode of a Matulorn of the Llama's layer sizes, beside that Llama (fp16), at the same batch sizes."""
+    from denograd_b200 import synth
+    from denograd_b200.matulorn import Matulorn
+    rig = Rig()
+    dev, K, W, P, peaks = rig.dev, args.steps, args.warmup, args.prompt, measured_peaks()
+    p, tied = arch(args.hybrid)
+    cfg = hybrid_config(args.hybrid, args.layers)
+    line = {"metric": "hybrid_tokens_per_second", "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W, "data": "synthetic", "dtype": "bf16, f32 stream and state",
+            "config": {"model": f"Matulorn, {args.hybrid} layer sizes", "layers": len(cfg["layers"]), "prompt_tokens": P,
+                       "l2": "inputs larger than L2: every step streams all weights once"}, "legs": {}}
+    batches = [int(b) for b in args.hybrid_batches.split(",")]
+    prefills = [int(n) for n in args.hybrid_prefills.split(",")]
+    ctx = max(max(prefills), P + 4 * K + W + 64)
+    with ClockSampler(rig.local_rank) as clocks:
+        for kind in ("matulorn", "llama"):
+            legs = line["legs"][kind] = {}
+            for B in batches:
+                if kind == "matulorn":
+                    llm = Matulorn(cfg, max_context=ctx, max_batch=B, device=rig.dev_name, temperature=0.0).load_synthetic()
+                else:
+                    llm = rig.llama(args.hybrid, "float16", (ctx + 63) // 64 * 64, B, n_layers=len(cfg["layers"]))
+                m = llm.model
+                if B == 1:
+                    for n in prefills:
+                        prompt = synth.prompt_tokens(n, p["vocab_size"])
+                        for _ in range(2):
+                            llm.reset(); llm.prefill(prompt)
+                        dev.synchronize(); dev.timer_start()
+                        for _ in range(3):
+                            llm.reset(); llm.prefill(prompt)
+                        s = dev.timer_stop() / 3
+                        fl = hybrid_flops(cfg, 1, n) if kind == "matulorn" else prefill_flops(p | {"n_layers": len(cfg["layers"])}, 1, n)
+                        leg = legs[f"prefill{n}"] = {"tok_s": n / s, "ms": s * 1e3, "frac_of_bf16_peak": fl / s / 1e12 / peaks["tflops"]}
+                        if not args.no_extra:
+                            llm.reset()
+                            leg["calls"] = time_calls(dev, record_calls(lambda: llm.prefill(prompt)), n, n, p if kind == "llama" else None)
+                prompt = synth.prompt_tokens(P, p["vocab_size"], batch=B)
+                llm.reset()
+                first, pos = llm.prefill(prompt).numpy(), llm.start_pos
+                m.decode_loop(first, pos, W, collect=False)
+                times, pos = [], pos + W
+                for _ in range(3):
+                    dev.synchronize(); dev.timer_start()
+                    m.decode_loop(first, pos, K, collect=False, resume=True)
+                    times.append(dev.timer_stop())
+                    pos += K
+                s, T = statistics.median(times), P + W + 1.5 * K
+                by = hybrid_bytes(cfg, B, T) if kind == "matulorn" else weight_bytes(p | {"n_layers": len(cfg["layers"])}, tied, False) + B * T * kv_bytes_per_token(p | {"n_layers": len(cfg["layers"])})
+                leg = legs[f"decode_bs{B}"] = {"tok_s": B * K / s, "ms_per_step": s / K * 1e3, "context": int(T), "bytes_per_step": by,
+                                               "frac_of_hbm_roofline": by / (s / K) / 1e9 / peaks["hbm_gbs"]}
+                if not args.no_extra:
+                    ws = m._workspace(B)
+                    if kind == "llama":
+                        m._step_plan = False  # the launch-per-op step, call by call
+                        m._step(ws)
+                    leg["calls"] = time_calls(dev, record_calls(lambda: m._step(ws)), B, T, p if kind == "llama" else None)
+                    ws = None
+                del m, llm
+                rig.release()
+    line["clocks"] = clocks.summary()
+    print(json.dumps(line))
+
+
 def strip(d: dict) -> dict:
     return {k: v for k, v in d.items() if not k.startswith("_")}
 
@@ -631,6 +835,10 @@ def main() -> None:
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU-baseline leg")
     ap.add_argument("--no-extra", action="store_true", help="skip the extra legs")
     ap.add_argument("--no-parity", action="store_true", help="skip the checks against the CPU checker (profiling captures only)")
+    ap.add_argument("--hybrid", default="", choices=["", "1B", "3B", "8B"],
+                    help="instead of the default workload: prefill and decode of a Matulorn with that Llama's layer sizes, beside the Llama")
+    ap.add_argument("--hybrid-batches", default="1,2,8,32")
+    ap.add_argument("--hybrid-prefills", default="512,2048")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
@@ -638,6 +846,8 @@ def main() -> None:
     LAYERS_OVERRIDE = args.layers
     if args.impl == "reference":
         run_reference(args)
+    elif args.hybrid:
+        run_hybrid(args)
     else:
         run_gpu(args)
 

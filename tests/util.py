@@ -90,3 +90,20 @@ def oracle_greedy(m: O.OracleModel, prompt: np.ndarray, n_new: int):
 # vocabulary shard (501 rows) does not divide by the number of CTAs.
 TP_STEP_ARCH = {"dim": 512, "n_heads": 8, "n_kv_heads": 2, "n_layers": 3, "norm_eps": 1e-5, "rope_theta": 500000,
                 "vocab_size": 1002, "hidden_dim": 13312}
+
+
+def write_safetensors_bf16(path: str, tensors: dict) -> None:
+    """A .safetensors file with every tensor as BF16 (float32 values, rounded to nearest even)."""
+    import json
+    import struct
+
+    from oracle.matulorn import bf16_round
+    header, data, at = {}, [], 0
+    for name, v in tensors.items():
+        raw = (bf16_round(np.asarray(v, np.float32)).view(np.uint32) >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(np.shape(v)), "data_offsets": [at, at + len(raw)]}
+        data.append(raw)
+        at += len(raw)
+    j = json.dumps(header).encode()
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(j)) + j + b"".join(data))

@@ -640,66 +640,76 @@ def record_calls(fn) -> list[tuple]:
     return calls
 
 
-def call_work(name: str, a: tuple, R: int, T: float) -> tuple[str, float, float] | None:
-    """(label, bytes, flops) of one recorded projection or mixer call on R rows with T cached positions."""
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12  # CUDA cores: the delta rule's state is fp32 and never meets a tensor core
+
+
+def call_work(name: str, a: tuple, B: int, Sc: int, T: float, p: dict | None) -> tuple[str, float, float, float] | None:
+    """(label, bytes, tensor-core flops, fp32 flops) of one recorded call on Sc tokens of B sequences, each with T positions in
+    the cache when the call is done (p: the Llama's sizes)."""
     from denograd_b200 import ffi
+    R = B * Sc
+    pairs = R * T if Sc == 1 else R * (T - Sc / 2.0)  # query-key pairs
     if name == "jg_dense":
         d = a[2]
-        nw = {ffi.DENSE_GLU: 2, ffi.DENSE_MINGRU: 3}.get(d.epilogue, 1)
-        n = nw * d.N
+        n, R = {ffi.DENSE_GLU: 2, ffi.DENSE_MINGRU: 3}.get(d.epilogue, 1) * d.N, a[1]._obj.B * a[1]._obj.Sc
         kind = {ffi.DENSE_GLU: "gate/up + GLU", ffi.DENSE_MINGRU: "minGRU gates + recurrence", ffi.DENSE_LOGITS: "logits"}.get(d.epilogue, "projection")
-        return f"{kind} {n}x{d.K}" + (" (norms fused)" if d.x == 0 else ""), 2.0 * n * d.K + R * (2.0 * d.K + 2.0 * d.N), 2.0 * R * n * d.K
+        return f"{kind} {n}x{d.K}" + (" (norms fused)" if d.x == 0 else ""), 2.0 * n * d.K + R * (2.0 * d.K + 2.0 * d.N), 2.0 * R * n * d.K, 0.0
     if name == "jg_latent_attn":
         d = a[2]
-        span = min(T, d.window) if d.window else T
-        ukv = d.heads * (d.dim + d.vdim) * d.kv_rank
-        pairs = span if R == 1 or span < R else span  # decode: every row sees `span`
-        return "latent attention", 2.0 * ukv + 2.0 * span * (d.kv_rank + d.rot_dim) * (R if T > R else 1), 2.0 * R * ukv + 2.0 * d.heads * R * pairs * (d.dim + d.rot_dim + d.vdim) * (0.5 if T <= R else 1.0)
+        w = d.window or 1 << 30
+        seen = min(T, w + Sc - 1.0)
+        pairs = R * min(T, w) if Sc == 1 else pairs if T <= w else R * float(w)
+        ukv, row = d.heads * (d.dim + d.vdim) * d.kv_rank, 2.0 * (d.kv_rank + d.rot_dim)
+        return "latent attention", 2.0 * ukv + B * seen * row + 2.0 * R * (d.ldp + d.ldo), 2.0 * R * ukv + 2.0 * d.heads * pairs * (d.dim + d.rot_dim + d.vdim), 0.0
     if name == "jg_delta_rule":
         d = a[2]
         st = d.heads * d.dim * d.vdim
-        return "delta rule", 8.0 * st + R * 2.0 * (d.ldp + d.ldo), 8.0 * R * st
+        return "delta rule", B * 8.0 * st + R * 2.0 * (d.ldp + d.ldo), 0.0, 7.0 * R * st
     if name == "jg_mingru_scan":
         d = a[2]
-        return "minGRU scan", R * 2.0 * (d.ldp + d.ldo) + 8.0 * d.width, 0.0
+        return "minGRU scan", R * 2.0 * (d.ldp + d.ldo) + B * 8.0 * d.width, 0.0, 0.0
+    if name == "jg_stream_norm":
+        d = a[2]
+        R = a[1]._obj.B * a[1]._obj.Sc
+        return "residual + norms", R * d.width * (4.0 + (8.0 if d.y else 0.0) + 2.0), 0.0, 0.0
+    if name == "jg_rmsnorm":
+        return "rmsnorm", 4.0 * a[-3] * a[-2], 0.0, 0.0
     if name in ("jg_norm_linear", "jg_linear", "jg_norm_swiglu", "jg_norm_logits_argmax_shard"):
-        M, N, K = {"jg_norm_linear": a[-3:], "jg_linear": a[-3:], "jg_norm_swiglu": a[-3:], "jg_norm_logits_argmax_shard": a[-4:-1]}[name]
+        M, N, K = a[-4:-1] if name.endswith("shard") else a[-3:]
         n = 2 * N if name == "jg_norm_swiglu" else N
-        return f"{name[3:]} {n}x{K}", 2.0 * n * K + M * (2.0 * K + 2.0 * N), 2.0 * M * n * K
-    if name in ("jg_attn_decode_fused", "jg_attn_chunk", "jg_rope_kvwrite_rows", "jg_rmsnorm", "jg_stream_norm", "jg_stream_embed", "jg_embed"):
-        return name[3:], 0.0, 0.0
+        return f"{name[3:]} {n}x{K}", 2.0 * n * K + M * (2.0 * K + 2.0 * N), 2.0 * M * n * K, 0.0
+    if name in ("jg_attn_decode_fused", "jg_attn_chunk") and p is not None:
+        hd, H, G = p["dim"] // p["n_heads"], p["n_heads"], p["n_kv_heads"]
+        return name[3:], B * 4.0 * T * G * hd + R * 4.0 * H * hd, 4.0 * H * hd * pairs, 0.0
+    if name == "jg_rope_kvwrite_rows" and p is not None:
+        hd = p["dim"] // p["n_heads"]
+        return name[3:], R * 4.0 * (p["n_heads"] + 2 * p["n_kv_heads"]) * hd, 0.0, 0.0
     return None
 
 
-def time_calls(dev, calls: list[tuple], R: int, T: float, p: dict | None = None) -> list[dict]:
+def time_calls(dev, calls: list[tuple], B: int, Sc: int, T: float, p: dict | None = None) -> list[dict]:
     """Each kind of call on its own: all layers' calls of that kind back to back (their weights are far larger than L2
-    together), CUDA events, against the measured copy bandwidth and bf16 rate."""
+    together), CUDA events, against the measured copy bandwidth, the measured bf16 rate and the fp32 rate of the CUDA cores."""
     from denograd_b200 import ffi
     peaks, groups = measured_peaks(), {}
     for name, a in calls:
-        w = call_work(name, a, R, T)
+        w = call_work(name, a, B, Sc, T, p)
         if w is None:
             continue
-        label, by, fl = w
-        if p is not None and name in ("jg_attn_decode_fused", "jg_attn_chunk"):
-            hd, G = p["dim"] // p["n_heads"], p["n_kv_heads"]
-            by = 4.0 * T * G * hd * (R if name == "jg_attn_decode_fused" else 1)
-            fl = 4.0 * p["n_heads"] * hd * R * (T if name == "jg_attn_decode_fused" else T / 2.0)
-        g = groups.setdefault(label, {"calls": [], "bytes": by, "flops": fl})
-        g["calls"].append((name, a))
+        t_min = max(w[1] / (peaks["hbm_gbs"] * 1e3), w[2] / (peaks["tflops"] * 1e6), w[3] / (FP32_TFLOPS * 1e6))
+        groups.setdefault(w[0], (t_min, []))[1].append((name, a))
     out = []
-    for label, g in groups.items():
-        reps = max(2, 48 // len(g["calls"]))
-        for n, a in g["calls"]:
+    for label, (t_min, group) in groups.items():
+        reps = max(2, 48 // len(group))
+        for n, a in group:
             ffi.call(n, *a)
         dev.synchronize()
         dev.timer_start()
         for _ in range(reps):
-            for n, a in g["calls"]:
+            for n, a in group:
                 ffi.call(n, *a)
-        us = dev.timer_stop() / (reps * len(g["calls"])) * 1e6
-        t_min = max(g["bytes"] / (peaks["hbm_gbs"] * 1e3), g["flops"] / (peaks["tflops"] * 1e6))
-        out.append({"call": label, "per_step": len(g["calls"]), "us": round(us, 2), "roofline_us": round(t_min, 2), "frac": round(t_min / us, 3)})
+        us = dev.timer_stop() / (reps * len(group)) * 1e6
+        out.append({"call": label, "per_step": len(group), "us": round(us, 2), "roofline_us": round(t_min, 2), "frac": round(t_min / us, 3)})
     return out
 
 
@@ -739,7 +749,7 @@ def run_hybrid(args) -> None:
                         leg = legs[f"prefill{n}"] = {"tok_s": n / s, "ms": s * 1e3, "frac_of_bf16_peak": fl / s / 1e12 / peaks["tflops"]}
                         if not args.no_extra:
                             llm.reset()
-                            leg["calls"] = time_calls(dev, record_calls(lambda: llm.prefill(prompt)), n, n, p if kind == "llama" else None)
+                            leg["calls"] = time_calls(dev, record_calls(lambda: llm.prefill(prompt)), 1, n, n, p if kind == "llama" else None)
                 prompt = synth.prompt_tokens(P, p["vocab_size"], batch=B)
                 llm.reset()
                 first, pos = llm.prefill(prompt).numpy(), llm.start_pos
@@ -759,7 +769,7 @@ def run_hybrid(args) -> None:
                     if kind == "llama":
                         m._step_plan = False  # the launch-per-op step, call by call
                         m._step(ws)
-                    leg["calls"] = time_calls(dev, record_calls(lambda: m._step(ws)), B, T, p if kind == "llama" else None)
+                    leg["calls"] = time_calls(dev, record_calls(lambda: m._step(ws)), B, 1, T, p if kind == "llama" else None)
                     ws = None
                 del m, llm
                 rig.release()

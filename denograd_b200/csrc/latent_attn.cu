@@ -1,14 +1,19 @@
 // Latent attention over a paged ring of (normed latent | rotated key part) rows: a sliding window, a learned sink in the
 // softmax's denominator, YaRN-scaled half-split rotary on the shared key part.
 //
-//   latent_write    per row: RMS norm of the latent, rotation of the key part, cache row
-//   decode, short portions, fp32 ("absorbed"): the per-head key and value projections are applied to the query and to
-//                   the attended latent instead of to every cached position —
-//                   latent_absorb   qt = [W_uk^T q_unrotated | rotated q]
-//                   latent_split    scores qt . cache row, softmax statistics and the weighted latent of a context slice
-//                   latent_combine  slices + sink -> latent, then W_uv
+//   absorbed (decoding, short portions, fp32): the per-head key and value projections are applied to the query and to the
+//   attended latent instead of to every cached position
+//       latent_pre      qt = [W_uk^T q_unrotated | rotated q] per head; norm, rotation and cache row of the new tokens
+//       latent_mma      bf16: scores qt . cache row, softmax statistics and the weighted latent of a context slice, for 16
+//                       or 32 heads at once on the tensor cores (all heads share the cached rows)
+//       latent_split    the same for one head on the CUDA cores (fp32, and shapes the other does not take)
+//       latent_combine  slices + sink -> latent, then W_uv
+//   expanded (bf16 prompt portions): keys and values of the window and the new tokens are projected once
+//       latent_write    cache rows of the new tokens, and the attended rows side by side in scratch
+//       dense           [W_uk | W_uv] on those rows
+//       latent_chunk    causal windowed attention, 64 queries of a head per CTA, one pass with running statistics
 //
-// Scores, softmax statistics and weights are fp32.
+// Scores, softmax statistics and weights are fp32; on the tensor cores the weights meet the values in bf16.
 #include <math.h>
 #include <stdlib.h>
 
@@ -21,17 +26,23 @@ struct LatentArgs {
   const int32_t* bt;
   const float *rot, *norm_w, *sink;
   const T *uk, *uv;
-  float *qt, *part;
+  T* qt;        // [R][H][lq]
+  float* part;  // [R][H][ns][rank + 2]: maximum, sum, weighted latent
+  T* ctx;       // expanded form: [B][T][ldc]
+  const T* kv;  // [B][T][ldkv]: keys of all heads, then values
   T* out;
   const int32_t *pos, *seq;
-  int B, Sc, H, dim, rd, vd, rank, window, ldp, ldo, ldc, ldu, page, page_shift, pps, rot_pairs, rot_rows, ns;
+  int B, Sc, H, dim, rd, vd, rank, window, ldp, ldo, ldc, ldu, page, page_shift, pps, rot_pairs, rot_rows, ns, lq;
+  int T_ctx, T_prev, start, ldkv;
+  int shift;  // tokens of this call ahead of its first row (a portion worked off in several passes)
   float eps, scale;
   __device__ __forceinline__ int qk() const { return dim + rd; }
-  __device__ __forceinline__ int lat() const { return rank + rd; }
+  __host__ __device__ __forceinline__ int lat() const { return rank + rd; }
   // cache row of position p of the slot whose block-table row is `t`
   __device__ __forceinline__ T* row(const int32_t* t, int p) const {
     return pool + ((size_t)t[(p >> page_shift) % pps] * page + (p & (page - 1))) * ldc;
   }
+  __device__ __forceinline__ int position(int r) const { return min(max(pos[r % B] + shift + r / B, 0), rot_rows - 1); }
 };
 
 // Entry i of a rotated vector: pairs (i, i + rot_pairs) turn, the rest passes.
@@ -43,46 +54,119 @@ __device__ __forceinline__ float rotated(const T* x, int i, const float* cs, int
   return i < pairs ? fmaf(u, c, -v * s) : fmaf(v, c, u * s);
 }
 
+// Cache row of the new token in row r, by one warp; `copy` (or null) receives it too.
 template <typename T>
-__global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a, int R) {
-  pdl_launch();
-  pdl_wait();
-  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (r >= R) return;
-  const int b = r % a.B, p = a.pos[b] + r / a.B;
+__device__ __forceinline__ void write_row(const LatentArgs<T>& a, int r, int lane, T* copy) {
+  const int b = r % a.B, p = a.pos[b] + a.shift + r / a.B;
   if (p < 0 || p >= a.rot_rows) return;  // outside the tables: left alone
   const T* c = a.proj + (size_t)r * a.ldp + a.H * a.qk();
   T* dst = a.row(a.bt + (size_t)a.seq[b] * a.pps, p);
   float ss = 0.f;
   for (int i = lane; i < a.rank; i += 32) { const float v = to_f32(c[i]); ss = fmaf(v, v, ss); }
   const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)a.rank + a.eps);
-  for (int i = lane; i < a.rank; i += 32) dst[i] = from_f32<T>(to_f32(c[i]) * rs * a.norm_w[i]);
   const float* cs = a.rot + (size_t)p * a.rot_pairs * 2;
-  for (int i = lane; i < a.rd; i += 32) dst[a.rank + i] = from_f32<T>(rotated(c + a.rank, i, cs, a.rot_pairs));
+  for (int i = lane; i < a.ldc; i += 32) {
+    const T v = from_f32<T>(i < a.rank ? to_f32(c[i]) * rs * a.norm_w[i] : (i < a.lat() ? rotated(c + a.rank, i - a.rank, cs, a.rot_pairs) : 0.f));
+    dst[i] = v;
+    if (copy) copy[i] = v;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a, int R) {
+  pdl_launch();
+  pdl_wait();
+  const int w = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (w < R) {
+    write_row(a, w, lane, a.ctx + ((size_t)(w % a.B) * a.T_ctx + a.T_prev + w / a.B) * a.ldc);
+  } else if (w < R + a.B * a.T_prev) {  // an earlier position that the window still reaches
+    const int b = (w - R) / a.T_prev, j = (w - R) % a.T_prev;
+    const uint4* src = reinterpret_cast<const uint4*>(a.row(a.bt + (size_t)a.seq[b] * a.pps, a.start - a.T_prev + j));
+    uint4* dst = reinterpret_cast<uint4*>(a.ctx + ((size_t)b * a.T_ctx + j) * a.ldc);
+    for (int i = lane; i < a.ldc / Elem<T>::VEC; i += 32) dst[i] = src[i];
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ absorbed form
+constexpr int LP_COLS = 64, LP_ROWS = 4;  // latent columns of a CTA, activation rows it serves with one read of the weights
+
+// Blocks 0 .. H * slices - 1: head and 64 latent columns of LP_ROWS rows; the last block along x writes those rows' cache
+// rows.  All warps run down W_uk together, each thread a 16-byte piece of a row.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentArgs<T> a) {
-  extern __shared__ float sq[];
+__global__ void __launch_bounds__(256) latent_pre_kernel(const LatentArgs<T> a, int R) {
+  constexpr int VEC = Elem<T>::VEC, TPR = LP_COLS / VEC, DR = 256 / TPR, AHEAD = 4;
+  extern __shared__ float sq[];  // [LP_ROWS][dim]
+  __shared__ float red[8][LP_ROWS][LP_COLS];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r0 = blockIdx.y * LP_ROWS, nr = min(LP_ROWS, R - r0);
   pdl_launch();
-  pdl_wait();
-  const int r = blockIdx.x, h = blockIdx.y, b = r % a.B, p = min(max(a.pos[b] + r / a.B, 0), a.rot_rows - 1);
-  const T* q = a.proj + (size_t)r * a.ldp + (size_t)h * a.qk();
-  for (int i = threadIdx.x; i < a.dim; i += 128) sq[i] = to_f32(q[i]);
-  __syncthreads();
-  float* qt = a.qt + ((size_t)r * a.H + h) * a.lat();
-  const T* uk = a.uk + (size_t)h * a.dim * a.ldu;
-  for (int i = threadIdx.x; i < a.rank; i += 128) {
-    float acc = 0.f;
-    for (int d = 0; d < a.dim; d++) acc = fmaf(sq[d], to_f32(uk[(size_t)d * a.ldu + i]), acc);
-    qt[i] = acc;
+  if (blockIdx.x == gridDim.x - 1) {
+    pdl_wait();
+    if (warp < nr) write_row(a, r0 + warp, lane, (T*)nullptr);
+    return;
   }
-  const float* cs = a.rot + (size_t)p * a.rot_pairs * 2;
-  for (int i = threadIdx.x; i < a.rd; i += 128) qt[a.rank + i] = rotated(q + a.dim, i, cs, a.rot_pairs);
+  const int slices = (a.rank + LP_COLS - 1) / LP_COLS, h = blockIdx.x / slices, c0 = (blockIdx.x % slices) * LP_COLS;
+  const int dr = tid / TPR, cc = c0 + (tid % TPR) * VEC;
+  const T* uk = a.uk + (size_t)h * a.dim * a.ldu + cc;
+  const bool in = cc < a.ldu;
+  uint4 ahead[AHEAD];  // parameters: requested before the dependency wait
+#pragma unroll
+  for (int i = 0; i < AHEAD; i++) ahead[i] = (in && dr + i * DR < a.dim) ? ld_128(uk + (size_t)(dr + i * DR) * a.ldu) : make_uint4(0, 0, 0, 0);
+  pdl_wait();
+  for (int i = tid; i < LP_ROWS * a.dim; i += 256) {
+    const int r = i / a.dim;
+    sq[i] = r < nr ? to_f32(a.proj[(size_t)(r0 + r) * a.ldp + (size_t)h * a.qk() + i % a.dim]) : 0.f;
+  }
+  __syncthreads();
+  float acc[LP_ROWS][VEC];
+#pragma unroll
+  for (int r = 0; r < LP_ROWS; r++)
+#pragma unroll
+    for (int k = 0; k < VEC; k++) acc[r][k] = 0.f;
+  auto use = [&](const uint4& raw, int d) {
+    float w[VEC];
+    unpack_chunk(raw, w);
+#pragma unroll
+    for (int r = 0; r < LP_ROWS; r++) {
+      const float q = sq[r * a.dim + d];
+#pragma unroll
+      for (int k = 0; k < VEC; k++) acc[r][k] = fmaf(q, w[k], acc[r][k]);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < AHEAD; i++)
+    if (dr + i * DR < a.dim) use(ahead[i], dr + i * DR);
+  for (int d = dr + AHEAD * DR; d < a.dim; d += DR)
+    if (in) use(ld_128(uk + (size_t)d * a.ldu), d);
+#pragma unroll
+  for (int r = 0; r < LP_ROWS; r++)
+#pragma unroll
+    for (int k = 0; k < VEC; k++) {
+      float v = acc[r][k];
+#pragma unroll
+      for (int o = TPR; o < 32; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+      if (lane < TPR) red[warp][r][lane * VEC + k] = v;
+    }
+  __syncthreads();
+  for (int i = tid; i < nr * LP_COLS; i += 256) {
+    const int r = i / LP_COLS, c = i % LP_COLS;
+    if (c0 + c >= a.rank) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) v += red[w][r][c];
+    a.qt[((size_t)(r0 + r) * a.H + h) * a.lq + c0 + c] = from_f32<T>(v);
+  }
+  if (c0 == 0) {  // the rotated part and the padding
+    const int n = a.lq - a.rank;
+    for (int i = tid; i < nr * n; i += 256) {
+      const int r = i / n, e = i % n;
+      const float* cs = a.rot + (size_t)a.position(r0 + r) * a.rot_pairs * 2;
+      const T* q = a.proj + (size_t)(r0 + r) * a.ldp + (size_t)h * a.qk() + a.dim;
+      a.qt[((size_t)(r0 + r) * a.H + h) * a.lq + a.rank + e] = from_f32<T>(e < a.rd ? rotated(q, e, cs, a.rot_pairs) : 0.f);
+    }
+  }
 }
 
-constexpr int LS_THREADS = 128, LS_TILE = 64, LS_MAX_RANK = 1024;
+constexpr int LS_THREADS = 128, LS_TILE = 64, LS_MAX_RANK = 1024, LS_MAX_NS = 32;
 
 template <typename T>
 __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentArgs<T> a) {
@@ -93,12 +177,12 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
   pdl_launch();
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int r = blockIdx.x, h = blockIdx.y, b = r % a.B, p = min(max(a.pos[b] + r / a.B, 0), a.rot_rows - 1), L = a.lat();
-  const int32_t* bt = a.bt + (size_t)a.seq[b] * a.pps;
+  const int r = blockIdx.x, h = blockIdx.y, p = a.position(r), L = a.lat();
+  const int32_t* bt = a.bt + (size_t)a.seq[r % a.B] * a.pps;
   const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0, n = p + 1 - lo;
   const int chunk = (n + a.ns - 1) / a.ns, t0 = lo + blockIdx.z * chunk, t1 = min(p + 1, t0 + chunk);
   float* part = a.part + (((size_t)r * a.H + h) * a.ns + blockIdx.z) * (a.rank + 2);
-  for (int i = tid; i < L; i += LS_THREADS) sq[i] = a.qt[((size_t)r * a.H + h) * L + i];
+  for (int i = tid; i < L; i += LS_THREADS) sq[i] = to_f32(a.qt[((size_t)r * a.H + h) * a.lq + i]);
   float acc[NR], m = -INFINITY, l = 0.f;
 #pragma unroll
   for (int k = 0; k < NR; k++) acc[k] = 0.f;
@@ -137,49 +221,518 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
     if (tid + k * LS_THREADS < a.rank) part[2 + tid + k * LS_THREADS] = acc[k];
 }
 
-template <typename T>
-__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs<T> a) {
-  extern __shared__ float so[];  // the attended latent
+// ---- tensor cores (mma.sync m16n8k16, bf16 in, fp32 out)
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+constexpr float LOG2E = 1.4426950408889634f;
+
+// One row, 16 * MT heads, one context slice: tiles of 64 cached rows; warp w scores 8 of them for all heads, two warps'
+// worth of heads get their softmax statistics per warp, and each warp owns NTW * 8 columns of the weighted latent.
+constexpr int LM_THREADS = 256, LM_TILE = 64;
+template <int MT>
+static constexpr size_t lm_smem(int lq, int stages) {
+  return (size_t)(stages * LM_TILE + 16 * MT) * (lq + 8) * 2 + (size_t)16 * MT * (LM_TILE * 4 + (LM_TILE + 8) * 2 + 12);
+}
+
+template <int MT, int NTW>
+__global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs<bf16> a, int stages) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  constexpr int HR = 16 * MT;
+  const int ld = a.lq + 8;  // row stride: an odd number of 16-byte pieces
+  bf16* tiles = reinterpret_cast<bf16*>(smem);
+  bf16* sQ = tiles + (size_t)stages * LM_TILE * ld;
+  float* sS = reinterpret_cast<float*>(sQ + (size_t)HR * ld);  // [HR][64]
+  bf16* sP = reinterpret_cast<bf16*>(sS + HR * LM_TILE);       // [HR][72]
+  float *sM = reinterpret_cast<float*>(sP + HR * (LM_TILE + 8)), *sL = sM + HR, *sA = sL + HR;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, z = blockIdx.x, h0 = blockIdx.y * HR, r = blockIdx.z;
   pdl_launch();
   pdl_wait();
-  const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const float* part = a.part + ((size_t)r * a.H + h) * a.ns * (a.rank + 2);
-  float M = a.sink[h];
-  for (int s = 0; s < a.ns; s++) M = fmaxf(M, part[(size_t)s * (a.rank + 2)]);
-  float l = expf(a.sink[h] - M);
-  for (int s = 0; s < a.ns; s++) l += part[(size_t)s * (a.rank + 2) + 1] * expf(part[(size_t)s * (a.rank + 2)] - M);
-  const float rl = 1.0f / l;
-  for (int i = threadIdx.x; i < a.rank; i += 128) {
-    float v = 0.f;
-    for (int s = 0; s < a.ns; s++) v = fmaf(part[(size_t)s * (a.rank + 2) + 2 + i], expf(part[(size_t)s * (a.rank + 2)] - M), v);
-    so[i] = v * rl;
+  const int p = a.position(r);
+  const int32_t* bt = a.bt + (size_t)a.seq[r % a.B] * a.pps;
+  const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0, n = p + 1 - lo;
+  const int chunk = ((n + a.ns - 1) / a.ns + LM_TILE - 1) / LM_TILE * LM_TILE, t0 = lo + z * chunk, t1 = min(p + 1, t0 + chunk);
+  const size_t pstride = a.rank + 2;
+  if (t0 >= t1) {  // an empty slice
+    if (tid < HR && h0 + tid < a.H) {
+      float* part = a.part + (((size_t)r * a.H + h0 + tid) * a.ns + z) * pstride;
+      part[0] = -INFINITY;
+      part[1] = 0.f;
+    }
+    return;
+  }
+  const int pieces = a.lq / 8, row_pieces = a.ldc / 8;
+  for (int i = tid; i < HR * pieces; i += LM_THREADS) {
+    const int h = i / pieces, c = i % pieces;
+    bf16* d = sQ + (size_t)h * ld + c * 8;
+    if (h0 + h < a.H) cp16(d, a.qt + ((size_t)r * a.H + h0 + h) * a.lq + c * 8);
+    else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+  }
+  auto load_tile = [&](int base, int s) {
+    bf16* t = tiles + (size_t)s * LM_TILE * ld;
+    for (int i = tid; i < LM_TILE * pieces; i += LM_THREADS) {
+      const int k = i / pieces, c = i % pieces;
+      bf16* d = t + (size_t)k * ld + c * 8;
+      if (base + k < t1 && c < row_pieces) cp16(d, a.row(bt, base + k) + c * 8);
+      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    }
+    cp_commit();
+  };
+  load_tile(t0, 0);
+  if (tid < HR) { sM[tid] = -INFINITY; sL[tid] = 0.f; }
+  float o[MT][NTW][4];
+#pragma unroll
+  for (int m = 0; m < MT; m++)
+#pragma unroll
+    for (int j = 0; j < NTW; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) o[m][j][i] = 0.f;
+  const int g = lane >> 2, tq = lane & 3;
+  int s = 0;
+  for (int base = t0; base < t1; base += LM_TILE) {
+    const bool more = base + LM_TILE < t1;
+    if (stages > 1 && more) { load_tile(base + LM_TILE, s ^ 1); cp_wait<1>(); }
+    else cp_wait<0>();
+    __syncthreads();
+    const bf16* t = tiles + (size_t)s * LM_TILE * ld;
+    float sc[MT][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) sc[m][i] = 0.f;
+    const bf16* kb = t + (size_t)(warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
+    const bf16* qb = sQ + (size_t)(lane & 15) * ld + (lane >> 4) * 8;
+    for (int k = 0; k < a.lq; k += 32) {
+      uint32_t bk[4];
+      ldsm4(bk, kb + k);
+#pragma unroll
+      for (int m = 0; m < MT; m++) {
+        uint32_t q0[4], q1[4];
+        ldsm4(q0, qb + (size_t)m * 16 * ld + k);
+        ldsm4(q1, qb + (size_t)m * 16 * ld + k + 16);
+        mma_bf16(sc[m], q0, bk[0], bk[1]);
+        mma_bf16(sc[m], q1, bk[2], bk[3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int c = warp * 8 + tq * 2 + (i & 1);
+        sS[(m * 16 + g + 8 * (i >> 1)) * LM_TILE + c] = base + c < t1 ? sc[m][i] * a.scale : -INFINITY;
+      }
+    __syncthreads();
+    for (int row = warp; row < HR; row += 8) {
+      const float x0 = sS[row * LM_TILE + lane], x1 = sS[row * LM_TILE + lane + 32], old = sM[row];
+      const float m = fmaxf(old, warp_max(fmaxf(x0, x1)));
+      const float e0 = expf(x0 - m), e1 = expf(x1 - m), sum = warp_sum(e0 + e1);
+      sP[row * (LM_TILE + 8) + lane] = __float2bfloat16_rn(e0);
+      sP[row * (LM_TILE + 8) + lane + 32] = __float2bfloat16_rn(e1);
+      if (lane == 0) {
+        const float al = expf(old - m);
+        sA[row] = al;
+        sL[row] = fmaf(sL[row], al, sum);
+        sM[row] = m;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; m++) {
+      const float a0 = sA[m * 16 + g], a1 = sA[m * 16 + g + 8];
+#pragma unroll
+      for (int j = 0; j < NTW; j++) { o[m][j][0] *= a0; o[m][j][1] *= a0; o[m][j][2] *= a1; o[m][j][3] *= a1; }
+    }
+#pragma unroll
+    for (int k = 0; k < LM_TILE; k += 16) {
+      uint32_t pf[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; m++) ldsm4(pf[m], sP + (size_t)(m * 16 + (lane & 15)) * (LM_TILE + 8) + k + (lane >> 4) * 8);
+#pragma unroll
+      for (int j = 0; j < NTW; j += 2) {
+        const int c = (warp * NTW + j) * 8;
+        if (c < a.rank) {  // a pair of column tiles may reach past the latent into the padding of the row, never past it
+          uint32_t v[4];
+          ldsm4t(v, t + (size_t)(k + (lane & 15)) * ld + c + (lane >> 4) * 8);
+#pragma unroll
+          for (int m = 0; m < MT; m++) {
+            mma_bf16(o[m][j], pf[m], v[0], v[1]);
+            mma_bf16(o[m][j + 1], pf[m], v[2], v[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+    if (stages > 1) s ^= 1;
+    else if (more) load_tile(base + LM_TILE, 0);
+  }
+  if (tid < HR && h0 + tid < a.H) {
+    float* part = a.part + (((size_t)r * a.H + h0 + tid) * a.ns + z) * pstride;
+    part[0] = sM[tid];
+    part[1] = sL[tid];
+  }
+#pragma unroll
+  for (int m = 0; m < MT; m++)
+#pragma unroll
+    for (int j = 0; j < NTW; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int h = h0 + m * 16 + g + 8 * (i >> 1), c = (warp * NTW + j) * 8 + tq * 2 + (i & 1);
+        if (h < a.H && c < a.rank) a.part[(((size_t)r * a.H + h) * a.ns + z) * pstride + 2 + c] = o[m][j][i];
+      }
+}
+
+// Slices and the sink -> the attended latent; then this CTA's LC_OUT values of the head, for LC_ROWS rows.
+constexpr int LC_OUT = 32, LC_ROWS = 4;
+template <typename T>
+__global__ void __launch_bounds__(256) latent_combine_kernel(const LatentArgs<T> a, int R) {
+  constexpr int VEC = Elem<T>::VEC;
+  extern __shared__ __align__(16) float so[];  // [LC_ROWS][ldu] attended latents
+  __shared__ float wgt[LC_ROWS][LS_MAX_NS];
+  const int h = blockIdx.x, j0 = blockIdx.y * LC_OUT, r0 = blockIdx.z * LC_ROWS, nr = min(LC_ROWS, R - r0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  pdl_launch();
+  // parameters: this warp's rows of W_uv travel to L2 while the predecessor drains
+  for (int q = 0; q < LC_OUT / 8; q++) {
+    const int j = j0 + warp + 8 * q;
+    if (j < a.vd)
+      for (size_t off = (size_t)lane * 128; off < (size_t)a.ldu * sizeof(T); off += 32 * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.uv + ((size_t)h * a.vd + j) * a.ldu) + off));
+  }
+  pdl_wait();
+  const size_t ps = a.rank + 2;
+  if (warp < nr) {
+    const float* part = a.part + ((size_t)(r0 + warp) * a.H + h) * a.ns * ps;
+    const float m = lane < a.ns ? part[lane * ps] : -INFINITY, l = lane < a.ns ? part[lane * ps + 1] : 0.f;
+    const float sink = a.sink[h], M = fmaxf(warp_max(m), sink), e = expf(m - M);
+    const float L = warp_sum(l * e) + expf(sink - M);
+    if (lane < a.ns) wgt[warp][lane] = e / L;
   }
   __syncthreads();
-  for (int j = warp; j < a.vd; j += 4) {
+  for (int i = tid; i < nr * a.ldu; i += 256) {
+    const int r = i / a.ldu, c = i % a.ldu;
+    float v = 0.f;
+    if (c < a.rank) {
+      const float* part = a.part + ((size_t)(r0 + r) * a.H + h) * a.ns * ps + 2 + c;
+#pragma unroll 4
+      for (int s = 0; s < a.ns; s++) {
+        const float w = wgt[r][s];
+        if (w != 0.f) v = fmaf(part[(size_t)s * ps], w, v);  // an empty slice has no latent to read
+      }
+    }
+    so[i] = v;
+  }
+  __syncthreads();
+  for (int q = 0; q < LC_OUT / 8; q++) {
+    const int j = j0 + warp + 8 * q;
+    if (j >= a.vd) continue;
     const T* w = a.uv + ((size_t)h * a.vd + j) * a.ldu;
-    float d = 0.f;
-    for (int i = lane; i < a.rank; i += 32) d = fmaf(to_f32(w[i]), so[i], d);
-    d = warp_sum(d);
-    if (lane == 0) a.out[(size_t)r * a.ldo + (size_t)h * a.vd + j] = from_f32<T>(d);
+    float acc[LC_ROWS];
+#pragma unroll
+    for (int r = 0; r < LC_ROWS; r++) acc[r] = 0.f;
+    for (int c = lane; c < a.ldu / VEC; c += 32) {
+      float f[VEC];
+      unpack_chunk(ld_128(w + (size_t)c * VEC), f);
+#pragma unroll
+      for (int r = 0; r < LC_ROWS; r++)
+        if (r < nr) {
+#pragma unroll
+          for (int k = 0; k < VEC; k++) acc[r] = fmaf(f[k], so[r * a.ldu + c * VEC + k], acc[r]);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < LC_ROWS; r++) {
+      const float v = warp_sum(acc[r]);
+      if (lane == 0 && r < nr) a.out[(size_t)(r0 + r) * a.ldo + (size_t)h * a.vd + j] = from_f32<T>(v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ expanded form
+// 64 consecutive tokens of a sequence x one head; warp w owns tokens 16 w .. 16 w + 15.
+constexpr int LX_Q = 64, LX_KV = 64, LX_THREADS = 128;
+
+template <int VT>  // value tiles of 8 columns, an even number
+__global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentArgs<bf16> a, int qkp) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  const int ldq = qkp + 8, ldv = VT * 8 + 8;
+  bf16* sQ = reinterpret_cast<bf16*>(smem);
+  bf16* sK = sQ + (size_t)LX_Q * ldq;
+  bf16* sV = sK + (size_t)2 * LX_KV * ldq;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, b = blockIdx.z;
+  // the last tokens have the longest context: first
+  const int q0 = (int)(gridDim.x - 1 - blockIdx.x) * LX_Q, nq = min(LX_Q, a.Sc - q0);
+  pdl_launch();
+  pdl_wait();
+  const bf16 zero = __float2bfloat16_rn(0.f);
+  for (int i = tid; i < LX_Q * qkp; i += LX_THREADS) {
+    const int t = i / qkp, e = i % qkp;
+    bf16 v = zero;
+    if (t < nq && e < a.qk()) {
+      const bf16* q = a.proj + ((size_t)(q0 + t) * a.B + b) * a.ldp + (size_t)h * a.qk();
+      v = e < a.dim ? q[e] : from_f32<bf16>(rotated(q + a.dim, e - a.dim, a.rot + (size_t)(a.start + q0 + t) * a.rot_pairs * 2, a.rot_pairs));
+    }
+    sQ[(size_t)t * ldq + e] = v;
+  }
+  // keys 0 .. T_ctx - 1 are positions start - T_prev ..; token q0 + t is key T_prev + q0 + t
+  const int own = a.T_prev + q0, last = own + nq - 1;
+  const int first = a.window > 0 ? max(0, own - a.window + 1) : 0;
+  const int kp = a.dim / 8, rp = a.rd / 8, pad = (qkp - a.qk()) / 8, vp = a.vd / 8, per = kp + rp + pad + VT;
+  auto load_tile = [&](int base, int s) {
+    bf16 *tk = sK + (size_t)s * LX_KV * ldq, *tv = sV + (size_t)s * LX_KV * ldv;
+    for (int i = tid; i < LX_KV * per; i += LX_THREADS) {
+      const int k = i / per, c = i % per;
+      const size_t row = (size_t)b * a.T_ctx + base + k;
+      const bool in = base + k <= last;
+      bf16* d = c < kp + rp + pad ? tk + (size_t)k * ldq + c * 8 : tv + (size_t)k * ldv + (c - kp - rp - pad) * 8;
+      if (!in || (c >= kp + rp && c < kp + rp + pad) || c >= kp + rp + pad + vp) { *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0); continue; }
+      const bf16* src;
+      if (c < kp) src = a.kv + row * a.ldkv + (size_t)h * a.dim + c * 8;
+      else if (c < kp + rp) src = a.ctx + row * a.ldc + a.rank + (c - kp) * 8;
+      else src = a.kv + row * a.ldkv + (size_t)a.H * a.dim + (size_t)h * a.vd + (c - kp - rp - pad) * 8;
+      cp16(d, src);
+    }
+    cp_commit();
+  };
+  load_tile(first, 0);
+  float o[VT][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+  for (int j = 0; j < VT; j++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) o[j][i] = 0.f;
+  const int g = lane >> 2, tq = lane & 3;
+  const int row0 = own + warp * 16 + g;  // key number of this thread's first token; the second is 8 further
+  const float sl2 = a.scale * LOG2E;
+  int s = 0;
+  for (int base = first; base <= last; base += LX_KV, s ^= 1) {
+    if (base + LX_KV <= last) { load_tile(base + LX_KV, s ^ 1); cp_wait<1>(); }
+    else cp_wait<0>();
+    __syncthreads();
+    const bf16 *tk = sK + (size_t)s * LX_KV * ldq, *tv = sV + (size_t)s * LX_KV * ldv;
+    float sc[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) sc[j][i] = 0.f;
+    for (int k = 0; k < qkp; k += 16) {
+      uint32_t qf[4];
+      ldsm4(qf, sQ + (size_t)(warp * 16 + (lane & 15)) * ldq + k + (lane >> 4) * 8);
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        uint32_t kf[4];
+        ldsm4(kf, tk + (size_t)(j * 8 + (lane >> 4) * 8 + (lane & 7)) * ldq + k + ((lane >> 3) & 1) * 8);
+        mma_bf16(sc[j], qf, kf[0], kf[1]);
+        mma_bf16(sc[j + 1], qf, kf[2], kf[3]);
+      }
+    }
+    float mx[2] = {m[0], m[1]};
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int back = row0 + 8 * (i >> 1) - (base + j * 8 + tq * 2 + (i & 1));
+        sc[j][i] = (back >= 0 && (a.window <= 0 || back < a.window)) ? sc[j][i] * sl2 : -INFINITY;
+        mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+      }
+    float al[2], mu[2];
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+      mu[i] = mx[i] == -INFINITY ? 0.f : mx[i];  // nothing seen yet: every weight below is exp2(-inf) = 0
+      al[i] = exp2f(m[i] - mu[i]);
+      m[i] = mx[i];
+      l[i] *= al[i];
+    }
+#pragma unroll
+    for (int j = 0; j < VT; j++) { o[j][0] *= al[0]; o[j][1] *= al[0]; o[j][2] *= al[1]; o[j][3] *= al[1]; }
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        sc[j][i] = exp2f(sc[j][i] - mu[i >> 1]);
+        l[i >> 1] += sc[j][i];
+      }
+#pragma unroll
+    for (int k = 0; k < 4; k++) {
+      const uint32_t pf[4] = {pack_bf16(sc[2 * k][0], sc[2 * k][1]), pack_bf16(sc[2 * k][2], sc[2 * k][3]), pack_bf16(sc[2 * k + 1][0], sc[2 * k + 1][1]),
+                              pack_bf16(sc[2 * k + 1][2], sc[2 * k + 1][3])};
+#pragma unroll
+      for (int j = 0; j < VT; j += 2) {
+        uint32_t vf[4];
+        ldsm4t(vf, tv + (size_t)(k * 16 + (lane & 15)) * ldv + j * 8 + (lane >> 4) * 8);
+        mma_bf16(o[j], pf, vf[0], vf[1]);
+        mma_bf16(o[j + 1], pf, vf[2], vf[3]);
+      }
+    }
+    __syncthreads();
+  }
+  const float sink = a.sink[h] * LOG2E;
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+    const float M = fmaxf(m[i], sink), e = exp2f(m[i] - M);
+    l[i] = e / fmaf(l[i], e, exp2f(sink - M));
+  }
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int t = warp * 16 + g + 8 * i;
+    if (t < nq) {
+      bf16* dst = a.out + ((size_t)(q0 + t) * a.B + b) * a.ldo + (size_t)h * a.vd;
+#pragma unroll
+      for (int j = 0; j < VT; j++)
+        if (j * 8 < a.vd) *reinterpret_cast<uint32_t*>(dst + j * 8 + tq * 2) = pack_bf16(o[j][2 * i] * l[i], o[j][2 * i + 1] * l[i]);
+    }
   }
 }
 
 // ------------------------------------------------------------------------------------------------ host side
-constexpr int LS_MAX_PARTS = 296;  // two CTAs per SM
-static int latent_splits(const jg_latent_desc* d, int R) {
-  const long long span = d->window > 0 ? d->window : d->rot_rows;
-  long long ns = LS_MAX_PARTS / ((long long)R * d->heads > 0 ? (long long)R * d->heads : 1);
+static int round32(int n) { return (n + 31) & ~31; }
+// tensor-core form of the absorbed path: heads per CTA / 16 (0: this shape stays on the CUDA cores)
+static int mma_tiles(const jg_dev* dev, const jg_latent_desc* d, int* stages) {
+  if (d->dtype != JG_BF16 || d->kv_rank > LS_MAX_RANK) return 0;
+  const int lq = round32(d->kv_rank + d->rot_dim);
+  const size_t limit = (size_t)dev->prop.sharedMemPerBlockOptin - 1024;
+  const int mt = d->heads > 16 && d->kv_rank <= 512 ? 2 : 1;
+  for (*stages = 2; *stages >= 1; (*stages)--)
+    if ((mt == 2 ? lm_smem<2>(lq, *stages) : lm_smem<1>(lq, *stages)) <= limit) return mt;
+  return 0;
+}
+constexpr int LATENT_MAX_PARTS = 32 * 160;  // (row, head, slice) triples of a call with few rows
+static int latent_splits(const jg_dev* dev, const jg_latent_desc* d, int R, int heads_per_cta) {
+  const long long span = d->window > 0 && d->window < d->rot_rows ? d->window : d->rot_rows;
+  const int groups = (d->heads + heads_per_cta - 1) / heads_per_cta;
+  long long ns = (heads_per_cta > 1 ? dev->sm_count : 2 * dev->sm_count) / ((long long)R * groups);
   if (ns > (span + 63) / 64) ns = (span + 63) / 64;
-  return ns < 1 ? 1 : (ns > 32 ? 32 : (int)ns);
+  if (ns > LATENT_MAX_PARTS / ((long long)R * d->heads)) ns = LATENT_MAX_PARTS / ((long long)R * d->heads);
+  return ns < 1 ? 1 : (ns > LS_MAX_NS ? LS_MAX_NS : (int)ns);
+}
+// whether a portion of Sc tokens runs in expanded form (when the host knows where it starts)
+constexpr int LATENT_MIN_EXPANDED = 16, LATENT_MAX_CTX = 16384;
+static bool expandable(const jg_latent_desc* d, int Sc) {
+  return d->dtype == JG_BF16 && Sc >= LATENT_MIN_EXPANDED && d->dim % 8 == 0 && d->rot_dim % 8 == 0 && d->vdim % 8 == 0 && d->kv_rank % 8 == 0 &&
+         d->dim + d->rot_dim <= 256 && d->vdim <= 256;
+}
+static long long longest_ctx(const jg_latent_desc* d, int Sc) {
+  long long prev = d->window > 0 ? (long long)d->window - 1 : d->rot_rows;
+  if (prev + Sc > d->rot_rows) prev = d->rot_rows - Sc;
+  if (prev < 0) prev = 0;
+  return prev + Sc > LATENT_MAX_CTX ? LATENT_MAX_CTX : prev + Sc;
 }
 
 JG_API int jg_latent_scratch_bytes(const jg_latent_desc* d, int32_t B, int32_t Sc, uint64_t* out) {
   JG_REQUIRE(d != nullptr && out != nullptr && B > 0 && Sc > 0, "latent_scratch_bytes: bad arguments");
-  const uint64_t RH = (uint64_t)B * Sc * d->heads;
-  // slices: one per (row, head), or up to LS_MAX_PARTS in all when there are fewer (any smaller call fits too)
-  *out = 4 * (RH * (uint64_t)(d->kv_rank + d->rot_dim) + (RH > LS_MAX_PARTS ? RH : LS_MAX_PARTS) * (uint64_t)(d->kv_rank + 2)) + 256;
+  uint64_t RH = (uint64_t)B * Sc * d->heads, wide = 0;
+  if (expandable(d, Sc)) {
+    wide = (uint64_t)B * longest_ctx(d, Sc) * 2 * (d->ldc + d->heads * (d->dim + d->vdim)) + 64;
+    // longer contexts, and starts the host does not know, take the absorbed form in passes of this many rows
+    const uint64_t few = (uint64_t)B * LATENT_MIN_EXPANDED * d->heads;
+    if (RH > few) RH = few;
+  }
+  const uint64_t parts = RH > LATENT_MAX_PARTS ? RH : LATENT_MAX_PARTS;
+  const uint64_t narrow = 4 * (RH * (uint64_t)round32(d->kv_rank + d->rot_dim) + parts * (uint64_t)(d->kv_rank + 2)) + 256;
+  *out = narrow > wide ? narrow : wide;
   return JG_OK;
 }
+
+template <int MT, int NTW>
+static int launch_mma(jg_dev* dev, const LatentArgs<bf16>& a, int R, int stages) {
+  auto kern = latent_mma_kernel<MT, NTW>;
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dev->prop.sharedMemPerBlockOptin - 1024));
+    set[dev->ordinal & 7] = true;
+  }
+  return jg_launch(dev, "latent_mma", kern, dim3((unsigned)a.ns, (unsigned)((a.H + 16 * MT - 1) / (16 * MT)), (unsigned)R), dim3(LM_THREADS), lm_smem<MT>(a.lq, stages), a, stages);
+}
+template <int MT>
+static int launch_mma_cols(jg_dev* dev, const LatentArgs<bf16>& a, int R, int stages) {
+  if (a.rank <= 128) return launch_mma<MT, 2>(dev, a, R, stages);
+  if (a.rank <= 256) return launch_mma<MT, 4>(dev, a, R, stages);
+  if (a.rank <= 512) return launch_mma<MT, 8>(dev, a, R, stages);
+  return launch_mma<1, 16>(dev, a, R, stages);
+}
+static int launch_scores(jg_dev* dev, const LatentArgs<float>& a, int R, int, int) {
+  return jg_launch(dev, "latent_split", latent_split_kernel<float>, dim3((unsigned)R, (unsigned)a.H, (unsigned)a.ns), dim3(LS_THREADS), (size_t)a.lat() * 4, a);
+}
+static int launch_scores(jg_dev* dev, const LatentArgs<bf16>& a, int R, int mt, int stages) {
+  if (mt == 2) return launch_mma_cols<2>(dev, a, R, stages);
+  if (mt == 1) return launch_mma_cols<1>(dev, a, R, stages);
+  return jg_launch(dev, "latent_split", latent_split_kernel<bf16>, dim3((unsigned)R, (unsigned)a.H, (unsigned)a.ns), dim3(LS_THREADS), (size_t)a.lat() * 4, a);
+}
+
+template <typename T>
+static int run_absorbed(jg_dev* dev, LatentArgs<T> a, const jg_latent_desc* d) {
+  const int R = a.B * a.Sc;
+  int stages = 1;
+  const int mt = mma_tiles(dev, d, &stages);
+  a.lq = round32(d->kv_rank + d->rot_dim);
+  a.ns = latent_splits(dev, d, R, mt ? 16 * mt : 1);
+  a.qt = (T*)d->scratch;
+  a.part = (float*)(d->scratch + 4ull * R * d->heads * a.lq);
+  const unsigned slices = (unsigned)((d->kv_rank + LP_COLS - 1) / LP_COLS), rg = (unsigned)((R + LP_ROWS - 1) / LP_ROWS);
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(latent_pre_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 4096 * LP_ROWS * 4));
+    set[dev->ordinal & 7] = true;
+  }
+  int rc = jg_launch(dev, "latent_pre", latent_pre_kernel<T>, dim3(d->heads * slices + 1, rg), dim3(256), (size_t)LP_ROWS * d->dim * 4, a, R);
+  if (rc) return rc;
+  rc = launch_scores(dev, a, R, mt, stages);
+  if (rc) return rc;
+  return jg_launch(dev, "latent_combine", latent_combine_kernel<T>, dim3((unsigned)d->heads, (unsigned)((d->vdim + LC_OUT - 1) / LC_OUT), (unsigned)((R + LC_ROWS - 1) / LC_ROWS)), dim3(256),
+                   (size_t)LC_ROWS * d->ld_u * 4, a, R);
+}
+
+template <int VT>
+static int launch_chunk(jg_dev* dev, const LatentArgs<bf16>& a, int qkp) {
+  auto kern = latent_chunk_kernel<VT>;
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dev->prop.sharedMemPerBlockOptin - 1024));
+    set[dev->ordinal & 7] = true;
+  }
+  const size_t smem = (size_t)2 * ((LX_Q + 2 * LX_KV) * (qkp + 8) + 2 * LX_KV * (VT * 8 + 8));
+  return jg_launch(dev, "latent_chunk", kern, dim3((unsigned)((a.Sc + LX_Q - 1) / LX_Q), (unsigned)a.H, (unsigned)a.B), dim3(LX_THREADS), smem, a, qkp);
+}
+
+static int run_expanded(jg_dev* dev, LatentArgs<bf16> a, const jg_latent_desc* d) {
+  const int R = a.B * a.Sc, N = d->heads * (d->dim + d->vdim), W = a.B * a.T_prev;
+  a.ctx = (bf16*)d->scratch;
+  a.kv = a.ctx + (((size_t)a.B * a.T_ctx * d->ldc + 31) & ~(size_t)31);
+  a.ldkv = N;
+  int rc = jg_launch(dev, "latent_write", latent_write_kernel<bf16>, dim3((unsigned)((R + W + 7) / 8)), dim3(256), 0, a, R);
+  if (rc) return rc;
+  DenseCall c = {};
+  c.dtype = JG_BF16; c.epilogue = JG_DENSE_STORE; c.M = a.B * a.T_ctx; c.N = N; c.K = d->kv_rank; c.x = a.ctx; c.ldx = d->ldc;
+  c.w[0] = a.uk; c.ldw = d->ld_u; c.y = (void*)a.kv; c.ldy = N;
+  rc = jg_dense_call(dev, c);
+  if (rc) return rc;
+  const int qkp = (d->dim + d->rot_dim + 15) & ~15;
+  if (d->vdim <= 64) return launch_chunk<8>(dev, a, qkp);
+  if (d->vdim <= 128) return launch_chunk<16>(dev, a, qkp);
+  return launch_chunk<32>(dev, a, qkp);
+}
+static int run_expanded(jg_dev*, const LatentArgs<float>&, const jg_latent_desc*) { return JG_ENOTSUP; }
 
 template <typename T>
 static int latent_run(jg_dev* dev, const jg_batch* bt, const jg_latent_desc* d) {
@@ -190,19 +743,27 @@ static int latent_run(jg_dev* dev, const jg_batch* bt, const jg_latent_desc* d) 
   a.pos = (const int32_t*)bt->pos; a.seq = (const int32_t*)bt->seq;
   a.B = bt->B; a.Sc = bt->Sc; a.H = d->heads; a.dim = d->dim; a.rd = d->rot_dim; a.vd = d->vdim; a.rank = d->kv_rank; a.window = d->window;
   a.ldp = d->ldp; a.ldo = d->ldo; a.ldc = d->ldc; a.ldu = d->ld_u; a.page = d->page; a.pps = d->pages_per_slot;
-  a.rot_pairs = d->rot_pairs; a.rot_rows = d->rot_rows; a.eps = d->eps; a.scale = d->scale;
+  a.rot_pairs = d->rot_pairs; a.rot_rows = d->rot_rows; a.eps = d->eps; a.scale = d->scale; a.start = bt->start;
   while ((1 << a.page_shift) < d->page) a.page_shift++;
-  const int R = bt->B * bt->Sc, L = d->kv_rank + d->rot_dim;
-  a.ns = latent_splits(d, R);
-  a.qt = (float*)d->scratch;
-  a.part = a.qt + (size_t)R * d->heads * L;
-  int rc = jg_launch(dev, "latent_write", latent_write_kernel<T>, dim3((unsigned)((R + 7) / 8)), dim3(256), 0, a, R);
-  if (rc) return rc;
-  rc = jg_launch(dev, "latent_absorb", latent_absorb_kernel<T>, dim3((unsigned)R, (unsigned)d->heads), dim3(128), (size_t)d->dim * 4, a);
-  if (rc) return rc;
-  rc = jg_launch(dev, "latent_split", latent_split_kernel<T>, dim3((unsigned)R, (unsigned)d->heads, (unsigned)a.ns), dim3(LS_THREADS), (size_t)L * 4, a);
-  if (rc) return rc;
-  return jg_launch(dev, "latent_combine", latent_combine_kernel<T>, dim3((unsigned)R, (unsigned)d->heads), dim3(128), (size_t)d->kv_rank * 4, a);
+  if (expandable(d, bt->Sc) && bt->start >= 0) {
+    JG_REQUIRE(bt->start + bt->Sc <= d->rot_rows, "latent_attn: positions %d .. %d are outside the tables", bt->start, bt->start + bt->Sc);
+    a.T_prev = d->window > 0 && d->window - 1 < bt->start ? d->window - 1 : bt->start;
+    a.T_ctx = a.T_prev + bt->Sc;
+    if (a.T_ctx <= LATENT_MAX_CTX) return run_expanded(dev, a, d);
+  }
+  if (!expandable(d, bt->Sc)) return run_absorbed(dev, a, d);
+  // absorbed form in passes of LATENT_MIN_EXPANDED tokens per sequence: rows of a pass are contiguous, positions shift
+  JG_REQUIRE(bt->start >= 0, "latent_attn: a portion of %d tokens needs its start on the host", bt->Sc);
+  for (int s = 0; s < bt->Sc; s += LATENT_MIN_EXPANDED) {
+    LatentArgs<T> q = a;
+    q.Sc = bt->Sc - s < LATENT_MIN_EXPANDED ? bt->Sc - s : LATENT_MIN_EXPANDED;
+    q.shift = s;
+    q.proj = a.proj + (size_t)s * a.B * a.ldp;
+    q.out = a.out + (size_t)s * a.B * a.ldo;
+    int rc = run_absorbed(dev, q, d);
+    if (rc) return rc;
+  }
+  return JG_OK;
 }
 
 JG_API int jg_latent_attn(jg_dev* dev, const jg_batch* b, const jg_latent_desc* d) {
@@ -210,15 +771,17 @@ JG_API int jg_latent_attn(jg_dev* dev, const jg_batch* b, const jg_latent_desc* 
   JG_REQUIRE(d != nullptr && b != nullptr && b->B > 0 && b->Sc > 0 && jg_aligned(b->pos, 4) && jg_aligned(b->seq, 4), "latent_attn: bad batch");
   JG_REQUIRE(d->dtype == JG_F32 || d->dtype == JG_BF16, "latent_attn: unknown element type %d", d->dtype);
   JG_REQUIRE(d->heads > 0 && d->heads <= 65535 && d->dim > 0 && d->rot_dim > 0 && d->vdim > 0 && d->kv_rank > 0 && d->window >= 0, "latent_attn: bad shape");
-  JG_REQUIRE(d->dim <= 4096 && d->kv_rank + d->rot_dim <= 8192, "latent_attn: heads of %d or latents of %d values are too large", d->dim, d->kv_rank);
+  JG_REQUIRE(d->dim <= 2048 && d->rot_dim <= 4096, "latent_attn: heads of %d + %d values are too large", d->dim, d->rot_dim);
   if (d->kv_rank > LS_MAX_RANK) { jg_set_error("latent_attn: latents of %d values (largest supported: %d)", d->kv_rank, LS_MAX_RANK); return JG_ENOTSUP; }
   JG_REQUIRE(d->rot_pairs >= 0 && 2 * d->rot_pairs <= d->rot_dim && d->rot_rows > 0, "latent_attn: bad rotary table");
-  JG_REQUIRE(d->ldp >= d->heads * (d->dim + d->rot_dim) + d->kv_rank + d->rot_dim && d->ldo >= d->heads * d->vdim && d->ldc >= d->kv_rank + d->rot_dim && d->ld_u >= d->kv_rank,
-             "latent_attn: row strides too small");
+  const int vec = d->dtype == JG_F32 ? 4 : 8;
+  JG_REQUIRE(d->ldp >= d->heads * (d->dim + d->rot_dim) + d->kv_rank + d->rot_dim && d->ldo >= d->heads * d->vdim && d->ldc >= d->kv_rank + d->rot_dim && d->ld_u >= d->kv_rank &&
+             d->ldc % vec == 0 && d->ld_u % vec == 0 && d->ldo % 2 == 0, "latent_attn: bad row strides");
   JG_REQUIRE(d->page > 0 && (d->page & (d->page - 1)) == 0 && d->pages_per_slot > 0, "latent_attn: page size must be a power of two");
   const long long span = d->window > 0 ? (long long)d->window - 1 + b->Sc : (long long)d->rot_rows, cap = (long long)d->page * d->pages_per_slot;
   JG_REQUIRE(cap >= span || cap >= d->rot_rows, "latent_attn: %lld cached positions do not hold a window of %d and %d new tokens", cap, d->window, b->Sc);
-  JG_REQUIRE(d->proj && d->pool && jg_aligned(d->block_table, 4) && jg_aligned(d->rot, 4) && d->norm_w && d->sink && d->ukv && jg_aligned(d->scratch, 16) && d->out, "latent_attn: null pointer");
+  JG_REQUIRE(d->proj && jg_aligned(d->pool, 16) && jg_aligned(d->block_table, 4) && jg_aligned(d->rot, 4) && d->norm_w && d->sink && jg_aligned(d->ukv, 16) && jg_aligned(d->scratch, 16) &&
+             jg_aligned(d->out, 4), "latent_attn: null or misaligned pointer");
   uint64_t need = 0;
   int rc = jg_latent_scratch_bytes(d, b->B, b->Sc, &need);
   if (rc) return rc;

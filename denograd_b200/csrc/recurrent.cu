@@ -11,11 +11,11 @@ namespace cg = cooperative_groups;
 // S_t = (1 - z_t) S_{t-1} + z_t c_t is, per channel, an affine map of the state; maps compose, so a portion is scanned in
 // blocks of MG_WARPS x MG_TOK tokens: warp w composes its MG_TOK consecutive tokens, the warps' maps meet in shared
 // memory, and each warp replays its tokens from the state its predecessors leave.  One CTA = 32 channels of a sequence.
-constexpr int MG_WARPS = 16, MG_TOK = 8, MG_THREADS = 32 * MG_WARPS;
+constexpr int MG_WARPS = 32, MG_TOK = 4, MG_THREADS = 32 * MG_WARPS;
 
 template <typename T>
-__global__ void __launch_bounds__(MG_THREADS) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
-                                                                 const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
+__global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
+                                                                    const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
   __shared__ float s_a[MG_WARPS][32], s_b[MG_WARPS][32], s_carry[2][32];
   pdl_launch();
   pdl_wait();
@@ -24,26 +24,30 @@ __global__ void __launch_bounds__(MG_THREADS) mingru_scan_kernel(const T* __rest
   float* st = state + (size_t)seq[b] * width + ch;
   if (warp == 0) s_carry[0][lane] = (ok && pos[b] > 0) ? *st : 0.f;
   int par = 0;
-  for (int t0 = 0; t0 < Sc; t0 += MG_WARPS * MG_TOK) {
-    float z[MG_TOK], c[MG_TOK], g[MG_TOK];
+  T nz[MG_TOK], nc[MG_TOK], ng[MG_TOK];  // the next block's inputs travel while this one is worked on
+  auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
       const int t = t0 + warp * MG_TOK + i;
-      const bool in = ok && t < Sc;
+      if (!ok || t >= Sc) continue;
       const T* p = proj + ((size_t)t * B + b) * ldp + ch;
-      z[i] = in ? to_f32(p[0]) : 0.f;
-      c[i] = in ? to_f32(p[width]) : 0.f;
-      g[i] = in ? to_f32(p[2 * width]) : 0.f;
+      nz[i] = p[0]; nc[i] = p[width]; ng[i] = p[2 * width];
     }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < Sc; t0 += MG_WARPS * MG_TOK) {
+    float z[MG_TOK], c[MG_TOK], g[MG_TOK];
     float A = 1.f, Bc = 0.f;
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
-      const bool in = t0 + warp * MG_TOK + i < Sc;
-      z[i] = in ? sigmoid_f32(z[i]) : 0.f;  // past the end: the identity map
-      c[i] = z[i] * mingru_candidate(c[i]);
+      const bool in = ok && t0 + warp * MG_TOK + i < Sc;
+      z[i] = in ? sigmoid_f32(to_f32(nz[i])) : 0.f;  // past the end: the identity map
+      c[i] = in ? z[i] * mingru_candidate(to_f32(nc[i])) : 0.f;
+      g[i] = in ? to_f32(ng[i]) : 0.f;
       A *= 1.0f - z[i];
       Bc = fmaf(1.0f - z[i], Bc, c[i]);
     }
+    fetch(t0 + MG_WARPS * MG_TOK);
     s_a[warp][lane] = A;
     s_b[warp][lane] = Bc;
     __syncthreads();
@@ -62,6 +66,31 @@ __global__ void __launch_bounds__(MG_THREADS) mingru_scan_kernel(const T* __rest
   if (warp == 0 && ok) *st = s_carry[par][lane];
 }
 
+// One token per sequence: one thread per channel.
+template <typename T>
+__global__ void __launch_bounds__(256) mingru_step_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
+                                                          const int32_t* __restrict__ seq, int width, int ldp, int ldo) {
+  pdl_launch();
+  pdl_wait();
+  const int ch = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y;
+  if (ch >= width) return;
+  const T* p = proj + (size_t)b * ldp + ch;
+  float* st = state + (size_t)seq[b] * width + ch;
+  const float z = sigmoid_f32(to_f32(p[0])), s = fmaf(z, mingru_candidate(to_f32(p[width])), (1.0f - z) * (pos[b] > 0 ? *st : 0.f));
+  *st = s;
+  out[(size_t)b * ldo + ch] = from_f32<T>(s * silu_f32(to_f32(p[2 * width])));
+}
+
+template <typename T>
+static int mingru_run(jg_dev* dev, const jg_batch* b, const jg_mingru_desc* d) {
+  const int32_t *pos = (const int32_t*)b->pos, *seq = (const int32_t*)b->seq;
+  if (b->Sc == 1)
+    return jg_launch(dev, "mingru_step", mingru_step_kernel<T>, dim3((unsigned)((d->width + 255) / 256), (unsigned)b->B), dim3(256), 0, (const T*)d->proj, (float*)d->state,
+                     (T*)d->out, pos, seq, d->width, d->ldp, d->ldo);
+  return jg_launch(dev, "mingru_scan", mingru_scan_kernel<T>, dim3((unsigned)((d->width + 31) / 32), (unsigned)b->B), dim3(MG_THREADS), 0, (const T*)d->proj, (float*)d->state,
+                   (T*)d->out, pos, seq, b->B, b->Sc, d->width, d->ldp, d->ldo);
+}
+
 static int check_rows(const char* name, const jg_batch* b, int dtype) {
   JG_REQUIRE(b != nullptr && b->B > 0 && b->Sc > 0 && jg_aligned(b->pos, 4) && jg_aligned(b->seq, 4), "%s: bad batch", name);
   JG_REQUIRE(dtype == JG_F32 || dtype == JG_BF16, "%s: unknown element type %d", name, dtype);
@@ -74,11 +103,7 @@ JG_API int jg_mingru_scan(jg_dev* dev, const jg_batch* b, const jg_mingru_desc* 
   int rc = check_rows("mingru_scan", b, d->dtype);
   if (rc) return rc;
   JG_REQUIRE(d->width > 0 && d->ldp >= 3 * d->width && d->ldo >= d->width && d->proj && d->out && jg_aligned(d->state, 4), "mingru_scan: bad shape or pointer");
-  const dim3 grid((unsigned)((d->width + 31) / 32), (unsigned)b->B);
-  const int32_t *pos = (const int32_t*)b->pos, *seq = (const int32_t*)b->seq;
-  if (d->dtype == JG_F32)
-    return jg_launch(dev, "mingru_scan", mingru_scan_kernel<float>, grid, dim3(MG_THREADS), 0, (const float*)d->proj, (float*)d->state, (float*)d->out, pos, seq, b->B, b->Sc, d->width, d->ldp, d->ldo);
-  return jg_launch(dev, "mingru_scan", mingru_scan_kernel<bf16>, grid, dim3(MG_THREADS), 0, (const bf16*)d->proj, (float*)d->state, (bf16*)d->out, pos, seq, b->B, b->Sc, d->width, d->ldp, d->ldo);
+  return d->dtype == JG_F32 ? mingru_run<float>(dev, b, d) : mingru_run<bf16>(dev, b, d);
 }
 
 // ------------------------------------------------------------------------------------------------ gated delta rule
@@ -88,7 +113,8 @@ struct DeltaArgs {
   const float *conv_w, *a_log, *dt_bias, *norm_w;
   float* state;
   T* tail;
-  float *qkv, *gates, *kq, *o;  // scratch: [R][C], [R][H][2] (decay, beta), [R][G], [R][H * vd]
+  // scratch: unit vectors [R][G][q | k][lds], [R][H][2] (decay, beta), v and then the read-outs [R][H * vd]
+  float *qk, *gates, *v, *o;
   T* out;
   const int32_t *pos, *seq;
   int B, Sc, H, G, dim, vd, taps, ldp, ldo, lds;  // lds: dim rounded up to 4
@@ -124,7 +150,7 @@ __device__ __forceinline__ float2 delta_gates(const DeltaArgs<T>& a, size_t row,
 }
 constexpr float DELTA_UNIT_EPS = 1e-6f;
 
-// Portions, step 1, one CTA per row: convolutions, unit vectors, gates and k.q into scratch.
+// Portions, step 1, one CTA per row: convolutions, unit vectors and gates into scratch.
 template <typename T>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs<T> a) {
   extern __shared__ __align__(16) float buf[];
@@ -132,24 +158,24 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs<T> a) {
   pdl_wait();
   const int r = blockIdx.x, b = r % a.B, s = r / a.B, C = a.channels(), p0 = a.pos[b];
   const T* tail = a.tail + (size_t)a.seq[b] * a.taps * C;
-  float* dst = a.qkv + (size_t)r * C;
   const int nqk = 2 * a.G * a.dim;
+  float* dv = a.v + (size_t)r * a.H * a.vd;
+#pragma unroll 2
   for (int c = threadIdx.x; c < C; c += 256) {
     const float v = delta_conv_silu(a, b, s, c, p0, tail);
     if (c < nqk) buf[c] = v;
-    else dst[c] = v;
+    else dv[c - nqk] = v;
   }
   for (int h = threadIdx.x; h < a.H; h += 256) *reinterpret_cast<float2*>(a.gates + ((size_t)r * a.H + h) * 2) = delta_gates(a, r, h);
   __syncthreads();
   const int lane = threadIdx.x & 31;
-  for (int g = threadIdx.x >> 5; g < a.G; g += 8) {
-    const float *q = buf + g * a.dim, *k = buf + (a.G + g) * a.dim;
-    float sq = 0.f, sk = 0.f, qk = 0.f;
-    for (int i = lane; i < a.dim; i += 32) { sq = fmaf(q[i], q[i], sq); sk = fmaf(k[i], k[i], sk); qk = fmaf(q[i], k[i], qk); }
-    sq = warp_sum(sq); sk = warp_sum(sk); qk = warp_sum(qk);
-    const float rq = 1.0f / sqrtf(sq + DELTA_UNIT_EPS) * (1.0f / sqrtf((float)a.dim)), rk = 1.0f / sqrtf(sk + DELTA_UNIT_EPS);
-    for (int i = lane; i < a.dim; i += 32) { dst[g * a.dim + i] = q[i] * rq; dst[(a.G + g) * a.dim + i] = k[i] * rk; }
-    if (lane == 0) a.kq[(size_t)r * a.G + g] = qk * rq * rk;
+  for (int g = threadIdx.x >> 5; g < 2 * a.G; g += 8) {  // q heads, then k heads
+    const float* x = buf + g * a.dim;
+    float ss = 0.f;
+    for (int i = lane; i < a.dim; i += 32) ss = fmaf(x[i], x[i], ss);
+    const float rs = 1.0f / sqrtf(warp_sum(ss) + DELTA_UNIT_EPS) * (g < a.G ? 1.0f / sqrtf((float)a.dim) : 1.0f);
+    float* dst = a.qk + (((size_t)r * a.G + (g < a.G ? g : g - a.G)) * 2 + (g < a.G ? 0 : 1)) * a.lds;
+    for (int i = lane; i < a.lds; i += 32) dst[i] = i < a.dim ? x[i] * rs : 0.f;
   }
 }
 
@@ -201,54 +227,165 @@ struct DeltaCol {
 };
 
 // Portions, step 2: the recurrence.  Columns of S never meet, so a CTA takes DS_COLS columns of one head of one sequence
-// and walks the tokens in blocks staged in shared memory (double-buffered through registers).
-constexpr int DS_LPC = 8, DS_COLS = 16, DS_THREADS = DS_LPC * DS_COLS, DS_TOK = 16;
+// and walks the tokens, DS_STEP at a time.  With D_i the product of the decays up to token i of such a group and w_j the
+// update of token j decayed to the present one,
+//   S_0^T k_i, S_0^T q_i          for all i at once, on the state before the group
+//   u_i = beta_i (v_i - D_i S_0^T k_i - sum_{j<i} (k_j . k_i) w_j),   o_i = D_i S_0^T q_i + sum_{j<=i} (k_j . q_i) w_j
+//   S   = D S_0 + sum_j k_j w_j^T
+// so that the reductions over the lanes of a column overlap instead of following one another.  Blocks of DS_TOK tokens are
+// staged by cp.async, one ahead; the products k_j . k_i and k_j . q_i of a block are worked out by all threads first.
+constexpr int DS_LPC = 8, DS_COLS = 16, DS_THREADS = DS_LPC * DS_COLS, DS_TOK = 16, DS_STEP = 4, DS_PAIRS = DS_STEP * DS_STEP;
+
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async8(void* smem, const void* gmem) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+// two fp32 FMAs in one instruction
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("{\n\t.reg .b64 ra, rb, rc, rd;\n\tmov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %5};\n\tmov.b64 rc, {%6, %7};\n\t"
+      "fma.rn.f32x2 rd, ra, rb, rc;\n\tmov.b64 {%0, %1}, rd;\n\t}"
+      : "=f"(d.x), "=f"(d.y)
+      : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return fma2(a, b, make_float2(-0.0f, -0.0f)); }
+
+template <int E>
+struct DeltaStage {
+  static constexpr int ROW = E * DS_LPC + 4;  // padded: the rows a warp compares start in different banks
+  float k[DS_TOK][ROW], q[DS_TOK][ROW], v[DS_TOK][DS_COLS], gate[DS_TOK][2];
+};
 
 template <typename T, int E>
 __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<T> a) {
-  constexpr int DP = E * DS_LPC;  // padded head size
-  __shared__ __align__(16) float sk[DS_TOK][DP], sq[DS_TOK][DP];
-  __shared__ float sv[DS_TOK][DS_COLS], sg[DS_TOK][3];
+  using Stage = DeltaStage<E>;
+  extern __shared__ __align__(16) unsigned char dsm[];
+  Stage* stages = reinterpret_cast<Stage*>(dsm);
+  __shared__ __align__(16) float pairs[DS_TOK / DS_STEP][2][DS_PAIRS];  // [group][k.k | k.q][i * DS_STEP + j]
   pdl_launch();
-  pdl_wait();
   const int tid = threadIdx.x, l = tid % DS_LPC, col = tid / DS_LPC, h = blockIdx.y, b = blockIdx.z;
-  const int j0 = blockIdx.x * DS_COLS, j = j0 + col, g = h / (a.H / a.G), C = a.channels(), slot = a.seq[b];
+  const int j0 = blockIdx.x * DS_COLS, j = j0 + col, g = h / (a.H / a.G), C = a.channels();
+  for (int i = tid; i < (int)(2 * sizeof(Stage) / 4); i += DS_THREADS) reinterpret_cast<float*>(dsm)[i] = 0.f;  // padding, columns past vd
+  __syncthreads();
+  pdl_wait();
+  const int slot = a.seq[b];
   const bool live = j < a.vd;
-  float* st = a.state + (((size_t)slot * a.H + h) * a.vd + (live ? j : 0)) * a.lds;
-  DeltaCol<DS_LPC, E> S;
-  S.load(st, l, a.lds, live && a.pos[b] > 0);
-  for (int t0 = 0; t0 < a.Sc; t0 += DS_TOK) {
+  const int c4 = a.lds / 4;
+  auto stage_block = [&](int t0, Stage& st) {
     const int nt = min(DS_TOK, a.Sc - t0);
-    for (int i = tid; i < nt * DP; i += DS_THREADS) {
-      const int t = i / DP, e = i % DP;
-      const float* src = a.qkv + ((size_t)(t0 + t) * a.B + b) * C;
-      sq[t][e] = e < a.dim ? src[g * a.dim + e] : 0.f;
-      sk[t][e] = e < a.dim ? src[(a.G + g) * a.dim + e] : 0.f;
+    for (int i = tid; i < DS_TOK * 2 * c4; i += DS_THREADS) {
+      const int t = i / (2 * c4), e = i % (2 * c4);
+      float* dst = e < c4 ? &st.q[t][e * 4] : &st.k[t][(e - c4) * 4];
+      if (t < nt) cp_async16(dst, a.qk + (((size_t)(t0 + t) * a.B + b) * a.G + g) * 2 * a.lds + e * 4);
+      else *reinterpret_cast<float4*>(dst) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    for (int i = tid; i < nt * DS_COLS; i += DS_THREADS) {
+    for (int i = tid; i < DS_TOK * DS_COLS; i += DS_THREADS) {
       const int t = i / DS_COLS, c = i % DS_COLS;
-      sv[t][c] = j0 + c < a.vd ? a.qkv[((size_t)(t0 + t) * a.B + b) * C + 2 * a.G * a.dim + h * a.vd + j0 + c] : 0.f;
+      if (t < nt && j0 + c < a.vd) cp_async4(&st.v[t][c], a.v + ((size_t)(t0 + t) * a.B + b) * a.H * a.vd + (size_t)h * a.vd + j0 + c);
     }
-    for (int t = tid; t < nt; t += DS_THREADS) {
-      const size_t r = (size_t)(t0 + t) * a.B + b;
-      sg[t][0] = a.gates[(r * a.H + h) * 2];
-      sg[t][1] = a.gates[(r * a.H + h) * 2 + 1];
-      sg[t][2] = a.kq[r * a.G + g];
+    if (tid < DS_TOK) {  // a token past the end keeps the state: decay 1, beta 0
+      if (tid < nt) cp_async8(st.gate[tid], a.gates + (((size_t)(t0 + tid) * a.B + b) * a.H + h) * 2);
+      else { st.gate[tid][0] = 1.f; st.gate[tid][1] = 0.f; }
     }
-    __syncthreads();
-    for (int t = 0; t < nt; t++) {
-      float4 kv[E / 4], qv[E / 4];
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  stage_block(0, stages[0]);
+  float* stp = a.state + (((size_t)slot * a.H + h) * a.vd + (live ? j : 0)) * a.lds;
+  DeltaCol<DS_LPC, E> col_s;
+  col_s.load(stp, l, a.lds, live && a.pos[b] > 0);
+  float2 S[E / 2];
 #pragma unroll
-      for (int i = 0; i < E / 4; i++) {
-        kv[i] = *reinterpret_cast<const float4*>(&sk[t][(l + DS_LPC * i) * 4]);
-        qv[i] = *reinterpret_cast<const float4*>(&sq[t][(l + DS_LPC * i) * 4]);
-      }
-      const float o = S.step(kv, qv, sv[t][col], sg[t][0], sg[t][1], sg[t][2]);
-      if (l == 0 && live) a.o[((size_t)(t0 + t) * a.B + b) * a.H * a.vd + h * a.vd + j] = o;
+  for (int i = 0; i < E / 2; i++) S[i] = make_float2(col_s.s[2 * i], col_s.s[2 * i + 1]);
+
+  int buf = 0;
+  for (int t0 = 0; t0 < a.Sc; t0 += DS_TOK, buf ^= 1) {
+    if (t0 + DS_TOK < a.Sc) {
+      stage_block(t0 + DS_TOK, stages[buf ^ 1]);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
+    const Stage& st = stages[buf];
+    // k_j . k_i and k_j . q_i: DS_TOK / DS_STEP groups x 16 pairs, two threads per pair (which share both products)
+    {
+      const int pr = tid >> 1, half = tid & 1, grp = pr / DS_PAIRS, i = (pr / DS_STEP) % DS_STEP, jj = pr % DS_STEP;
+      float dk = 0.f, dq = 0.f;
+      if (jj <= i) {
+        const float *kj = st.k[grp * DS_STEP + jj], *ki = st.k[grp * DS_STEP + i], *qi = st.q[grp * DS_STEP + i];
+        for (int e = half; e < c4; e += 2) {
+          const float4 x = *reinterpret_cast<const float4*>(kj + e * 4), y = *reinterpret_cast<const float4*>(ki + e * 4), z = *reinterpret_cast<const float4*>(qi + e * 4);
+          dk = fmaf(x.x, y.x, dk); dk = fmaf(x.y, y.y, dk); dk = fmaf(x.z, y.z, dk); dk = fmaf(x.w, y.w, dk);
+          dq = fmaf(x.x, z.x, dq); dq = fmaf(x.y, z.y, dq); dq = fmaf(x.z, z.z, dq); dq = fmaf(x.w, z.w, dq);
+        }
+      }
+      dk += __shfl_xor_sync(0xffffffffu, dk, 1);
+      dq += __shfl_xor_sync(0xffffffffu, dq, 1);
+      if (half == 0) { pairs[grp][0][i * DS_STEP + jj] = dk; pairs[grp][1][i * DS_STEP + jj] = dq; }
+    }
+    __syncthreads();
+    for (int grp = 0; grp < DS_TOK / DS_STEP; grp++) {
+      const int tb = grp * DS_STEP;
+      float sk[DS_STEP], sq[DS_STEP];
+#pragma unroll
+      for (int i = 0; i < DS_STEP; i++) {
+        float2 ak = make_float2(0.f, 0.f), aq = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int e = 0; e < E / 4; e++) {
+          const float4 kv = *reinterpret_cast<const float4*>(&st.k[tb + i][(l + DS_LPC * e) * 4]), qv = *reinterpret_cast<const float4*>(&st.q[tb + i][(l + DS_LPC * e) * 4]);
+          ak = fma2(S[2 * e], make_float2(kv.x, kv.y), ak); ak = fma2(S[2 * e + 1], make_float2(kv.z, kv.w), ak);
+          aq = fma2(S[2 * e], make_float2(qv.x, qv.y), aq); aq = fma2(S[2 * e + 1], make_float2(qv.z, qv.w), aq);
+        }
+        sk[i] = ak.x + ak.y;
+        sq[i] = aq.x + aq.y;
+      }
+#pragma unroll
+      for (int o = DS_LPC / 2; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < DS_STEP; i++) { sk[i] += __shfl_xor_sync(0xffffffffu, sk[i], o); sq[i] += __shfl_xor_sync(0xffffffffu, sq[i], o); }
+      float w[DS_STEP], D = 1.f, mine = 0.f;
+#pragma unroll
+      for (int i = 0; i < DS_STEP; i++) {
+        const float2 gt = *reinterpret_cast<const float2*>(st.gate[tb + i]);
+        D *= gt.x;
+        float pre = D * sk[i], o = D * sq[i];
+#pragma unroll
+        for (int jj = 0; jj < i; jj++) {
+          w[jj] *= gt.x;
+          pre = fmaf(pairs[grp][0][i * DS_STEP + jj], w[jj], pre);
+          o = fmaf(pairs[grp][1][i * DS_STEP + jj], w[jj], o);
+        }
+        w[i] = gt.y * (st.v[tb + i][col] - pre);
+        o = fmaf(pairs[grp][1][i * DS_STEP + i], w[i], o);
+        if (l == i) mine = o;
+      }
+      const float2 D2 = make_float2(D, D);
+#pragma unroll
+      for (int e = 0; e < E / 2; e++) S[e] = mul2(S[e], D2);
+#pragma unroll
+      for (int i = 0; i < DS_STEP; i++) {
+        const float2 w2 = make_float2(w[i], w[i]);
+#pragma unroll
+        for (int e = 0; e < E / 4; e++) {
+          const float4 kv = *reinterpret_cast<const float4*>(&st.k[tb + i][(l + DS_LPC * e) * 4]);
+          S[2 * e] = fma2(make_float2(kv.x, kv.y), w2, S[2 * e]);
+          S[2 * e + 1] = fma2(make_float2(kv.z, kv.w), w2, S[2 * e + 1]);
+        }
+      }
+      const int t = t0 + tb + l;
+      if (l < DS_STEP && live && t < a.Sc) a.o[((size_t)t * a.B + b) * a.H * a.vd + (size_t)h * a.vd + j] = mine;
+    }
+    __syncthreads();  // the other stage is refilled next, and `pairs` is rewritten
   }
-  if (live) S.store(st, l, a.lds);
+#pragma unroll
+  for (int i = 0; i < E / 2; i++) { col_s.s[2 * i] = S[i].x; col_s.s[2 * i + 1] = S[i].y; }
+  if (live) col_s.store(stp, l, a.lds);
   // the convolution's last inputs: entry position % taps, which no row of this call reads any more
   T* tail = a.tail + (size_t)slot * a.taps * C;
   const int cta = blockIdx.y * gridDim.x + blockIdx.x, ctas = gridDim.x * gridDim.y, keep = min(a.taps - 1, a.Sc);
@@ -340,12 +477,14 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<
     const int j = jb + col;
     const bool live = j < j1;
     float* st = st0 + (size_t)(live ? j : j0) * a.lds;
-    if (jb != j0) S.load(st, l, a.lds, live && p0 > 0);
+    DeltaCol<DS_LPC, E> next;
+    if (jb + DD_COLS < j1) next.load(st0 + (size_t)min(j + DD_COLS, j1 - 1) * a.lds, l, a.lds, p0 > 0);
     const float o = S.step(k4, q4, live ? dyn[j - j0] : 0.f, gt.x, gt.y, tqk * rq * rk);
     if (live) {
       S.store(st, l, a.lds);
       if (l == 0) { dyn[j - j0] = o; ss = fmaf(o, o, ss); }
     }
+    if (jb + DD_COLS < j1) S = next;
     __syncwarp();
   }
   ss = warp_sum(ss);
@@ -370,16 +509,16 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<
 JG_API int jg_delta_scratch_floats(const jg_delta_desc* d, int32_t rows, uint64_t* out) {
   JG_REQUIRE(d != nullptr && out != nullptr && rows > 0, "delta_scratch_floats: bad arguments");
   const uint64_t R = (uint64_t)rows;
-  *out = R * (2ull * d->kv_heads * d->dim + 2ull * d->heads * d->vdim + 2ull * d->heads + d->kv_heads + 8);
+  *out = R * (2ull * d->kv_heads * ((d->dim + 3) & ~3) + 2ull * d->heads * d->vdim + 2ull * d->heads) + 16;
   return JG_OK;
 }
 
 template <typename T, int E>
 static int delta_launch(jg_dev* dev, const DeltaArgs<T>& a) {
-  const int R = a.B * a.Sc, C = 2 * a.G * a.dim + a.H * a.vd;
+  const int R = a.B * a.Sc;
   if (a.Sc == 1) {
     int cs = 1;
-    while (cs < DD_MAX_CLUSTER && cs * DD_COLS < a.vd) cs *= 2;
+    while (cs < DD_MAX_CLUSTER && cs * DD_COLS < a.vd && R * a.H * cs < 2 * dev->sm_count) cs *= 2;
     const size_t smem = (size_t)((a.vd + cs - 1) / cs) * sizeof(float);
     return jg_launch_cluster(dev, "delta_step", delta_step_kernel<T, E>, dim3((unsigned)cs, (unsigned)a.H, (unsigned)R), dim3(DD_THREADS), smem, cs, a);
   }
@@ -389,10 +528,15 @@ static int delta_launch(jg_dev* dev, const DeltaArgs<T>& a) {
     JG_CUDA(cudaFuncSetAttribute(delta_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dev->prop.sharedMemPerBlockOptin - 1024));
     set[dev->ordinal & 7] = true;
   }
-  (void)C;
   int rc = jg_launch(dev, "delta_prep", delta_prep_kernel<T>, dim3((unsigned)R), dim3(256), smem, a);
   if (rc) return rc;
-  rc = jg_launch(dev, "delta_scan", delta_scan_kernel<T, E>, dim3((unsigned)((a.vd + DS_COLS - 1) / DS_COLS), (unsigned)a.H, (unsigned)a.B), dim3(DS_THREADS), 0, a);
+  static bool scan_set[8] = {};
+  if (!scan_set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(delta_scan_kernel<T, E>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * sizeof(DeltaStage<E>))));
+    scan_set[dev->ordinal & 7] = true;
+  }
+  rc = jg_launch(dev, "delta_scan", delta_scan_kernel<T, E>, dim3((unsigned)((a.vd + DS_COLS - 1) / DS_COLS), (unsigned)a.H, (unsigned)a.B), dim3(DS_THREADS),
+                 2 * sizeof(DeltaStage<E>), a);
   if (rc) return rc;
   return jg_launch(dev, "delta_out", delta_out_kernel<T>, dim3((unsigned)(((long long)R * a.H + 7) / 8)), dim3(256), 0, a, R);
 }
@@ -405,11 +549,11 @@ static int delta_run(jg_dev* dev, const jg_batch* b, const jg_delta_desc* d) {
   a.pos = (const int32_t*)b->pos; a.seq = (const int32_t*)b->seq;
   a.B = b->B; a.Sc = b->Sc; a.H = d->heads; a.G = d->kv_heads; a.dim = d->dim; a.vd = d->vdim; a.taps = d->taps;
   a.ldp = d->ldp; a.ldo = d->ldo; a.lds = (d->dim + 3) & ~3; a.eps = d->eps;
-  const size_t R = (size_t)b->B * b->Sc, C = (size_t)2 * d->kv_heads * d->dim + (size_t)d->heads * d->vdim;
-  a.gates = (float*)d->scratch;  // 8-byte aligned pairs first
-  a.qkv = a.gates + ((R * d->heads * 2 + 3) & ~(size_t)3);
-  a.o = a.qkv + R * C;
-  a.kq = a.o + R * d->heads * d->vdim;
+  const size_t R = (size_t)b->B * b->Sc;
+  a.qk = (float*)d->scratch;  // 16-byte rows first, 8-byte pairs next
+  a.gates = a.qk + R * d->kv_heads * 2 * a.lds;
+  a.v = a.gates + R * d->heads * 2;
+  a.o = a.v + R * d->heads * d->vdim;
   if (d->dim <= 32) return delta_launch<T, 4>(dev, a);
   if (d->dim <= 64) return delta_launch<T, 8>(dev, a);
   if (d->dim <= 128) return delta_launch<T, 16>(dev, a);

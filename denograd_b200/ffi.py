@@ -50,7 +50,7 @@ def _fields(spec: str) -> list:
 
 
 class Batch(C.Structure):
-    _fields_ = _fields("i32 B Sc; u64 pos seq")
+    _fields_ = _fields("i32 B Sc; u64 pos seq; i32 start reserved")
 
 
 class StreamDesc(C.Structure):

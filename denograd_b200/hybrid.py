@@ -318,7 +318,7 @@ class _Rows:
         self.ffn = Tensor.zeros((cap, ffn * (2 if m.dtype == "float32" else 1)), m.dtype, dev) if ffn else None
         Sc = max(1, cap // B)
         self.scratch = Tensor.empty((max(max(l.mixer.scratch(B, s) for l in layers for s in {1, Sc}), 16),), "uint8", dev)
-        self.batch = ffi.Batch(B, 1, self.pos.ptr, self.seq.ptr)
+        self.batch = ffi.Batch(B, 1, self.pos.ptr, self.seq.ptr, -1, 0)
         self.plans: dict[tuple, Plan] = {}
         self.heads: dict[tuple, tuple] = {}
         self.logits = None
@@ -428,8 +428,9 @@ class HybridTransformer(Decoder):
             ws.plans[key] = p
         return ws.plans[key]
 
-    def _run_layers(self, ws: _Rows, B: int, Sc: int) -> Plan:
-        ws.batch.B, ws.batch.Sc = B, Sc
+    def _run_layers(self, ws: _Rows, B: int, Sc: int, start: int = -1) -> Plan:
+        """`start`: the position the rows begin at, or -1 when only the device knows it (a step that is captured)."""
+        ws.batch.B, ws.batch.Sc, ws.batch.start = B, Sc, start
         p = self._plan(ws, B * Sc, Sc == 1)
         p.run(ws.batch)
         return p
@@ -445,7 +446,7 @@ class HybridTransformer(Decoder):
                 d.stream = st
             else:
                 d.ldx = self.ld_width
-            ws.heads[hk] = (st, d, ffi.Batch(n, 1, ws.pos.ptr, ws.seq.ptr))
+            ws.heads[hk] = (st, d, ffi.Batch(n, 1, ws.pos.ptr, ws.seq.ptr, -1, 0))
         st, d, batch = ws.heads[hk]
         d.y, d.key = logits.ptr, key.ptr
         if n > 2:
@@ -493,7 +494,7 @@ class HybridTransformer(Decoder):
             ws.tokens.assign(buf)
             ws.pos.assign(np.full((B,), start_pos + s0, np.int32))
             ws.seq.assign(slots)
-            p = self._run_layers(ws, B, Sc)
+            p = self._run_layers(ws, B, Sc, start_pos + s0)
             if want is None:
                 if s0 + Sc >= S:
                     wsb = self._workspace(B)
@@ -576,7 +577,7 @@ class HybridTransformer(Decoder):
         ws.tokens.assign(buf)
         ws.pos.assign(np.array([start_pos], np.int32))
         ws.seq.assign(np.array([slot], np.int32))
-        ws.batch.B, ws.batch.Sc = 1, S
+        ws.batch.B, ws.batch.Sc, ws.batch.start = 1, S, start_pos
         out, peek = [], Plan(self, ws, S <= 2, S == 1)
         if S <= 2 and len(ws.x) < 2:
             ws.x.append(Tensor.zeros(ws.x[0].shape, "float32", self.dev))

@@ -401,6 +401,8 @@ int jg_dequant_nf4_f16(jg_dev* dev, uint64_t dst, uint64_t w, uint64_t scale, in
 typedef struct {
   int32_t B, Sc;
   uint64_t pos, seq; /* device int32 [B] each */
+  int32_t start;     /* the value of every pos[b], when the host knows it; -1 otherwise (a captured step) */
+  int32_t reserved;
 } jg_batch;
 
 /* x <- x + norm(y) * w_add (y = 0: nothing), stored to x_out (0: not); h = norm(x) * w_norm (0: nothing).  norm divides each
@@ -447,7 +449,8 @@ typedef struct {
  * [i * page, (i + 1) * page) of slot s live on page block_table[s][i % pages_per_slot], so that a window needs only as many
  * pages as it and one call's tokens span.  rot: fp32 [rot_rows][rot_pairs][2] (cos, sin).  window = 0: every earlier
  * position.  The denominator of the softmax also contains exp(sink[h]).  uk, uv: [heads * dim][ld_u], [heads * vdim][ld_u]
- * contiguous (uv = uk + heads * dim rows).  scratch: jg_latent_scratch_bytes(desc, B, Sc) bytes. */
+ * contiguous (uv = uk + heads * dim rows).  scratch: jg_latent_scratch_bytes(desc, B, Sc) bytes
+ * (enough for every smaller call too). */
 typedef struct {
   int32_t dtype, heads, dim, rot_dim, vdim, kv_rank, window, ldp, ldo, ldc, ld_u, page, pages_per_slot, n_slots, rot_pairs, rot_rows;
   float eps, scale;

@@ -152,7 +152,7 @@ def test_stream_step(dev, D, groups, R):
     ld = (D + 7) // 8 * 8
     tx, ty, ta, tn, tr = (Tensor(v, device=dev) for v in (x, y, wa, wn, rows))
     out, h = Tensor.zeros((R + 2, D), "float32", dev), Tensor.zeros((R, ld), "float32", dev)
-    b = ffi.Batch(R, 1, 0, 0)
+    b = ffi.Batch(R, 1, 0, 0, -1, 0)
     for use_rows in (False, True):
         st = ffi.StreamDesc(D, groups, 1e-3, 0, tx.ptr, ty.ptr, ta.ptr, out.ptr, tn.ptr, tr.ptr if use_rows else 0)
         dev.call("jg_stream_norm", C.byref(b), st, h.ptr, ld, ffi.JG_F32)
@@ -182,7 +182,7 @@ def test_projection(dev, M, N, K, dtype, glu):
     y = Tensor.zeros((2 * M, ldy), dtype if glu else "float32", dev)
     d = ffi.DenseDesc(DTYPES[dtype], ffi.DENSE_GLU if glu else ffi.DENSE_STORE, N, K, ld, ld, ldy, 0 if glu else 1, 0.7, 0, tx.ptr, tw[0].ptr, tw[1].ptr, 0,
                       tb[0].ptr, tb[1].ptr, 0, y.ptr)
-    dev.call("jg_dense", C.byref(ffi.Batch(M, 1, 0, 0)), d)
+    dev.call("jg_dense", C.byref(ffi.Batch(M, 1, 0, 0, -1, 0)), d)
     a, b = (x.astype(np.float64) @ w[i].T.astype(np.float64) + bias[i] for i in range(2))
     if glu:
         g, u = np.minimum(a, 0.7), np.clip(b, -0.7, 0.7)
@@ -252,11 +252,13 @@ def test_batch_rows_against_each_alone(B, dtype):
     m = build(MIXED, params, dtype)
     toks = np.array([tokens(MIXED, 60, seed=30 + b) for b in range(B)], np.int32)
     want = [O.forward(params, MIXED, t) for t in toks]
-    at = 0
+    at, got, ref = 0, [], []
     for n in (23, 2, 1, 1, 1, 20, 1, 1):
         m.call(toks[:, at:at + n], at)
         at += n
-        check(m.last_logits(B), np.stack([w[at - 1] for w in want]), dtype, at)
+        got.append(m.last_logits(B))
+        ref.append(np.stack([w[at - 1] for w in want]))
+    check(np.concatenate(got), np.concatenate(ref), dtype)
 
 
 def test_state_goes_on_from_where_it_is_or_starts_anew():

@@ -27,12 +27,14 @@ struct LatentArgs {
   const float *rot, *norm_w, *sink;
   const T *uk, *uv;
   T* qt;        // [R][H][lq]
-  float* part;  // [R][H][ns][rank + 2]: maximum, sum, weighted latent
+  float* part;  // [R][H][ns][lat4] weighted latents of the slices (lat4: the latent rounded up to 4)
+  float2* stat;  // [R][H][ns] their maxima and sums
   T* ctx;       // expanded form: [B][T][ldc]
   const T* kv;  // [B][T][ldkv]: keys of all heads, then values
   T* out;
   const int32_t *pos, *seq;
-  int B, Sc, H, dim, rd, vd, rank, window, ldp, ldo, ldc, ldu, page, page_shift, pps, rot_pairs, rot_rows, ns, lq;
+  int B, Sc, H, dim, rd, vd, rank, window, ldp, ldo, ldc, ldu, page, page_shift, pps, rot_pairs, rot_rows, ns, lq, lat4;
+  int slice_round;  // slices are multiples of this many positions
   int T_ctx, T_prev, start, ldkv;
   int shift;  // tokens of this call ahead of its first row (a portion worked off in several passes)
   float eps, scale;
@@ -42,6 +44,8 @@ struct LatentArgs {
   __device__ __forceinline__ T* row(const int32_t* t, int p) const {
     return pool + ((size_t)t[(p >> page_shift) % pps] * page + (p & (page - 1))) * ldc;
   }
+  // positions per slice when a row sees n of them
+  __device__ __forceinline__ int slice(int n) const { return ((n + ns - 1) / ns + slice_round - 1) / slice_round * slice_round; }
   __device__ __forceinline__ int position(int r) const { return min(max(pos[r % B] + shift + r / B, 0), rot_rows - 1); }
 };
 
@@ -74,7 +78,6 @@ __device__ __forceinline__ void write_row(const LatentArgs<T>& a, int r, int lan
 
 template <typename T>
 __global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a, int R) {
-  pdl_launch();
   pdl_wait();
   const int w = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (w < R) {
@@ -88,11 +91,11 @@ __global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a
 }
 
 // ------------------------------------------------------------------------------------------------ absorbed form
-constexpr int LP_COLS = 64, LP_ROWS = 4;  // latent columns of a CTA, activation rows it serves with one read of the weights
+constexpr int LP_COLS = 64;  // latent columns of a CTA; it serves LP_ROWS activation rows with one read of the weights
 
 // Blocks 0 .. H * slices - 1: head and 64 latent columns of LP_ROWS rows; the last block along x writes those rows' cache
 // rows.  All warps run down W_uk together, each thread a 16-byte piece of a row.
-template <typename T>
+template <typename T, int LP_ROWS>
 __global__ void __launch_bounds__(256) latent_pre_kernel(const LatentArgs<T> a, int R) {
   constexpr int VEC = Elem<T>::VEC, TPR = LP_COLS / VEC, DR = 256 / TPR, AHEAD = 4;
   extern __shared__ float sq[];  // [LP_ROWS][dim]
@@ -180,8 +183,10 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
   const int r = blockIdx.x, h = blockIdx.y, p = a.position(r), L = a.lat();
   const int32_t* bt = a.bt + (size_t)a.seq[r % a.B] * a.pps;
   const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0, n = p + 1 - lo;
-  const int chunk = (n + a.ns - 1) / a.ns, t0 = lo + blockIdx.z * chunk, t1 = min(p + 1, t0 + chunk);
-  float* part = a.part + (((size_t)r * a.H + h) * a.ns + blockIdx.z) * (a.rank + 2);
+  const int chunk = a.slice(n), t0 = lo + blockIdx.z * chunk, t1 = min(p + 1, t0 + chunk);
+  if (t0 >= t1) return;  // nobody reads an empty slice
+  const size_t id = ((size_t)r * a.H + h) * a.ns + blockIdx.z;
+  float* part = a.part + id * a.lat4;
   for (int i = tid; i < L; i += LS_THREADS) sq[i] = to_f32(a.qt[((size_t)r * a.H + h) * a.lq + i]);
   float acc[NR], m = -INFINITY, l = 0.f;
 #pragma unroll
@@ -215,10 +220,10 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
         if (tid + k * LS_THREADS < a.rank) acc[k] = fmaf(e, to_f32(c[tid + k * LS_THREADS]), acc[k]);
     }
   }
-  if (tid == 0) { part[0] = m; part[1] = l; }
+  if (tid == 0) a.stat[id] = make_float2(m, l);
 #pragma unroll
   for (int k = 0; k < NR; k++)
-    if (tid + k * LS_THREADS < a.rank) part[2 + tid + k * LS_THREADS] = acc[k];
+    if (tid + k * LS_THREADS < a.lat4) part[tid + k * LS_THREADS] = acc[k];  // zeros past the latent
 }
 
 // ---- tensor cores (mma.sync m16n8k16, bf16 in, fp32 out)
@@ -243,6 +248,11 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 __device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
   return *reinterpret_cast<const uint32_t*>(&v);
+}
+__device__ __forceinline__ float ex2(float x) {  // 2^x by the hardware's approximation (2^-22 relative), 0 for -inf
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -270,16 +280,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
   const int p = a.position(r);
   const int32_t* bt = a.bt + (size_t)a.seq[r % a.B] * a.pps;
   const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0, n = p + 1 - lo;
-  const int chunk = ((n + a.ns - 1) / a.ns + LM_TILE - 1) / LM_TILE * LM_TILE, t0 = lo + z * chunk, t1 = min(p + 1, t0 + chunk);
-  const size_t pstride = a.rank + 2;
-  if (t0 >= t1) {  // an empty slice
-    if (tid < HR && h0 + tid < a.H) {
-      float* part = a.part + (((size_t)r * a.H + h0 + tid) * a.ns + z) * pstride;
-      part[0] = -INFINITY;
-      part[1] = 0.f;
-    }
-    return;
-  }
+  const int chunk = a.slice(n), t0 = lo + z * chunk, t1 = min(p + 1, t0 + chunk);
+  if (t0 >= t1) return;  // nobody reads an empty slice
   const int pieces = a.lq / 8, row_pieces = a.ldc / 8;
   for (int i = tid; i < HR * pieces; i += LM_THREADS) {
     const int h = i / pieces, c = i % pieces;
@@ -384,70 +386,65 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
     if (stages > 1) s ^= 1;
     else if (more) load_tile(base + LM_TILE, 0);
   }
-  if (tid < HR && h0 + tid < a.H) {
-    float* part = a.part + (((size_t)r * a.H + h0 + tid) * a.ns + z) * pstride;
-    part[0] = sM[tid];
-    part[1] = sL[tid];
-  }
+  if (tid < HR && h0 + tid < a.H) a.stat[((size_t)r * a.H + h0 + tid) * a.ns + z] = make_float2(sM[tid], sL[tid]);
 #pragma unroll
   for (int m = 0; m < MT; m++)
 #pragma unroll
     for (int j = 0; j < NTW; j++)
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
-        const int h = h0 + m * 16 + g + 8 * (i >> 1), c = (warp * NTW + j) * 8 + tq * 2 + (i & 1);
-        if (h < a.H && c < a.rank) a.part[(((size_t)r * a.H + h) * a.ns + z) * pstride + 2 + c] = o[m][j][i];
+      for (int i = 0; i < 2; i++) {
+        const int h = h0 + m * 16 + g + 8 * i, c = (warp * NTW + j) * 8 + tq * 2;
+        if (h < a.H && c < a.lat4) *reinterpret_cast<float2*>(a.part + (((size_t)r * a.H + h) * a.ns + z) * a.lat4 + c) = make_float2(o[m][j][2 * i], o[m][j][2 * i + 1]);
       }
 }
 
-// Slices and the sink -> the attended latent; then this CTA's LC_OUT values of the head, for LC_ROWS rows.
-constexpr int LC_OUT = 32, LC_ROWS = 4;
+// Slices and the sink -> the attended latent; then `outs` values of the head per CTA, for LC_ROWS rows.
+constexpr int LC_ROWS = 4;
 template <typename T>
-__global__ void __launch_bounds__(256) latent_combine_kernel(const LatentArgs<T> a, int R) {
+__global__ void __launch_bounds__(256) latent_combine_kernel(const LatentArgs<T> a, int R, int outs) {
   constexpr int VEC = Elem<T>::VEC;
-  extern __shared__ __align__(16) float so[];  // [LC_ROWS][ldu] attended latents
+  extern __shared__ __align__(16) float so[];  // [LC_ROWS][lds] attended latents
   __shared__ float wgt[LC_ROWS][LS_MAX_NS];
-  const int h = blockIdx.x, j0 = blockIdx.y * LC_OUT, r0 = blockIdx.z * LC_ROWS, nr = min(LC_ROWS, R - r0);
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  __shared__ int active[LC_ROWS];
+  const int h = blockIdx.x, j0 = blockIdx.y * outs, j1 = min(a.vd, j0 + outs), r0 = blockIdx.z * LC_ROWS, nr = min(LC_ROWS, R - r0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, lds = (a.ldu + 3) & ~3;
   pdl_launch();
   // parameters: this warp's rows of W_uv travel to L2 while the predecessor drains
-  for (int q = 0; q < LC_OUT / 8; q++) {
-    const int j = j0 + warp + 8 * q;
-    if (j < a.vd)
-      for (size_t off = (size_t)lane * 128; off < (size_t)a.ldu * sizeof(T); off += 32 * 128)
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.uv + ((size_t)h * a.vd + j) * a.ldu) + off));
-  }
+  for (int j = j0 + warp; j < j1; j += 8)
+    for (size_t off = (size_t)lane * 128; off < (size_t)a.ldu * sizeof(T); off += 32 * 128)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(a.uv + ((size_t)h * a.vd + j) * a.ldu) + off));
   pdl_wait();
-  const size_t ps = a.rank + 2;
   if (warp < nr) {
-    const float* part = a.part + ((size_t)(r0 + warp) * a.H + h) * a.ns * ps;
-    const float m = lane < a.ns ? part[lane * ps] : -INFINITY, l = lane < a.ns ? part[lane * ps + 1] : 0.f;
-    const float sink = a.sink[h], M = fmaxf(warp_max(m), sink), e = expf(m - M);
-    const float L = warp_sum(l * e) + expf(sink - M);
-    if (lane < a.ns) wgt[warp][lane] = e / L;
+    const int p = a.position(r0 + warp), n = a.window > 0 ? min(p + 1, a.window) : p + 1, chunk = a.slice(n), na = (n + chunk - 1) / chunk;
+    const float2 st = lane < na ? a.stat[((size_t)(r0 + warp) * a.H + h) * a.ns + lane] : make_float2(-INFINITY, 0.f);
+    const float sink = a.sink[h], M = fmaxf(warp_max(st.x), sink), e = expf(st.x - M);
+    const float L = warp_sum(st.y * e) + expf(sink - M);
+    wgt[warp][lane] = e / L;
+    if (lane == 0) active[warp] = na;
   }
   __syncthreads();
-  for (int i = tid; i < nr * a.ldu; i += 256) {
-    const int r = i / a.ldu, c = i % a.ldu;
-    float v = 0.f;
-    if (c < a.rank) {
-      const float* part = a.part + ((size_t)(r0 + r) * a.H + h) * a.ns * ps + 2 + c;
-#pragma unroll 4
-      for (int s = 0; s < a.ns; s++) {
+  for (int i = tid; i < nr * (lds / 4); i += 256) {
+    const int r = i / (lds / 4), c = i % (lds / 4) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < a.lat4) {
+      const float* part = a.part + ((size_t)(r0 + r) * a.H + h) * a.ns * a.lat4 + c;
+      const int na = active[r];
+#pragma unroll 8
+      for (int s = 0; s < na; s++) {
+        const float4 x = *reinterpret_cast<const float4*>(part + (size_t)s * a.lat4);
         const float w = wgt[r][s];
-        if (w != 0.f) v = fmaf(part[(size_t)s * ps], w, v);  // an empty slice has no latent to read
+        v.x = fmaf(x.x, w, v.x); v.y = fmaf(x.y, w, v.y); v.z = fmaf(x.z, w, v.z); v.w = fmaf(x.w, w, v.w);
       }
     }
-    so[i] = v;
+    *reinterpret_cast<float4*>(so + (size_t)r * lds + c) = v;  // what lies past the latent meets zeros of W_uv
   }
   __syncthreads();
-  for (int q = 0; q < LC_OUT / 8; q++) {
-    const int j = j0 + warp + 8 * q;
-    if (j >= a.vd) continue;
+  for (int j = j0 + warp; j < j1; j += 8) {
     const T* w = a.uv + ((size_t)h * a.vd + j) * a.ldu;
     float acc[LC_ROWS];
 #pragma unroll
     for (int r = 0; r < LC_ROWS; r++) acc[r] = 0.f;
+#pragma unroll 2
     for (int c = lane; c < a.ldu / VEC; c += 32) {
       float f[VEC];
       unpack_chunk(ld_128(w + (size_t)c * VEC), f);
@@ -455,7 +452,10 @@ __global__ void __launch_bounds__(256) latent_combine_kernel(const LatentArgs<T>
       for (int r = 0; r < LC_ROWS; r++)
         if (r < nr) {
 #pragma unroll
-          for (int k = 0; k < VEC; k++) acc[r] = fmaf(f[k], so[r * a.ldu + c * VEC + k], acc[r]);
+          for (int k = 0; k < VEC; k += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(so + (size_t)r * lds + c * VEC + k);
+            acc[r] = fmaf(f[k], x.x, acc[r]); acc[r] = fmaf(f[k + 1], x.y, acc[r]); acc[r] = fmaf(f[k + 2], x.z, acc[r]); acc[r] = fmaf(f[k + 3], x.w, acc[r]);
+          }
         }
     }
 #pragma unroll
@@ -480,26 +480,17 @@ __global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentAr
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, b = blockIdx.z;
   // the last tokens have the longest context: first
   const int q0 = (int)(gridDim.x - 1 - blockIdx.x) * LX_Q, nq = min(LX_Q, a.Sc - q0);
-  pdl_launch();
   pdl_wait();
-  const bf16 zero = __float2bfloat16_rn(0.f);
-  for (int i = tid; i < LX_Q * qkp; i += LX_THREADS) {
-    const int t = i / qkp, e = i % qkp;
-    bf16 v = zero;
-    if (t < nq && e < a.qk()) {
-      const bf16* q = a.proj + ((size_t)(q0 + t) * a.B + b) * a.ldp + (size_t)h * a.qk();
-      v = e < a.dim ? q[e] : from_f32<bf16>(rotated(q + a.dim, e - a.dim, a.rot + (size_t)(a.start + q0 + t) * a.rot_pairs * 2, a.rot_pairs));
-    }
-    sQ[(size_t)t * ldq + e] = v;
-  }
   // keys 0 .. T_ctx - 1 are positions start - T_prev ..; token q0 + t is key T_prev + q0 + t
   const int own = a.T_prev + q0, last = own + nq - 1;
   const int first = a.window > 0 ? max(0, own - a.window + 1) : 0;
   const int kp = a.dim / 8, rp = a.rd / 8, pad = (qkp - a.qk()) / 8, vp = a.vd / 8, per = kp + rp + pad + VT;
   auto load_tile = [&](int base, int s) {
     bf16 *tk = sK + (size_t)s * LX_KV * ldq, *tv = sV + (size_t)s * LX_KV * ldv;
-    for (int i = tid; i < LX_KV * per; i += LX_THREADS) {
-      const int k = i / per, c = i % per;
+    int k = tid / per, c = tid % per;
+    const int dk = LX_THREADS / per, dc = LX_THREADS % per;
+    for (; k < LX_KV; k += dk, c += dc) {
+      if (c >= per) { c -= per; k++; if (k >= LX_KV) break; }
       const size_t row = (size_t)b * a.T_ctx + base + k;
       const bool in = base + k <= last;
       bf16* d = c < kp + rp + pad ? tk + (size_t)k * ldq + c * 8 : tv + (size_t)k * ldv + (c - kp - rp - pad) * 8;
@@ -513,6 +504,30 @@ __global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentAr
     cp_commit();
   };
   load_tile(first, 0);
+  // queries: 16-byte pieces as they are, the first 2 * rot_pairs values behind the unrotated ones turned
+  {
+    const int qp = qkp / 8, turned = 2 * a.rot_pairs;
+    for (int i = tid; i < LX_Q * qp; i += LX_THREADS) {
+      const int t = i / qp, e = i % qp * 8;
+      bf16* d = sQ + (size_t)t * ldq + e;
+      if (t >= nq || e >= a.qk()) *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+      else if (e < a.dim || e >= a.dim + turned) *reinterpret_cast<uint4*>(d) = ld_128(a.proj + ((size_t)(q0 + t) * a.B + b) * a.ldp + (size_t)h * a.qk() + e);
+      else if (e + 8 > a.dim + turned) {  // a piece that turns in part
+        for (int k = 0; k < 8; k++)
+          if (e + k >= a.dim + turned) d[k] = a.proj[((size_t)(q0 + t) * a.B + b) * a.ldp + (size_t)h * a.qk() + e + k];
+      }
+    }
+#pragma unroll 4
+    for (int i = tid; i < nq * a.rot_pairs; i += LX_THREADS) {
+      const int t = i / a.rot_pairs, k = i % a.rot_pairs;
+      const bf16* q = a.proj + ((size_t)(q0 + t) * a.B + b) * a.ldp + (size_t)h * a.qk() + a.dim;
+      const float2 cs = *reinterpret_cast<const float2*>(a.rot + ((size_t)(a.start + q0 + t) * a.rot_pairs + k) * 2);
+      const float u = to_f32(q[k]), v = to_f32(q[k + a.rot_pairs]);
+      bf16* d = sQ + (size_t)t * ldq + a.dim + k;
+      d[0] = __float2bfloat16_rn(fmaf(u, cs.x, -v * cs.y));
+      d[a.rot_pairs] = __float2bfloat16_rn(fmaf(v, cs.x, u * cs.y));
+    }
+  }
   float o[VT][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
   for (int j = 0; j < VT; j++)
@@ -544,21 +559,32 @@ __global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentAr
       }
     }
     float mx[2] = {m[0], m[1]};
+    const int w0 = own + warp * 16;  // this warp's tokens are keys w0 .. w0 + 15
+    if (base + LX_KV - 1 <= w0 && (a.window <= 0 || w0 + 15 - base < a.window)) {  // every key of the tile is seen by all of them
 #pragma unroll
-    for (int j = 0; j < 8; j++)
+      for (int j = 0; j < 8; j++)
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
-        const int back = row0 + 8 * (i >> 1) - (base + j * 8 + tq * 2 + (i & 1));
-        sc[j][i] = (back >= 0 && (a.window <= 0 || back < a.window)) ? sc[j][i] * sl2 : -INFINITY;
-        mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
-      }
+        for (int i = 0; i < 4; i++) {
+          sc[j][i] *= sl2;
+          mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+        }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; j++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+          const int back = row0 + 8 * (i >> 1) - (base + j * 8 + tq * 2 + (i & 1));
+          sc[j][i] = (back >= 0 && (a.window <= 0 || back < a.window)) ? sc[j][i] * sl2 : -INFINITY;
+          mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+        }
+    }
     float al[2], mu[2];
 #pragma unroll
     for (int i = 0; i < 2; i++) {
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
       mu[i] = mx[i] == -INFINITY ? 0.f : mx[i];  // nothing seen yet: every weight below is exp2(-inf) = 0
-      al[i] = exp2f(m[i] - mu[i]);
+      al[i] = ex2(m[i] - mu[i]);
       m[i] = mx[i];
       l[i] *= al[i];
     }
@@ -568,7 +594,7 @@ __global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentAr
     for (int j = 0; j < 8; j++)
 #pragma unroll
       for (int i = 0; i < 4; i++) {
-        sc[j][i] = exp2f(sc[j][i] - mu[i >> 1]);
+        sc[j][i] = ex2(sc[j][i] - mu[i >> 1]);
         l[i >> 1] += sc[j][i];
       }
 #pragma unroll
@@ -585,6 +611,7 @@ __global__ void __launch_bounds__(LX_THREADS) latent_chunk_kernel(const LatentAr
     }
     __syncthreads();
   }
+  pdl_launch();
   const float sink = a.sink[h] * LOG2E;
 #pragma unroll
   for (int i = 0; i < 2; i++) {
@@ -649,7 +676,7 @@ JG_API int jg_latent_scratch_bytes(const jg_latent_desc* d, int32_t B, int32_t S
     if (RH > few) RH = few;
   }
   const uint64_t parts = RH > LATENT_MAX_PARTS ? RH : LATENT_MAX_PARTS;
-  const uint64_t narrow = 4 * (RH * (uint64_t)round32(d->kv_rank + d->rot_dim) + parts * (uint64_t)(d->kv_rank + 2)) + 256;
+  const uint64_t narrow = 4 * (RH * (uint64_t)round32(d->kv_rank + d->rot_dim) + parts * (uint64_t)(((d->kv_rank + 3) & ~3) + 2)) + 256;
   *out = narrow > wide ? narrow : wide;
   return JG_OK;
 }
@@ -680,6 +707,18 @@ static int launch_scores(jg_dev* dev, const LatentArgs<bf16>& a, int R, int mt, 
   return jg_launch(dev, "latent_split", latent_split_kernel<bf16>, dim3((unsigned)R, (unsigned)a.H, (unsigned)a.ns), dim3(LS_THREADS), (size_t)a.lat() * 4, a);
 }
 
+template <typename T, int ROWS>
+static int launch_pre(jg_dev* dev, const LatentArgs<T>& a, const jg_latent_desc* d, int R) {
+  auto kern = latent_pre_kernel<T, ROWS>;
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 2048 * ROWS * 4));
+    set[dev->ordinal & 7] = true;
+  }
+  const unsigned slices = (unsigned)((d->kv_rank + LP_COLS - 1) / LP_COLS);
+  return jg_launch(dev, "latent_pre", kern, dim3(d->heads * slices + 1, (unsigned)((R + ROWS - 1) / ROWS)), dim3(256), (size_t)ROWS * d->dim * 4, a, R);
+}
+
 template <typename T>
 static int run_absorbed(jg_dev* dev, LatentArgs<T> a, const jg_latent_desc* d) {
   const int R = a.B * a.Sc;
@@ -687,20 +726,20 @@ static int run_absorbed(jg_dev* dev, LatentArgs<T> a, const jg_latent_desc* d) {
   const int mt = mma_tiles(dev, d, &stages);
   a.lq = round32(d->kv_rank + d->rot_dim);
   a.ns = latent_splits(dev, d, R, mt ? 16 * mt : 1);
+  a.lat4 = (d->kv_rank + 3) & ~3;
+  a.slice_round = mt ? LM_TILE : 1;
   a.qt = (T*)d->scratch;
   a.part = (float*)(d->scratch + 4ull * R * d->heads * a.lq);
-  const unsigned slices = (unsigned)((d->kv_rank + LP_COLS - 1) / LP_COLS), rg = (unsigned)((R + LP_ROWS - 1) / LP_ROWS);
-  static bool set[8] = {};
-  if (!set[dev->ordinal & 7]) {
-    JG_CUDA(cudaFuncSetAttribute(latent_pre_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 4096 * LP_ROWS * 4));
-    set[dev->ordinal & 7] = true;
-  }
-  int rc = jg_launch(dev, "latent_pre", latent_pre_kernel<T>, dim3(d->heads * slices + 1, rg), dim3(256), (size_t)LP_ROWS * d->dim * 4, a, R);
+  a.stat = (float2*)(a.part + (size_t)R * d->heads * a.ns * a.lat4);
+  int rc = R == 1 ? launch_pre<T, 1>(dev, a, d, R) : (R <= 4 ? launch_pre<T, 4>(dev, a, d, R) : launch_pre<T, 8>(dev, a, d, R));
   if (rc) return rc;
   rc = launch_scores(dev, a, R, mt, stages);
   if (rc) return rc;
-  return jg_launch(dev, "latent_combine", latent_combine_kernel<T>, dim3((unsigned)d->heads, (unsigned)((d->vdim + LC_OUT - 1) / LC_OUT), (unsigned)((R + LC_ROWS - 1) / LC_ROWS)), dim3(256),
-                   (size_t)LC_ROWS * d->ld_u * 4, a, R);
+  const int rg = (R + LC_ROWS - 1) / LC_ROWS;
+  int outs = 32;  // as many CTAs as fill the machine, no more: each of them merges the slices anew
+  while (outs < d->vdim && (long long)rg * d->heads * ((d->vdim + 2 * outs - 1) / (2 * outs)) >= dev->sm_count) outs *= 2;
+  return jg_launch(dev, "latent_combine", latent_combine_kernel<T>, dim3((unsigned)d->heads, (unsigned)((d->vdim + outs - 1) / outs), (unsigned)rg), dim3(256),
+                   (size_t)LC_ROWS * ((d->ld_u + 3) & ~3) * 4, a, R, outs);
 }
 
 template <int VT>

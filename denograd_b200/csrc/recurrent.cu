@@ -17,8 +17,7 @@ template <typename T>
 __global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
                                                                     const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
   __shared__ float s_a[MG_WARPS][32], s_b[MG_WARPS][32], s_carry[2][32];
-  pdl_launch();
-  pdl_wait();
+  pdl_wait();  // no early trigger: the next kernel's CTAs would sit on this one's SMs for its whole length
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, b = blockIdx.y, ch = blockIdx.x * 32 + lane;
   const bool ok = ch < width;
   float* st = state + (size_t)seq[b] * width + ch;
@@ -63,6 +62,7 @@ __global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __r
     par ^= 1;
     __syncthreads();
   }
+  pdl_launch();
   if (warp == 0 && ok) *st = s_carry[par][lane];
 }
 
@@ -150,32 +150,88 @@ __device__ __forceinline__ float2 delta_gates(const DeltaArgs<T>& a, size_t row,
 }
 constexpr float DELTA_UNIT_EPS = 1e-6f;
 
-// Portions, step 1, one CTA per row: convolutions, unit vectors and gates into scratch.
-template <typename T>
+// Portions, step 1: convolutions, unit vectors and gates into scratch.  A warp takes one q or k head, or a run of value
+// channels, and walks DP_TOK consecutive tokens of a sequence with the taps and the last inputs in registers; the last unit
+// is the gates.  NI * 32 channels per unit; TAPS = 0: any number of taps, inputs read again for every token.
+constexpr int DP_TOK = 16;
+template <typename T, int NI, int TAPS>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs<T> a) {
-  extern __shared__ __align__(16) float buf[];
-  pdl_launch();
+  constexpr int KEEP = TAPS > 0 ? TAPS : 1;
   pdl_wait();
-  const int r = blockIdx.x, b = r % a.B, s = r / a.B, C = a.channels(), p0 = a.pos[b];
-  const T* tail = a.tail + (size_t)a.seq[b] * a.taps * C;
-  const int nqk = 2 * a.G * a.dim;
-  float* dv = a.v + (size_t)r * a.H * a.vd;
-#pragma unroll 2
-  for (int c = threadIdx.x; c < C; c += 256) {
-    const float v = delta_conv_silu(a, b, s, c, p0, tail);
-    if (c < nqk) buf[c] = v;
-    else dv[c - nqk] = v;
+  const int lane = threadIdx.x & 31, C = a.channels(), nqk = 2 * a.G * a.dim, run = NI * 32;
+  const int n_units = 2 * a.G + (a.H * a.vd + run - 1) / run + 1, unit = blockIdx.x * 8 + (threadIdx.x >> 5), b = blockIdx.z;
+  const int s0 = blockIdx.y * DP_TOK, s1 = min(a.Sc, s0 + DP_TOK), p0 = a.pos[b];
+  if (unit >= n_units) return;
+  if (unit == n_units - 1) {
+    for (int i = lane; i < (s1 - s0) * a.H; i += 32) {
+      const size_t r = (size_t)(s0 + i / a.H) * a.B + b;
+      *reinterpret_cast<float2*>(a.gates + (r * a.H + i % a.H) * 2) = delta_gates(a, r, i % a.H);
+    }
+    return;
   }
-  for (int h = threadIdx.x; h < a.H; h += 256) *reinterpret_cast<float2*>(a.gates + ((size_t)r * a.H + h) * 2) = delta_gates(a, r, h);
-  __syncthreads();
-  const int lane = threadIdx.x & 31;
-  for (int g = threadIdx.x >> 5; g < 2 * a.G; g += 8) {  // q heads, then k heads
-    const float* x = buf + g * a.dim;
-    float ss = 0.f;
-    for (int i = lane; i < a.dim; i += 32) ss = fmaf(x[i], x[i], ss);
-    const float rs = 1.0f / sqrtf(warp_sum(ss) + DELTA_UNIT_EPS) * (g < a.G ? 1.0f / sqrtf((float)a.dim) : 1.0f);
-    float* dst = a.qk + (((size_t)r * a.G + (g < a.G ? g : g - a.G)) * 2 + (g < a.G ? 0 : 1)) * a.lds;
-    for (int i = lane; i < a.lds; i += 32) dst[i] = i < a.dim ? x[i] * rs : 0.f;
+  const bool head = unit < 2 * a.G;  // q heads, then k heads, then value channels
+  const int c0 = head ? unit * a.dim : nqk + (unit - 2 * a.G) * run, n = head ? a.dim : min(run, C - c0);
+  const T* tail = a.tail + (size_t)a.seq[b] * a.taps * C;
+  auto input = [&](int s, int c) -> float {  // token s of this call, or one before it
+    if (s >= 0) return to_f32(a.proj[((size_t)s * a.B + b) * a.ldp + c]);
+    return p0 + s >= 0 ? to_f32(tail[(size_t)((p0 + s) % a.taps) * C + c]) : 0.f;
+  };
+  float w[NI][KEEP], x[NI][KEEP];  // x[i][KEEP - 1]: the newest input
+  if (TAPS > 0) {
+#pragma unroll
+    for (int i = 0; i < NI; i++)
+#pragma unroll
+      for (int j = 0; j < KEEP; j++) {
+        const bool in = i * 32 + lane < n;
+        w[i][j] = in ? a.conv_w[(size_t)(c0 + i * 32 + lane) * a.taps + j] : 0.f;
+        x[i][j] = in && j > 0 ? input(s0 - KEEP + j, c0 + i * 32 + lane) : 0.f;
+      }
+  }
+  T ahead[NI];
+  auto fetch = [&](int s) {
+#pragma unroll
+    for (int i = 0; i < NI; i++)
+      if (s < s1 && i * 32 + lane < n) ahead[i] = a.proj[((size_t)s * a.B + b) * a.ldp + c0 + i * 32 + lane];
+  };
+  if (TAPS > 0) fetch(s0);
+  const float unit_scale = head && unit < a.G ? 1.0f / sqrtf((float)a.dim) : 1.0f;
+  for (int s = s0; s < s1; s++) {
+    float y[NI], ss = 0.f;
+    if (TAPS > 0) {
+#pragma unroll
+      for (int i = 0; i < NI; i++) {
+#pragma unroll
+        for (int j = 0; j + 1 < KEEP; j++) x[i][j] = x[i][j + 1];
+        x[i][KEEP - 1] = i * 32 + lane < n ? to_f32(ahead[i]) : 0.f;
+      }
+      fetch(s + 1);
+    }
+#pragma unroll
+    for (int i = 0; i < NI; i++) {
+      float acc = 0.f;
+      if (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < KEEP; j++) acc = fmaf(w[i][j], x[i][j], acc);
+      } else if (i * 32 + lane < n) {
+        const int c = c0 + i * 32 + lane;
+        for (int j = 0; j < a.taps; j++) acc = fmaf(a.conv_w[(size_t)c * a.taps + j], input(s - (a.taps - 1 - j), c), acc);
+      }
+      y[i] = silu_f32(acc);
+      ss = fmaf(y[i], y[i], ss);
+    }
+    const size_t r = (size_t)s * a.B + b;
+    if (head) {
+      const float rs = unit_scale / sqrtf(warp_sum(ss) + DELTA_UNIT_EPS);
+      float* dst = a.qk + ((r * a.G + (unit < a.G ? unit : unit - a.G)) * 2 + (unit < a.G ? 0 : 1)) * a.lds;
+#pragma unroll
+      for (int i = 0; i < NI; i++)
+        if (i * 32 + lane < a.lds) dst[i * 32 + lane] = i * 32 + lane < n ? y[i] * rs : 0.f;
+    } else {
+      float* dst = a.v + r * a.H * a.vd + c0 - nqk;
+#pragma unroll
+      for (int i = 0; i < NI; i++)
+        if (i * 32 + lane < n) dst[i * 32 + lane] = y[i];
+    }
   }
 }
 
@@ -234,7 +290,11 @@ struct DeltaCol {
 //   S   = D S_0 + sum_j k_j w_j^T
 // so that the reductions over the lanes of a column overlap instead of following one another.  Blocks of DS_TOK tokens are
 // staged by cp.async, one ahead; the products k_j . k_i and k_j . q_i of a block are worked out by all threads first.
-constexpr int DS_LPC = 8, DS_COLS = 16, DS_THREADS = DS_LPC * DS_COLS, DS_TOK = 16, DS_STEP = 4, DS_PAIRS = DS_STEP * DS_STEP;
+// A lane holds E elements of each of four columns (so that a loaded piece of k or q serves four), 16 lanes a group of
+// four columns; the partial sums are exchanged so that each lane ends up with one column's, solves that one, and hands the
+// updates back to the group.
+constexpr int DL_LPC = 8;  // lanes per column of the decode kernel below
+constexpr int DS_LPC = 16, DS_NC = 4, DS_THREADS = 128, DS_COLS = DS_THREADS / DS_LPC * DS_NC, DS_TOK = 16, DS_STEP = 4, DS_PAIRS = DS_STEP * DS_STEP;
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
@@ -268,14 +328,14 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<
   extern __shared__ __align__(16) unsigned char dsm[];
   Stage* stages = reinterpret_cast<Stage*>(dsm);
   __shared__ __align__(16) float pairs[DS_TOK / DS_STEP][2][DS_PAIRS];  // [group][k.k | k.q][i * DS_STEP + j]
-  pdl_launch();
-  const int tid = threadIdx.x, l = tid % DS_LPC, col = tid / DS_LPC, h = blockIdx.y, b = blockIdx.z;
-  const int j0 = blockIdx.x * DS_COLS, j = j0 + col, g = h / (a.H / a.G), C = a.channels();
+  constexpr int V = E < 4 ? 2 : 4;  // elements of a lane's contiguous pieces
+  const int tid = threadIdx.x, l = tid % DS_LPC, h = blockIdx.y, b = blockIdx.z;
+  // columns of the CTA: j0 ..; of this lane's group: jc .. jc + 3; the one this lane solves: j0 + col
+  const int j0 = blockIdx.x * DS_COLS, jc = j0 + tid / DS_LPC * DS_NC, col = tid / DS_LPC * DS_NC + (l >> 2), g = h / (a.H / a.G), C = a.channels();
   for (int i = tid; i < (int)(2 * sizeof(Stage) / 4); i += DS_THREADS) reinterpret_cast<float*>(dsm)[i] = 0.f;  // padding, columns past vd
   __syncthreads();
   pdl_wait();
   const int slot = a.seq[b];
-  const bool live = j < a.vd;
   const int c4 = a.lds / 4;
   auto stage_block = [&](int t0, Stage& st) {
     const int nt = min(DS_TOK, a.Sc - t0);
@@ -296,12 +356,18 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   stage_block(0, stages[0]);
-  float* stp = a.state + (((size_t)slot * a.H + h) * a.vd + (live ? j : 0)) * a.lds;
-  DeltaCol<DS_LPC, E> col_s;
-  col_s.load(stp, l, a.lds, live && a.pos[b] > 0);
-  float2 S[E / 2];
+  // chunk e of a lane: V elements from (l + DS_LPC * e) * V on
+  const bool cont = a.pos[b] > 0;
+  float2 S[DS_NC][E / 2];
 #pragma unroll
-  for (int i = 0; i < E / 2; i++) S[i] = make_float2(col_s.s[2 * i], col_s.s[2 * i + 1]);
+  for (int c = 0; c < DS_NC; c++) {
+    const float* sp = a.state + (((size_t)slot * a.H + h) * a.vd + min(jc + c, a.vd - 1)) * a.lds;
+#pragma unroll
+    for (int e = 0; e < E / 2; e++) {
+      const int off = (l + DS_LPC * (2 * e / V)) * V + 2 * e % V;
+      S[c][e] = (cont && jc + c < a.vd && off < a.lds) ? *reinterpret_cast<const float2*>(sp + off) : make_float2(0.f, 0.f);
+    }
+  }
 
   int buf = 0;
   for (int t0 = 0; t0 < a.Sc; t0 += DS_TOK, buf ^= 1) {
@@ -332,29 +398,56 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<
     __syncthreads();
     for (int grp = 0; grp < DS_TOK / DS_STEP; grp++) {
       const int tb = grp * DS_STEP;
-      float sk[DS_STEP], sq[DS_STEP];
+      float sk[DS_NC][DS_STEP], sq[DS_NC][DS_STEP];
+      float2 kr[DS_STEP][E / 2];
 #pragma unroll
       for (int i = 0; i < DS_STEP; i++) {
-        float2 ak = make_float2(0.f, 0.f), aq = make_float2(0.f, 0.f);
+        float2 qr[E / 2];
 #pragma unroll
-        for (int e = 0; e < E / 4; e++) {
-          const float4 kv = *reinterpret_cast<const float4*>(&st.k[tb + i][(l + DS_LPC * e) * 4]), qv = *reinterpret_cast<const float4*>(&st.q[tb + i][(l + DS_LPC * e) * 4]);
-          ak = fma2(S[2 * e], make_float2(kv.x, kv.y), ak); ak = fma2(S[2 * e + 1], make_float2(kv.z, kv.w), ak);
-          aq = fma2(S[2 * e], make_float2(qv.x, qv.y), aq); aq = fma2(S[2 * e + 1], make_float2(qv.z, qv.w), aq);
+        for (int e = 0; e < E / V; e++) {
+          const float *kp = &st.k[tb + i][(l + DS_LPC * e) * V], *qp = &st.q[tb + i][(l + DS_LPC * e) * V];
+          if constexpr (V == 4) {
+            const float4 kv = *reinterpret_cast<const float4*>(kp), qv = *reinterpret_cast<const float4*>(qp);
+            kr[i][2 * e] = make_float2(kv.x, kv.y); kr[i][2 * e + 1] = make_float2(kv.z, kv.w);
+            qr[2 * e] = make_float2(qv.x, qv.y); qr[2 * e + 1] = make_float2(qv.z, qv.w);
+          } else {
+            kr[i][e] = *reinterpret_cast<const float2*>(kp);
+            qr[e] = *reinterpret_cast<const float2*>(qp);
+          }
         }
-        sk[i] = ak.x + ak.y;
-        sq[i] = aq.x + aq.y;
+#pragma unroll
+        for (int c = 0; c < DS_NC; c++) {
+          float2 ak = make_float2(0.f, 0.f), aq = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int e = 0; e < E / 2; e++) { ak = fma2(S[c][e], kr[i][e], ak); aq = fma2(S[c][e], qr[e], aq); }
+          sk[c][i] = ak.x + ak.y;
+          sq[c][i] = aq.x + aq.y;
+        }
+      }
+      // exchange: lanes with bit 3 keep columns 2 and 3, then those with bit 2 the upper of their two; then all-reduce over 4
+      const bool up8 = l & 8, up4 = l & 4;
+      float mk[DS_STEP], mq[DS_STEP];
+#pragma unroll
+      for (int i = 0; i < DS_STEP; i++) {
+        float k2[2], q2[2];
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+          k2[c] = (up8 ? sk[c + 2][i] : sk[c][i]) + __shfl_xor_sync(0xffffffffu, up8 ? sk[c][i] : sk[c + 2][i], 8);
+          q2[c] = (up8 ? sq[c + 2][i] : sq[c][i]) + __shfl_xor_sync(0xffffffffu, up8 ? sq[c][i] : sq[c + 2][i], 8);
+        }
+        mk[i] = (up4 ? k2[1] : k2[0]) + __shfl_xor_sync(0xffffffffu, up4 ? k2[0] : k2[1], 4);
+        mq[i] = (up4 ? q2[1] : q2[0]) + __shfl_xor_sync(0xffffffffu, up4 ? q2[0] : q2[1], 4);
       }
 #pragma unroll
-      for (int o = DS_LPC / 2; o > 0; o >>= 1)
+      for (int o = 2; o > 0; o >>= 1)
 #pragma unroll
-        for (int i = 0; i < DS_STEP; i++) { sk[i] += __shfl_xor_sync(0xffffffffu, sk[i], o); sq[i] += __shfl_xor_sync(0xffffffffu, sq[i], o); }
+        for (int i = 0; i < DS_STEP; i++) { mk[i] += __shfl_xor_sync(0xffffffffu, mk[i], o); mq[i] += __shfl_xor_sync(0xffffffffu, mq[i], o); }
       float w[DS_STEP], D = 1.f, mine = 0.f;
 #pragma unroll
       for (int i = 0; i < DS_STEP; i++) {
         const float2 gt = *reinterpret_cast<const float2*>(st.gate[tb + i]);
         D *= gt.x;
-        float pre = D * sk[i], o = D * sq[i];
+        float pre = D * mk[i], o = D * mq[i];
 #pragma unroll
         for (int jj = 0; jj < i; jj++) {
           w[jj] *= gt.x;
@@ -363,29 +456,37 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<
         }
         w[i] = gt.y * (st.v[tb + i][col] - pre);
         o = fmaf(pairs[grp][1][i * DS_STEP + i], w[i], o);
-        if (l == i) mine = o;
+        if ((l & 3) == i) mine = o;
       }
       const float2 D2 = make_float2(D, D);
 #pragma unroll
-      for (int e = 0; e < E / 2; e++) S[e] = mul2(S[e], D2);
+      for (int c = 0; c < DS_NC; c++) {
 #pragma unroll
-      for (int i = 0; i < DS_STEP; i++) {
-        const float2 w2 = make_float2(w[i], w[i]);
+        for (int e = 0; e < E / 2; e++) S[c][e] = mul2(S[c][e], D2);
 #pragma unroll
-        for (int e = 0; e < E / 4; e++) {
-          const float4 kv = *reinterpret_cast<const float4*>(&st.k[tb + i][(l + DS_LPC * e) * 4]);
-          S[2 * e] = fma2(make_float2(kv.x, kv.y), w2, S[2 * e]);
-          S[2 * e + 1] = fma2(make_float2(kv.z, kv.w), w2, S[2 * e + 1]);
+        for (int i = 0; i < DS_STEP; i++) {
+          const float wc = __shfl_sync(0xffffffffu, w[i], c * 4, DS_LPC);
+          const float2 w2 = make_float2(wc, wc);
+#pragma unroll
+          for (int e = 0; e < E / 2; e++) S[c][e] = fma2(kr[i][e], w2, S[c][e]);
         }
       }
-      const int t = t0 + tb + l;
-      if (l < DS_STEP && live && t < a.Sc) a.o[((size_t)t * a.B + b) * a.H * a.vd + (size_t)h * a.vd + j] = mine;
+      const int t = t0 + tb + (l & 3);
+      if (j0 + col < a.vd && t < a.Sc) a.o[((size_t)t * a.B + b) * a.H * a.vd + (size_t)h * a.vd + j0 + col] = mine;
     }
     __syncthreads();  // the other stage is refilled next, and `pairs` is rewritten
   }
+  pdl_launch();
 #pragma unroll
-  for (int i = 0; i < E / 2; i++) { col_s.s[2 * i] = S[i].x; col_s.s[2 * i + 1] = S[i].y; }
-  if (live) col_s.store(stp, l, a.lds);
+  for (int c = 0; c < DS_NC; c++) {
+    if (jc + c >= a.vd) continue;
+    float* sp = a.state + (((size_t)slot * a.H + h) * a.vd + jc + c) * a.lds;
+#pragma unroll
+    for (int e = 0; e < E / 2; e++) {
+      const int off = (l + DS_LPC * (2 * e / V)) * V + 2 * e % V;
+      if (off < a.lds) *reinterpret_cast<float2*>(sp + off) = S[c][e];
+    }
+  }
   // the convolution's last inputs: entry position % taps, which no row of this call reads any more
   T* tail = a.tail + (size_t)slot * a.taps * C;
   const int cta = blockIdx.y * gridDim.x + blockIdx.x, ctas = gridDim.x * gridDim.y, keep = min(a.taps - 1, a.Sc);
@@ -398,7 +499,6 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs<
 // Portions, step 3, one warp per (row, head): norm over the value dimension, norm weight, output gate.
 template <typename T>
 __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs<T> a, int R) {
-  pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -414,17 +514,17 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs<T> a, in
 
 // One token per row, everything in one launch: a cluster of CTAs shares a (row, head), each CTA takes a run of columns of
 // S; the sum of squares of the output norm crosses through distributed shared memory.
-constexpr int DD_THREADS = 256, DD_COLS = DD_THREADS / DS_LPC, DD_MAX_CLUSTER = 8;
+constexpr int DD_THREADS = 256, DD_COLS = DD_THREADS / DL_LPC, DD_MAX_CLUSTER = 8;
 
 template <typename T, int E>
 __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<T> a) {
-  constexpr int DP = E * DS_LPC;
+  constexpr int DP = E * DL_LPC;
   extern __shared__ __align__(16) float dyn[];  // this CTA's columns: v, then o
   __shared__ __align__(16) float sk[DP], sq[DP];
   __shared__ float red[3][DD_THREADS / 32], s_ss[DD_MAX_CLUSTER];
   cg::cluster_group cluster = cg::this_cluster();
   const int cr = (int)cluster.block_rank(), cs = (int)cluster.num_blocks();
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, l = tid % DS_LPC, col = tid / DS_LPC, h = blockIdx.y, r = blockIdx.z;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, l = tid % DL_LPC, col = tid / DL_LPC, h = blockIdx.y, r = blockIdx.z;
   const int g = h / (a.H / a.G), C = a.channels();
   const int per = (a.vd + cs - 1) / cs, j0 = min(a.vd, cr * per), j1 = min(a.vd, j0 + per);
   asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // every CTA of the cluster has started ...
@@ -435,7 +535,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<
   T* tail_now = tail + (size_t)(p0 % a.taps) * C;  // no CTA reads this entry: it holds position p0 - taps
   const T* row = a.proj + (size_t)r * a.ldp;
   // the first columns of the state are requested before the convolutions
-  DeltaCol<DS_LPC, E> S;
+  DeltaCol<DL_LPC, E> S;
   float* st0 = a.state + ((size_t)slot * a.H + h) * a.vd * a.lds;
   S.load(st0 + (size_t)min(j0 + col, a.vd - 1) * a.lds, l, a.lds, p0 > 0);
   float qv = 0.f, kv = 0.f, pq = 0.f, pk = 0.f, pqk = 0.f;
@@ -467,8 +567,8 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<
   float4 k4[E / 4], q4[E / 4];
 #pragma unroll
   for (int i = 0; i < E / 4; i++) {
-    k4[i] = *reinterpret_cast<const float4*>(&sk[(l + DS_LPC * i) * 4]);
-    q4[i] = *reinterpret_cast<const float4*>(&sq[(l + DS_LPC * i) * 4]);
+    k4[i] = *reinterpret_cast<const float4*>(&sk[(l + DL_LPC * i) * 4]);
+    q4[i] = *reinterpret_cast<const float4*>(&sq[(l + DL_LPC * i) * 4]);
     k4[i].x *= rk; k4[i].y *= rk; k4[i].z *= rk; k4[i].w *= rk;
     q4[i].x *= rq; q4[i].y *= rq; q4[i].z *= rq; q4[i].w *= rq;
   }
@@ -477,7 +577,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaArgs<
     const int j = jb + col;
     const bool live = j < j1;
     float* st = st0 + (size_t)(live ? j : j0) * a.lds;
-    DeltaCol<DS_LPC, E> next;
+    DeltaCol<DL_LPC, E> next;
     if (jb + DD_COLS < j1) next.load(st0 + (size_t)min(j + DD_COLS, j1 - 1) * a.lds, l, a.lds, p0 > 0);
     const float o = S.step(k4, q4, live ? dyn[j - j0] : 0.f, gt.x, gt.y, tqk * rq * rk);
     if (live) {
@@ -513,22 +613,18 @@ JG_API int jg_delta_scratch_floats(const jg_delta_desc* d, int32_t rows, uint64_
   return JG_OK;
 }
 
-template <typename T, int E>
+template <typename T, int DP>  // DP: head size rounded up to 32, 64, 128 or 256
 static int delta_launch(jg_dev* dev, const DeltaArgs<T>& a) {
   const int R = a.B * a.Sc;
   if (a.Sc == 1) {
     int cs = 1;
     while (cs < DD_MAX_CLUSTER && cs * DD_COLS < a.vd && R * a.H * cs < 2 * dev->sm_count) cs *= 2;
     const size_t smem = (size_t)((a.vd + cs - 1) / cs) * sizeof(float);
-    return jg_launch_cluster(dev, "delta_step", delta_step_kernel<T, E>, dim3((unsigned)cs, (unsigned)a.H, (unsigned)R), dim3(DD_THREADS), smem, cs, a);
+    return jg_launch_cluster(dev, "delta_step", delta_step_kernel<T, DP / DL_LPC>, dim3((unsigned)cs, (unsigned)a.H, (unsigned)R), dim3(DD_THREADS), smem, cs, a);
   }
-  const size_t smem = (size_t)2 * a.G * a.dim * sizeof(float);
-  static bool set[8] = {};
-  if (!set[dev->ordinal & 7]) {
-    JG_CUDA(cudaFuncSetAttribute(delta_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dev->prop.sharedMemPerBlockOptin - 1024));
-    set[dev->ordinal & 7] = true;
-  }
-  int rc = jg_launch(dev, "delta_prep", delta_prep_kernel<T>, dim3((unsigned)R), dim3(256), smem, a);
+  constexpr int E = DP / DS_LPC, NI = DP <= 128 ? 4 : 8;
+  const dim3 pg((unsigned)((2 * a.G + (a.H * a.vd + NI * 32 - 1) / (NI * 32) + 1 + 7) / 8), (unsigned)((a.Sc + DP_TOK - 1) / DP_TOK), (unsigned)a.B);
+  int rc = a.taps == 4 ? jg_launch(dev, "delta_prep", delta_prep_kernel<T, NI, 4>, pg, dim3(256), 0, a) : jg_launch(dev, "delta_prep", delta_prep_kernel<T, NI, 0>, pg, dim3(256), 0, a);
   if (rc) return rc;
   static bool scan_set[8] = {};
   if (!scan_set[dev->ordinal & 7]) {
@@ -554,10 +650,10 @@ static int delta_run(jg_dev* dev, const jg_batch* b, const jg_delta_desc* d) {
   a.gates = a.qk + R * d->kv_heads * 2 * a.lds;
   a.v = a.gates + R * d->heads * 2;
   a.o = a.v + R * d->heads * d->vdim;
-  if (d->dim <= 32) return delta_launch<T, 4>(dev, a);
-  if (d->dim <= 64) return delta_launch<T, 8>(dev, a);
-  if (d->dim <= 128) return delta_launch<T, 16>(dev, a);
-  if (d->dim <= 256) return delta_launch<T, 32>(dev, a);
+  if (d->dim <= 32) return delta_launch<T, 32>(dev, a);
+  if (d->dim <= 64) return delta_launch<T, 64>(dev, a);
+  if (d->dim <= 128) return delta_launch<T, 128>(dev, a);
+  if (d->dim <= 256) return delta_launch<T, 256>(dev, a);
   jg_set_error("delta_rule: query / key heads of %d values (largest supported: 256)", d->dim);
   return JG_ENOTSUP;
 }

@@ -90,6 +90,36 @@ __global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a
   }
 }
 
+// ---- tensor cores (mma.sync m16n8k16, bf16 in, fp32 out)
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+__device__ __forceinline__ float ex2(float x) {  // 2^x by the hardware's approximation (2^-22 relative), 0 for -inf
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+
 // ------------------------------------------------------------------------------------------------ absorbed form
 constexpr int LP_COLS = 64;  // latent columns of a CTA; it serves LP_ROWS activation rows with one read of the weights
 
@@ -169,6 +199,63 @@ __global__ void __launch_bounds__(256) latent_pre_kernel(const LatentArgs<T> a, 
   }
 }
 
+// The same for up to 16 rows on the tensor cores (bf16, three rows and more): [16 rows][dim] x [dim][64 latent columns].
+constexpr int LPM_ROWS = 16, LPM_THREADS = 128;
+static constexpr size_t lpm_smem(int dp) { return (size_t)2 * (dp * (LP_COLS + 8) + LPM_ROWS * (dp + 8)); }
+
+__global__ void __launch_bounds__(LPM_THREADS) latent_pre_mma_kernel(const LatentArgs<bf16> a, int R, int dp) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  bf16 *sW = reinterpret_cast<bf16*>(smem), *sQ = sW + (size_t)dp * (LP_COLS + 8);  // dp: dim rounded up to 16
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r0 = blockIdx.y * LPM_ROWS, nr = min(LPM_ROWS, R - r0);
+  pdl_launch();
+  if (blockIdx.x == gridDim.x - 1) {
+    pdl_wait();
+    for (int r = warp; r < nr; r += LPM_THREADS / 32) write_row(a, r0 + r, lane, (bf16*)nullptr);
+    return;
+  }
+  const int slices = (a.rank + LP_COLS - 1) / LP_COLS, h = blockIdx.x / slices, c0 = (blockIdx.x % slices) * LP_COLS;
+  for (int i = tid; i < dp * (LP_COLS / 8); i += LPM_THREADS) {  // parameters: ahead of the dependency wait
+    const int d = i / (LP_COLS / 8), c = i % (LP_COLS / 8) * 8;
+    bf16* dst = sW + (size_t)d * (LP_COLS + 8) + c;
+    if (d < a.dim && c0 + c < a.ldu) cp16(dst, a.uk + ((size_t)h * a.dim + d) * a.ldu + c0 + c);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+  }
+  cp_commit();
+  pdl_wait();
+#pragma unroll 4
+  for (int i = tid; i < LPM_ROWS * dp; i += LPM_THREADS) {
+    const int r = i / dp, d = i % dp;
+    sQ[(size_t)r * (dp + 8) + d] = (r < nr && d < a.dim) ? a.proj[(size_t)(r0 + r) * a.ldp + (size_t)h * a.qk() + d] : __float2bfloat16_rn(0.f);
+  }
+  cp_wait<0>();
+  __syncthreads();
+  float acc[2][4] = {};
+  for (int k = 0; k < dp; k += 16) {
+    uint32_t q[4], w[4];
+    ldsm4(q, sQ + (size_t)(lane & 15) * (dp + 8) + k + (lane >> 4) * 8);
+    ldsm4t(w, sW + (size_t)(k + (lane & 15)) * (LP_COLS + 8) + warp * 16 + (lane >> 4) * 8);
+    mma_bf16(acc[0], q, w[0], w[1]);
+    mma_bf16(acc[1], q, w[2], w[3]);
+  }
+  const int g = lane >> 2, tq = lane & 3;
+#pragma unroll
+  for (int j = 0; j < 2; j++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int r = g + 8 * (i >> 1), c = c0 + warp * 16 + j * 8 + tq * 2 + (i & 1);
+      if (r < nr && c < a.rank) a.qt[((size_t)(r0 + r) * a.H + h) * a.lq + c] = __float2bfloat16_rn(acc[j][i]);
+    }
+  if (c0 == 0) {
+    const int n = a.lq - a.rank;
+    for (int i = tid; i < nr * n; i += LPM_THREADS) {
+      const int r = i / n, e = i % n;
+      const float* cs = a.rot + (size_t)a.position(r0 + r) * a.rot_pairs * 2;
+      const bf16* q = a.proj + (size_t)(r0 + r) * a.ldp + (size_t)h * a.qk() + a.dim;
+      a.qt[((size_t)(r0 + r) * a.H + h) * a.lq + a.rank + e] = from_f32<bf16>(e < a.rd ? rotated(q, e, cs, a.rot_pairs) : 0.f);
+    }
+  }
+}
+
 constexpr int LS_THREADS = 128, LS_TILE = 64, LS_MAX_RANK = 1024, LS_MAX_NS = 32;
 
 template <typename T>
@@ -225,36 +312,6 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
   for (int k = 0; k < NR; k++)
     if (tid + k * LS_THREADS < a.lat4) part[tid + k * LS_THREADS] = acc[k];  // zeros past the latent
 }
-
-// ---- tensor cores (mma.sync m16n8k16, bf16 in, fp32 out)
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(void* smem, const void* gmem) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-__device__ __forceinline__ float ex2(float x) {  // 2^x by the hardware's approximation (2^-22 relative), 0 for -inf
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-constexpr float LOG2E = 1.4426950408889634f;
 
 // One row, 16 * MT heads, one context slice: tiles of 64 cached rows; warp w scores 8 of them for all heads, two warps'
 // worth of heads get their softmax statistics per warp, and each warp owns NTW * 8 columns of the weighted latent.
@@ -464,6 +521,80 @@ __global__ void __launch_bounds__(256) latent_combine_kernel(const LatentArgs<T>
       if (lane == 0 && r < nr) a.out[(size_t)(r0 + r) * a.ldo + (size_t)h * a.vd + j] = from_f32<T>(v);
     }
   }
+}
+
+// The same for up to 16 rows on the tensor cores: the merged latents [16][rank], rounded to bf16, x W_uv of `LCM_OUT` values.
+constexpr int LCM_ROWS = 16, LCM_OUT = 64, LCM_THREADS = 256;
+static constexpr size_t lcm_smem(int rp) { return (size_t)2 * (LCM_ROWS + LCM_OUT) * (rp + 8); }
+
+__global__ void __launch_bounds__(LCM_THREADS) latent_combine_mma_kernel(const LatentArgs<bf16> a, int R, int rp) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  bf16 *sW = reinterpret_cast<bf16*>(smem), *sO = sW + (size_t)LCM_OUT * (rp + 8);  // rp: rank rounded up to 16
+  __shared__ float wgt[LCM_ROWS][LS_MAX_NS];
+  __shared__ int active[LCM_ROWS];
+  __shared__ float red[4][2][32][4];
+  const int h = blockIdx.x, j0 = blockIdx.y * LCM_OUT, r0 = blockIdx.z * LCM_ROWS, nr = min(LCM_ROWS, R - r0);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  pdl_launch();
+  for (int i = tid; i < LCM_OUT * (rp / 8); i += LCM_THREADS) {  // parameters: ahead of the dependency wait
+    const int j = i / (rp / 8), c = i % (rp / 8) * 8;
+    bf16* dst = sW + (size_t)j * (rp + 8) + c;
+    if (j0 + j < a.vd && c < a.ldu) cp16(dst, a.uv + ((size_t)h * a.vd + j0 + j) * a.ldu + c);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+  }
+  cp_commit();
+  pdl_wait();
+  for (int r = warp; r < nr; r += LCM_THREADS / 32) {
+    const int p = a.position(r0 + r), n = a.window > 0 ? min(p + 1, a.window) : p + 1, chunk = a.slice(n), na = (n + chunk - 1) / chunk;
+    const float2 st = lane < na ? a.stat[((size_t)(r0 + r) * a.H + h) * a.ns + lane] : make_float2(-INFINITY, 0.f);
+    const float sink = a.sink[h], M = fmaxf(warp_max(st.x), sink), e = expf(st.x - M);
+    const float L = warp_sum(st.y * e) + expf(sink - M);
+    wgt[r][lane] = e / L;
+    if (lane == 0) active[r] = na;
+  }
+  __syncthreads();
+  for (int i = tid; i < LCM_ROWS * (rp / 4); i += LCM_THREADS) {
+    const int r = i / (rp / 4), c = i % (rp / 4) * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r < nr && c < a.lat4) {
+      const float* part = a.part + ((size_t)(r0 + r) * a.H + h) * a.ns * a.lat4 + c;
+      const int na = active[r];
+#pragma unroll 8
+      for (int s = 0; s < na; s++) {
+        const float4 x = *reinterpret_cast<const float4*>(part + (size_t)s * a.lat4);
+        const float w = wgt[r][s];
+        v.x = fmaf(x.x, w, v.x); v.y = fmaf(x.y, w, v.y); v.z = fmaf(x.z, w, v.z); v.w = fmaf(x.w, w, v.w);
+      }
+    }
+    *reinterpret_cast<uint2*>(sO + (size_t)r * (rp + 8) + c) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+  }
+  cp_wait<0>();
+  __syncthreads();
+  // warps 0-3 take 16 values each over the first half of the latent, warps 4-7 over the second
+  const int cg = warp & 3, half = warp >> 2, kh = (rp / 32) * 16, k0 = half ? kh : 0, k1 = half ? rp : kh;
+  float acc[2][4] = {};
+  for (int k = k0; k < k1; k += 16) {
+    uint32_t o[4], w[4];
+    ldsm4(o, sO + (size_t)(lane & 15) * (rp + 8) + k + (lane >> 4) * 8);
+    ldsm4(w, sW + (size_t)(cg * 16 + (lane >> 4) * 8 + (lane & 7)) * (rp + 8) + k + ((lane >> 3) & 1) * 8);
+    mma_bf16(acc[0], o, w[0], w[1]);
+    mma_bf16(acc[1], o, w[2], w[3]);
+  }
+  if (half)
+#pragma unroll
+    for (int j = 0; j < 2; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) red[cg][j][lane][i] = acc[j][i];
+  __syncthreads();
+  if (half) return;
+  const int g = lane >> 2, tq = lane & 3;
+#pragma unroll
+  for (int j = 0; j < 2; j++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int r = g + 8 * (i >> 1), c = j0 + cg * 16 + j * 8 + tq * 2 + (i & 1);
+      if (r < nr && c < a.vd) a.out[(size_t)(r0 + r) * a.ldo + (size_t)h * a.vd + c] = __float2bfloat16_rn(acc[j][i] + red[cg][j][lane][i]);
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ expanded form
@@ -719,6 +850,30 @@ static int launch_pre(jg_dev* dev, const LatentArgs<T>& a, const jg_latent_desc*
   return jg_launch(dev, "latent_pre", kern, dim3(d->heads * slices + 1, (unsigned)((R + ROWS - 1) / ROWS)), dim3(256), (size_t)ROWS * d->dim * 4, a, R);
 }
 
+// Three rows and more in bf16: all three stages on the tensor cores; 1 = not this call.
+static int launch_rows(jg_dev*, const LatentArgs<float>&, const jg_latent_desc*, int, int, int) { return 1; }
+static int launch_rows(jg_dev* dev, const LatentArgs<bf16>& a0, const jg_latent_desc* d, int R, int mt, int stages) {
+  const int dp = (d->dim + 15) & ~15, rp = (d->kv_rank + 15) & ~15;
+  const size_t limit = (size_t)dev->prop.sharedMemPerBlockOptin - 8192;
+  if (R < 3 || mt == 0 || lpm_smem(dp) > limit || lcm_smem(rp) > limit) return 1;
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    if (cudaFuncSetAttribute(latent_pre_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit) != cudaSuccess ||
+        cudaFuncSetAttribute(latent_combine_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit) != cudaSuccess)
+      return jg_cuda_fail(cudaGetLastError(), "latent_pre_mma attributes", __FILE__, __LINE__);
+    set[dev->ordinal & 7] = true;
+  }
+  LatentArgs<bf16> a = a0;
+  a.slice_round = 2 * LM_TILE;  // fewer slices to merge
+  const unsigned slices = (unsigned)((d->kv_rank + LP_COLS - 1) / LP_COLS);
+  int rc = jg_launch(dev, "latent_pre_mma", latent_pre_mma_kernel, dim3(d->heads * slices + 1, (unsigned)((R + LPM_ROWS - 1) / LPM_ROWS)), dim3(LPM_THREADS), lpm_smem(dp), a, R, dp);
+  if (rc) return rc;
+  rc = launch_scores(dev, a, R, mt, stages);
+  if (rc) return rc;
+  return jg_launch(dev, "latent_combine_mma", latent_combine_mma_kernel, dim3((unsigned)d->heads, (unsigned)((d->vdim + LCM_OUT - 1) / LCM_OUT), (unsigned)((R + LCM_ROWS - 1) / LCM_ROWS)),
+                   dim3(LCM_THREADS), lcm_smem(rp), a, R, rp);
+}
+
 template <typename T>
 static int run_absorbed(jg_dev* dev, LatentArgs<T> a, const jg_latent_desc* d) {
   const int R = a.B * a.Sc;
@@ -731,7 +886,9 @@ static int run_absorbed(jg_dev* dev, LatentArgs<T> a, const jg_latent_desc* d) {
   a.qt = (T*)d->scratch;
   a.part = (float*)(d->scratch + 4ull * R * d->heads * a.lq);
   a.stat = (float2*)(a.part + (size_t)R * d->heads * a.ns * a.lat4);
-  int rc = R == 1 ? launch_pre<T, 1>(dev, a, d, R) : (R <= 4 ? launch_pre<T, 4>(dev, a, d, R) : launch_pre<T, 8>(dev, a, d, R));
+  int rc = launch_rows(dev, a, d, R, mt, stages);
+  if (rc != 1) return rc;
+  rc = R == 1 ? launch_pre<T, 1>(dev, a, d, R) : (R <= 4 ? launch_pre<T, 4>(dev, a, d, R) : launch_pre<T, 8>(dev, a, d, R));
   if (rc) return rc;
   rc = launch_scores(dev, a, R, mt, stages);
   if (rc) return rc;

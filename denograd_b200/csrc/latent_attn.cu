@@ -208,9 +208,10 @@ __global__ void __launch_bounds__(LPM_THREADS) latent_pre_mma_kernel(const Laten
   bf16 *sW = reinterpret_cast<bf16*>(smem), *sQ = sW + (size_t)dp * (LP_COLS + 8);  // dp: dim rounded up to 16
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r0 = blockIdx.y * LPM_ROWS, nr = min(LPM_ROWS, R - r0);
   pdl_launch();
-  if (blockIdx.x == gridDim.x - 1) {
+  if (blockIdx.x >= gridDim.x - LPM_ROWS / 4) {  // the last blocks write the cache rows, one per warp
+    const int r = (int)(blockIdx.x - (gridDim.x - LPM_ROWS / 4)) * 4 + warp;
     pdl_wait();
-    for (int r = warp; r < nr; r += LPM_THREADS / 32) write_row(a, r0 + r, lane, (bf16*)nullptr);
+    if (r < nr) write_row(a, r0 + r, lane, (bf16*)nullptr);
     return;
   }
   const int slices = (a.rank + LP_COLS - 1) / LP_COLS, h = blockIdx.x / slices, c0 = (blockIdx.x % slices) * LP_COLS;
@@ -222,10 +223,12 @@ __global__ void __launch_bounds__(LPM_THREADS) latent_pre_mma_kernel(const Laten
   }
   cp_commit();
   pdl_wait();
+#pragma unroll
+  for (int k = 0; k < LPM_ROWS / 4; k++) {
+    const int r = k * 4 + warp;
+    const bf16* src = a.proj + (size_t)(r0 + min(r, nr - 1)) * a.ldp + (size_t)h * a.qk();
 #pragma unroll 4
-  for (int i = tid; i < LPM_ROWS * dp; i += LPM_THREADS) {
-    const int r = i / dp, d = i % dp;
-    sQ[(size_t)r * (dp + 8) + d] = (r < nr && d < a.dim) ? a.proj[(size_t)(r0 + r) * a.ldp + (size_t)h * a.qk() + d] : __float2bfloat16_rn(0.f);
+    for (int d = lane; d < dp; d += 32) sQ[(size_t)r * (dp + 8) + d] = (r < nr && d < a.dim) ? src[d] : __float2bfloat16_rn(0.f);
   }
   cp_wait<0>();
   __syncthreads();
@@ -340,19 +343,29 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
   const int chunk = a.slice(n), t0 = lo + z * chunk, t1 = min(p + 1, t0 + chunk);
   if (t0 >= t1) return;  // nobody reads an empty slice
   const int pieces = a.lq / 8, row_pieces = a.ldc / 8;
-  for (int i = tid; i < HR * pieces; i += LM_THREADS) {
-    const int h = i / pieces, c = i % pieces;
-    bf16* d = sQ + (size_t)h * ld + c * 8;
-    if (h0 + h < a.H) cp16(d, a.qt + ((size_t)r * a.H + h0 + h) * a.lq + c * 8);
-    else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+#pragma unroll
+  for (int k = 0; k < HR / 8; k++) {  // a warp takes whole rows: one address calculation each
+    const int h = k * 8 + warp;
+    const bf16* src = a.qt + ((size_t)r * a.H + min(h0 + h, a.H - 1)) * a.lq;
+    for (int c = lane; c < pieces; c += 32) {
+      bf16* d = sQ + (size_t)h * ld + c * 8;
+      if (h0 + h < a.H) cp16(d, src + c * 8);
+      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    }
   }
   auto load_tile = [&](int base, int s) {
     bf16* t = tiles + (size_t)s * LM_TILE * ld;
-    for (int i = tid; i < LM_TILE * pieces; i += LM_THREADS) {
-      const int k = i / pieces, c = i % pieces;
-      bf16* d = t + (size_t)k * ld + c * 8;
-      if (base + k < t1 && c < row_pieces) cp16(d, a.row(bt, base + k) + c * 8);
-      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    const bf16* src[LM_TILE / 8];
+#pragma unroll
+    for (int k = 0; k < LM_TILE / 8; k++) src[k] = a.row(bt, min(base + k * 8 + warp, t1 - 1));
+#pragma unroll
+    for (int k = 0; k < LM_TILE / 8; k++) {
+      const bool in = base + k * 8 + warp < t1;
+      bf16* d = t + (size_t)(k * 8 + warp) * ld;
+      for (int c = lane; c < pieces; c += 32) {
+        if (in && c < row_pieces) cp16(d + c * 8, src[k] + c * 8);
+        else *reinterpret_cast<uint4*>(d + c * 8) = make_uint4(0, 0, 0, 0);
+      }
     }
     cp_commit();
   };
@@ -400,17 +413,43 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
         sS[(m * 16 + g + 8 * (i >> 1)) * LM_TILE + c] = base + c < t1 ? sc[m][i] * a.scale : -INFINITY;
       }
     __syncthreads();
-    for (int row = warp; row < HR; row += 8) {
-      const float x0 = sS[row * LM_TILE + lane], x1 = sS[row * LM_TILE + lane + 32], old = sM[row];
-      const float m = fmaxf(old, warp_max(fmaxf(x0, x1)));
-      const float e0 = expf(x0 - m), e1 = expf(x1 - m), sum = warp_sum(e0 + e1);
-      sP[row * (LM_TILE + 8) + lane] = __float2bfloat16_rn(e0);
-      sP[row * (LM_TILE + 8) + lane + 32] = __float2bfloat16_rn(e1);
-      if (lane == 0) {
-        const float al = expf(old - m);
-        sA[row] = al;
-        sL[row] = fmaf(sL[row], al, sum);
-        sM[row] = m;
+    {  // the warp's heads side by side: their reductions overlap
+      constexpr int NH = HR / 8;
+      float x0[NH], x1[NH], old[NH], mx[NH], sum[NH];
+#pragma unroll
+      for (int k = 0; k < NH; k++) {
+        const int row = k * 8 + warp;
+        x0[k] = sS[row * LM_TILE + lane];
+        x1[k] = sS[row * LM_TILE + lane + 32];
+        old[k] = sM[row];
+        mx[k] = fmaxf(x0[k], x1[k]);
+      }
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1)
+#pragma unroll
+        for (int k = 0; k < NH; k++) mx[k] = fmaxf(mx[k], __shfl_xor_sync(0xffffffffu, mx[k], w));
+#pragma unroll
+      for (int k = 0; k < NH; k++) {
+        mx[k] = fmaxf(mx[k], old[k]);
+        x0[k] = expf(x0[k] - mx[k]);
+        x1[k] = expf(x1[k] - mx[k]);
+        sum[k] = x0[k] + x1[k];
+      }
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1)
+#pragma unroll
+        for (int k = 0; k < NH; k++) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], w);
+#pragma unroll
+      for (int k = 0; k < NH; k++) {
+        const int row = k * 8 + warp;
+        sP[row * (LM_TILE + 8) + lane] = __float2bfloat16_rn(x0[k]);
+        sP[row * (LM_TILE + 8) + lane + 32] = __float2bfloat16_rn(x1[k]);
+        if (lane == 0) {
+          const float al = expf(old[k] - mx[k]);
+          sA[row] = al;
+          sL[row] = fmaf(sL[row], al, sum[k]);
+          sM[row] = mx[k];
+        }
       }
     }
     __syncthreads();
@@ -536,12 +575,12 @@ __global__ void __launch_bounds__(LCM_THREADS) latent_combine_mma_kernel(const L
   const int h = blockIdx.x, j0 = blockIdx.y * LCM_OUT, r0 = blockIdx.z * LCM_ROWS, nr = min(LCM_ROWS, R - r0);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   pdl_launch();
-  for (int i = tid; i < LCM_OUT * (rp / 8); i += LCM_THREADS) {  // parameters: ahead of the dependency wait
-    const int j = i / (rp / 8), c = i % (rp / 8) * 8;
-    bf16* dst = sW + (size_t)j * (rp + 8) + c;
-    if (j0 + j < a.vd && c < a.ldu) cp16(dst, a.uv + ((size_t)h * a.vd + j0 + j) * a.ldu + c);
-    else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-  }
+  for (int j = warp; j < LCM_OUT; j += LCM_THREADS / 32)  // parameters: ahead of the dependency wait
+    for (int c = lane * 8; c < rp; c += 256) {
+      bf16* dst = sW + (size_t)j * (rp + 8) + c;
+      if (j0 + j < a.vd && c < a.ldu) cp16(dst, a.uv + ((size_t)h * a.vd + j0 + j) * a.ldu + c);
+      else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    }
   cp_commit();
   pdl_wait();
   for (int r = warp; r < nr; r += LCM_THREADS / 32) {
@@ -553,20 +592,31 @@ __global__ void __launch_bounds__(LCM_THREADS) latent_combine_mma_kernel(const L
     if (lane == 0) active[r] = na;
   }
   __syncthreads();
-  for (int i = tid; i < LCM_ROWS * (rp / 4); i += LCM_THREADS) {
-    const int r = i / (rp / 4), c = i % (rp / 4) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < nr && c < a.lat4) {
-      const float* part = a.part + ((size_t)(r0 + r) * a.H + h) * a.ns * a.lat4 + c;
-      const int na = active[r];
-#pragma unroll 8
+  for (int r = warp; r < LCM_ROWS; r += LCM_THREADS / 32) {
+    const int na = r < nr ? active[r] : 0;
+    const float* part = a.part + ((size_t)(r0 + min(r, nr - 1)) * a.H + h) * a.ns * a.lat4;
+    for (int c0 = 0; c0 < rp; c0 += 512) {  // four pieces of a row per lane: their loads overlap
+      float4 v[4];
+#pragma unroll
+      for (int k = 0; k < 4; k++) v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
       for (int s = 0; s < na; s++) {
-        const float4 x = *reinterpret_cast<const float4*>(part + (size_t)s * a.lat4);
         const float w = wgt[r][s];
-        v.x = fmaf(x.x, w, v.x); v.y = fmaf(x.y, w, v.y); v.z = fmaf(x.z, w, v.z); v.w = fmaf(x.w, w, v.w);
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+          const int c = c0 + k * 128 + lane * 4;
+          if (c < a.lat4) {
+            const float4 x = *reinterpret_cast<const float4*>(part + (size_t)s * a.lat4 + c);
+            v[k].x = fmaf(x.x, w, v[k].x); v[k].y = fmaf(x.y, w, v[k].y); v[k].z = fmaf(x.z, w, v[k].z); v[k].w = fmaf(x.w, w, v[k].w);
+          }
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 4; k++) {
+        const int c = c0 + k * 128 + lane * 4;
+        if (c < rp) *reinterpret_cast<uint2*>(sO + (size_t)r * (rp + 8) + c) = make_uint2(pack_bf16(v[k].x, v[k].y), pack_bf16(v[k].z, v[k].w));
       }
     }
-    *reinterpret_cast<uint2*>(sO + (size_t)r * (rp + 8) + c) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
   }
   cp_wait<0>();
   __syncthreads();
@@ -866,7 +916,7 @@ static int launch_rows(jg_dev* dev, const LatentArgs<bf16>& a0, const jg_latent_
   LatentArgs<bf16> a = a0;
   a.slice_round = 2 * LM_TILE;  // fewer slices to merge
   const unsigned slices = (unsigned)((d->kv_rank + LP_COLS - 1) / LP_COLS);
-  int rc = jg_launch(dev, "latent_pre_mma", latent_pre_mma_kernel, dim3(d->heads * slices + 1, (unsigned)((R + LPM_ROWS - 1) / LPM_ROWS)), dim3(LPM_THREADS), lpm_smem(dp), a, R, dp);
+  int rc = jg_launch(dev, "latent_pre_mma", latent_pre_mma_kernel, dim3(d->heads * slices + LPM_ROWS / 4, (unsigned)((R + LPM_ROWS - 1) / LPM_ROWS)), dim3(LPM_THREADS), lpm_smem(dp), a, R, dp);
   if (rc) return rc;
   rc = launch_scores(dev, a, R, mt, stages);
   if (rc) return rc;

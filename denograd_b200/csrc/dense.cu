@@ -367,13 +367,15 @@ static int launch_stream(jg_dev* dev, const StreamArgs& st, T* h, int ldh, int R
 }
 
 template <typename T>
-__global__ void stream_embed_kernel(float* __restrict__ out, const int32_t* __restrict__ tokens, const T* __restrict__ table, int n, int dim, int ld, int vocab) {
+__global__ void __launch_bounds__(256) stream_embed_kernel(float* __restrict__ out, const int32_t* __restrict__ tokens, const T* __restrict__ table, int dim, int ld, int vocab) {
   pdl_launch();
   pdl_wait();
-  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < (long long)n * dim; i += (long long)gridDim.x * blockDim.x) {
-    const int r = (int)(i / dim), c = (int)(i % dim), tok = tokens[r];
-    out[i] = (tok >= 0 && tok < vocab) ? to_f32(table[(size_t)tok * ld + c]) : 0.f;  // an id outside the table reads as zeros
-  }
+  const int tok = tokens[blockIdx.x];
+  const T* row = table + (size_t)(tok >= 0 && tok < vocab ? tok : 0) * ld;
+  const bool in = tok >= 0 && tok < vocab;  // an id outside the table reads as zeros
+  float* o = out + (size_t)blockIdx.x * dim;
+#pragma unroll 4
+  for (int c = threadIdx.x; c < dim; c += 256) o[c] = in ? to_f32(row[c]) : 0.f;
 }
 
 // ------------------------------------------------------------------------------------------------ dispatch
@@ -440,12 +442,10 @@ JG_API int jg_stream_embed(jg_dev* dev, const jg_batch* b, uint64_t out, uint64_
   if (rc) return rc;
   JG_REQUIRE(dim > 0 && ld >= dim && vocab > 0 && (dtype == JG_F32 || dtype == JG_BF16), "stream_embed: bad shape");
   JG_REQUIRE(jg_aligned(out, 4) && jg_aligned(tokens, 4) && table != 0, "stream_embed: null or misaligned pointer");
-  const int n = b->B * b->Sc;
-  long long blocks = ((long long)n * dim + 255) / 256;
-  if (blocks > dev->sm_count * 8) blocks = dev->sm_count * 8;
+  const dim3 grid((unsigned)(b->B * b->Sc));
   if (dtype == JG_F32)
-    return jg_launch(dev, "stream_embed", stream_embed_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, (float*)out, (const int32_t*)tokens, (const float*)table, n, dim, ld, vocab);
-  return jg_launch(dev, "stream_embed", stream_embed_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, (float*)out, (const int32_t*)tokens, (const bf16*)table, n, dim, ld, vocab);
+    return jg_launch(dev, "stream_embed", stream_embed_kernel<float>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const float*)table, dim, ld, vocab);
+  return jg_launch(dev, "stream_embed", stream_embed_kernel<bf16>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const bf16*)table, dim, ld, vocab);
 }
 
 JG_API int jg_stream_norm(jg_dev* dev, const jg_batch* b, const jg_stream_desc* s, uint64_t h, int32_t ldh, int32_t dtype) {

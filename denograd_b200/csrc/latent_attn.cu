@@ -58,22 +58,37 @@ __device__ __forceinline__ float rotated(const T* x, int i, const float* cs, int
   return i < pairs ? fmaf(u, c, -v * s) : fmaf(v, c, u * s);
 }
 
-// Cache row of the new token in row r, by one warp; `copy` (or null) receives it too.
+// Cache row of the new token in row r, by one warp; `copy` (or null) receives it too.  Up to 512 latent values stay in
+// registers between the norm and the store, their loads all in flight at once.
 template <typename T>
 __device__ __forceinline__ void write_row(const LatentArgs<T>& a, int r, int lane, T* copy) {
+  constexpr int KEEP = 16;
   const int b = r % a.B, p = a.pos[b] + a.shift + r / a.B;
-  if (p < 0 || p >= a.rot_rows) return;  // outside the tables: left alone
   const T* c = a.proj + (size_t)r * a.ldp + a.H * a.qk();
-  T* dst = a.row(a.bt + (size_t)a.seq[b] * a.pps, p);
-  float ss = 0.f;
-  for (int i = lane; i < a.rank; i += 32) { const float v = to_f32(c[i]); ss = fmaf(v, v, ss); }
-  const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)a.rank + a.eps);
-  const float* cs = a.rot + (size_t)p * a.rot_pairs * 2;
-  for (int i = lane; i < a.ldc; i += 32) {
-    const T v = from_f32<T>(i < a.rank ? to_f32(c[i]) * rs * a.norm_w[i] : (i < a.lat() ? rotated(c + a.rank, i - a.rank, cs, a.rot_pairs) : 0.f));
-    dst[i] = v;
-    if (copy) copy[i] = v;
+  float v[KEEP], w[KEEP], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; k++) {
+    const int i = lane + 32 * k;
+    v[k] = i < a.rank ? to_f32(c[i]) : 0.f;
+    w[k] = i < a.rank ? a.norm_w[i] : 0.f;
   }
+#pragma unroll
+  for (int k = 0; k < KEEP; k++) ss = fmaf(v[k], v[k], ss);
+  for (int i = lane + 32 * KEEP; i < a.rank; i += 32) { const float x = to_f32(c[i]); ss = fmaf(x, x, ss); }
+  const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)a.rank + a.eps);
+  if (p < 0 || p >= a.rot_rows) return;  // outside the tables: left alone
+  T* dst = a.row(a.bt + (size_t)a.seq[b] * a.pps, p);
+  auto put = [&](int i, float x) {
+    const T t = from_f32<T>(x);
+    dst[i] = t;
+    if (copy) copy[i] = t;
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; k++)
+    if (lane + 32 * k < a.rank) put(lane + 32 * k, v[k] * rs * w[k]);
+  for (int i = lane + 32 * KEEP; i < a.rank; i += 32) put(i, to_f32(c[i]) * rs * a.norm_w[i]);
+  const float* cs = a.rot + (size_t)p * a.rot_pairs * 2;
+  for (int i = lane; i < a.ldc - a.rank; i += 32) put(a.rank + i, i < a.rd ? rotated(c + a.rank, i, cs, a.rot_pairs) : 0.f);
 }
 
 template <typename T>

@@ -10,19 +10,19 @@ namespace cg = cooperative_groups;
 // ------------------------------------------------------------------------------------------------ minGRU
 // S_t = (1 - z_t) S_{t-1} + z_t c_t is, per channel, an affine map of the state; maps compose, so a portion is scanned in
 // blocks of MG_WARPS x MG_TOK tokens: warp w composes its MG_TOK consecutive tokens, the warps' maps meet in shared
-// memory, and each warp replays its tokens from the state its predecessors leave.  One CTA = 32 channels of a sequence.
+// memory, warp 0 runs through them, and each warp replays its tokens from the state its predecessors leave.  One CTA = 32
+// channels of a sequence.
 constexpr int MG_WARPS = 32, MG_TOK = 4, MG_THREADS = 32 * MG_WARPS;
 
 template <typename T>
 __global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
                                                                     const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
-  __shared__ float s_a[MG_WARPS][32], s_b[MG_WARPS][32], s_carry[2][32];
+  __shared__ float s_a[MG_WARPS][32], s_b[MG_WARPS][32], s_in[MG_WARPS][32];
   pdl_wait();  // no early trigger: the next kernel's CTAs would sit on this one's SMs for its whole length
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, b = blockIdx.y, ch = blockIdx.x * 32 + lane;
   const bool ok = ch < width;
   float* st = state + (size_t)seq[b] * width + ch;
-  if (warp == 0) s_carry[0][lane] = (ok && pos[b] > 0) ? *st : 0.f;
-  int par = 0;
+  float carry = (warp == 0 && ok && pos[b] > 0) ? *st : 0.f;  // warp 0: the state ahead of the block
   T nz[MG_TOK], nc[MG_TOK], ng[MG_TOK];  // the next block's inputs travel while this one is worked on
   auto fetch = [&](int t0) {
 #pragma unroll
@@ -50,20 +50,24 @@ __global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __r
     s_a[warp][lane] = A;
     s_b[warp][lane] = Bc;
     __syncthreads();
-    float s = s_carry[par][lane];
-    for (int w = 0; w < warp; w++) s = fmaf(s_a[w][lane], s, s_b[w][lane]);
-    if (warp == MG_WARPS - 1) s_carry[par ^ 1][lane] = fmaf(A, s, Bc);
+    if (warp == 0) {
+#pragma unroll 8
+      for (int w = 0; w < MG_WARPS; w++) {
+        s_in[w][lane] = carry;
+        carry = fmaf(s_a[w][lane], carry, s_b[w][lane]);
+      }
+    }
+    __syncthreads();
+    float s = s_in[warp][lane];
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
       const int t = t0 + warp * MG_TOK + i;
       s = fmaf(1.0f - z[i], s, c[i]);
       if (ok && t < Sc) out[((size_t)t * B + b) * ldo + ch] = from_f32<T>(s * silu_f32(g[i]));
     }
-    par ^= 1;
-    __syncthreads();
   }
   pdl_launch();
-  if (warp == 0 && ok) *st = s_carry[par][lane];
+  if (warp == 0 && ok) *st = carry;
 }
 
 // One token per sequence: one thread per channel.

@@ -186,16 +186,13 @@ static int launch_dt(jg_dev* dev, const DenseCall& c, const DtArgs& a) {
     JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
     attr_set[dev->ordinal & 7] = true;
   }
-  const CUtensorMap* p;
-  int rc = jg_tensor_map(&p, c.w[0], c.N, c.K, c.ldw, DT_BM, "weights", 2, true);
+  CUtensorMap tw0, tw1, tx;
+  int rc = jg_tensor_map(&tw0, c.w[0], c.N, c.K, c.ldw, DT_BM, "weights", 2, true);
   if (rc) return rc;
-  const CUtensorMap tw0 = *p;
-  rc = jg_tensor_map(&p, c.w[GLU ? 1 : 0], c.N, c.K, c.ldw, DT_BM, "weights (second matrix)", 2, true);
+  rc = jg_tensor_map(&tw1, c.w[GLU ? 1 : 0], c.N, c.K, c.ldw, DT_BM, "weights (second matrix)", 2, true);
   if (rc) return rc;
-  const CUtensorMap tw1 = *p;
-  rc = jg_tensor_map(&p, c.x, c.M, c.K, c.ldx, TN, "activations", 2, true);
+  rc = jg_tensor_map(&tx, c.x, c.M, c.K, c.ldx, TN, "activations", 2, true);
   if (rc) return rc;
-  const CUtensorMap tx = *p;
   const int n_ft = (c.N + DT_BM - 1) / DT_BM, n_tt = (c.M + TN - 1) / TN, tiles = n_ft * n_tt, n_kb = (c.K + DT_BK - 1) / DT_BK;
   int ks = 1;
   if (c.M > 128) {  // the split with the smallest waves x (k-blocks at the tensor peak + fixed cost) estimate, as in gemm_tc.cu

@@ -466,7 +466,7 @@ __global__ void __launch_bounds__(Tc2Cfg<EPI>::THREADS) gemm_tc_pair_kernel(cons
 }
 
 // ------------------------------------------------------------------------------------------------ host side
-static int cached_map(const CUtensorMap** out, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, const char* what, int bytes = 2) {
+static int cached_map(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint32_t box_rows, const char* what, int bytes = 2) {
   return jg_tensor_map(out, base, rows, cols, cols, box_rows, what, bytes);
 }
 
@@ -480,14 +480,13 @@ static int launch_tc(jg_dev* dev, const void* x, const void* w0, const void* w1,
     JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
     attr_set[slot] = true;
   }
-  const CUtensorMap *pw0, *pw1, *px;
-  int rc = cached_map(&pw0, w0, a.N, a.K, TC_BM, "weights", W8 ? 1 : 2);
+  CUtensorMap tw0, tw1, tx;
+  int rc = cached_map(&tw0, w0, a.N, a.K, TC_BM, "weights", W8 ? 1 : 2);
   if (rc) return rc;
-  rc = cached_map(&pw1, Cfg::NW == 2 ? w1 : w0, a.N, a.K, TC_BM, "weights (second matrix)", W8 ? 1 : 2);
+  rc = cached_map(&tw1, Cfg::NW == 2 ? w1 : w0, a.N, a.K, TC_BM, "weights (second matrix)", W8 ? 1 : 2);
   if (rc) return rc;
-  rc = cached_map(&px, x, a.M, a.K, TN, "activations");
+  rc = cached_map(&tx, x, a.M, a.K, TN, "activations");
   if (rc) return rc;
-  const CUtensorMap tw0 = *pw0, tw1 = *pw1, tx = *px;
   // up to 128 rows (weight streaming): split K over a cluster until the launch has CTAs for about two thirds of the
   // SMs, keeping at least 8 k-blocks per CTA and the peers' partial sums within rank 0's pipeline buffers
   const int tiles = ((a.M + TN - 1) / TN) * (a.N / TC_BM), n_kb = a.K / TC_BK;
@@ -554,14 +553,13 @@ static int launch_tc_pair(jg_dev* dev, const void* x, const void* w0, const void
     JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
     attr_set[slot] = true;
   }
-  const CUtensorMap *pw0, *pw1, *px;
-  int rc = cached_map(&pw0, w0, a.N, a.K, TC_BM, "weights");
+  CUtensorMap tw0, tw1, tx;
+  int rc = cached_map(&tw0, w0, a.N, a.K, TC_BM, "weights");
   if (rc) return rc;
-  rc = cached_map(&pw1, Cfg::NW == 2 ? w1 : w0, a.N, a.K, TC_BM, "weights (second matrix)");
+  rc = cached_map(&tw1, Cfg::NW == 2 ? w1 : w0, a.N, a.K, TC_BM, "weights (second matrix)");
   if (rc) return rc;
-  rc = cached_map(&px, x, a.M, a.K, Cfg::TN / 2, "activations (half tile)");
+  rc = cached_map(&tx, x, a.M, a.K, Cfg::TN / 2, "activations (half tile)");
   if (rc) return rc;
-  const CUtensorMap tw0 = *pw0, tw1 = *pw1, tx = *px;
   dev->tc_pending = true;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(2 * ((a.M + Cfg::TN - 1) / Cfg::TN), a.N / (2 * TC_BM), 1);

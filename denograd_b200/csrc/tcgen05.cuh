@@ -92,6 +92,7 @@ __device__ __forceinline__ void st_cluster_f32(uint32_t addr, float v) {
 #endif
 
 // Tensor map of a row-major [rows][cols] matrix of 16-bit elements (or int8 when bytes == 1) with `ld` elements between
-// rows, cut into boxes of box_rows x 64; out-of-range elements read as zero.  Maps are cached per argument set.
-int jg_tensor_map(const CUtensorMap** out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
+// rows, cut into boxes of box_rows x 64; out-of-range elements read as zero.  Maps are kept per argument set; `out` is a
+// copy, because the next call may reuse the slot this one came from.
+int jg_tensor_map(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
                   const char* what, int bytes = 2, bool bf16 = false);

@@ -39,23 +39,23 @@ static int make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t co
 // step after the first finds all of its maps here instead of encoding three per launch.
 struct MapKey { const void* base; uint64_t rows, cols, ld; uint32_t box_rows; int bytes; bool bf16; };
 struct MapSlot { MapKey k; CUtensorMap m; bool used; };
-constexpr int MAP_SLOTS = 1024;
+constexpr int MAP_SLOTS = 8192;
 static MapSlot g_maps[MAP_SLOTS];
 
-int jg_tensor_map(const CUtensorMap** out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows, const char* what,
+int jg_tensor_map(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows, const char* what,
                   int bytes, bool bf16) {
   uint64_t h = (uint64_t)(uintptr_t)base * 0x9E3779B97F4A7C15ull ^ (rows * 0xBF58476D1CE4E5B9ull) ^ (cols << 20) ^ (ld << 4) ^ box_rows ^ ((uint64_t)bytes << 40) ^ ((uint64_t)bf16 << 43);
   h ^= h >> 29;
   for (int probe = 0; probe < 8; probe++) {
     MapSlot& s = g_maps[(h + probe) % MAP_SLOTS];
     if (s.used && s.k.base == base && s.k.rows == rows && s.k.cols == cols && s.k.ld == ld && s.k.box_rows == box_rows && s.k.bytes == bytes &&
-        s.k.bf16 == bf16) { *out = &s.m; return JG_OK; }
+        s.k.bf16 == bf16) { *out = s.m; return JG_OK; }
     if (!s.used) {
       int rc = make_map(&s.m, base, rows, cols, ld, box_rows, what, bytes, bf16);
       if (rc) return rc;
       s.k = MapKey{base, rows, cols, ld, box_rows, bytes, bf16};
       s.used = true;
-      *out = &s.m;
+      *out = s.m;
       return JG_OK;
     }
   }
@@ -64,6 +64,6 @@ int jg_tensor_map(const CUtensorMap** out, const void* base, uint64_t rows, uint
   if (rc) { s.used = false; return rc; }
   s.k = MapKey{base, rows, cols, ld, box_rows, bytes, bf16};
   s.used = true;
-  *out = &s.m;
+  *out = s.m;
   return JG_OK;
 }

@@ -57,3 +57,20 @@ def test_cta_pairs_forced_for_every_epilogue():
                         f"test_dense_projection_all_epilogues and ({pick})"], env=dict(os.environ, JG_TC_PAIR="2"),
                        capture_output=True, text=True, timeout=900, cwd=os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
     assert r.returncode == 0 and "4 passed" in r.stdout, r.stdout[-2000:] + r.stderr[-2000:]
+
+
+def test_more_operands_than_kept_tensor_maps(dev):
+    """A process that projects with more distinct matrices than the library keeps tensor maps for: slots are reused, also
+    between the maps of one launch."""
+    n, M, N, K = 9000, 3, 128, 64
+    rng = np.random.default_rng(7)
+    w = rng.standard_normal((n * 8 + N, K)).astype(np.float16)
+    x = rng.standard_normal((n + M, K)).astype(np.float16)
+    wt, xt, y = Tensor(w, device=dev), Tensor(x, device=dev), Tensor.zeros((n, M, N), "float16", dev)
+    for _ in range(2):
+        for i in range(n):  # matrix i: rows 8 i .. of one allocation; its activation rows: i ..
+            dev.call("jg_linear", y.ptr + 2 * i * M * N, xt.ptr + 2 * i * K, wt.ptr + 2 * 8 * i * K, 0, 0, M, N, K)
+    got = y.numpy()
+    for i in range(0, n, 37):
+        ref = (x[i:i + M].astype(np.float32) @ w[8 * i:8 * i + N].astype(np.float32).T).astype(np.float16)
+        assert_reduction_close(got[i], ref, max_ulp=1, max_frac=0.08, what=f"matrix {i}")

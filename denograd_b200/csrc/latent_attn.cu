@@ -331,12 +331,13 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
     if (tid + k * LS_THREADS < a.lat4) part[tid + k * LS_THREADS] = acc[k];  // zeros past the latent
 }
 
-// One row, 16 * MT heads, one context slice: tiles of 64 cached rows; warp w scores 8 of them for all heads, two warps'
-// worth of heads get their softmax statistics per warp, and each warp owns NTW * 8 columns of the weighted latent.
+// One row, 16 * MT heads, one context slice: tiles of 64 cached rows; a warp scores 16 of them for all heads over one half
+// of the latent (two partial score tiles), the heads' softmax statistics are dealt over the warps, and each warp owns
+// NTW * 8 columns of the weighted latent.
 constexpr int LM_THREADS = 256, LM_TILE = 64;
 template <int MT>
 static constexpr size_t lm_smem(int lq, int stages) {
-  return (size_t)(stages * LM_TILE + 16 * MT) * (lq + 8) * 2 + (size_t)16 * MT * (LM_TILE * 4 + (LM_TILE + 8) * 2 + 12);
+  return (size_t)(stages * LM_TILE + 16 * MT) * (lq + 8) * 2 + (size_t)16 * MT * (2 * LM_TILE * 4 + (LM_TILE + 8) * 2 + 12);
 }
 
 template <int MT, int NTW>
@@ -346,8 +347,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
   const int ld = a.lq + 8;  // row stride: an odd number of 16-byte pieces
   bf16* tiles = reinterpret_cast<bf16*>(smem);
   bf16* sQ = tiles + (size_t)stages * LM_TILE * ld;
-  float* sS = reinterpret_cast<float*>(sQ + (size_t)HR * ld);  // [HR][64]
-  bf16* sP = reinterpret_cast<bf16*>(sS + HR * LM_TILE);       // [HR][72]
+  float* sS = reinterpret_cast<float*>(sQ + (size_t)HR * ld);  // [2][HR][64]
+  bf16* sP = reinterpret_cast<bf16*>(sS + 2 * HR * LM_TILE);   // [HR][72]
   float *sM = reinterpret_cast<float*>(sP + HR * (LM_TILE + 8)), *sL = sM + HR, *sA = sL + HR;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, z = blockIdx.x, h0 = blockIdx.y * HR, r = blockIdx.z;
   pdl_launch();
@@ -401,32 +402,38 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
     else cp_wait<0>();
     __syncthreads();
     const bf16* t = tiles + (size_t)s * LM_TILE * ld;
-    float sc[MT][4];
+    float sc[MT][2][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
-      for (int i = 0; i < 4; i++) sc[m][i] = 0.f;
-    const bf16* kb = t + (size_t)(warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
+      for (int j = 0; j < 2; j++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) sc[m][j][i] = 0.f;
+    const int pg = warp & 3, kh = warp >> 2;
+    const bf16* kb = t + (size_t)(pg * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;
     const bf16* qb = sQ + (size_t)(lane & 15) * ld + (lane >> 4) * 8;
-    for (int k = 0; k < a.lq; k += 32) {
+#pragma unroll 2
+    for (int k = kh * (a.lq / 2); k < (kh + 1) * (a.lq / 2); k += 16) {
       uint32_t bk[4];
       ldsm4(bk, kb + k);
 #pragma unroll
       for (int m = 0; m < MT; m++) {
-        uint32_t q0[4], q1[4];
-        ldsm4(q0, qb + (size_t)m * 16 * ld + k);
-        ldsm4(q1, qb + (size_t)m * 16 * ld + k + 16);
-        mma_bf16(sc[m], q0, bk[0], bk[1]);
-        mma_bf16(sc[m], q1, bk[2], bk[3]);
+        uint32_t q[4];
+        ldsm4(q, qb + (size_t)m * 16 * ld + k);
+        mma_bf16(sc[m][0], q, bk[0], bk[1]);
+        mma_bf16(sc[m][1], q, bk[2], bk[3]);
       }
     }
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
-        const int c = warp * 8 + tq * 2 + (i & 1);
-        sS[(m * 16 + g + 8 * (i >> 1)) * LM_TILE + c] = base + c < t1 ? sc[m][i] * a.scale : -INFINITY;
-      }
+      for (int j = 0; j < 2; j++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+          const int c = pg * 16 + j * 8 + tq * 2;
+          *reinterpret_cast<float2*>(sS + (size_t)kh * HR * LM_TILE + (m * 16 + g + 8 * i) * LM_TILE + c) =
+              make_float2(base + c < t1 ? sc[m][j][2 * i] * a.scale : -INFINITY, base + c + 1 < t1 ? sc[m][j][2 * i + 1] * a.scale : -INFINITY);
+        }
     __syncthreads();
     {  // the warp's heads side by side: their reductions overlap
       constexpr int NH = HR / 8;
@@ -434,8 +441,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
 #pragma unroll
       for (int k = 0; k < NH; k++) {
         const int row = k * 8 + warp;
-        x0[k] = sS[row * LM_TILE + lane];
-        x1[k] = sS[row * LM_TILE + lane + 32];
+        x0[k] = sS[row * LM_TILE + lane] + sS[(HR + row) * LM_TILE + lane];
+        x1[k] = sS[row * LM_TILE + lane + 32] + sS[(HR + row) * LM_TILE + lane + 32];
         old[k] = sM[row];
         mx[k] = fmaxf(x0[k], x1[k]);
       }

@@ -9,65 +9,65 @@ namespace cg = cooperative_groups;
 
 // ------------------------------------------------------------------------------------------------ minGRU
 // S_t = (1 - z_t) S_{t-1} + z_t c_t is, per channel, an affine map of the state; maps compose, so a portion is scanned in
-// blocks of MG_WARPS x MG_TOK tokens: warp w composes its MG_TOK consecutive tokens, the warps' maps meet in shared
-// memory, warp 0 runs through them, and each warp replays its tokens from the state its predecessors leave.  One CTA = 32
-// channels of a sequence.
-constexpr int MG_WARPS = 32, MG_TOK = 4, MG_THREADS = 32 * MG_WARPS;
+// blocks of MG_GROUPS x MG_TOK tokens: a group of lanes composes its MG_TOK consecutive tokens, the groups' maps meet in
+// shared memory, the first group runs through them, and each group replays its tokens from the state its predecessors
+// leave.  One CTA = 16 channels of a sequence.
+constexpr int MG_CH = 16, MG_GROUPS = 32, MG_TOK = 4, MG_THREADS = MG_CH * MG_GROUPS;
 
 template <typename T>
-__global__ void __launch_bounds__(MG_THREADS, 1) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
-                                                                    const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
-  __shared__ float s_a[MG_WARPS][32], s_b[MG_WARPS][32], s_in[MG_WARPS][32];
+__global__ void __launch_bounds__(MG_THREADS) mingru_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, T* __restrict__ out, const int32_t* __restrict__ pos,
+                                                                 const int32_t* __restrict__ seq, int B, int Sc, int width, int ldp, int ldo) {
+  __shared__ float s_a[MG_GROUPS][MG_CH], s_b[MG_GROUPS][MG_CH], s_in[MG_GROUPS][MG_CH];
   pdl_wait();  // no early trigger: the next kernel's CTAs would sit on this one's SMs for its whole length
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, b = blockIdx.y, ch = blockIdx.x * 32 + lane;
+  const int c = threadIdx.x % MG_CH, grp = threadIdx.x / MG_CH, b = blockIdx.y, ch = blockIdx.x * MG_CH + c;
   const bool ok = ch < width;
   float* st = state + (size_t)seq[b] * width + ch;
-  float carry = (warp == 0 && ok && pos[b] > 0) ? *st : 0.f;  // warp 0: the state ahead of the block
+  float carry = (grp == 0 && ok && pos[b] > 0) ? *st : 0.f;  // first group: the state ahead of the block
   T nz[MG_TOK], nc[MG_TOK], ng[MG_TOK];  // the next block's inputs travel while this one is worked on
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
-      const int t = t0 + warp * MG_TOK + i;
+      const int t = t0 + grp * MG_TOK + i;
       if (!ok || t >= Sc) continue;
       const T* p = proj + ((size_t)t * B + b) * ldp + ch;
       nz[i] = p[0]; nc[i] = p[width]; ng[i] = p[2 * width];
     }
   };
   fetch(0);
-  for (int t0 = 0; t0 < Sc; t0 += MG_WARPS * MG_TOK) {
-    float z[MG_TOK], c[MG_TOK], g[MG_TOK];
+  for (int t0 = 0; t0 < Sc; t0 += MG_GROUPS * MG_TOK) {
+    float z[MG_TOK], u[MG_TOK], g[MG_TOK];
     float A = 1.f, Bc = 0.f;
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
-      const bool in = ok && t0 + warp * MG_TOK + i < Sc;
+      const bool in = ok && t0 + grp * MG_TOK + i < Sc;
       z[i] = in ? sigmoid_f32(to_f32(nz[i])) : 0.f;  // past the end: the identity map
-      c[i] = in ? z[i] * mingru_candidate(to_f32(nc[i])) : 0.f;
+      u[i] = in ? z[i] * mingru_candidate(to_f32(nc[i])) : 0.f;
       g[i] = in ? to_f32(ng[i]) : 0.f;
       A *= 1.0f - z[i];
-      Bc = fmaf(1.0f - z[i], Bc, c[i]);
+      Bc = fmaf(1.0f - z[i], Bc, u[i]);
     }
-    fetch(t0 + MG_WARPS * MG_TOK);
-    s_a[warp][lane] = A;
-    s_b[warp][lane] = Bc;
+    fetch(t0 + MG_GROUPS * MG_TOK);
+    s_a[grp][c] = A;
+    s_b[grp][c] = Bc;
     __syncthreads();
-    if (warp == 0) {
+    if (grp == 0) {
 #pragma unroll 8
-      for (int w = 0; w < MG_WARPS; w++) {
-        s_in[w][lane] = carry;
-        carry = fmaf(s_a[w][lane], carry, s_b[w][lane]);
+      for (int w = 0; w < MG_GROUPS; w++) {
+        s_in[w][c] = carry;
+        carry = fmaf(s_a[w][c], carry, s_b[w][c]);
       }
     }
     __syncthreads();
-    float s = s_in[warp][lane];
+    float s = s_in[grp][c];
 #pragma unroll
     for (int i = 0; i < MG_TOK; i++) {
-      const int t = t0 + warp * MG_TOK + i;
-      s = fmaf(1.0f - z[i], s, c[i]);
+      const int t = t0 + grp * MG_TOK + i;
+      s = fmaf(1.0f - z[i], s, u[i]);
       if (ok && t < Sc) out[((size_t)t * B + b) * ldo + ch] = from_f32<T>(s * silu_f32(g[i]));
     }
   }
   pdl_launch();
-  if (warp == 0 && ok) *st = carry;
+  if (grp == 0 && ok) *st = carry;
 }
 
 // One token per sequence: one thread per channel.
@@ -91,7 +91,7 @@ static int mingru_run(jg_dev* dev, const jg_batch* b, const jg_mingru_desc* d) {
   if (b->Sc == 1)
     return jg_launch(dev, "mingru_step", mingru_step_kernel<T>, dim3((unsigned)((d->width + 255) / 256), (unsigned)b->B), dim3(256), 0, (const T*)d->proj, (float*)d->state,
                      (T*)d->out, pos, seq, d->width, d->ldp, d->ldo);
-  return jg_launch(dev, "mingru_scan", mingru_scan_kernel<T>, dim3((unsigned)((d->width + 31) / 32), (unsigned)b->B), dim3(MG_THREADS), 0, (const T*)d->proj, (float*)d->state,
+  return jg_launch(dev, "mingru_scan", mingru_scan_kernel<T>, dim3((unsigned)((d->width + MG_CH - 1) / MG_CH), (unsigned)b->B), dim3(MG_THREADS), 0, (const T*)d->proj, (float*)d->state,
                    (T*)d->out, pos, seq, b->B, b->Sc, d->width, d->ldp, d->ldo);
 }
 

@@ -36,7 +36,7 @@ __device__ __forceinline__ void unpack_chunk(const uint4& v, float (&o)[8]) {
   o[6] = __uint_as_float(v.w << 16); o[7] = __uint_as_float(v.w & 0xFFFF0000u);
 }
 
-__device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f32(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }  // division within 2 ulp; 0 below -87
 __device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // minGRU: candidate state of a pre-activation

@@ -331,24 +331,25 @@ __global__ void __launch_bounds__(LS_THREADS) latent_split_kernel(const LatentAr
     if (tid + k * LS_THREADS < a.lat4) part[tid + k * LS_THREADS] = acc[k];  // zeros past the latent
 }
 
-// One row, 16 * MT heads, one context slice: tiles of 64 cached rows; a warp scores 16 of them for all heads over one half
-// of the latent (two partial score tiles), the heads' softmax statistics are dealt over the warps, and each warp owns
-// NTW * 8 columns of the weighted latent.
-constexpr int LM_THREADS = 256, LM_TILE = 64;
-template <int MT>
+// One row, 16 * MT heads, one context slice: tiles of 64 cached rows; a warp scores 16 of them for all heads over one part
+// of the latent (NW / 4 partial score tiles), the heads' softmax statistics are dealt over the NW warps, and each warp owns
+// NTW * 8 columns of the weighted latent.  A CTA fills an SM's shared memory: with 16 warps instead of 8 more of a tile's
+// latencies overlap.
+constexpr int LM_TILE = 64;
+template <int MT, int NW>
 static constexpr size_t lm_smem(int lq, int stages) {
-  return (size_t)(stages * LM_TILE + 16 * MT) * (lq + 8) * 2 + (size_t)16 * MT * (2 * LM_TILE * 4 + (LM_TILE + 8) * 2 + 12);
+  return (size_t)(stages * LM_TILE + 16 * MT) * (lq + 8) * 2 + (size_t)16 * MT * ((NW / 4) * LM_TILE * 4 + (LM_TILE + 8) * 2 + 12);
 }
 
-template <int MT, int NTW>
-__global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs<bf16> a, int stages) {
+template <int MT, int NTW, int NW>
+__global__ void __launch_bounds__(32 * NW) latent_mma_kernel(const LatentArgs<bf16> a, int stages) {
   extern __shared__ __align__(16) unsigned char smem[];
-  constexpr int HR = 16 * MT;
+  constexpr int HR = 16 * MT, KS = NW / 4;
   const int ld = a.lq + 8;  // row stride: an odd number of 16-byte pieces
   bf16* tiles = reinterpret_cast<bf16*>(smem);
   bf16* sQ = tiles + (size_t)stages * LM_TILE * ld;
-  float* sS = reinterpret_cast<float*>(sQ + (size_t)HR * ld);  // [2][HR][64]
-  bf16* sP = reinterpret_cast<bf16*>(sS + 2 * HR * LM_TILE);   // [HR][72]
+  float* sS = reinterpret_cast<float*>(sQ + (size_t)HR * ld);  // [KS][HR][64]
+  bf16* sP = reinterpret_cast<bf16*>(sS + KS * HR * LM_TILE);  // [HR][72]
   float *sM = reinterpret_cast<float*>(sP + HR * (LM_TILE + 8)), *sL = sM + HR, *sA = sL + HR;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, z = blockIdx.x, h0 = blockIdx.y * HR, r = blockIdx.z;
   pdl_launch();
@@ -360,8 +361,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
   if (t0 >= t1) return;  // nobody reads an empty slice
   const int pieces = a.lq / 8, row_pieces = a.ldc / 8;
 #pragma unroll
-  for (int k = 0; k < HR / 8; k++) {  // a warp takes whole rows: one address calculation each
-    const int h = k * 8 + warp;
+  for (int k = 0; k < HR / NW; k++) {  // a warp takes whole rows: one address calculation each
+    const int h = k * NW + warp;
     const bf16* src = a.qt + ((size_t)r * a.H + min(h0 + h, a.H - 1)) * a.lq;
     for (int c = lane; c < pieces; c += 32) {
       bf16* d = sQ + (size_t)h * ld + c * 8;
@@ -371,13 +372,13 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
   }
   auto load_tile = [&](int base, int s) {
     bf16* t = tiles + (size_t)s * LM_TILE * ld;
-    const bf16* src[LM_TILE / 8];
+    const bf16* src[LM_TILE / NW];
 #pragma unroll
-    for (int k = 0; k < LM_TILE / 8; k++) src[k] = a.row(bt, min(base + k * 8 + warp, t1 - 1));
+    for (int k = 0; k < LM_TILE / NW; k++) src[k] = a.row(bt, min(base + k * NW + warp, t1 - 1));
 #pragma unroll
-    for (int k = 0; k < LM_TILE / 8; k++) {
-      const bool in = base + k * 8 + warp < t1;
-      bf16* d = t + (size_t)(k * 8 + warp) * ld;
+    for (int k = 0; k < LM_TILE / NW; k++) {
+      const bool in = base + k * NW + warp < t1;
+      bf16* d = t + (size_t)(k * NW + warp) * ld;
       for (int c = lane; c < pieces; c += 32) {
         if (in && c < row_pieces) cp16(d + c * 8, src[k] + c * 8);
         else *reinterpret_cast<uint4*>(d + c * 8) = make_uint4(0, 0, 0, 0);
@@ -412,8 +413,9 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
     const int pg = warp & 3, kh = warp >> 2;
     const bf16* kb = t + (size_t)(pg * 16 + (lane >> 4) * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;
     const bf16* qb = sQ + (size_t)(lane & 15) * ld + (lane >> 4) * 8;
+    const int k0 = a.lq / 16 * kh / KS * 16, k1 = a.lq / 16 * (kh + 1) / KS * 16;
 #pragma unroll 2
-    for (int k = kh * (a.lq / 2); k < (kh + 1) * (a.lq / 2); k += 16) {
+    for (int k = k0; k < k1; k += 16) {
       uint32_t bk[4];
       ldsm4(bk, kb + k);
 #pragma unroll
@@ -436,13 +438,17 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
         }
     __syncthreads();
     {  // the warp's heads side by side: their reductions overlap
-      constexpr int NH = HR / 8;
+      constexpr int NH = HR / NW;
       float x0[NH], x1[NH], old[NH], mx[NH], sum[NH];
 #pragma unroll
       for (int k = 0; k < NH; k++) {
-        const int row = k * 8 + warp;
-        x0[k] = sS[row * LM_TILE + lane] + sS[(HR + row) * LM_TILE + lane];
-        x1[k] = sS[row * LM_TILE + lane + 32] + sS[(HR + row) * LM_TILE + lane + 32];
+        const int row = k * NW + warp;
+        x0[k] = x1[k] = 0.f;
+#pragma unroll
+        for (int q = 0; q < KS; q++) {
+          x0[k] += sS[(q * HR + row) * LM_TILE + lane];
+          x1[k] += sS[(q * HR + row) * LM_TILE + lane + 32];
+        }
         old[k] = sM[row];
         mx[k] = fmaxf(x0[k], x1[k]);
       }
@@ -463,7 +469,7 @@ __global__ void __launch_bounds__(LM_THREADS) latent_mma_kernel(const LatentArgs
         for (int k = 0; k < NH; k++) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], w);
 #pragma unroll
       for (int k = 0; k < NH; k++) {
-        const int row = k * 8 + warp;
+        const int row = k * NW + warp;
         sP[row * (LM_TILE + 8) + lane] = __float2bfloat16_rn(x0[k]);
         sP[row * (LM_TILE + 8) + lane + 32] = __float2bfloat16_rn(x1[k]);
         if (lane == 0) {
@@ -844,7 +850,7 @@ static int mma_tiles(const jg_dev* dev, const jg_latent_desc* d, int* stages) {
   const size_t limit = (size_t)dev->prop.sharedMemPerBlockOptin - 1024;
   const int mt = d->heads > 16 && d->kv_rank <= 512 ? 2 : 1;
   for (*stages = 2; *stages >= 1; (*stages)--)
-    if ((mt == 2 ? lm_smem<2>(lq, *stages) : lm_smem<1>(lq, *stages)) <= limit) return mt;
+    if ((mt == 2 ? lm_smem<2, 8>(lq, *stages) : lm_smem<1, 8>(lq, *stages)) <= limit) return mt;
   return 0;
 }
 constexpr int LATENT_MAX_PARTS = 32 * 160;  // (row, head, slice) triples of a call with few rows
@@ -884,22 +890,23 @@ JG_API int jg_latent_scratch_bytes(const jg_latent_desc* d, int32_t B, int32_t S
   return JG_OK;
 }
 
-template <int MT, int NTW>
+template <int MT, int NTW, int NW>
 static int launch_mma(jg_dev* dev, const LatentArgs<bf16>& a, int R, int stages) {
-  auto kern = latent_mma_kernel<MT, NTW>;
+  auto kern = latent_mma_kernel<MT, NTW, NW>;
   static bool set[8] = {};
   if (!set[dev->ordinal & 7]) {
     JG_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dev->prop.sharedMemPerBlockOptin - 1024));
     set[dev->ordinal & 7] = true;
   }
-  return jg_launch(dev, "latent_mma", kern, dim3((unsigned)a.ns, (unsigned)((a.H + 16 * MT - 1) / (16 * MT)), (unsigned)R), dim3(LM_THREADS), lm_smem<MT>(a.lq, stages), a, stages);
+  return jg_launch(dev, "latent_mma", kern, dim3((unsigned)a.ns, (unsigned)((a.H + 16 * MT - 1) / (16 * MT)), (unsigned)R), dim3(32 * NW), lm_smem<MT, NW>(a.lq, stages), a, stages);
 }
 template <int MT>
 static int launch_mma_cols(jg_dev* dev, const LatentArgs<bf16>& a, int R, int stages) {
-  if (a.rank <= 128) return launch_mma<MT, 2>(dev, a, R, stages);
-  if (a.rank <= 256) return launch_mma<MT, 4>(dev, a, R, stages);
-  if (a.rank <= 512) return launch_mma<MT, 8>(dev, a, R, stages);
-  return launch_mma<1, 16>(dev, a, R, stages);
+  if (a.rank <= 128) return launch_mma<MT, 2, 8>(dev, a, R, stages);
+  const bool wide = lm_smem<MT, 16>(a.lq, stages) <= (size_t)dev->prop.sharedMemPerBlockOptin - 1024;
+  if (a.rank <= 256) return wide ? launch_mma<MT, 2, 16>(dev, a, R, stages) : launch_mma<MT, 4, 8>(dev, a, R, stages);
+  if (a.rank <= 512) return wide ? launch_mma<MT, 4, 16>(dev, a, R, stages) : launch_mma<MT, 8, 8>(dev, a, R, stages);
+  return launch_mma<1, 16, 8>(dev, a, R, stages);
 }
 static int launch_scores(jg_dev* dev, const LatentArgs<float>& a, int R, int, int) {
   return jg_launch(dev, "latent_split", latent_split_kernel<float>, dim3((unsigned)R, (unsigned)a.H, (unsigned)a.ns), dim3(LS_THREADS), (size_t)a.lat() * 4, a);

@@ -108,6 +108,9 @@ SINGLE = {
     "latent, odd sizes": config(latent(heads=1, dim=7, rot_dim=6, rot={"base": 50.0, "dims": 6, "scaling": YARN}, vdim=5, kv_rank=9)),
     "latent, wide": config(latent(heads=4, dim=64, rot_dim=32, rot={"base": 1e4, "dims": 32, "scaling": YARN}, vdim=64, kv_rank=160, mask={"size": 40}),
                            width=128, groups=2),
+    "latent, many heads": config(latent(heads=20, dim=16, rot_dim=8, rot={"base": 1e4, "dims": 8, "scaling": YARN}, vdim=72, kv_rank=264, mask={"size": 50})),
+    "latent, many heads, short latent": config(latent(heads=33, dim=8, rot_dim=8, rot={"base": 1e4, "dims": 8, "scaling": YARN}, vdim=8, kv_rank=72)),
+    "latent, long latent": config(latent(heads=2, dim=16, kv_rank=600)),
     "mlp with a tight clamp": config(with_mlp(mingru(24), ff=40, limit=0.3)),
 }
 
@@ -122,6 +125,7 @@ def test_one_layer(name, dtype):
     m = build(cfg, params, dtype)
     check(run(m, toks, [70]), want, dtype)
     check(run(m, toks, [33, 1]), want, dtype)
+    check(run(m, toks, [5, 9, 15]), want, dtype)  # portions below the size that expands keys and values
 
 
 def test_layer_outputs():

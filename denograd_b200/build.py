@@ -13,9 +13,9 @@ LIB = os.path.join(OUT_DIR, "libjsgrad_cuda.so")
 # The whole library is every source below.  A component is the part one model family needs on its own, linked as a
 # library of that name, so that a fresh checkout which serves one model does not compile the other families' kernels.
 CORE = ["device.cu", "comm.cu", "elementwise.cu", "sample.cu", "tensor_map.cu"]
-COMPONENTS = {"hybrid": CORE + ["dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu"]}
+COMPONENTS = {"hybrid": CORE + ["dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu", "linear_state.cu", "window_attn.cu"]}
 SOURCES = CORE + ["gemv.cu", "matvec_w8.cu", "gemm_small.cu", "gemm_tc.cu", "attention.cu", "attention_chunk.cu", "step.cu", "program.cu",
-                  "dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu"]
+                  "dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu", "linear_state.cu", "window_attn.cu"]
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC,-fvisibility=hidden", "--expt-relaxed-constexpr"]
 

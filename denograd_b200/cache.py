@@ -1,7 +1,7 @@
 """Per-request state of the layer-list models (hybrid.py): slots, and what every layer keeps per slot.
 
-A request owns one slot.  Recurrent layers keep fixed-size state per slot; a latent-attention layer keeps a ring of pages per
-slot, taken from the layer's pool when the slot is acquired and given back with it.  Nothing is cleared in between: the
+A request owns one slot.  Recurrent layers keep fixed-size state per slot; an attention layer keeps a ring of pages per
+slot, and pages for the first tokens where those stay visible, taken from the layer's pool when the slot is acquired and given back with it.  Nothing is cleared in between: the
 kernels never read a slot's old contents for a sequence that starts at position 0.
 """
 from __future__ import annotations
@@ -14,11 +14,13 @@ from .device import CUDA, Tensor
 class PageRing:
     """One layer's paged store: T [n_pages][page][ld], and the block table int32 [slots][pages_per_slot].  Position p of a
     slot lives on page table[slot][(p / page) % pages_per_slot], so `pages_per_slot` pages serve any length as long as the
-    positions that are still looked at, and the tokens of one call, span no more than they hold."""
+    positions that are still looked at, and the tokens of one call, span no more than they hold.  The first `pinned` pages of a
+    slot are no part of the ring: they keep the sequence's first positions, table[slot][p / page], and the ring runs over the
+    others, table[slot][pinned + (p / page - pinned) % (pages_per_slot - pinned)]."""
 
-    def __init__(self, dev: CUDA, slots: int, span: int, row: int, dtype: str, page: int):
-        self.page, self.row = page, row
-        self.pages_per_slot = (span + page - 1) // page
+    def __init__(self, dev: CUDA, slots: int, span: int, row: int, dtype: str, page: int, pinned: int = 0):
+        self.page, self.row, self.pinned = page, row, pinned
+        self.pages_per_slot = pinned + (span + page - 1) // page
         self.n_pages = slots * self.pages_per_slot
         self.pool = Tensor.zeros((self.n_pages, page, row), dtype, dev)
         self._free = list(range(self.n_pages))[::-1]
@@ -52,10 +54,13 @@ class SlotStates:
         self.tensors.append(t)
         return t
 
-    def ring(self, row: int, dtype: str, window: int) -> PageRing:
-        """Pages for rows of `row` elements, `window` positions looked back on (0: all of them)."""
+    def ring(self, row: int, dtype: str, window: int, keep: int = 0) -> PageRing:
+        """Pages for rows of `row` elements, `window` positions looked back on (0: all of them), the first `keep` ones for good."""
         span = self.max_context if window <= 0 else min(self.max_context, window - 1 + self.max_rows)
-        r = PageRing(self.dev, self.slots, span, row, dtype, self.page)
+        pinned = (keep + self.page - 1) // self.page
+        if pinned * self.page + span >= self.max_context:  # every position has a place of its own
+            span, pinned = self.max_context, 0
+        r = PageRing(self.dev, self.slots, span, row, dtype, self.page, pinned)
         self.rings.append(r)
         return r
 

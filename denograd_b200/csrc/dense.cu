@@ -7,7 +7,9 @@
 //              new stream to a second buffer.
 //   more rows  bf16: tcgen05 kernel (dense_tc.cu); float: a register-tiled fp32 kernel (no reduced-precision modes).
 //
-// Epilogues: STORE (T or fp32), GLU (clamped gate x linear, two matrices with biases), MINGRU (three matrices: update gate,
+// The prologue can also finish a linear recurrence (division, norm and output gate of jg_gated_norm).
+//
+// Epilogues: STORE (T or fp32; activation on some columns, some columns in fp32 elsewhere), GLU (clamped gate x linear, two matrices with biases), MINGRU (three matrices: update gate,
 // candidate, output gate; advances the recurrence by one token and gates it), LOGITS (fp32 + argmax key).
 #include "dense.cuh"
 
@@ -15,6 +17,8 @@ template <typename T>
 struct MvArgs {
   const T* x;
   StreamArgs st;
+  GatedArgs<T> gated;
+  DenseOut out;
   const T* w[3];
   const float* bias[3];
   T* y;
@@ -22,9 +26,11 @@ struct MvArgs {
   float* state;
   const int32_t *pos, *seq;
   unsigned long long* key;
-  int M, N, ldx, ldw, ldy;
+  int M, N, ldx, ldw, ldy, lead;
   float limit;
 };
+// where the rows of a matrix-vector call come from
+constexpr int ROWS_GIVEN = 0, ROWS_STREAM = 1, ROWS_GATED = 2;
 
 constexpr int MV_THREADS = 256;
 constexpr int MV_WARPS = MV_THREADS / 32;
@@ -39,7 +45,7 @@ __device__ __forceinline__ float dot_chunk(float acc, const uint4& w, const uint
   return acc;
 }
 
-template <typename T, int MT, int EPI, bool NORM>
+template <typename T, int MT, int EPI, int FROM>
 __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T> a) {
   constexpr int VEC = Elem<T>::VEC;
   constexpr int NW = EPI == JG_DENSE_GLU ? 2 : (EPI == JG_DENSE_MINGRU ? 3 : 1);
@@ -79,7 +85,15 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
     T* xm = xs + (size_t)m * a.ldw;
     if (m >= a.M) {
       for (int c = tid; c < KC; c += MV_THREADS) reinterpret_cast<uint4*>(xm)[c] = make_uint4(0, 0, 0, 0);
-    } else if (NORM) {
+    } else if (FROM == ROWS_GATED) {
+      float* buf = reinterpret_cast<float*>(smem_raw + (size_t)MT * row_bytes);
+      const int n = a.gated.H * a.gated.vd;
+      const T* xg = a.x + (size_t)m * a.ldx;
+      for (int c = tid; c < a.lead; c += MV_THREADS) xm[c] = xg[c];
+      for (int c = a.lead + n + tid; c < a.ldw; c += MV_THREADS) xm[c] = from_f32<T>(0.f);
+      if (m > 0) __syncthreads();
+      gated_row<MV_THREADS>(a.gated, (size_t)m, buf, buf + ((n + 3) & ~3), [&](int i, float v) { xm[a.lead + i] = from_f32<T>(v); });
+    } else if (FROM == ROWS_STREAM) {
       float* buf = reinterpret_cast<float*>(smem_raw + (size_t)MT * row_bytes);
       float* red = buf + ((a.st.D + 3) & ~3);
       const size_t src = a.st.rows ? (size_t)a.st.rows[m] : (size_t)m;
@@ -105,7 +119,9 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
     if (a.bias[0]) s0 += a.bias[0][row];
     const size_t o = (size_t)m * a.ldy + row;
     if (EPI == JG_DENSE_STORE) {
-      if (a.y32) a.y32[o] = s0;
+      s0 = dense_act<T>(a.out, m, row, s0);
+      if (row >= a.out.split) a.out.y2[(size_t)m * a.out.ld2 + row - a.out.split] = s0;
+      else if (a.y32) a.y32[o] = s0;
       else a.y[o] = from_f32<T>(s0);
     } else if (EPI == JG_DENSE_GLU) {
       if (a.bias[1]) s1 += a.bias[1][row];
@@ -222,9 +238,18 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
   }
 }
 
-template <typename T, int MT, int EPI, bool NORM>
+template <typename T>
+static GatedArgs<T> gated_args(const jg_gated_desc& d) {
+  GatedArgs<T> g = {};
+  g.o = (const float*)d.o; g.den = (const float*)d.den; g.w = (const float*)d.norm_w; g.gate = (const T*)d.gate;
+  g.H = d.heads; g.vd = d.vdim; g.groups = d.groups; g.ldp = d.ldp; g.eps = d.eps; g.scale = d.scale;
+  return g;
+}
+static size_t gated_smem_floats(const jg_gated_desc& d, int warps) { return (size_t)((d.heads * d.vdim + 3) & ~3) + stream_units(d.groups, warps); }
+
+template <typename T, int MT, int EPI, int FROM>
 static int launch_mv(jg_dev* dev, const DenseCall& c) {
-  auto kern = dense_mv_kernel<T, MT, EPI, NORM>;
+  auto kern = dense_mv_kernel<T, MT, EPI, FROM>;
   constexpr int RW = (EPI == JG_DENSE_GLU || EPI == JG_DENSE_MINGRU) ? 1 : 2;
   MvArgs<T> a = {};
   a.x = (const T*)c.x; a.st = c.st;
@@ -232,8 +257,10 @@ static int launch_mv(jg_dev* dev, const DenseCall& c) {
   if (c.out_f32) a.y32 = (float*)c.y;
   else a.y = (T*)c.y;
   a.state = c.state; a.pos = c.pos; a.seq = c.seq; a.key = c.key;
-  a.M = c.M; a.N = c.N; a.ldx = c.ldx; a.ldw = c.ldw; a.ldy = c.ldy; a.limit = c.limit;
-  const size_t smem = (size_t)MT * c.ldw * sizeof(T) + (NORM ? stream_smem_floats(c.st.D, c.st.groups, MV_WARPS) * sizeof(float) : 0);
+  a.M = c.M; a.N = c.N; a.ldx = c.ldx; a.ldw = c.ldw; a.ldy = c.ldy; a.limit = c.limit; a.out = c.out; a.lead = c.lead;
+  if (FROM == ROWS_GATED) a.gated = gated_args<T>(*c.gated);
+  const size_t smem = (size_t)MT * c.ldw * sizeof(T) + (FROM == ROWS_STREAM  ? stream_smem_floats(c.st.D, c.st.groups, MV_WARPS) * sizeof(float)
+                                                        : FROM == ROWS_GATED ? gated_smem_floats(*c.gated, MV_WARPS) * sizeof(float) : 0);
   const size_t limit = (size_t)dev->prop.sharedMemPerBlockOptin - 8192;
   if (smem > limit) {
     jg_set_error("dense: %d rows of K=%d need %zu B of shared memory (limit %zu)", MT, c.K, smem, limit);
@@ -262,7 +289,7 @@ static int launch_mv(jg_dev* dev, const DenseCall& c) {
 // ------------------------------------------------------------------------------------------------ fp32, many rows
 // 64 x 64 output tile, 4 x 4 per thread, plain fp32 FMAs in ascending k.
 __global__ void __launch_bounds__(256) dense_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
-                                                        float* __restrict__ y, int M, int N, int K, int ldx, int ldw, int ldy) {
+                                                        float* __restrict__ y, int M, int N, int K, int ldx, int ldw, int ldy, const DenseOut out) {
   __shared__ float xs[16][65], ws[16][65];
   pdl_launch();
   pdl_wait();
@@ -288,7 +315,10 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const float* __restrict_
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int m = m0 + tm + 16 * i, n = n0 + tn + 16 * j;
-      if (m < M && n < N) y[(size_t)m * ldy + n] = acc[i][j] + (bias ? bias[n] : 0.f);
+      if (m >= M || n >= N) continue;
+      const float v = dense_act<float>(out, m, n, acc[i][j] + (bias ? bias[n] : 0.f));
+      if (n >= out.split) out.y2[(size_t)m * out.ld2 + n - out.split] = v;
+      else y[(size_t)m * ldy + n] = v;
     }
 }
 
@@ -334,7 +364,7 @@ __global__ void __launch_bounds__(256) stream_step_kernel(const StreamArgs a, T*
   pdl_wait();
   const size_t r = blockIdx.x, src = a.rows ? (size_t)a.rows[r] : r;
   T* hr = h + r * ldh;
-  if (a.w_norm)
+  if (a.w_norm || a.plain)
     for (int i = a.D + threadIdx.x; i < ldh; i += 256) hr[i] = from_f32<T>(0.f);
   stream_row<256>(a, src, a.x_out ? a.x_out + src * a.D : nullptr, sbuf, sbuf + ((a.D + 3) & ~3), [&](int i, const auto& v) {
     constexpr int V = sizeof(v) / sizeof(float);
@@ -367,7 +397,8 @@ static int launch_stream(jg_dev* dev, const StreamArgs& st, T* h, int ldh, int R
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) stream_embed_kernel(float* __restrict__ out, const int32_t* __restrict__ tokens, const T* __restrict__ table, int dim, int ld, int vocab) {
+__global__ void __launch_bounds__(256) stream_embed_kernel(float* __restrict__ out, const int32_t* __restrict__ tokens, const T* __restrict__ table, int dim, int ld, int vocab,
+                                                           float scale) {
   pdl_launch();
   pdl_wait();
   const int tok = tokens[blockIdx.x];
@@ -375,22 +406,24 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(float* __restrict__ o
   const bool in = tok >= 0 && tok < vocab;  // an id outside the table reads as zeros
   float* o = out + (size_t)blockIdx.x * dim;
 #pragma unroll 4
-  for (int c = threadIdx.x; c < dim; c += 256) o[c] = in ? to_f32(row[c]) : 0.f;
+  for (int c = threadIdx.x; c < dim; c += 256) o[c] = in ? to_f32(row[c]) * scale : 0.f;
 }
 
 // ------------------------------------------------------------------------------------------------ dispatch
-template <typename T, int EPI, bool NORM>
+template <typename T, int EPI, int FROM>
 static int mv_rows(jg_dev* dev, const DenseCall& c) {
-  return c.M == 1 ? launch_mv<T, 1, EPI, NORM>(dev, c) : launch_mv<T, 2, EPI, NORM>(dev, c);
+  return c.M == 1 ? launch_mv<T, 1, EPI, FROM>(dev, c) : launch_mv<T, 2, EPI, FROM>(dev, c);
 }
 template <typename T>
 static int mv_dispatch(jg_dev* dev, const DenseCall& c) {
   const bool norm = c.x == nullptr;
   switch (c.epilogue) {
-    case JG_DENSE_STORE: return norm ? mv_rows<T, JG_DENSE_STORE, true>(dev, c) : mv_rows<T, JG_DENSE_STORE, false>(dev, c);
-    case JG_DENSE_GLU: return norm ? mv_rows<T, JG_DENSE_GLU, true>(dev, c) : mv_rows<T, JG_DENSE_GLU, false>(dev, c);
-    case JG_DENSE_LOGITS: return norm ? mv_rows<T, JG_DENSE_LOGITS, true>(dev, c) : mv_rows<T, JG_DENSE_LOGITS, false>(dev, c);
-    case JG_DENSE_MINGRU: if (norm) return mv_rows<T, JG_DENSE_MINGRU, true>(dev, c);
+    case JG_DENSE_STORE:
+      if (c.gated) return mv_rows<T, JG_DENSE_STORE, ROWS_GATED>(dev, c);
+      return norm ? mv_rows<T, JG_DENSE_STORE, ROWS_STREAM>(dev, c) : mv_rows<T, JG_DENSE_STORE, ROWS_GIVEN>(dev, c);
+    case JG_DENSE_GLU: return norm ? mv_rows<T, JG_DENSE_GLU, ROWS_STREAM>(dev, c) : mv_rows<T, JG_DENSE_GLU, ROWS_GIVEN>(dev, c);
+    case JG_DENSE_LOGITS: return norm ? mv_rows<T, JG_DENSE_LOGITS, ROWS_STREAM>(dev, c) : mv_rows<T, JG_DENSE_LOGITS, ROWS_GIVEN>(dev, c);
+    case JG_DENSE_MINGRU: if (norm) return mv_rows<T, JG_DENSE_MINGRU, ROWS_STREAM>(dev, c);
   }
   jg_set_error("dense: epilogue %d has no kernel for these operands", c.epilogue);
   return JG_ENOTSUP;
@@ -398,11 +431,12 @@ static int mv_dispatch(jg_dev* dev, const DenseCall& c) {
 
 static int f32_gemm(jg_dev* dev, const DenseCall& c, const void* w, const float* bias, float* y, int ldy) {
   const dim3 grid((unsigned)((c.N + 63) / 64), (unsigned)((c.M + 63) / 64));
-  return jg_launch(dev, "dense_f32", dense_f32_kernel, grid, dim3(256), 0, (const float*)c.x, (const float*)w, bias, y, c.M, c.N, c.K, c.ldx, c.ldw, ldy);
+  return jg_launch(dev, "dense_f32", dense_f32_kernel, grid, dim3(256), 0, (const float*)c.x, (const float*)w, bias, y, c.M, c.N, c.K, c.ldx, c.ldw, ldy, c.out);
 }
 
 int jg_dense_call(jg_dev* dev, const DenseCall& c) {
   if (c.M <= 2) return c.dtype == JG_F32 ? mv_dispatch<float>(dev, c) : mv_dispatch<bf16>(dev, c);
+  JG_REQUIRE(c.gated == nullptr, "dense: %d rows: run jg_gated_norm first and pass its rows", c.M);
   JG_REQUIRE(c.x != nullptr, "dense: %d rows: run the stream step first (jg_stream_norm) and pass its rows", c.M);
   JG_REQUIRE(c.epilogue != JG_DENSE_MINGRU, "dense: the recurrent epilogue takes 1-2 rows (M=%d)", c.M);
   int rc;
@@ -430,13 +464,14 @@ static int check_batch(const char* name, const jg_batch* b) {
 static int fill_stream(const char* name, const jg_stream_desc& s, StreamArgs* a) {
   JG_REQUIRE(s.width > 0 && s.groups > 0 && s.width % s.groups == 0, "%s: %d values do not divide into %d groups", name, s.width, s.groups);
   JG_REQUIRE(jg_aligned(s.x, 16) && (s.y == 0) == (s.w_add == 0), "%s: bad stream pointers", name);
+  a->plain = s.plain;
   for (uint64_t p : {s.y, s.w_add, s.x_out, s.w_norm, s.rows}) JG_REQUIRE(p % (p == s.rows ? 4 : 16) == 0, "%s: misaligned pointer", name);
   a->x = (const float*)s.x; a->y = (const float*)s.y; a->w_add = (const float*)s.w_add; a->x_out = (float*)s.x_out;
   a->w_norm = (const float*)s.w_norm; a->rows = (const int32_t*)s.rows; a->D = s.width; a->groups = s.groups; a->eps = s.eps;
   return JG_OK;
 }
 
-JG_API int jg_stream_embed(jg_dev* dev, const jg_batch* b, uint64_t out, uint64_t tokens, uint64_t table, int32_t dtype, int32_t dim, int32_t ld, int32_t vocab) {
+JG_API int jg_stream_embed(jg_dev* dev, const jg_batch* b, uint64_t out, uint64_t tokens, uint64_t table, int32_t dtype, int32_t dim, int32_t ld, int32_t vocab, float scale) {
   JG_ENTER(dev);
   int rc = check_batch("stream_embed", b);
   if (rc) return rc;
@@ -444,8 +479,8 @@ JG_API int jg_stream_embed(jg_dev* dev, const jg_batch* b, uint64_t out, uint64_
   JG_REQUIRE(jg_aligned(out, 4) && jg_aligned(tokens, 4) && table != 0, "stream_embed: null or misaligned pointer");
   const dim3 grid((unsigned)(b->B * b->Sc));
   if (dtype == JG_F32)
-    return jg_launch(dev, "stream_embed", stream_embed_kernel<float>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const float*)table, dim, ld, vocab);
-  return jg_launch(dev, "stream_embed", stream_embed_kernel<bf16>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const bf16*)table, dim, ld, vocab);
+    return jg_launch(dev, "stream_embed", stream_embed_kernel<float>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const float*)table, dim, ld, vocab, scale);
+  return jg_launch(dev, "stream_embed", stream_embed_kernel<bf16>, grid, dim3(256), 0, (float*)out, (const int32_t*)tokens, (const bf16*)table, dim, ld, vocab, scale);
 }
 
 JG_API int jg_stream_norm(jg_dev* dev, const jg_batch* b, const jg_stream_desc* s, uint64_t h, int32_t ldh, int32_t dtype) {
@@ -456,9 +491,51 @@ JG_API int jg_stream_norm(jg_dev* dev, const jg_batch* b, const jg_stream_desc* 
   StreamArgs a = {};
   rc = fill_stream("stream_norm", *s, &a);
   if (rc) return rc;
-  JG_REQUIRE(s->w_norm == 0 || (jg_aligned(h, 16) && ldh >= s->width), "stream_norm: bad output");
+  JG_REQUIRE((s->w_norm == 0 && !s->plain) || (jg_aligned(h, 16) && ldh >= s->width), "stream_norm: bad output");
   const int R = b->B * b->Sc;
   return dtype == JG_F32 ? launch_stream<float>(dev, a, (float*)h, ldh, R) : launch_stream<bf16>(dev, a, (bf16*)h, ldh, R);
+}
+
+static int check_gated(const char* name, const jg_gated_desc& d) {
+  JG_REQUIRE(d.dtype == JG_F32 || d.dtype == JG_BF16, "%s: unknown element type %d", name, d.dtype);
+  JG_REQUIRE(d.heads > 0 && d.vdim > 0 && d.groups > 0 && d.heads * d.vdim % d.groups == 0 && d.ldp >= d.heads * d.vdim, "%s: bad gated row", name);
+  JG_REQUIRE(jg_aligned(d.o, 4) && d.den % 4 == 0 && d.gate && jg_aligned(d.norm_w, 4), "%s: null or misaligned pointer", name);
+  return JG_OK;
+}
+
+// Gated rows on their own (more rows than the matrix-vector kernel takes).
+template <typename T>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedArgs<T> a, T* __restrict__ out, int ldo) {
+  extern __shared__ __align__(16) float sbuf[];
+  pdl_launch();
+  pdl_wait();
+  const size_t r = blockIdx.x;
+  gated_row<256>(a, r, sbuf, sbuf + ((a.H * a.vd + 3) & ~3), [&](int i, float v) { out[r * ldo + i] = from_f32<T>(v); });
+}
+template <typename T>
+static int launch_gated(jg_dev* dev, const jg_gated_desc& d, T* out, int ldo, int R) {
+  const size_t smem = gated_smem_floats(d, 8) * sizeof(float), limit = (size_t)dev->prop.sharedMemPerBlockOptin - 1024;
+  if (smem > limit) {
+    jg_set_error("gated_norm: rows of %d values need %zu B of shared memory (limit %zu)", d.heads * d.vdim, smem, limit);
+    return JG_ENOTSUP;
+  }
+  static bool set[8] = {};
+  if (!set[dev->ordinal & 7]) {
+    JG_CUDA(cudaFuncSetAttribute(gated_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit));
+    set[dev->ordinal & 7] = true;
+  }
+  return jg_launch(dev, "gated_norm", gated_norm_kernel<T>, dim3((unsigned)R), dim3(256), smem, gated_args<T>(d), out, ldo);
+}
+JG_API int jg_gated_norm(jg_dev* dev, const jg_batch* b, const jg_gated_desc* d, uint64_t out, int32_t ldo) {
+  JG_ENTER(dev);
+  int rc = check_batch("gated_norm", b);
+  if (rc) return rc;
+  JG_REQUIRE(d != nullptr, "gated_norm: null descriptor");
+  rc = check_gated("gated_norm", *d);
+  if (rc) return rc;
+  JG_REQUIRE(out != 0 && out % (d->dtype == JG_F32 ? 4 : 2) == 0 && ldo >= d->heads * d->vdim, "gated_norm: bad output");
+  const int R = b->B * b->Sc;
+  return d->dtype == JG_F32 ? launch_gated<float>(dev, *d, (float*)out, ldo, R) : launch_gated<bf16>(dev, *d, (bf16*)out, ldo, R);
 }
 
 JG_API int jg_dense(jg_dev* dev, const jg_batch* b, const jg_dense_desc* d) {
@@ -480,12 +557,27 @@ JG_API int jg_dense(jg_dev* dev, const jg_batch* b, const jg_dense_desc* d) {
   }
   JG_REQUIRE(d->y != 0 && d->y % 4 == 0, "dense: null or misaligned output");
   c.y = (void*)d->y;
-  if (d->x) {
+  c.out.act = d->act; c.out.lo = d->act_lo; c.out.hi = d->act_hi > 0 ? d->act_hi : d->N; c.out.split = d->split > 0 ? d->split : d->N;
+  c.out.ld2 = d->ld2; c.out.y2 = (float*)d->y2; c.out.side = (const void*)d->side; c.out.tokens = (const int32_t*)d->tokens;
+  c.out.ld_side = d->ld_side; c.out.col_side = d->col_side; c.out.vocab = d->vocab;
+  if (d->epilogue == JG_DENSE_STORE) {
+    JG_REQUIRE(d->act >= JG_ACT_NONE && d->act <= JG_ACT_GELU_SIDE && d->act_lo >= 0 && d->split >= 0, "dense: bad activation or split");
+    JG_REQUIRE(c.out.split >= d->N || (jg_aligned(d->y2, 4) && d->ld2 >= d->N - c.out.split), "dense: bad fp32 columns");
+    JG_REQUIRE(d->act != JG_ACT_GELU_SIDE || (d->side && jg_aligned(d->tokens, 4) && d->col_side >= 0 && d->vocab > 0 && d->ld_side >= d->col_side + d->N), "dense: bad side table");
+  }
+  if (d->gated.o) {
+    const jg_gated_desc& g = d->gated;
+    rc = check_gated("dense", g);
+    if (rc) return rc;
+    JG_REQUIRE(d->epilogue == JG_DENSE_STORE && g.dtype == d->dtype && d->lead >= 0 && d->lead + g.heads * g.vdim == d->K, "dense: the gated prologue needs K = lead + heads * vdim");
+    JG_REQUIRE(d->lead == 0 || (jg_aligned(d->x, 16) && d->ldx >= d->lead), "dense: bad leading columns");
+    c.gated = &g; c.lead = d->lead;
+  } else if (d->x) {
     JG_REQUIRE(jg_aligned(d->x, 16) && d->ldx >= d->ldw && d->ldx % vec == 0, "dense: misaligned rows or row stride (ldx=%d, ldw=%d)", d->ldx, d->ldw);
   } else {
     rc = fill_stream("dense", d->stream, &c.st);
     if (rc) return rc;
-    JG_REQUIRE(c.st.D == d->K && c.st.w_norm != nullptr && c.st.x_out != c.st.x, "dense: the stream prologue needs K-wide rows and a second stream buffer");
+    JG_REQUIRE(c.st.D == d->K && (c.st.w_norm != nullptr || c.st.plain) && c.st.x_out != c.st.x, "dense: the stream prologue needs K-wide rows and a second stream buffer");
   }
   if (d->epilogue == JG_DENSE_LOGITS) {
     JG_REQUIRE(jg_aligned(d->key, 8) && d->out_f32, "dense: logits are fp32 and need their keys");

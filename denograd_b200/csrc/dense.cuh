@@ -2,6 +2,24 @@
 #pragma once
 #include "stream.cuh"
 
+// What STORE does beyond the bias: an activation on columns [lo, hi), and columns from `split` on in fp32 elsewhere.
+struct DenseOut {
+  int act = JG_ACT_NONE, lo = 0, hi = 0, split = 1 << 30, ld2 = 0, ld_side = 0, col_side = 0, vocab = 0;
+  float* y2 = nullptr;
+  const void* side = nullptr;  // T [vocab][ld_side]
+  const int32_t* tokens = nullptr;
+};
+#ifdef __CUDACC__
+template <typename T>
+__device__ __forceinline__ float dense_act(const DenseOut& o, int row, int col, float v) {
+  if (o.act == JG_ACT_NONE || col < o.lo || col >= o.hi) return v;
+  if (o.act == JG_ACT_SILU) return silu_f32(v);
+  if (o.act == JG_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
+  const int tok = o.tokens[row];  // an id outside the table reads as zeros
+  return tok >= 0 && tok < o.vocab ? gelu_tanh_f32(v) * to_f32(reinterpret_cast<const T*>(o.side)[(size_t)tok * o.ld_side + o.col_side + col]) : 0.f;
+}
+#endif
+
 struct DenseCall {
   int dtype;             // JG_F32 / JG_BF16
   int epilogue;          // JG_DENSE_*
@@ -9,11 +27,14 @@ struct DenseCall {
   const void* x;         // T [M][ldx], or null: rows come from the residual stream through `st`
   int ldx;
   StreamArgs st;
+  const jg_gated_desc* gated;  // or null; columns from `lead` on (1-2 rows)
+  int lead;
   const void* w[3];      // T [N][ldw], zero between K and ldw
   int ldw;
   const float* bias[3];  // fp32 [N] or null
   void* y;               // T or (out_f32) float [M][ldy]
   int ldy, out_f32;
+  DenseOut out;          // STORE
   float limit;                        // GLU
   float* state;                       // MINGRU: [slots][N]
   const int32_t *pos, *seq;           // MINGRU: [M]

@@ -21,6 +21,7 @@ struct DtArgs {
   int* err;
   int M, N, K, ldy, w_late;
   float limit;
+  DenseOut out;
 };
 
 template <int TN, bool GLU, bool HALF>
@@ -162,8 +163,12 @@ __global__ void __launch_bounds__(DtCfg<TN, GLU, HALF>::THREADS, HALF ? 2 : 1)
           if (tok < a.M) {
             const size_t o = (size_t)tok * a.ldy + feat;
             if (GLU) a.y[o] = __float2bfloat16_rn(clamped_glu(r0[j] + bias0, r1[j] + bias1, a.limit));
-            else if (a.y32) a.y32[o] = r0[j] + bias0;
-            else a.y[o] = __float2bfloat16_rn(r0[j] + bias0);
+            else {
+              const float v = dense_act<bf16>(a.out, tok, feat, r0[j] + bias0);
+              if (feat >= a.out.split) a.out.y2[(size_t)tok * a.out.ld2 + feat - a.out.split] = v;
+              else if (a.y32) a.y32[o] = v;
+              else a.y[o] = __float2bfloat16_rn(v);
+            }
           }
         }
       }
@@ -242,7 +247,7 @@ int jg_dense_tc(jg_dev* dev, const DenseCall& c) {
   DtArgs a = {};
   if (c.out_f32) a.y32 = (float*)c.y;
   else a.y = (bf16*)c.y;
-  a.b0 = c.bias[0]; a.b1 = c.bias[1]; a.err = dev->err_word; a.M = c.M; a.N = c.N; a.K = c.K; a.ldy = c.ldy; a.limit = c.limit;
+  a.b0 = c.bias[0]; a.b1 = c.bias[1]; a.err = dev->err_word; a.M = c.M; a.N = c.N; a.K = c.K; a.ldy = c.ldy; a.limit = c.limit; a.out = c.out;
   a.w_late = jg_is_fresh(dev, c.w[0]) || jg_is_fresh(dev, c.w[1]);
   if (c.epilogue == JG_DENSE_GLU) {
     if (c.M <= 16) return launch_dt<16, true, false>(dev, c, a);

@@ -18,6 +18,7 @@
 #include <stdlib.h>
 
 #include "dense.cuh"
+#include "mma.cuh"
 
 template <typename T>
 struct LatentArgs {
@@ -104,36 +105,6 @@ __global__ void __launch_bounds__(256) latent_write_kernel(const LatentArgs<T> a
     for (int i = lane; i < a.ldc / Elem<T>::VEC; i += 32) dst[i] = src[i];
   }
 }
-
-// ---- tensor cores (mma.sync m16n8k16, bf16 in, fp32 out)
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(void* smem, const void* gmem) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-__device__ __forceinline__ float ex2(float x) {  // 2^x by the hardware's approximation (2^-22 relative), 0 for -inf
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-constexpr float LOG2E = 1.4426950408889634f;
 
 // ------------------------------------------------------------------------------------------------ absorbed form
 constexpr int LP_COLS = 64;  // latent columns of a CTA; it serves LP_ROWS activation rows with one read of the weights

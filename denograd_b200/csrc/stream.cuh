@@ -38,6 +38,8 @@ __device__ __forceinline__ void unpack_chunk(const uint4& v, float (&o)[8]) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }  // division within 2 ulp; 0 below -87
 __device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
+__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
+__device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // minGRU: candidate state of a pre-activation
 __device__ __forceinline__ float mingru_candidate(float u) { return u >= 0.0f ? u + 0.5f : sigmoid_f32(u); }
@@ -59,7 +61,7 @@ __device__ __forceinline__ unsigned long long argmax_key_f32(float v, uint32_t i
 // ------------------------------------------------------------------------------------------------ between two sublayers
 // x <- x + norm(y) * w_add (skipped when y is null), then h = norm(x) * w_norm (skipped when w_norm is null): the norm
 // after one sublayer, the residual sum and the norm before the next one, on one row.  norm divides each of `groups` equal
-// consecutive parts by its own sqrt(mean(part^2) + eps).
+// consecutive parts by its own sqrt(mean(part^2) + eps).  A sublayer that reads the stream itself takes h = x (`plain`).
 struct StreamArgs {
   const float* x;       // [R][D] residual stream
   const float* y;       // [R][D] what the sublayer returned, or null
@@ -69,6 +71,7 @@ struct StreamArgs {
   const int32_t* rows;  // row indirection into x and y, or null
   int D, groups;
   float eps;
+  int plain;            // h = x, whatever w_norm is
 };
 
 static inline int stream_units(int groups, int warps) { return groups >= warps ? groups : (warps / groups) * groups; }
@@ -134,6 +137,17 @@ __device__ __forceinline__ void stream_row_v(const StreamArgs& a, size_t src, fl
     }
     __syncthreads();
   }
+  if (a.plain) {
+    for (int u = warp; u < units; u += W) {
+      const int g = u / P, lo = g * gs + (u % P) * plen, hi = min((g + 1) * gs, lo + plen);
+      for (int i = lo + lane * V; i < hi; i += 32 * V) {
+        float v[V];
+        load(buf + i, v);
+        store(i, v);
+      }
+    }
+    return;
+  }
   if (a.w_norm == nullptr) return;
   for (int u = warp; u < units; u += W) {
     const int g = u / P, lo = g * gs + (u % P) * plen, hi = min((g + 1) * gs, lo + plen);
@@ -152,5 +166,45 @@ template <int NT, typename Store>
 __device__ __forceinline__ void stream_row(const StreamArgs& a, size_t src, float* x_out_row, float* buf, float* red, Store store) {
   if ((a.D / a.groups) % 4 == 0) stream_row_v<NT, 4>(a, src, x_out_row, buf, red, store);
   else stream_row_v<NT, 1>(a, src, x_out_row, buf, red, store);
+}
+
+// ------------------------------------------------------------------------------------------------ after a linear recurrence
+// One row of o / den / rms(group) * w * sigmoid(gate) * scale (jg_gated_norm) by the NT threads of a CTA; buf holds H * vd floats,
+// red stream_units of them.  store(i, value) for every i.
+template <typename T>
+struct GatedArgs {
+  const float *o, *den, *w;
+  const T* gate;
+  int H, vd, groups, ldp;
+  float eps, scale;
+};
+template <int NT, typename T, typename Store>
+__device__ __forceinline__ void gated_row(const GatedArgs<T>& a, size_t r, float* buf, float* red, Store store) {
+  constexpr int W = NT / 32;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = a.H * a.vd;
+  const int gs = n / a.groups, P = a.groups >= W ? 1 : W / a.groups, units = a.groups * P, plen = (gs + P - 1) / P;
+  const float *o = a.o + r * n, *den = a.den ? a.den + r * a.H : nullptr;
+  const T* gate = a.gate + r * a.ldp;
+  for (int u = warp; u < units; u += W) {
+    const int g = u / P, lo = g * gs + (u % P) * plen, hi = min((g + 1) * gs, lo + plen);
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = lo + lane; i < hi; i += 32) {
+      const float v = den ? o[i] / den[i / a.vd] : o[i];
+      buf[i] = v;
+      ss = fmaf(v, v, ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) red[u] = ss;
+  }
+  __syncthreads();
+  for (int u = warp; u < units; u += W) {
+    const int g = u / P, lo = g * gs + (u % P) * plen, hi = min((g + 1) * gs, lo + plen);
+    float t = 0.f;
+    for (int p = 0; p < P; p++) t += red[g * P + p];
+    const float rs = a.scale / sqrtf(t / (float)gs + a.eps);
+#pragma unroll 4
+    for (int i = lo + lane; i < hi; i += 32) store(i, buf[i] * rs * a.w[i] * sigmoid_f32(to_f32(gate[i])));
+  }
 }
 #endif

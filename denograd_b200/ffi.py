@@ -41,6 +41,7 @@ class StepDesc(C.Structure):
 
 JG_F32, JG_BF16 = 0, 1
 DENSE_STORE, DENSE_GLU, DENSE_MINGRU, DENSE_LOGITS = 0, 1, 2, 3
+ACT_NONE, ACT_SILU, ACT_RELU2, ACT_GELU_SIDE = 0, 1, 2, 3
 
 
 def _fields(spec: str) -> list:
@@ -54,12 +55,17 @@ class Batch(C.Structure):
 
 
 class StreamDesc(C.Structure):
-    _fields_ = _fields("i32 width groups; f32 eps; i32 reserved; u64 x y w_add x_out w_norm rows")
+    _fields_ = _fields("i32 width groups; f32 eps; i32 plain; u64 x y w_add x_out w_norm rows")
+
+
+class GatedDesc(C.Structure):
+    _fields_ = _fields("i32 dtype heads vdim groups ldp reserved; f32 eps scale; u64 o den gate norm_w")
 
 
 class DenseDesc(C.Structure):
     _fields_ = _fields("i32 dtype epilogue N K ldx ldw ldy out_f32; f32 limit; i32 reserved; "
-                       "u64 x w0 w1 w2 b0 b1 b2 y key state") + [("stream", StreamDesc)]
+                       "u64 x w0 w1 w2 b0 b1 b2 y key state") + [("stream", StreamDesc), ("gated", GatedDesc)] + \
+               _fields("i32 act act_lo act_hi split ld2 ld_side col_side vocab lead reserved2; u64 y2 side tokens")
 
 
 class MinGruDesc(C.Structure):
@@ -74,6 +80,15 @@ class DeltaDesc(C.Structure):
 class LatentDesc(C.Structure):
     _fields_ = _fields("i32 dtype heads dim rot_dim vdim kv_rank window ldp ldo ldc ld_u page pages_per_slot n_slots rot_pairs rot_rows; "
                        "f32 eps scale; u64 proj pool block_table rot norm_w sink ukv scratch out scratch_bytes")
+
+
+class LinearDesc(C.Structure):
+    _fields_ = _fields("i32 dtype heads dim vdim ldp reserved; f32 q_scale cap; u64 q k v gates decay state m scratch o den")
+
+
+class WindowDesc(C.Structure):
+    _fields_ = _fields("i32 dtype heads kv_heads dim vdim window keep ldp ldo page pages_per_slot pinned rot_pairs rot_rows; f32 eps scale out_scale; i32 reserved; "
+                       "u64 q k v q_norm k_norm rot pool block_table scratch scratch_bytes out")
 
 
 _vp, _i32, _i64, _u64, _f32, _f64, _sz = C.c_void_p, C.c_int32, C.c_int64, C.c_uint64, C.c_float, C.c_double, C.c_size_t
@@ -166,7 +181,7 @@ SIGNATURES: dict[str, list] = {
     "jg_comm_group_end": [],
     "jg_linear_partial": [_vp, _u64, _u64, _u64, _u64, _i32, _i32, _i32],
     "jg_residual_add_f32": [_vp, _u64, _u64, _i64],
-    "jg_stream_embed": [_vp, _P(Batch), _u64, _u64, _u64, _i32, _i32, _i32, _i32],
+    "jg_stream_embed": [_vp, _P(Batch), _u64, _u64, _u64, _i32, _i32, _i32, _i32, _f32],
     "jg_stream_norm": [_vp, _P(Batch), _P(StreamDesc), _u64, _i32, _i32],
     "jg_dense": [_vp, _P(Batch), _P(DenseDesc)],
     "jg_mingru_scan": [_vp, _P(Batch), _P(MinGruDesc)],
@@ -174,6 +189,11 @@ SIGNATURES: dict[str, list] = {
     "jg_delta_rule": [_vp, _P(Batch), _P(DeltaDesc)],
     "jg_latent_scratch_bytes": [_P(LatentDesc), _i32, _i32, _P(_u64)],
     "jg_latent_attn": [_vp, _P(Batch), _P(LatentDesc)],
+    "jg_linear_scratch_bytes": [_P(LinearDesc), _i32, _P(_u64)],
+    "jg_linear_state": [_vp, _P(Batch), _P(LinearDesc)],
+    "jg_gated_norm": [_vp, _P(Batch), _P(GatedDesc), _u64, _i32],
+    "jg_window_scratch_bytes": [_P(WindowDesc), _i32, _i32, _P(_u64)],
+    "jg_window_attn": [_vp, _P(Batch), _P(WindowDesc)],
     "jg_sample_f32": [_vp, _u64, _u64, _u64, _u64, _i32, _i32, _f32, _i32, _f32, _f32, _f32],
     "jg_norm_logits_argmax_shard": [_vp, _u64, _u64, _u64, _u64, _f32, _u64, _u64, _i32, _i32, _i32, _i32],
 }

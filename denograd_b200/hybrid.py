@@ -1,24 +1,32 @@
-"""Decoders given as a list of layers, each with its own kind of mixer and an optional feed-forward.
+"""Decoders given as a list of layers, each with its own kind of mixer, an optional feed-forward and an optional token input.
 
-  stream x (fp32) = embedding rows
-  per layer   x <- x + norm_b(mixer(norm(x)));  with a feed-forward: x <- x + norm_b(ff(norm(x)))
+  stream x (fp32) = embedding rows * scale
+  per layer   x <- x + norm_b(mixer(norm(x)));  with a feed-forward: x <- x + norm_b(ff(norm(x)));  with a token input
+              x <- x + norm_b(W_proj (gelu(W_gate x) * the layer's part of the token's row in a second table))
   logits      = head norm(x)
 
+What differs between architectures beyond sizes is a `Design` (`DESIGNS`): whether sublayers read a normed stream or the stream
+itself, whether norm weights are stored around zero, a head of its own or the embedding table, and which feed-forward a
+"dense" one is.
+
 Mixers (`MIXERS`): ``mingru`` (gated linear recurrence), ``latent_attention`` (low-rank keys and values, sliding window,
-sinks, YaRN rotary), ``delta`` (gated delta rule with short convolutions).  Feed-forwards (`FEED_FORWARDS`): ``dense`` (clamped
-gated unit with biases).  Norms divide groups of channels by their own root mean square.  A model's configuration gives
-every size; `ARCHITECTURES` (registry.py) maps a configuration to the model.
+sinks, YaRN rotary), ``delta`` (gated delta rule with short convolutions), and mixers made of one or more `Branches` side by
+side: ``window_attention`` (grouped heads, sliding window and kept first tokens), ``lightning`` (linear attention with a decay
+per head), ``mlstm`` (exponentially gated matrix memory), ``parallel`` (the first two of these).  Norms divide groups of
+channels by their own root mean square.  A model's configuration gives every size; `ARCHITECTURES` (registry.py) maps a
+configuration to the model.
 
 How a step runs: each layer contributes library calls to a *plan* — descriptors of device addresses, made once per
 workspace — and a step walks the plan with the batch (sequences, tokens per sequence, positions, slots) as the only
 argument that changes.  With 1-2 rows the plan has no calls for norms and residual sums: the projection that follows takes
-the fp32 stream and does them in its prologue, and the minGRU recurrence is the epilogue of its projections.  A decode step
-is captured into a CUDA graph.
+the fp32 stream and does them in its prologue, the minGRU recurrence is the epilogue of its projections, and the norm and
+output gate after a linear recurrence are the prologue of the output projection.  A decode step is captured into a CUDA graph.
 """
 from __future__ import annotations
 
 import ctypes as C
 import math
+from dataclasses import dataclass
 
 import numpy as np
 
@@ -37,13 +45,18 @@ def round_up(n: int, m: int) -> int:
 
 # ------------------------------------------------------------------------------------------------ parameters
 class Param:
-    """Where one checkpoint tensor goes: `shape` values, rows of `cols` in device rows `ld` apart (zeros in between)."""
+    """Where one checkpoint tensor goes: `shape` values plus `offset`, rows of `cols` in device rows `ld` apart (zeros in
+    between)."""
 
-    def __init__(self, tensor: Tensor, shape: tuple, ld: int | None = None):
-        self.tensor, self.shape, self.ld = tensor, tuple(shape), ld
+    def __init__(self, tensor: Tensor, shape: tuple, ld: int | None = None, offset: float = 0.0):
+        self.tensor, self.shape, self.ld, self.offset = tensor, tuple(shape), ld, offset
+
+    @property
+    def ptr(self) -> int:
+        return self.tensor.ptr
 
     def assign(self, arr: np.ndarray) -> None:
-        arr = np.asarray(arr, np.float32)
+        arr = np.asarray(arr, np.float32) + np.float32(self.offset)
         if self.ld is not None and self.ld != self.shape[-1]:
             wide = np.zeros(self.shape[:-1] + (self.ld,), np.float32)
             wide[..., :self.shape[-1]] = arr
@@ -51,16 +64,35 @@ class Param:
         self.tensor.assign(arr)
 
 
-class Matrix:
-    """Projection weights [N][ld] of the model's element type; `parts` names runs of rows after checkpoint tensors."""
+class ColumnParam(Param):
+    """Columns [at, at + shape[1]) of a matrix whose columns come from several checkpoint tensors (`Columns`)."""
 
-    def __init__(self, m: "HybridTransformer", params: dict, parts: list[tuple[str, int]], K: int):
-        self.N, self.K, self.ld = sum(n for _, n in parts), K, round_up(K, 8)
+    def __init__(self, owner: "Columns", shape: tuple, at: int):
+        super().__init__(owner.weight, shape, owner.ld)
+        self.owner, self.at = owner, at
+
+    @property
+    def ptr(self) -> int:
+        return self.tensor.ptr + self.at * self.tensor.nbytes // self.tensor.numel()
+
+    def assign(self, arr: np.ndarray) -> None:
+        self.owner.put(self, np.asarray(arr, np.float32))
+
+
+class Matrix:
+    """Projection weights [N][ld] of the model's element type; `parts` names runs of rows after checkpoint tensors: (name,
+    rows), or (name, rows, alignment of the first row) with rows of zeros in between."""
+
+    def __init__(self, m: "HybridTransformer", params: dict, parts: list[tuple], K: int):
+        self.K, self.ld, self.row0, r = K, round_up(K, 8), {}, 0
+        for name, n, *align in parts:
+            self.row0[name] = r = round_up(r, align[0] if align else 1)
+            r += n
+        self.N = r
         self.weight = Tensor.zeros((self.N, self.ld), m.dtype, m.dev)
-        self.row0, r = {}, 0
-        for name, n in parts:
+        for name, n, *_ in parts:
+            r = self.row0[name]
             params[name] = Param(self.weight.view_rows(r, r + n), (n, K), self.ld)
-            self.row0[name], r = r, r + n
 
     @property
     def ptr(self) -> int:
@@ -70,15 +102,54 @@ class Matrix:
         return self.weight.ptr + self.row0[name] * self.ld * self.weight.nbytes // self.weight.numel()
 
 
-def vector(m: "HybridTransformer", params: dict, parts: list[tuple[str, tuple]], pad: int = 0) -> Tensor:
-    """fp32 parameters of consecutive checkpoint tensors (scalars per channel, taps, ...), `pad` zeros behind them."""
+class Columns:
+    """Projection weights [N][ld] whose columns are those of several checkpoint tensors (name, columns), each from a multiple
+    of 8 on, zeros in between: one projection of several inputs side by side.  `col0`: where each starts."""
+
+    def __init__(self, m: "HybridTransformer", params: dict, parts: list[tuple[str, int]], N: int):
+        self.N, self.col0, c = N, {}, 0
+        for name, n in parts:
+            self.col0[name] = c = round_up(c, 8)
+            c += n
+        self.K, self.ld = c, round_up(c, 8)
+        self.weight = Tensor.zeros((N, self.ld), m.dtype, m.dev)
+        self.params = [ColumnParam(self, (N, n), self.col0[name]) for name, n in parts]
+        params.update({name: q for (name, _), q in zip(parts, self.params)})
+        self._host: np.ndarray | None = None
+        self._missing: set[int] = set()
+
+    @property
+    def ptr(self) -> int:
+        return self.weight.ptr
+
+    def put(self, param: ColumnParam, arr: np.ndarray) -> None:
+        """The matrix goes to the device when the last of its tensors has come."""
+        if self._host is None:
+            self._host, self._missing = np.zeros((self.N, self.ld), np.float32), {q.at for q in self.params}
+        self._host[:, param.at:param.at + param.shape[1]] = arr
+        self._missing.discard(param.at)
+        if not self._missing:
+            self.weight.assign(self._host)
+            self._host = None
+
+
+def vector(m: "HybridTransformer", params: dict, parts: list[tuple[str, tuple]], pad: int = 0, offset: float = 0.0) -> Tensor:
+    """fp32 parameters of consecutive checkpoint tensors (scalars per channel, taps, ...) plus `offset`, `pad` zeros behind."""
     width = parts[0][1][1:]
     n = sum(s[0] for _, s in parts)
     t = Tensor.zeros((n + pad,) + width, "float32", m.dev)
     r = 0
     for name, s in parts:
-        params[name] = Param(t.view_rows(r, r + s[0]), s)
+        params[name] = Param(t.view_rows(r, r + s[0]), s, offset=offset)
         r += s[0]
+    return t
+
+
+def row_vector(m: "HybridTransformer", params: dict, w: Matrix, parts: list[tuple[str, str, int]]) -> Tensor:
+    """fp32, one value per row of `w`: (name, part of w it belongs to, rows); zeros elsewhere."""
+    t = Tensor.zeros((w.N,), "float32", m.dev)
+    for name, part, n in parts:
+        params[name] = Param(t.view_rows(w.row0[part], w.row0[part] + n), (n,))
     return t
 
 
@@ -98,7 +169,7 @@ class Plan:
     def call(self, name: str, *args) -> None:
         self.calls.append((name,) + args)
 
-    def stream(self, w_norm: Tensor | None, rows: int = 0, keep: bool = True) -> ffi.StreamDesc:
+    def stream(self, w_norm: Tensor | None, rows: int = 0, keep: bool = True, plain: bool = False) -> ffi.StreamDesc:
         m, ws = self.model, self.ws
         out = 0
         src = ws.x[self.cur].ptr
@@ -108,29 +179,34 @@ class Plan:
                 self.cur ^= 1
             out = ws.x[self.cur].ptr
             self.pending = None
-        return ffi.StreamDesc(m.width, m.groups, m.eps, 0, src, y, w_add, out, w_norm.ptr if w_norm is not None else 0, rows)
+        return ffi.StreamDesc(m.width, m.groups, m.eps, int(plain), src, y, w_add, out, w_norm.ptr if w_norm is not None else 0, rows)
 
-    def dense(self, desc: ffi.DenseDesc, w_norm: Tensor) -> None:
-        """A projection of the normed stream."""
+    def dense(self, desc: ffi.DenseDesc, w_norm: Tensor | None) -> None:
+        """A projection of the normed stream, or (w_norm None) of the stream itself."""
         if self.fused:
-            desc.stream = self.stream(w_norm)
+            desc.stream = self.stream(w_norm, plain=w_norm is None)
         else:
-            self.call("jg_stream_norm", self.stream(w_norm), self.ws.h.ptr, self.model.ld_width, self.model.dt)
+            self.call("jg_stream_norm", self.stream(w_norm, plain=w_norm is None), self.ws.h.ptr, self.model.ld_width, self.model.dt)
             desc.x, desc.ldx = self.ws.h.ptr, self.model.ld_width
         self.call("jg_dense", desc)
 
-    def project(self, w: Matrix, w_norm: Tensor, bias: int = 0) -> int:
-        """Normed stream -> ws.proj; returns the row stride."""
+    def project(self, w: Matrix, w_norm: Tensor | None, bias: int = 0, **kw) -> int:
+        """Normed stream -> ws.proj; returns the row stride.  kw: further fields of the descriptor."""
         ld = round_up(w.N, 8)
-        self.dense(ffi.DenseDesc(self.model.dt, ffi.DENSE_STORE, w.N, w.K, 0, w.ld, ld, 0, 0.0, 0, 0, w.ptr, 0, 0, bias, 0, 0,
-                                 self.ws.proj.ptr), w_norm)
+        desc = ffi.DenseDesc(self.model.dt, ffi.DENSE_STORE, w.N, w.K, 0, w.ld, ld, 0, 0.0, 0, 0, w.ptr, 0, 0, bias, 0, 0, self.ws.proj.ptr)
+        for k, v in kw.items():
+            setattr(desc, k, v)
+        self.dense(desc, w_norm)
         return ld
 
-    def output(self, w: Matrix, x: int, ldx: int, w_add: Tensor, bias: int = 0) -> None:
-        """The sublayer's last projection -> ws.y, to be normed with w_add and added to the stream."""
+    def output(self, w: "Matrix | Columns", x: int, ldx: int, w_add: Tensor, bias: int = 0, gated: ffi.GatedDesc | None = None, lead: int = 0) -> None:
+        """The sublayer's last projection -> ws.y, to be normed with w_add and added to the stream.  `gated`: columns of x from
+        `lead` on are still to be made from a linear recurrence's read-out."""
         m = self.model
-        self.call("jg_dense", ffi.DenseDesc(m.dt, ffi.DENSE_STORE, w.N, w.K, ldx, w.ld, m.width, 1, 0.0, 0, x, w.ptr, 0, 0, bias, 0, 0,
-                                            self.ws.y.ptr))
+        desc = ffi.DenseDesc(m.dt, ffi.DENSE_STORE, w.N, w.K, ldx, w.ld, m.width, 1, 0.0, 0, x, w.ptr, 0, 0, bias, 0, 0, self.ws.y.ptr)
+        if gated is not None:
+            desc.gated, desc.lead = gated, lead
+        self.call("jg_dense", desc)
         self.pending = w_add
 
     def finish_layer(self) -> None:
@@ -257,6 +333,162 @@ class LatentAttention:
         p.output(self.o, p.ws.act.ptr, self.act_ld, w_add)
 
 
+# ------------------------------------------------------------------------------------------------ branches
+class WindowBranch:
+    """Grouped-head attention over a sliding window and the first tokens; query and key norms over the whole projection."""
+
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str):
+        self.name, self.H, self.G, self.dim, self.vd = name, *(int(cfg[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+        if self.H % self.G:
+            raise ValueError(f"{self.H} heads do not divide among {self.G} key / value heads")
+        mask, rot = cfg.get("mask") or {}, cfg["rot"]
+        self.window, self.keep, self.scale = int(mask.get("size") or 0), int(mask.get("keep_first") or 0), float(cfg["scale"])
+        self.pairs = int(rot["dims"]) // 2
+        if 2 * self.pairs > self.dim:
+            raise ValueError(f"rotary over {rot['dims']} of {self.dim} dimensions")
+        self.rot = m.shared_table(("yarn", rot["dims"], rot["base"], ()), lambda: yarn_table(int(rot["dims"]), float(rot["base"]), None, m.max_context))
+        self.ring = m.states.ring(self.G * (round_up(self.dim, 8) + round_up(self.vd, 8)), m.dtype, self.window, self.keep)
+        self.eps, self.dt, self.max_context = m.eps, m.dt, m.max_context
+        self.sizes = [("q", self.H * self.dim), ("k", self.G * self.dim), ("v", self.G * self.vd)]
+        self.parts, self.width, self.fp32, self.silu = [(name + n, r, 8) for n, r in self.sizes], self.H * self.vd, 0, None
+
+    def bind(self, m: "HybridTransformer", params: dict, w: Matrix) -> list[tuple[str, str, int]]:
+        self.col = [w.row0[self.name + n] for n in "qkv"]
+        self.qn, self.kn = (vector(m, params, [(self.name + n + ".norm", (r,))]) for n, r in self.sizes[:2])
+        return [(self.name + n + ".b", self.name + n, r) for n, r in self.sizes]
+
+    def desc(self) -> ffi.WindowDesc:
+        r = self.ring
+        return ffi.WindowDesc(self.dt, self.H, self.G, self.dim, self.vd, self.window, self.keep, 0, 0, r.page, r.pages_per_slot, r.pinned, self.pairs,
+                              self.max_context, self.eps, self.scale, 1.0, 0, 0, 0, 0, self.qn.ptr, self.kn.ptr, self.rot.ptr, r.pool.ptr, r.table.ptr)
+
+    def scratch(self, B: int, Sc: int) -> int:
+        n = C.c_uint64(0)
+        ffi.call("jg_window_scratch_bytes", C.byref(self.desc()), B, Sc, C.byref(n))
+        return n.value
+
+    def plan(self, p: Plan, proj, ld: int, scratch: int, nbytes: int, out: int, ldo: int, scale: float) -> None:
+        d = self.desc()
+        d.q, d.k, d.v = (proj(c) for c in self.col)
+        d.ldp, d.ldo, d.out, d.out_scale, d.scratch, d.scratch_bytes = ld, ldo, out, scale, scratch, nbytes
+        p.call("jg_window_attn", d)
+
+
+class LinearBranch:
+    """A linear recurrence with a matrix state per head, its norm and output gate.  `gated`: mLSTM (gates i and f, a norm per head);
+    else a constant decay per head, silu on queries, keys and values, one norm over all heads."""
+
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, gated: bool):
+        self.H, self.dim, self.vd = H, d, v = tuple(int(cfg[k]) for k in ("heads", "dim", "vdim"))
+        self.name, self.gated, self.eps, self.dt = name, gated, m.eps, m.dt
+        self.q_scale, self.cap = (d ** -0.5, float(cfg["gate_cap"])) if gated else (1.0, 0.0)
+        self.state = m.states.per_slot((H, v + int(gated), round_up(d, 4)), "float32")
+        self.m = m.states.per_slot((2, H), "float32") if gated else None
+        self.decay = None
+        if not gated:
+            if len(cfg["decay"]) != H:
+                raise ValueError(f"{len(cfg['decay'])} decays for {H} heads")
+            self.decay = Tensor(np.asarray(cfg["decay"], np.float32), device=m.dev)
+        self.parts = [(name + "q", H * d, 8), (name + "k", H * d, 8), (name + "v", H * v, 8), (name + "g", H * v, 8)]
+        if gated:
+            self.parts += [(name + "i", H, 8), (name + "f", H)]
+        self.width, self.fp32, self.silu = H * v, 2 * H if gated else 0, None if gated else (name + "q", name + "g")
+
+    def bind(self, m: "HybridTransformer", params: dict, w: Matrix) -> list[tuple[str, str, int]]:
+        self.col = [w.row0[self.name + n] for n in "qkvg"]
+        self.norm = vector(m, params, [(self.name + "norm", (self.width,))])
+        return [(self.name + n + ".b", self.name + n, self.H) for n in "if"] if self.gated else []
+
+    def _layout(self, rows: int) -> tuple[int, int, int]:
+        """Where the divisors and the tokens' weights begin behind the read-outs, and the end."""
+        n = C.c_uint64(0)
+        ffi.call("jg_linear_scratch_bytes", C.byref(ffi.LinearDesc(self.dt, self.H, self.dim, self.vd)), rows, C.byref(n))
+        den = round_up(4 * rows * self.width, 256)
+        tok = den + round_up(4 * rows * self.H, 256)
+        return den, tok, tok + n.value
+
+    def scratch(self, B: int, Sc: int) -> int:
+        return self._layout(B * Sc)[2]
+
+    def plan(self, p: Plan, proj, ld: int, scratch: int, nbytes: int, out: int, ldo: int, scale: float) -> ffi.GatedDesc:
+        den, tok, _ = self._layout(p.ws.cap)
+        q, k, v, g = (proj(c) for c in self.col)
+        d = ffi.LinearDesc(self.dt, self.H, self.dim, self.vd, ld, 0, self.q_scale, self.cap, q, k, v, 0, 0, self.state.ptr, 0, scratch + tok, scratch, 0)
+        if self.gated:
+            d.gates, d.m, d.den = p.ws.aux.ptr, self.m.ptr, scratch + den
+        else:
+            d.decay = self.decay.ptr
+        p.call("jg_linear_state", d)
+        return ffi.GatedDesc(self.dt, self.H, self.vd, self.H if self.gated else 1, ld, 0, self.eps, scale, scratch, d.den, g, self.norm.ptr)
+
+
+class Branches:
+    """A mixer of one or more branches that read the same input: one projection for all of them, one output projection over
+    their results side by side.  branches: (branch, factor on its result, name of its output matrix)."""
+
+    def __init__(self, m: "HybridTransformer", branches: list[tuple], params: dict):
+        self.branches = [b for b, _, _ in branches]
+        self.scales = [f for _, f, _ in branches]
+        last = self.branches[-1]
+        if any(b.fp32 for b in self.branches[:-1]):
+            raise ValueError("a branch with gates in 32 bits comes last")
+        parts = [q for b in self.branches for q in b.parts]
+        self.w = Matrix(m, params, parts, m.width)
+        bias = [q for b in self.branches for q in b.bind(m, params, self.w)]
+        self.bias = row_vector(m, params, self.w, bias) if bias else None
+        self.o = Columns(m, params, [(name, b.width) for b, _, name in branches], m.width)
+        self.at = [self.o.col0[name] for _, _, name in branches]
+        self.aux_ld, self.split = last.fp32, self.w.N - last.fp32 if last.fp32 else 0
+        silu = [b.silu for b in self.branches if b.silu]
+        if len(silu) > 1:
+            raise ValueError("one branch of a mixer may have silu in its projection")
+        self.silu = tuple(self.w.row0[n] for n in silu[0]) if silu else None
+        self.proj_ld, self.act_ld = round_up(self.w.N, 8), round_up(self.o.K, 8)
+
+    def _scratch(self, B: int, Sc: int) -> list[int]:
+        return [round_up(b.scratch(B, Sc), 256) for b in self.branches]
+
+    def scratch(self, B: int, Sc: int) -> int:
+        return sum(self._scratch(B, Sc))
+
+    def plan(self, p: Plan, w_norm: Tensor | None, w_add: Tensor) -> None:
+        m, ws = p.model, p.ws
+        size = ws.act.nbytes // ws.act.numel()
+        kw = {}
+        if self.silu:
+            kw.update(act=ffi.ACT_SILU, act_lo=self.silu[0], act_hi=self.silu[1])
+        if self.split:
+            kw.update(split=self.split, y2=ws.aux.ptr, ld2=self.aux_ld)
+        ld = p.project(self.w, w_norm, self.bias.ptr if self.bias is not None else 0, **kw)
+        scratch, gated = ws.scratch.ptr, None
+        for i, (b, f, at, n) in enumerate(zip(self.branches, self.scales, self.at, self._scratch(ws.B, max(1, ws.cap // ws.B)))):
+            out = ws.act.ptr + at * size
+            gated = b.plan(p, lambda c: ws.proj.ptr + c * size, ld, scratch, n, out, self.act_ld, f)
+            scratch += n
+            if gated is not None and not (p.fused and i == len(self.branches) - 1):
+                p.call("jg_gated_norm", gated, out, self.act_ld)
+                gated = None
+        p.output(self.o, ws.act.ptr, self.act_ld, w_add, gated=gated, lead=self.at[-1])
+
+
+def window_attention(m: "HybridTransformer", cfg: dict, name: str, params: dict) -> Branches:
+    return Branches(m, [(WindowBranch(m, cfg, name), 1.0, name + "o")], params)
+
+
+def lightning(m: "HybridTransformer", cfg: dict, name: str, params: dict) -> Branches:
+    return Branches(m, [(LinearBranch(m, cfg, name, False), 1.0, name + "o")], params)
+
+
+def mlstm(m: "HybridTransformer", cfg: dict, name: str, params: dict) -> Branches:
+    return Branches(m, [(LinearBranch(m, cfg, name, True), 1.0, name + "o")], params)
+
+
+def parallel(m: "HybridTransformer", cfg: dict, name: str, params: dict) -> Branches:
+    return Branches(m, [(WindowBranch(m, cfg["left"], name + "left."), float(cfg["left_scale"]), name + "left.o"),
+                        (LinearBranch(m, cfg["right"], name + "right.", False), float(cfg["right_scale"]), name + "right.o")], params)
+
+
+# ------------------------------------------------------------------------------------------------ feed-forwards
 class DenseGLU:
     def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
         f = int(cfg["ff"])
@@ -274,29 +506,83 @@ class DenseGLU:
         p.output(self.down, p.ws.ffn.ptr, self.ffn_ld, w_add, self.down_b.ptr)
 
 
-MIXERS = {"mingru": MinGRU, "latent_attention": LatentAttention, "delta": GatedDelta}
-FEED_FORWARDS = {"dense": DenseGLU}
+class SquaredReLU:
+    """W_down max(W_up h, 0)^2."""
+
+    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
+        f = int(cfg["ff"])
+        self.up, self.down = Matrix(m, params, [(name + "up", f)], m.width), Matrix(m, params, [(name + "down", m.width)], f)
+        self.ffn_ld = round_up(f, 8)
+
+    def plan(self, p: Plan, w_norm: Tensor | None, w_add: Tensor) -> None:
+        u = self.up
+        d = ffi.DenseDesc(p.model.dt, ffi.DENSE_STORE, u.N, u.K, 0, u.ld, self.ffn_ld, 0, 0.0, 0, 0, u.ptr, 0, 0, 0, 0, 0, p.ws.ffn.ptr)
+        d.act = ffi.ACT_RELU2
+        p.dense(d, w_norm)
+        p.output(self.down, p.ws.ffn.ptr, self.ffn_ld, w_add)
+
+
+class TokenSide:
+    """Per-layer token input: W_proj (gelu(W_gate x) * e), e the layer's part of the token's row in `table`."""
+
+    def __init__(self, m: "HybridTransformer", table: Matrix, layer: int, dim: int, name: str, params: dict):
+        self.table, self.at, self.vocab = table, layer * dim, m.vocab_size
+        self.gate, self.proj = Matrix(m, params, [(name + "gate", dim)], m.width), Matrix(m, params, [(name + "proj", m.width)], dim)
+        self.norm = vector(m, params, [(name + "norm", (m.width,))])
+        self.ld = round_up(dim, 8)
+
+    def plan(self, p: Plan) -> None:
+        g, t, out = self.gate, self.table, p.ws.side.ptr
+        d = ffi.DenseDesc(p.model.dt, ffi.DENSE_STORE, g.N, g.K, 0, g.ld, self.ld, 0, 0.0, 0, 0, g.ptr, 0, 0, 0, 0, 0, out)
+        d.act, d.side, d.tokens, d.ld_side, d.col_side, d.vocab = ffi.ACT_GELU_SIDE, t.ptr, p.ws.tokens.ptr, t.ld, self.at, self.vocab
+        p.dense(d, None)
+        p.output(self.proj, out, self.ld, self.norm)
+
+
+MIXERS = {"mingru": MinGRU, "latent_attention": LatentAttention, "delta": GatedDelta, "window_attention": window_attention, "lightning": lightning,
+          "mlstm": mlstm, "parallel": parallel}
+
+
+@dataclass(frozen=True)
+class Design:
+    """What an architecture fixes beyond the sizes and constants of its configuration."""
+    norms: tuple = (("norm1", "norm1b"), ("norm2", "norm2b"))  # before (None: the sublayer reads the stream) and after mixer and feed-forward
+    norm_offset: float = 0.0        # these norms' weights, and the final one's, are stored minus this
+    tied_head: bool = False         # logits from the embedding table
+    feed_forwards: tuple = (("dense", DenseGLU),)
+
+
+DESIGNS = {"Matulorn": Design(),
+           "Rigazen": Design(norms=((None, "norm1"), (None, "norm2")), norm_offset=1.0, tied_head=True, feed_forwards=(("dense", SquaredReLU),))}
 
 
 class Layer:
-    def __init__(self, m: "HybridTransformer", cfg: dict, name: str, params: dict):
-        D = m.width
+    def __init__(self, m: "HybridTransformer", cfg: dict, index: int, params: dict):
+        name, kinds = f"l{index}.", dict(m.design.feed_forwards)
         if cfg["type"] not in MIXERS:
             raise ValueError(f"unknown mixer {cfg['type']!r} (known: {', '.join(MIXERS)})")
         self.mixer = MIXERS[cfg["type"]](m, cfg["mixer"], name + "mix.", params)
-        self.norm1, self.norm1b = (vector(m, params, [(name + n, (D,))]) for n in ("norm1", "norm1b"))
-        self.mlp = None
+        self.norm1 = self._norms(m, name, m.design.norms[0], params)
+        self.mlp = self.side = None
         if cfg.get("mlp"):
             kind = cfg["mlp"].get("kind", "dense")
-            if kind not in FEED_FORWARDS:
-                raise ValueError(f"unknown feed-forward {kind!r} (known: {', '.join(FEED_FORWARDS)})")
-            self.mlp = FEED_FORWARDS[kind](m, cfg["mlp"], name + "mlp.", params)
-            self.norm2, self.norm2b = (vector(m, params, [(name + n, (D,))]) for n in ("norm2", "norm2b"))
+            if kind not in kinds:
+                raise ValueError(f"unknown feed-forward {kind!r} (known: {', '.join(kinds)})")
+            self.mlp = kinds[kind](m, cfg["mlp"], name + "mlp.", params)
+            self.norm2 = self._norms(m, name, m.design.norms[1], params)
+        if m.side is not None:
+            self.side = TokenSide(m, m.side, index, m.side_dim, name + "side.", params)
+
+    @staticmethod
+    def _norms(m: "HybridTransformer", name: str, which: tuple, params: dict) -> list:
+        return [vector(m, params, [(name + n, (m.width,))], offset=m.design.norm_offset) if n else None for n in which]
 
     def plan(self, p: Plan) -> None:
-        self.mixer.plan(p, self.norm1, self.norm1b)
+        self.mixer.plan(p, *self.norm1)
         if self.mlp is not None:
-            self.mlp.plan(p, self.norm2, self.norm2b)
+            self.mlp.plan(p, *self.norm2)
+        if self.side is not None:
+            self.side.plan(p)
         p.finish_layer()
 
 
@@ -316,6 +602,9 @@ class _Rows:
         self.act = Tensor.zeros((cap, max(l.mixer.act_ld for l in layers)), m.dtype, dev)
         ffn = max((l.mlp.ffn_ld for l in layers if l.mlp is not None), default=0)
         self.ffn = Tensor.zeros((cap, ffn * (2 if m.dtype == "float32" else 1)), m.dtype, dev) if ffn else None
+        aux = max(getattr(l.mixer, "aux_ld", 0) for l in layers)  # columns of the projection kept in 32 bits
+        self.aux = Tensor.zeros((cap, aux), "float32", dev) if aux else None
+        self.side = Tensor.zeros((cap, layers[0].side.ld), m.dtype, dev) if m.side is not None else None
         Sc = max(1, cap // B)
         self.scratch = Tensor.empty((max(max(l.mixer.scratch(B, s) for l in layers for s in {1, Sc}), 16),), "uint8", dev)
         self.batch = ffi.Batch(B, 1, self.pos.ptr, self.seq.ptr, -1, 0)
@@ -345,7 +634,8 @@ class _Step(_Rows):
 
 
 class HybridTransformer(Decoder):
-    """A decoder over `config` (`width`, `vocab`, `norm`, `layers`).  dtype: 'bfloat16' or 'float32'."""
+    """A decoder over `config` (`width`, `vocab`, `norm`, `layers`; optional: `embedding.scale`, `token_side.dim`) under the
+    conventions of its `architecture` (DESIGNS).  dtype: 'bfloat16' or 'float32'."""
 
     def __init__(self, config: dict, dtype: str = "bfloat16", max_context: int = 8192, max_batch: int = 1, jit: bool = True, device=None,
                  page_size: int = 64, max_rows: int = 2048):
@@ -354,6 +644,10 @@ class HybridTransformer(Decoder):
         dev = _dev(device)
         self.dev, self.dtype, self.dt = dev, dtype, DTYPES[dtype]
         self.width, self.vocab_size = int(config["width"]), int(config["vocab"])
+        name = config.get("architecture", "Matulorn")
+        if name not in DESIGNS:
+            raise ValueError(f"unknown architecture {name!r} (known: {', '.join(DESIGNS)})")
+        self.design = DESIGNS[name]
         self.groups, self.eps = int(config["norm"].get("groups", 1)), float(config["norm"]["eps"])
         if self.width % self.groups:
             raise ValueError(f"width {self.width} does not divide into {self.groups} norm groups")
@@ -363,9 +657,13 @@ class HybridTransformer(Decoder):
         self._tables: dict = {}
         self.params: dict[str, Param] = {}
         self.embed = Matrix(self, self.params, [("embed", self.vocab_size)], self.width)
-        self.layers = [Layer(self, c, f"l{i}.", self.params) for i, c in enumerate(config["layers"])]
-        self.norm = vector(self, self.params, [("final.norm", (self.width,))])
-        self.head = Matrix(self, self.params, [("head", self.vocab_size)], self.width)
+        self.embed_scale = float((config.get("embedding") or {}).get("scale", 1.0))
+        self.side, self.side_dim = None, int((config.get("token_side") or {}).get("dim", 0))
+        if self.side_dim:
+            self.side = Matrix(self, self.params, [("side.embed", self.vocab_size)], self.side_dim * len(config["layers"]))
+        self.layers = [Layer(self, c, i, self.params) for i, c in enumerate(config["layers"])]
+        self.norm = vector(self, self.params, [("final.norm", (self.width,))], offset=self.design.norm_offset)
+        self.head = self.embed if self.design.tied_head else Matrix(self, self.params, [("head", self.vocab_size)], self.width)
         self._steps: dict[int, _Step] = {}
         self._chunks: dict[tuple[int, int], _Rows] = {}
         self._row_slots: list[int] = []
@@ -422,7 +720,7 @@ class HybridTransformer(Decoder):
             p = Plan(self, ws, *key)
             if fused and len(ws.x) < 2:
                 ws.x.append(Tensor.zeros(ws.x[0].shape, "float32", self.dev))
-            p.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size)
+            p.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size, self.embed_scale)
             for layer in self.layers:
                 layer.plan(p)
             ws.plans[key] = p
@@ -581,7 +879,7 @@ class HybridTransformer(Decoder):
         out, peek = [], Plan(self, ws, S <= 2, S == 1)
         if S <= 2 and len(ws.x) < 2:
             ws.x.append(Tensor.zeros(ws.x[0].shape, "float32", self.dev))
-        peek.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size)
+        peek.call("jg_stream_embed", ws.x[0].ptr, ws.tokens.ptr, self.embed.ptr, self.dt, self.width, self.embed.ld, self.vocab_size, self.embed_scale)
         res = Tensor.zeros((ws.cap, self.width), "float32", self.dev)
         for layer in self.layers:
             layer.plan(peek)

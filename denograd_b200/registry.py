@@ -18,11 +18,13 @@ def _weights_path(folder: str) -> str:
     raise FileNotFoundError(f"{folder}: no model.safetensors")
 
 
-def _matulorn(config: dict, folder: str, dtype: str | None, max_context: int, max_batch: int, **kw):
+def _hybrid(config: dict, folder: str, dtype: str | None, max_context: int, max_batch: int, **kw):
     from . import ffi
     ffi.use_component(HYBRID)
     from .matulorn import Matulorn
-    return Matulorn(config, dtype or "bfloat16", max_context, max_batch, **kw).load_weights(_weights_path(folder))
+    from .rigazen import Rigazen
+    cls = {c.architecture: c for c in (Matulorn, Rigazen)}[architecture(config)]
+    return cls(config, dtype or "bfloat16", max_context, max_batch, **kw).load_weights(_weights_path(folder))
 
 
 def _llama(config: dict, folder: str, dtype: str | None, max_context: int, max_batch: int, **kw):
@@ -38,7 +40,7 @@ def _llama(config: dict, folder: str, dtype: str | None, max_context: int, max_b
 
 
 # architecture name in config.json -> loader
-ARCHITECTURES = {"Matulorn": _matulorn, "LlamaForCausalLM": _llama}
+ARCHITECTURES = {"Matulorn": _hybrid, "Rigazen": _hybrid, "LlamaForCausalLM": _llama}
 
 
 def architecture(config: dict) -> str:

@@ -94,13 +94,13 @@ def fill_hybrid(model, base_seed: int = BASE_SEED) -> None:
         seed = name_seed(name, base_seed)
         if p.ld is not None:
             t = p.tensor
-            t.dev.call("jg_fill_normal", t.ptr, model.dt, seed, p.shape[0], p.shape[1], p.ld, WEIGHT_STD)
+            t.dev.call("jg_fill_normal", p.ptr, model.dt, seed, p.shape[0], p.shape[1], p.ld, WEIGHT_STD)
             continue
         n = int(np.prod(p.shape))
         u = (_word(seed, np.arange(n, dtype=np.uint64)) >> np.uint64(40)).astype(np.float64) / 2.0 ** 24
         leaf = name.rsplit(".", 1)[-1]
         if "norm" in leaf:
-            v = np.ones(n)
+            v = np.full(n, 1.0 - p.offset)
         elif leaf == "A_log":
             v = np.log(0.02 + u)
         elif leaf == "conv":

@@ -87,7 +87,7 @@ export const SYMBOLS = {
   jg_fill_scale_f16: fn([ptr, u64, u64, u64, u64, f32]),
   jg_fill_const_f16: fn([ptr, u64, u64, f32]),
   jg_fill_normal: fn([ptr, u64, i32, u64, u64, u64, u64, f32]),
-  jg_stream_embed: fn([ptr, buf, u64, u64, u64, i32, i32, i32, i32]),
+  jg_stream_embed: fn([ptr, buf, u64, u64, u64, i32, i32, i32, i32, f32]),
   jg_stream_norm: fn([ptr, buf, buf, u64, i32, i32]),
   jg_dense: fn([ptr, buf, buf]),
   jg_mingru_scan: fn([ptr, buf, buf]),
@@ -95,6 +95,11 @@ export const SYMBOLS = {
   jg_delta_rule: fn([ptr, buf, buf]),
   jg_latent_scratch_bytes: fn([buf, i32, i32, buf]),
   jg_latent_attn: fn([ptr, buf, buf]),
+  jg_linear_scratch_bytes: fn([buf, i32, buf]),
+  jg_linear_state: fn([ptr, buf, buf]),
+  jg_gated_norm: fn([ptr, buf, buf, u64, i32]),
+  jg_window_scratch_bytes: fn([buf, i32, i32, buf]),
+  jg_window_attn: fn([ptr, buf, buf]),
   jg_sample_f32: fn([ptr, u64, u64, u64, u64, i32, i32, f32, i32, f32, f32, f32]),
   jg_fill_normal_f16_2d: fn([ptr, u64, u64, u64, u64, u64, u64, u64, f32]),
   jg_fill_uniform_i8_2d: fn([ptr, u64, u64, u64, u64, u64, u64, u64]),

@@ -397,6 +397,11 @@ int jg_dequant_nf4_f16(jg_dev* dev, uint64_t dst, uint64_t w, uint64_t scale, in
 #define JG_DENSE_GLU 1     /* g = min(x W0^T + b0, limit), u = clamp(x W1^T + b1, +-limit); y = g sigmoid(1.702 g) (u + 1) */
 #define JG_DENSE_MINGRU 2  /* W0, W1, W2 = update gate, candidate, output gate: one token of jg_mingru_scan per row */
 #define JG_DENSE_LOGITS 3  /* y = x W0^T in fp32, and (value, lowest index) keys for jg_argmax_finalize */
+/* activations of JG_DENSE_STORE, on columns [act_lo, act_hi) (act_hi = 0: all) */
+#define JG_ACT_NONE 0
+#define JG_ACT_SILU 1
+#define JG_ACT_RELU2 2       /* max(v, 0)^2 */
+#define JG_ACT_GELU_SIDE 3   /* gelu_tanh(v) * side[tokens[row]][col_side + column] */
 
 typedef struct {
   int32_t B, Sc;
@@ -405,23 +410,37 @@ typedef struct {
   int32_t reserved;
 } jg_batch;
 
-/* x <- x + norm(y) * w_add (y = 0: nothing), stored to x_out (0: not); h = norm(x) * w_norm (0: nothing).  norm divides each
- * of `groups` equal parts of a row by sqrt(mean(part^2) + eps).  rows (0 = identity): device int32 row numbers into x, y. */
+/* x <- x + norm(y) * w_add (y = 0: nothing), stored to x_out (0: not); h = norm(x) * w_norm (0: nothing), or x itself with
+ * `plain`.  norm divides each of `groups` equal parts of a row by sqrt(mean(part^2) + eps).  rows (0 = identity): device
+ * int32 row numbers into x, y. */
 typedef struct {
   int32_t width, groups;
   float eps;
-  int32_t reserved;
+  int32_t plain;
   uint64_t x, y, w_add, x_out, w_norm, rows;
 } jg_stream_desc;
 
-/* x = 0: the rows are h of `stream` (1-2 rows; x_out must be another buffer than x).  fp32 GLU of 3+ rows uses the rows M
- * .. 2M of y as scratch. */
+/* What follows a linear recurrence: out[i] = o[i] / den[head] / rms(group) * norm_w[i] * sigmoid(gate[i]) * scale over the
+ * heads * vdim values of a row (den = 0: no division; `groups` equal parts, each with its own root mean square; eps inside).
+ * o: fp32 [R][heads * vdim], den: fp32 [R][heads], gate: T, rows ldp apart. */
+typedef struct {
+  int32_t dtype, heads, vdim, groups, ldp, reserved;
+  float eps, scale;
+  uint64_t o, den, gate, norm_w;
+} jg_gated_desc;
+
+/* x = 0: the rows are h of `stream` (1-2 rows; x_out must be another buffer than x).  gated.o != 0 (1-2 rows): the first
+ * `lead` columns come from x, the others are jg_gated_norm's.  fp32 GLU of 3+ rows uses the rows M .. 2M of y as scratch.
+ * STORE: columns from `split` on (0: none) go to y2 in fp32, [M][ld2], column `split` first. */
 typedef struct {
   int32_t dtype, epilogue, N, K, ldx, ldw, ldy, out_f32;
   float limit;
   int32_t reserved;
   uint64_t x, w0, w1, w2, b0, b1, b2, y, key, state;
   jg_stream_desc stream;
+  jg_gated_desc gated;
+  int32_t act, act_lo, act_hi, split, ld2, ld_side, col_side, vocab, lead, reserved2;
+  uint64_t y2, side, tokens;
 } jg_dense_desc;
 
 /* minGRU: z = sigmoid(zin), c = u >= 0 ? u + 1/2 : sigmoid(u); S <- (1 - z) S + z c; out = S silu(g), element by element.
@@ -458,9 +477,36 @@ typedef struct {
   uint64_t scratch_bytes;
 } jg_latent_desc;
 
-/* embedding rows (T [vocab][ld]) widened into the fp32 residual stream */
+/* Linear recurrence with a matrix state per head: S <- a S + b k v^T, o = S^T (q_scale q).
+ * Constant decay (gates = 0): a = decay[head], b = 1.  Gated (mLSTM): i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)),
+ * m' = max(f + m, i) from m = 0, a = exp(f + m - m'), b = exp(i - m'); a further column of S sums k alone (n), and
+ * den = max(|n . q|, exp(-m')) + 1e-6.  q, k, v: addresses inside T rows ldp apart (heads x dim, heads x dim, heads x vdim).
+ * gates: fp32 [R][2 heads] = z_i | z_f.  state: fp32 [slots][heads][vdim (+ 1 when gated)][dim4], m: fp32 [slots][2][heads]
+ * (entry: position & 1).  o: fp32 [R][heads * vdim] before the division, den: fp32 [R][heads].
+ * scratch: jg_linear_scratch_bytes(desc, R). */
+typedef struct {
+  int32_t dtype, heads, dim, vdim, ldp, reserved;
+  float q_scale, cap;
+  uint64_t q, k, v, gates, decay, state, m, scratch, o, den;
+} jg_linear_desc;
+
+/* Attention over a sliding window and the sequence's first tokens, grouped heads, normed queries and keys.  q (heads x dim),
+ * k (kv_heads x dim), v (kv_heads x vdim): addresses inside T rows ldp apart.  q and k: each divided by the root mean square
+ * of all of its values in the row, times q_norm / k_norm (fp32), then pairs (i, i + rot_pairs) of every head turn by the
+ * angles of `rot`, fp32 [rot_rows][rot_pairs][2] (cos, sin).  Position i sees j <= i with i - j < window (0: any) or j < keep.
+ * out: T [R][ldo], times out_scale.  Cache row: kv_heads keys of dim8, then kv_heads values of vdim8 (sizes rounded up to 8,
+ * zeros behind).  Positions of the first `pinned` pages stay on block_table[slot][p / page]; page i >= pinned lies on
+ * block_table[slot][pinned + (i - pinned) % (pages_per_slot - pinned)]. */
+typedef struct {
+  int32_t dtype, heads, kv_heads, dim, vdim, window, keep, ldp, ldo, page, pages_per_slot, pinned, rot_pairs, rot_rows;
+  float eps, scale, out_scale;
+  int32_t reserved;
+  uint64_t q, k, v, q_norm, k_norm, rot, pool, block_table, scratch, scratch_bytes, out;
+} jg_window_desc;
+
+/* embedding rows (T [vocab][ld]), times scale, widened into the fp32 residual stream */
 int jg_stream_embed(jg_dev* dev, const jg_batch* batch, uint64_t out, uint64_t tokens, uint64_t table, int32_t dtype, int32_t dim,
-                    int32_t ld, int32_t vocab);
+                    int32_t ld, int32_t vocab, float scale);
 int jg_stream_norm(jg_dev* dev, const jg_batch* batch, const jg_stream_desc* s, uint64_t h, int32_t ldh, int32_t dtype);
 int jg_dense(jg_dev* dev, const jg_batch* batch, const jg_dense_desc* d);
 int jg_mingru_scan(jg_dev* dev, const jg_batch* batch, const jg_mingru_desc* d);
@@ -468,6 +514,11 @@ int jg_delta_scratch_floats(const jg_delta_desc* d, int32_t rows, uint64_t* out)
 int jg_delta_rule(jg_dev* dev, const jg_batch* batch, const jg_delta_desc* d);
 int jg_latent_scratch_bytes(const jg_latent_desc* d, int32_t B, int32_t Sc, uint64_t* out);
 int jg_latent_attn(jg_dev* dev, const jg_batch* batch, const jg_latent_desc* d);
+int jg_linear_scratch_bytes(const jg_linear_desc* d, int32_t rows, uint64_t* out);
+int jg_linear_state(jg_dev* dev, const jg_batch* batch, const jg_linear_desc* d);
+int jg_gated_norm(jg_dev* dev, const jg_batch* batch, const jg_gated_desc* d, uint64_t out, int32_t ldo);
+int jg_window_scratch_bytes(const jg_window_desc* d, int32_t B, int32_t Sc, uint64_t* out);
+int jg_window_attn(jg_dev* dev, const jg_batch* batch, const jg_window_desc* d);
 /* jg_sample over fp32 logits */
 int jg_sample_f32(jg_dev* dev, uint64_t tokens_out, uint64_t logits, uint64_t u, uint64_t alpha_counter, int32_t B, int32_t V,
                   float temp, int32_t k, float p, float af, float ap);

@@ -107,14 +107,15 @@ def test_descriptor_sizes_match_the_header():
     from tests.test_abi import HEADER
     src = re.sub(r"/\*.*?\*/", "", open(HEADER).read(), flags=re.S)
     for name, cls in (("jg_batch", ffi.Batch), ("jg_stream_desc", ffi.StreamDesc), ("jg_dense_desc", ffi.DenseDesc), ("jg_mingru_desc", ffi.MinGruDesc),
-                      ("jg_delta_desc", ffi.DeltaDesc), ("jg_latent_desc", ffi.LatentDesc)):
+                      ("jg_delta_desc", ffi.DeltaDesc), ("jg_latent_desc", ffi.LatentDesc), ("jg_gated_desc", ffi.GatedDesc),
+                      ("jg_linear_desc", ffi.LinearDesc), ("jg_window_desc", ffi.WindowDesc)):
         body = re.search(r"typedef struct \{([^}]*)\} " + name + ";", src).group(1)
         want = []
         for decl in body.split(";"):
             if decl.strip():
                 kind, rest = decl.split(None, 1)
                 want += [(n.strip(), kind) for n in rest.split(",")]
-        kinds = {C.c_int32: "int32_t", C.c_uint64: "uint64_t", C.c_float: "float", ffi.StreamDesc: "jg_stream_desc"}
+        kinds = {C.c_int32: "int32_t", C.c_uint64: "uint64_t", C.c_float: "float", ffi.StreamDesc: "jg_stream_desc", ffi.GatedDesc: "jg_gated_desc"}
         assert [(n, kinds[t]) for n, t in cls._fields_] == want, name
 
 

@@ -42,7 +42,7 @@ def mlstm(h, p, cfg, eps, faults=()):
     gate_i = cap * np.tanh((h @ p["i"].T + p["i.b"]) / cap)
     gate_f = log_sigmoid(cap * np.tanh((h @ p["f"].T + p["f.b"]) / cap))
     S, n = np.zeros((H, d, vd), F), np.zeros((H, d), F)
-    m = np.full(H, -1e30 if "m_from_minus_infinity" in faults else 0.0)
+    m = np.zeros(H, F)
     o = np.empty((T, H, vd), F)
     for t in range(T):
         if "state_lost" in faults and t % 7 == 3:

@@ -24,7 +24,7 @@ in the KV cache, greedy decoding.  One JSON line is printed by rank 0:
   cpu_baseline  the CPU restatement of the reference's CLANG path (oracle/), timed on this host's cores on a bounded
              sample: full-width 1-, 4- and 8-layer slices with 512 positions in the cache, extrapolated in depth.
 
-`--hybrid SIZE` runs another workload in place of the default one: a layer-list model (Matulorn) with the layer sizes of the
+`--hybrid SIZE` runs another workload in place of the default one: layer-list models (`--hybrid-models`) with the layer sizes of the
 Llama of that size, prefill and decode at several batch sizes, call by call, with the Llama at the same sizes beside it.
 
 `--impl reference` times that CPU restatement as the reference arm (the reference itself needs a JS runtime and
@@ -567,12 +567,21 @@ def run_gpu(args) -> None:
 
 
 # ------------------------------------------------------------------------------------------------ layer-list models
-def hybrid_config(size: str, layers: int = 0) -> dict:
-    """A Matulorn configuration with the layer sizes of the Llama of that size: same width, depth, feed-forward and
-    vocabulary; of every four layers one is latent attention, one minGRU and two are gated delta."""
+def hybrid_config(size: str, layers: int = 0, design: str = "matulorn") -> dict:
+    """A configuration with the layer sizes of the Llama of that size: same width, depth, feed-forward and vocabulary.
+    matulorn: of every four layers one is latent attention, one minGRU and two are gated delta.  rigazen: mLSTM layers and
+    parallel ones (window attention with the Llama's heads beside lightning attention) take turns."""
     p, _ = arch(size)
     d, ff, L = p["dim"], p["hidden_dim"], layers or p["n_layers"]
     H = d // 128
+    if design == "rigazen":
+        mixers = [{"type": "mlstm", "mixer": {"heads": d // 512, "dim": 256, "vdim": 512, "gate_cap": 15.0}},
+                  {"type": "parallel", "mixer": {
+                      "left": {"heads": H, "kv_heads": p["n_kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096, "keep_first": 64},
+                               "rot": {"base": 500000.0, "dims": 128}},
+                      "right": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1 - 8.0 * (i + 1) / H) for i in range(H)]}, "left_scale": 0.8, "right_scale": 1.1}}]
+        return {"architecture": "Rigazen", "width": d, "vocab": p["vocab_size"], "norm": {"eps": 1e-6}, "embedding": {"scale": d ** 0.5}, "token_side": {"dim": 256},
+                "layers": [dict(mixers[i % 2], mlp={"kind": "dense", "ff": ff}) for i in range(L)]}
     mixers = [{"type": "latent_attention", "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "mask": {"size": 4096},
                                                      "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}},
                                                      "scale": 192 ** -0.5}},
@@ -587,9 +596,20 @@ def hybrid_config(size: str, layers: int = 0) -> dict:
 def hybrid_bytes(cfg: dict, B: int, T: float) -> float:
     """Bytes one decode step has to move: every matrix once, recurrent state read and written, the cached window read."""
     d, by = cfg["width"], 2.0 * cfg["vocab"] * cfg["width"]
+    ffs = 2 if cfg["architecture"] == "Rigazen" else 3
     for lc in cfg["layers"]:
         m = lc["mixer"]
-        if lc["type"] == "mingru":
+        by += 4.0 * d * (cfg.get("token_side") or {"dim": 0})["dim"]
+        if lc["type"] in ("mlstm", "parallel"):
+            r = m["right"] if lc["type"] == "parallel" else m
+            by += 2.0 * d * r["heads"] * (2 * r["dim"] + 3 * r["vdim"]) + B * 8.0 * r["heads"] * r["dim"] * r["vdim"]
+            if lc["type"] == "mlstm":
+                by += 4.0 * d * r["heads"] + B * 8.0 * r["heads"] * r["dim"]
+            else:
+                a = m["left"]
+                by += 2.0 * d * (a["heads"] * (a["dim"] + a["vdim"]) + a["kv_heads"] * (a["dim"] + a["vdim"]))
+                by += B * 2.0 * min(T, a["mask"]["size"] + a["mask"]["keep_first"]) * a["kv_heads"] * (a["dim"] + a["vdim"])
+        elif lc["type"] == "mingru":
             by += 2.0 * 4 * d * m["width"] + B * 8.0 * m["width"]
         elif lc["type"] == "delta":
             qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
@@ -598,7 +618,7 @@ def hybrid_bytes(cfg: dict, B: int, T: float) -> float:
             H, r = m["heads"], m["kv_rank"]
             by += 2.0 * (d * (H * (m["dim"] + m["rot_dim"]) + r + m["rot_dim"]) + H * (m["dim"] + m["vdim"]) * r + d * H * m["vdim"])
             by += B * 2.0 * min(T, m["mask"]["size"]) * (r + m["rot_dim"])
-        by += 2.0 * 3 * d * lc["mlp"]["ff"]
+        by += 2.0 * ffs * d * lc["mlp"]["ff"]
     return by
 
 
@@ -606,9 +626,24 @@ def hybrid_flops(cfg: dict, B: int, S: int) -> float:
     """Flops of a prompt of S tokens from an empty state: projections on all rows, the head on the last ones, windowed causal
     attention over expanded keys and values, 8 flops per state element and token of the delta rule."""
     d, fl = cfg["width"], 2.0 * B * cfg["vocab"] * cfg["width"]
+    ffs, side = 2.0 if cfg["architecture"] == "Rigazen" else 3.0, (cfg.get("token_side") or {"dim": 0})["dim"]
+
+    def pairs(W: int) -> float:
+        return S * S / 2.0 if S <= W else W * W / 2.0 + (S - W) * float(W)
+
     for lc in cfg["layers"]:
         m = lc["mixer"]
-        if lc["type"] == "mingru":
+        if lc["type"] in ("mlstm", "parallel"):
+            r = m["right"] if lc["type"] == "parallel" else m
+            w = d * r["heads"] * (2.0 * r["dim"] + 3 * r["vdim"]) + 2.0 * d * side
+            fl += 4.0 * B * S * r["heads"] * r["dim"] * r["vdim"]
+            if lc["type"] == "mlstm":
+                w += 2.0 * d * r["heads"]
+            else:
+                a = m["left"]
+                w += d * (a["heads"] + a["kv_heads"]) * (a["dim"] + a["vdim"])
+                fl += 2.0 * B * a["heads"] * pairs(a["mask"]["size"]) * (a["dim"] + a["vdim"])
+        elif lc["type"] == "mingru":
             w = 4.0 * d * m["width"]
         elif lc["type"] == "delta":
             qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
@@ -617,9 +652,8 @@ def hybrid_flops(cfg: dict, B: int, S: int) -> float:
         else:
             H, r, W = m["heads"], m["kv_rank"], m["mask"]["size"]
             w = d * (H * (m["dim"] + m["rot_dim"]) + r + m["rot_dim"]) + H * (m["dim"] + m["vdim"]) * r + d * H * m["vdim"]
-            pairs = S * S / 2.0 if S <= W else W * W / 2.0 + (S - W) * float(W)
-            fl += 2.0 * B * H * pairs * (m["dim"] + m["rot_dim"] + m["vdim"])
-        fl += 2.0 * B * S * (w + 3.0 * d * lc["mlp"]["ff"])
+            fl += 2.0 * B * H * pairs(W) * (m["dim"] + m["rot_dim"] + m["vdim"])
+        fl += 2.0 * B * S * (w + ffs * d * lc["mlp"]["ff"])
     return fl
 
 
@@ -652,8 +686,11 @@ def call_work(name: str, a: tuple, B: int, Sc: int, T: float, p: dict | None) ->
     if name == "jg_dense":
         d = a[2]
         n, R = {ffi.DENSE_GLU: 2, ffi.DENSE_MINGRU: 3}.get(d.epilogue, 1) * d.N, a[1]._obj.B * a[1]._obj.Sc
-        kind = {ffi.DENSE_GLU: "gate/up + GLU", ffi.DENSE_MINGRU: "minGRU gates + recurrence", ffi.DENSE_LOGITS: "logits"}.get(d.epilogue, "projection")
-        return f"{kind} {n}x{d.K}" + (" (norms fused)" if d.x == 0 else ""), 2.0 * n * d.K + R * (2.0 * d.K + 2.0 * d.N), 2.0 * R * n * d.K, 0.0
+        kind = {ffi.DENSE_GLU: "gate/up + GLU", ffi.DENSE_MINGRU: "minGRU gates + recurrence", ffi.DENSE_LOGITS: "logits"}.get(d.epilogue)
+        if kind is None:
+            kind = {ffi.ACT_RELU2: "up + squared ReLU", ffi.ACT_GELU_SIDE: "token side gate"}.get(d.act, "projection")
+        fused = " (norm and gate fused)" if d.gated.o else " (norms fused)" if d.x == 0 else ""
+        return f"{kind} {n}x{d.K}{fused}", 2.0 * n * d.K + R * (2.0 * d.K + 2.0 * d.N), 2.0 * R * n * d.K, 0.0
     if name == "jg_latent_attn":
         d = a[2]
         w = d.window or 1 << 30
@@ -668,6 +705,18 @@ def call_work(name: str, a: tuple, B: int, Sc: int, T: float, p: dict | None) ->
     if name == "jg_mingru_scan":
         d = a[2]
         return "minGRU scan", R * 2.0 * (d.ldp + d.ldo) + B * 8.0 * d.width, 0.0, 0.0
+    if name == "jg_linear_state":
+        d = a[2]
+        st = d.heads * d.dim * (d.vdim + (1 if d.gates else 0))
+        return ("mLSTM" if d.gates else "lightning") + " recurrence", B * 8.0 * st + R * d.heads * (4.0 * d.dim + 6.0 * d.vdim), 0.0 if Sc == 1 else 4.0 * R * st, 4.0 * R * st if Sc == 1 else 0.0
+    if name == "jg_gated_norm":
+        d = a[2]
+        return "gated norm", R * 8.0 * d.heads * d.vdim, 0.0, 0.0
+    if name == "jg_window_attn":
+        d = a[2]
+        w, kv = d.window or 1 << 30, 2.0 * d.kv_heads * (d.dim + d.vdim)
+        pairs = R * min(T, w + d.keep) if Sc == 1 else pairs if T <= w else R * float(w + d.keep)
+        return "window attention", B * min(T, w + d.keep + Sc - 1.0) * kv + R * (kv + 2.0 * d.heads * (d.dim + d.vdim)), 2.0 * d.heads * pairs * (d.dim + d.vdim), 0.0
     if name == "jg_stream_norm":
         d = a[2]
         R = a[1]._obj.B * a[1]._obj.Sc
@@ -714,27 +763,33 @@ def time_calls(dev, calls: list[tuple], B: int, Sc: int, T: float, p: dict | Non
 
 
 def run_hybrid(args) -> None:
-    """Prefill and decode of a Matulorn of the Llama's layer sizes, beside that Llama (fp16), at the same batch sizes."""
+    """Prefill and decode of layer-list models of the Llama's layer sizes, beside that Llama (fp16), at the same batch sizes."""
     from denograd_b200 import synth
     from denograd_b200.matulorn import Matulorn
+    from denograd_b200.rigazen import Rigazen
+    models = {"matulorn": Matulorn, "rigazen": Rigazen}
+    kinds = args.hybrid_models.split(",")
+    if not kinds or any(k not in (*models, "llama") for k in kinds):
+        raise SystemExit(f"--hybrid-models: any of {', '.join((*models, 'llama'))}")
     rig = Rig()
     dev, K, W, P, peaks = rig.dev, args.steps, args.warmup, args.prompt, measured_peaks()
     p, tied = arch(args.hybrid)
-    cfg = hybrid_config(args.hybrid, args.layers)
+    L = args.layers or p["n_layers"]
     line = {"metric": "hybrid_tokens_per_second", "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W, "data": "synthetic", "dtype": "bf16, f32 stream and state",
-            "config": {"model": f"Matulorn, {args.hybrid} layer sizes", "layers": len(cfg["layers"]), "prompt_tokens": P,
+            "config": {"model": f"{', '.join(kinds)}: {args.hybrid} layer sizes", "layers": L, "prompt_tokens": P,
                        "l2": "inputs larger than L2: every step streams all weights once"}, "legs": {}}
     batches = [int(b) for b in args.hybrid_batches.split(",")]
     prefills = [int(n) for n in args.hybrid_prefills.split(",")]
     ctx = max(max(prefills), P + 4 * K + W + 64)
     with ClockSampler(rig.local_rank) as clocks:
-        for kind in ("matulorn", "llama"):
+        for kind in kinds:
+            cfg = hybrid_config(args.hybrid, args.layers, kind) if kind != "llama" else None
             legs = line["legs"][kind] = {}
             for B in batches:
-                if kind == "matulorn":
-                    llm = Matulorn(cfg, max_context=ctx, max_batch=B, device=rig.dev_name, temperature=0.0).load_synthetic()
+                if kind != "llama":
+                    llm = models[kind](cfg, max_context=ctx, max_batch=B, device=rig.dev_name, temperature=0.0).load_synthetic()
                 else:
-                    llm = rig.llama(args.hybrid, "float16", (ctx + 63) // 64 * 64, B, n_layers=len(cfg["layers"]))
+                    llm = rig.llama(args.hybrid, "float16", (ctx + 63) // 64 * 64, B, n_layers=L)
                 m = llm.model
                 if B == 1:
                     for n in prefills:
@@ -745,7 +800,7 @@ def run_hybrid(args) -> None:
                         for _ in range(3):
                             llm.reset(); llm.prefill(prompt)
                         s = dev.timer_stop() / 3
-                        fl = hybrid_flops(cfg, 1, n) if kind == "matulorn" else prefill_flops(p | {"n_layers": len(cfg["layers"])}, 1, n)
+                        fl = hybrid_flops(cfg, 1, n) if kind != "llama" else prefill_flops(p | {"n_layers": L}, 1, n)
                         leg = legs[f"prefill{n}"] = {"tok_s": n / s, "ms": s * 1e3, "frac_of_bf16_peak": fl / s / 1e12 / peaks["tflops"]}
                         if not args.no_extra:
                             llm.reset()
@@ -761,7 +816,7 @@ def run_hybrid(args) -> None:
                     times.append(dev.timer_stop())
                     pos += K
                 s, T = statistics.median(times), P + W + 1.5 * K
-                by = hybrid_bytes(cfg, B, T) if kind == "matulorn" else weight_bytes(p | {"n_layers": len(cfg["layers"])}, tied, False) + B * T * kv_bytes_per_token(p | {"n_layers": len(cfg["layers"])})
+                by = hybrid_bytes(cfg, B, T) if kind != "llama" else weight_bytes(p | {"n_layers": L}, tied, False) + B * T * kv_bytes_per_token(p | {"n_layers": L})
                 leg = legs[f"decode_bs{B}"] = {"tok_s": B * K / s, "ms_per_step": s / K * 1e3, "context": int(T), "bytes_per_step": by,
                                                "frac_of_hbm_roofline": by / (s / K) / 1e9 / peaks["hbm_gbs"]}
                 if not args.no_extra:
@@ -846,7 +901,8 @@ def main() -> None:
     ap.add_argument("--no-extra", action="store_true", help="skip the extra legs")
     ap.add_argument("--no-parity", action="store_true", help="skip the checks against the CPU checker (profiling captures only)")
     ap.add_argument("--hybrid", default="", choices=["", "1B", "3B", "8B"],
-                    help="instead of the default workload: prefill and decode of a Matulorn with that Llama's layer sizes, beside the Llama")
+                    help="instead of the default workload: prefill and decode of layer-list models with that Llama's layer sizes, beside the Llama")
+    ap.add_argument("--hybrid-models", default="matulorn,llama", help="with --hybrid: which of matulorn, rigazen, llama, in order")
     ap.add_argument("--hybrid-batches", default="1,2,8,32")
     ap.add_argument("--hybrid-prefills", default="512,2048")
     args = ap.parse_args()

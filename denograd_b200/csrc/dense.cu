@@ -92,7 +92,10 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
       for (int c = tid; c < a.lead; c += MV_THREADS) xm[c] = xg[c];
       for (int c = a.lead + n + tid; c < a.ldw; c += MV_THREADS) xm[c] = from_f32<T>(0.f);
       if (m > 0) __syncthreads();
-      gated_row<MV_THREADS>(a.gated, (size_t)m, buf, buf + ((n + 3) & ~3), [&](int i, float v) { xm[a.lead + i] = from_f32<T>(v); });
+      gated_row<MV_THREADS>(a.gated, (size_t)m, buf, [&](int i, const auto& v) {
+#pragma unroll
+        for (size_t k = 0; k < sizeof(v) / sizeof(float); k++) xm[a.lead + i + k] = from_f32<T>(v[k]);
+      });
     } else if (FROM == ROWS_STREAM) {
       float* buf = reinterpret_cast<float*>(smem_raw + (size_t)MT * row_bytes);
       float* red = buf + ((a.st.D + 3) & ~3);
@@ -243,9 +246,10 @@ static GatedArgs<T> gated_args(const jg_gated_desc& d) {
   GatedArgs<T> g = {};
   g.o = (const float*)d.o; g.den = (const float*)d.den; g.w = (const float*)d.norm_w; g.gate = (const T*)d.gate;
   g.H = d.heads; g.vd = d.vdim; g.groups = d.groups; g.ldp = d.ldp; g.eps = d.eps; g.scale = d.scale;
+  g.vec = d.vdim % 4 == 0 && d.heads * d.vdim / d.groups % 4 == 0 && d.ldp % 4 == 0 && d.gate % (4 * sizeof(T)) == 0 && d.o % 16 == 0 && d.norm_w % 16 == 0;
   return g;
 }
-static size_t gated_smem_floats(const jg_gated_desc& d, int warps) { return (size_t)((d.heads * d.vdim + 3) & ~3) + stream_units(d.groups, warps); }
+static size_t gated_smem_floats(const jg_gated_desc& d, int warps) { return 2 * (size_t)((d.heads * d.vdim + 3) & ~3) + stream_units(d.groups, warps); }
 
 template <typename T, int MT, int EPI, int FROM>
 static int launch_mv(jg_dev* dev, const DenseCall& c) {
@@ -510,7 +514,18 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedArgs<T> a, T
   pdl_launch();
   pdl_wait();
   const size_t r = blockIdx.x;
-  gated_row<256>(a, r, sbuf, sbuf + ((a.H * a.vd + 3) & ~3), [&](int i, float v) { out[r * ldo + i] = from_f32<T>(v); });
+  gated_row<256>(a, r, sbuf, [&](int i, const auto& v) {
+    constexpr int V = sizeof(v) / sizeof(float);
+    if constexpr (V == 4 && sizeof(T) == 2) {
+      if (ldo % 4 == 0 && (uintptr_t)out % 8 == 0) {
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(v[0], v[1]), p1 = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(out + r * ldo + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&p0), *reinterpret_cast<const uint32_t*>(&p1));
+        return;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; k++) out[r * ldo + i + k] = from_f32<T>(v[k]);
+  });
 }
 template <typename T>
 static int launch_gated(jg_dev* dev, const jg_gated_desc& d, T* out, int ldo, int R) {

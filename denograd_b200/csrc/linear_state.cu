@@ -199,13 +199,13 @@ __global__ void __launch_bounds__(LI_THREADS) linear_scan_kernel(const LinArgs<T
 }
 
 // ------------------------------------------------------------------------------------------------ tensor cores
-// A CTA keeps 32 columns of a head's state, transposed, in the accumulators of its four warps (16 columns x half of the head
-// each) and walks the sequence 64 tokens at a time.  With D the tokens' weights (jg_linear_desc, products of decays),
-//   A[t][s]  = D[t][s] (k_s . q_t) for s <= t                    q, k in shared memory, one warp per 16 rows
+// A CTA keeps 32 columns of a head's state, transposed, in the accumulators of its eight warps (16 columns x a quarter of the
+// head each) and walks the sequence 64 tokens at a time.  With D the tokens' weights (jg_linear_desc, products of decays),
+//   A[t][s]  = D[t][s] (k_s . q_t) for s <= t                    q, k in shared memory, two warps per 16 rows
 //   O^T      = (S^T q_t) dec_t + V^T A^T                          S^T straight from the accumulators as A fragments
 //   S^T      = g S^T + (w V)^T K
-// The halves of the head add up their O^T through shared memory.
-constexpr int LK_TOK = 64, LK_COLS = 32, LK_THREADS = 128, LK_LDA = LK_TOK + 8, LK_LDV = LK_COLS + 8, LK_LDR = LK_TOK + 4;
+// The quarters of the head add up their O^T through shared memory.
+constexpr int LK_TOK = 64, LK_COLS = 32, LK_WARPS = 8, LK_THREADS = 32 * LK_WARPS, LK_LDA = LK_TOK + 8, LK_LDV = LK_COLS + 8, LK_LDR = LK_COLS + 4;
 template <int DP>
 struct LinStage {
   bf16 q[LK_TOK][DP + 8], k[LK_TOK][DP + 8], v[LK_TOK][LK_LDV];
@@ -215,22 +215,23 @@ template <int DP>
 struct LinShared {
   LinStage<DP> st[2];
   bf16 hi[LK_TOK][LK_LDA], lo[LK_TOK][LK_LDA];
-  float red[LK_COLS][LK_LDR];
+  float red[4][LK_TOK][LK_LDR];
   float dec[LK_TOK], w[LK_TOK], pw[LK_TOK + 1];
 };
-// 16-byte pieces in the stages, 4- and 8-byte pairs elsewhere
+// 16-byte pieces in the stages, pairs of 8 bytes among the factors
 static_assert(offsetof(LinStage<64>, g) % 16 == 0 && sizeof(LinStage<64>) % 16 == 0 && sizeof(LinStage<128>) % 16 == 0 && sizeof(LinStage<256>) % 16 == 0, "stage layout");
-static_assert(offsetof(LinShared<64>, hi) % 16 == 0 && offsetof(LinShared<64>, lo) % 16 == 0 && offsetof(LinShared<64>, red) % 8 == 0 && LK_LDR % 2 == 0, "weight layout");
+static_assert(offsetof(LinShared<64>, hi) % 16 == 0 && offsetof(LinShared<64>, lo) % 16 == 0 , "weight layout");
 static_assert(offsetof(LinShared<64>, dec) % 8 == 0 && offsetof(LinShared<64>, w) % 8 == 0, "factor layout");
 
 template <int DP, bool GATED>
 __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<bf16> a) {
-  constexpr int NT = DP / 16;  // 8-wide tiles of a warp's half of the head
+  constexpr int NT = DP / 32;  // 8-wide tiles of a warp's quarter of the head
   extern __shared__ __align__(16) unsigned char lk_smem[];
   LinShared<DP>& sh = *reinterpret_cast<LinShared<DP>*>(lk_smem);
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3, cg = warp & 1, dh = warp >> 1;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3, cg = warp & 1, dq = warp >> 1;
   const int h = blockIdx.y, b = blockIdx.z, j0 = blockIdx.x * LK_COLS;
-  for (int i = tid; i < (int)(sizeof(sh.st) / 16); i += LK_THREADS) reinterpret_cast<uint4*>(sh.st)[i] = make_uint4(0, 0, 0, 0);
+  if (a.dim < DP)  // what lies past the head
+    for (int i = tid; i < (int)(sizeof(sh.st) / 16); i += LK_THREADS) reinterpret_cast<uint4*>(sh.st)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
   pdl_wait();
   const int slot = a.seq[b], dpc = a.dim / 8, per = 2 * dpc + LK_COLS / 8;
@@ -238,15 +239,16 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
   auto load = [&](int t0, int s) {
     LinStage<DP>& st = sh.st[s];
     const int nt = min(LK_TOK, a.Sc - t0);
-    for (int i = tid; i < LK_TOK * per; i += LK_THREADS) {
-      const int t = i / per, c = i % per;
+    for (int t = warp; t < LK_TOK; t += LK_WARPS) {
       const size_t row = ((size_t)(t0 + t) * a.B + b) * a.ldp;
-      const int vc = (c - 2 * dpc) * 8;
-      bf16* d = c < dpc ? &st.q[t][c * 8] : c < 2 * dpc ? &st.k[t][(c - dpc) * 8] : &st.v[t][vc];
-      if (t < nt && (c < 2 * dpc || j0 + vc < a.vd))
-        cp16(d, c < dpc ? a.q + row + h * a.dim + c * 8 : c < 2 * dpc ? a.k + row + h * a.dim + (c - dpc) * 8 : a.v + row + h * a.vd + j0 + vc);
-      else  // past the end; the normaliser's column holds ones
-        *reinterpret_cast<uint4*>(d) = make_uint4(GATED && t < nt && c >= 2 * dpc && j0 + vc == a.vd ? 0x3F80u : 0u, 0, 0, 0);
+      for (int c = lane; c < per; c += 32) {
+        const int vc = (c - 2 * dpc) * 8;
+        bf16* d = c < dpc ? &st.q[t][c * 8] : c < 2 * dpc ? &st.k[t][(c - dpc) * 8] : &st.v[t][vc];
+        if (t < nt && (c < 2 * dpc || j0 + vc < a.vd))
+          cp16(d, c < dpc ? a.q + row + h * a.dim + c * 8 : c < 2 * dpc ? a.k + row + h * a.dim + (c - dpc) * 8 : a.v + row + h * a.vd + j0 + vc);
+        else  // past the end; the normaliser's column holds ones
+          *reinterpret_cast<uint4*>(d) = make_uint4(GATED && t < nt && c >= 2 * dpc && j0 + vc == a.vd ? 0x3F80u : 0u, 0, 0, 0);
+      }
     }
     if (GATED && tid < nt) cp16(&st.g[tid], a.tok + ((size_t)(t0 + tid) * a.B + b) * a.H + h);
     cp_commit();
@@ -254,7 +256,7 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
   load(0, 0);
   float S[NT][4];
   const bool cont = a.pos[b] > 0;
-  const int d0 = dh * (DP / 2), c0 = j0 + cg * 16 + g;
+  const int d0 = dq * (DP / 4), c0 = j0 + cg * 16 + g;
   float* state = a.state + ((size_t)slot * a.H + h) * a.cols * a.lds;
 #pragma unroll
   for (int j = 0; j < NT; j++)
@@ -282,97 +284,96 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
         sh.w[tid] = !in ? 0.f : GATED ? expf(last.x + st.g[tid].y) : sh.pw[nt - 1 - tid];
       }
     }
-    {  // A: this warp's 16 tokens against the tokens up to them
-      float sc[8][4];
+    {  // A: 16 tokens against the tokens up to them, every other pair of tiles
+      const int rg = warp & 3, half = warp >> 2;
+      float sc[2][2][4];
 #pragma unroll
-      for (int j = 0; j < 8; j++)
+      for (int j = 0; j < 2; j++)
 #pragma unroll
-        for (int i = 0; i < 4; i++) sc[j][i] = 0.f;
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+          for (int i = 0; i < 4; i++) sc[j][n][i] = 0.f;
+      if (half <= rg) {
 #pragma unroll 4
-      for (int k = 0; k < DP; k += 16) {
-        uint32_t qf[4];
-        ldsm4(qf, &st.q[warp * 16 + (lane & 15)][k + (lane >> 4) * 8]);
+        for (int k = 0; k < DP; k += 16) {
+          uint32_t qf[4];
+          ldsm4(qf, &st.q[rg * 16 + (lane & 15)][k + (lane >> 4) * 8]);
 #pragma unroll
-        for (int j = 0; j < 8; j += 2)
-          if (j <= 2 * warp) {
-            uint32_t kf[4];
-            ldsm4(kf, &st.k[j * 8 + (lane >> 4) * 8 + (lane & 7)][k + ((lane >> 3) & 1) * 8]);
-            mma_bf16(sc[j], qf, kf[0], kf[1]);
-            mma_bf16(sc[j + 1], qf, kf[2], kf[3]);
-          }
-      }
-#pragma unroll
-      for (int j = 0; j < 8; j++)
-        if (j <= 2 * warp + 1)
-#pragma unroll
-          for (int i = 0; i < 2; i++) {
-            const int t = warp * 16 + g + 8 * i, e = j * 8 + tq * 2;
-            float x[2];
-#pragma unroll
-            for (int k = 0; k < 2; k++) {
-              const bool in = e + k <= t && t < nt;
-              const float w = !in ? 0.f : GATED ? expf(st.g[t].x + st.g[e + k].y) : sh.pw[t - e - k];
-              x[k] = in ? sc[j][2 * i + k] * (w * a.q_scale) : 0.f;
+          for (int j = 0; j < 2; j++)
+            if (2 * j + half <= rg) {
+              uint32_t kf[4];
+              ldsm4(kf, &st.k[(2 * j + half) * 16 + (lane >> 4) * 8 + (lane & 7)][k + ((lane >> 3) & 1) * 8]);
+              mma_bf16(sc[j][0], qf, kf[0], kf[1]);
+              mma_bf16(sc[j][1], qf, kf[2], kf[3]);
             }
-            uint32_t hi, lo;
-            split_bf16(x[0], x[1], hi, lo);
-            *reinterpret_cast<uint32_t*>(&sh.hi[t][e]) = hi;
-            *reinterpret_cast<uint32_t*>(&sh.lo[t][e]) = lo;
-          }
+        }
+#pragma unroll
+        for (int j = 0; j < 2; j++)
+          if (2 * j + half <= rg)
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+              for (int i = 0; i < 2; i++) {
+                const int t = rg * 16 + g + 8 * i, e = (2 * j + half) * 16 + n * 8 + tq * 2;
+                float x[2];
+#pragma unroll
+                for (int k = 0; k < 2; k++) {
+                  const bool in = e + k <= t && t < nt;
+                  const float w = !in ? 0.f : GATED ? expf(st.g[t].x + st.g[e + k].y) : sh.pw[t - e - k];
+                  x[k] = in ? sc[j][n][2 * i + k] * (w * a.q_scale) : 0.f;
+                }
+                uint32_t hi, lo;
+                split_bf16(x[0], x[1], hi, lo);
+                *reinterpret_cast<uint32_t*>(&sh.hi[t][e]) = hi;
+                *reinterpret_cast<uint32_t*>(&sh.lo[t][e]) = lo;
+              }
+      }
     }
-    __syncthreads();
     float o[8][4];
 #pragma unroll
     for (int j = 0; j < 8; j++)
 #pragma unroll
       for (int i = 0; i < 4; i++) o[j][i] = 0.f;
-    // S^T q over this warp's half of the head
+    // S^T q over this warp's quarter of the head
 #pragma unroll
     for (int k = 0; k < NT / 2; k++) {
-      uint32_t hi[4], lo[4];
+      uint32_t hi[4], lo[4], qf[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; j++) ldsm4(qf[j], &st.q[j * 16 + (lane >> 4) * 8 + (lane & 7)][d0 + k * 16 + ((lane >> 3) & 1) * 8]);
       split_bf16(S[2 * k][0], S[2 * k][1], hi[0], lo[0]);
       split_bf16(S[2 * k][2], S[2 * k][3], hi[1], lo[1]);
       split_bf16(S[2 * k + 1][0], S[2 * k + 1][1], hi[2], lo[2]);
       split_bf16(S[2 * k + 1][2], S[2 * k + 1][3], hi[3], lo[3]);
 #pragma unroll
-      for (int j = 0; j < 8; j += 2) {
-        uint32_t qf[4];
-        ldsm4(qf, &st.q[j * 8 + (lane >> 4) * 8 + (lane & 7)][d0 + k * 16 + ((lane >> 3) & 1) * 8]);
-        mma_bf16(o[j], hi, qf[0], qf[1]);
-        mma_bf16(o[j + 1], hi, qf[2], qf[3]);
-        mma_bf16(o[j], lo, qf[0], qf[1]);
-        mma_bf16(o[j + 1], lo, qf[2], qf[3]);
-      }
+      for (int j = 0; j < 4; j++) { mma_bf16(o[2 * j], hi, qf[j][0], qf[j][1]); mma_bf16(o[2 * j + 1], hi, qf[j][2], qf[j][3]); }
+#pragma unroll
+      for (int j = 0; j < 4; j++) { mma_bf16(o[2 * j], lo, qf[j][0], qf[j][1]); mma_bf16(o[2 * j + 1], lo, qf[j][2], qf[j][3]); }
     }
+    __syncthreads();  // A, the decays and the weights are there
 #pragma unroll
     for (int j = 0; j < 8; j++) {
       const float2 d = *reinterpret_cast<const float2*>(&sh.dec[j * 8 + tq * 2]);
       o[j][0] *= d.x; o[j][1] *= d.y; o[j][2] *= d.x; o[j][3] *= d.y;
     }
-    // V^T A^T over this warp's half of the block's tokens
-#pragma unroll
-    for (int kk = 0; kk < 2; kk++) {
-      const int ks = dh * 2 + kk;
+    {  // V^T A^T over this warp's quarter of the block's tokens
       uint32_t vf[4];
-      ldsm4t(vf, &st.v[ks * 16 + (lane >> 4) * 8 + (lane & 7)][cg * 16 + ((lane >> 3) & 1) * 8]);
+      ldsm4t(vf, &st.v[dq * 16 + (lane >> 4) * 8 + (lane & 7)][cg * 16 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-      for (int j = 0; j < 8; j += 2)
-        if (ks * 2 <= j) {
+      for (int j = 0; j < 4; j++)
+        if (dq <= j) {
           uint32_t hi[4], lo[4];
-          ldsm4(hi, &sh.hi[j * 8 + (lane >> 4) * 8 + (lane & 7)][ks * 16 + ((lane >> 3) & 1) * 8]);
-          ldsm4(lo, &sh.lo[j * 8 + (lane >> 4) * 8 + (lane & 7)][ks * 16 + ((lane >> 3) & 1) * 8]);
-          mma_bf16(o[j], vf, hi[0], hi[1]);
-          mma_bf16(o[j + 1], vf, hi[2], hi[3]);
-          mma_bf16(o[j], vf, lo[0], lo[1]);
-          mma_bf16(o[j + 1], vf, lo[2], lo[3]);
+          ldsm4(hi, &sh.hi[j * 16 + (lane >> 4) * 8 + (lane & 7)][dq * 16 + ((lane >> 3) & 1) * 8]);
+          ldsm4(lo, &sh.lo[j * 16 + (lane >> 4) * 8 + (lane & 7)][dq * 16 + ((lane >> 3) & 1) * 8]);
+          mma_bf16(o[2 * j], vf, hi[0], hi[1]);
+          mma_bf16(o[2 * j + 1], vf, hi[2], hi[3]);
+          mma_bf16(o[2 * j], vf, lo[0], lo[1]);
+          mma_bf16(o[2 * j + 1], vf, lo[2], lo[3]);
         }
     }
-    if (dh == 1) {
 #pragma unroll
-      for (int j = 0; j < 8; j++)
+    for (int j = 0; j < 8; j++)
 #pragma unroll
-        for (int i = 0; i < 2; i++) *reinterpret_cast<float2*>(&sh.red[cg * 16 + g + 8 * i][j * 8 + tq * 2]) = make_float2(o[j][2 * i], o[j][2 * i + 1]);
-    }
+      for (int i = 0; i < 4; i++) sh.red[dq][j * 8 + tq * 2 + (i & 1)][cg * 16 + g + 8 * (i >> 1)] = o[j][i];
     // the state moves on by the block
 #pragma unroll
     for (int j = 0; j < NT; j++)
@@ -380,8 +381,10 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
       for (int i = 0; i < 4; i++) S[j][i] *= decay;
 #pragma unroll
     for (int ks = 0; ks < LK_TOK / 16; ks++) {
-      uint32_t vf[4], hi[4], lo[4];
+      uint32_t vf[4], hi[4], lo[4], kf[NT / 2][4];
       ldsm4t(vf, &st.v[ks * 16 + (lane >> 4) * 8 + (lane & 7)][cg * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+      for (int j = 0; j < NT / 2; j++) ldsm4t(kf[j], &st.k[ks * 16 + (lane & 15)][d0 + j * 16 + (lane >> 4) * 8]);
       const float2 w0 = *reinterpret_cast<const float2*>(&sh.w[ks * 16 + tq * 2]), w1 = *reinterpret_cast<const float2*>(&sh.w[ks * 16 + 8 + tq * 2]);
 #pragma unroll
       for (int i = 0; i < 4; i++) {
@@ -389,29 +392,20 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
         split_bf16(__uint_as_float(vf[i] << 16) * w.x, __uint_as_float(vf[i] & 0xFFFF0000u) * w.y, hi[i], lo[i]);
       }
 #pragma unroll
-      for (int j = 0; j < NT; j += 2) {
-        uint32_t kf[4];
-        ldsm4t(kf, &st.k[ks * 16 + (lane & 15)][d0 + j * 8 + (lane >> 4) * 8]);
-        mma_bf16(S[j], hi, kf[0], kf[1]);
-        mma_bf16(S[j + 1], hi, kf[2], kf[3]);
-        mma_bf16(S[j], lo, kf[0], kf[1]);
-        mma_bf16(S[j + 1], lo, kf[2], kf[3]);
-      }
+      for (int j = 0; j < NT / 2; j++) { mma_bf16(S[2 * j], hi, kf[j][0], kf[j][1]); mma_bf16(S[2 * j + 1], hi, kf[j][2], kf[j][3]); }
+#pragma unroll
+      for (int j = 0; j < NT / 2; j++) { mma_bf16(S[2 * j], lo, kf[j][0], kf[j][1]); mma_bf16(S[2 * j + 1], lo, kf[j][2], kf[j][3]); }
     }
     __syncthreads();
-    if (dh == 0) {
-#pragma unroll
-      for (int j = 0; j < 8; j++)
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-          const int t = j * 8 + tq * 2 + (i & 1), cl = cg * 16 + g + 8 * (i >> 1), c = j0 + cl;
-          if (t >= nt || c >= a.cols) continue;
-          const float x = o[j][i] + sh.red[cl][t];
-          const size_t r = (size_t)(t0 + t) * a.B + b;
-          if (c < a.vd) a.o[(r * a.H + h) * a.vd + c] = x;
-          else a.den[r * a.H + h] = linear_den(x, st.g[t].z);
-        }
-    }
+    const int c = j0 + lane;  // a warp writes 32 columns of a token
+    if (c < a.cols)
+#pragma unroll 2
+      for (int t = warp; t < nt; t += LK_WARPS) {
+        const float x = sh.red[0][t][lane] + sh.red[1][t][lane] + sh.red[2][t][lane] + sh.red[3][t][lane];
+        const size_t r = (size_t)(t0 + t) * a.B + b;
+        if (c < a.vd) a.o[(r * a.H + h) * a.vd + c] = x;
+        else a.den[r * a.H + h] = linear_den(x, st.g[t].z);
+      }
   }
   pdl_launch();
 #pragma unroll

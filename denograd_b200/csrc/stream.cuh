@@ -169,31 +169,53 @@ __device__ __forceinline__ void stream_row(const StreamArgs& a, size_t src, floa
 }
 
 // ------------------------------------------------------------------------------------------------ after a linear recurrence
-// One row of o / den / rms(group) * w * sigmoid(gate) * scale (jg_gated_norm) by the NT threads of a CTA; buf holds H * vd floats,
-// red stream_units of them.  store(i, value) for every i.
+// One row of o / den / rms(group) * w * sigmoid(gate) * scale (jg_gated_norm) by the NT threads of a CTA; buf holds
+// gated_smem_floats.  Everything comes in at once: the divided read-outs and the factors behind the norm go to shared memory,
+// where the groups' sums are taken.  store(i, v) receives the V values from element i on.
 template <typename T>
 struct GatedArgs {
   const float *o, *den, *w;
   const T* gate;
-  int H, vd, groups, ldp;
+  int H, vd, groups, ldp, vec;  // vec: rows and heads come in pieces of four
   float eps, scale;
 };
-template <int NT, typename T, typename Store>
-__device__ __forceinline__ void gated_row(const GatedArgs<T>& a, size_t r, float* buf, float* red, Store store) {
+template <int NT, int V, typename T, typename Store>
+__device__ __forceinline__ void gated_row_v(const GatedArgs<T>& a, size_t r, float* buf, Store store) {
   constexpr int W = NT / 32;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = a.H * a.vd;
-  const int gs = n / a.groups, P = a.groups >= W ? 1 : W / a.groups, units = a.groups * P, plen = (gs + P - 1) / P;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = a.H * a.vd, n4 = (n + 3) & ~3;
+  const int gs = n / a.groups, P = a.groups >= W ? 1 : W / a.groups, units = a.groups * P, plen = ((gs + P - 1) / P + V - 1) / V * V;
   const float *o = a.o + r * n, *den = a.den ? a.den + r * a.H : nullptr;
   const T* gate = a.gate + r * a.ldp;
+  float *fac = buf + n4, *red = fac + n4;
+#pragma unroll 4
+  for (int i = threadIdx.x * V; i < n; i += NT * V) {
+    const float d = den ? den[i / a.vd] : 1.f;
+    if constexpr (V == 4) {
+      float4 x = *reinterpret_cast<const float4*>(o + i), w = *reinterpret_cast<const float4*>(a.w + i);
+      float g[4];
+      if constexpr (sizeof(T) == 2) {
+        const uint2 t = *reinterpret_cast<const uint2*>(gate + i);
+        g[0] = __uint_as_float(t.x << 16); g[1] = __uint_as_float(t.x & 0xFFFF0000u); g[2] = __uint_as_float(t.y << 16); g[3] = __uint_as_float(t.y & 0xFFFF0000u);
+      } else {
+        const float4 t = *reinterpret_cast<const float4*>(gate + i);
+        g[0] = t.x; g[1] = t.y; g[2] = t.z; g[3] = t.w;
+      }
+      if (den) { x.x /= d; x.y /= d; x.z /= d; x.w /= d; }
+      w.x *= sigmoid_f32(g[0]); w.y *= sigmoid_f32(g[1]); w.z *= sigmoid_f32(g[2]); w.w *= sigmoid_f32(g[3]);
+      *reinterpret_cast<float4*>(buf + i) = x;
+      *reinterpret_cast<float4*>(fac + i) = w;
+    } else {
+      buf[i] = den ? o[i] / d : o[i];
+      fac[i] = a.w[i] * sigmoid_f32(to_f32(gate[i]));
+    }
+  }
+  __syncthreads();
   for (int u = warp; u < units; u += W) {
     const int g = u / P, lo = g * gs + (u % P) * plen, hi = min((g + 1) * gs, lo + plen);
     float ss = 0.f;
-#pragma unroll 4
-    for (int i = lo + lane; i < hi; i += 32) {
-      const float v = den ? o[i] / den[i / a.vd] : o[i];
-      buf[i] = v;
-      ss = fmaf(v, v, ss);
-    }
+    for (int i = lo + lane * V; i < hi; i += 32 * V)
+#pragma unroll
+      for (int k = 0; k < V; k++) ss = fmaf(buf[i + k], buf[i + k], ss);
     ss = warp_sum(ss);
     if (lane == 0) red[u] = ss;
   }
@@ -203,8 +225,17 @@ __device__ __forceinline__ void gated_row(const GatedArgs<T>& a, size_t r, float
     float t = 0.f;
     for (int p = 0; p < P; p++) t += red[g * P + p];
     const float rs = a.scale / sqrtf(t / (float)gs + a.eps);
-#pragma unroll 4
-    for (int i = lo + lane; i < hi; i += 32) store(i, buf[i] * rs * a.w[i] * sigmoid_f32(to_f32(gate[i])));
+    for (int i = lo + lane * V; i < hi; i += 32 * V) {
+      float v[V];
+#pragma unroll
+      for (int k = 0; k < V; k++) v[k] = buf[i + k] * rs * fac[i + k];
+      store(i, v);
+    }
   }
+}
+template <int NT, typename T, typename Store>
+__device__ __forceinline__ void gated_row(const GatedArgs<T>& a, size_t r, float* buf, Store store) {
+  if (a.vec) gated_row_v<NT, 4>(a, r, buf, store);
+  else gated_row_v<NT, 1>(a, r, buf, store);
 }
 #endif

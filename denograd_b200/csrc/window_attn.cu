@@ -234,7 +234,8 @@ __global__ void __launch_bounds__(WM_THREADS) window_mma_kernel(const WinArgs<bf
   WinShared<KS, VT>& sh = *reinterpret_cast<WinShared<KS, VT>*>(wm_smem);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
   const int per = a.H / a.G, zg = (per + 15) / 16, kv = blockIdx.y / zg, hb = kv * per + blockIdx.y % zg * 16, nh = min(16, kv * per + per - hb), r = blockIdx.z;
-  for (int i = tid; i < (int)(sizeof(sh.t) / 16); i += WM_THREADS) reinterpret_cast<uint4*>(sh.t)[i] = make_uint4(0, 0, 0, 0);  // what lies past the heads
+  if (a.dk8 < KS * 16)  // what lies past the head in a key (a value's columns past the head are never used)
+    for (int i = tid; i < (int)(sizeof(sh.t) / 16); i += WM_THREADS) reinterpret_cast<uint4*>(sh.t)[i] = make_uint4(0, 0, 0, 0);
   for (int i = tid; i < (int)(sizeof(sh.q) / 16); i += WM_THREADS) reinterpret_cast<uint4*>(sh.q)[i] = make_uint4(0, 0, 0, 0);
   pdl_launch();
   pdl_wait();

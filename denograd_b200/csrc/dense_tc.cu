@@ -203,7 +203,7 @@ static int launch_dt(jg_dev* dev, const DenseCall& c, const DtArgs& a) {
   if (c.M > 128) {  // the split with the smallest waves x (k-blocks at the tensor peak + fixed cost) estimate, as in gemm_tc.cu
     float best = 0.f;
     for (int s = 1; s <= Cfg::MAX_KS && s <= 8 && n_kb / s >= 8; s++) {
-      const int waves = (tiles * s + dev->sm_count - 1) / dev->sm_count;
+      const int slots = dev->sm_count * (HALF ? 2 : 1), waves = (tiles * s + slots - 1) / slots;
       const float t = (float)waves * ((float)(n_kb / s) * 0.28f + 18.f);
       if (s == 1 || t < best) { best = t; ks = s; }
     }
@@ -258,6 +258,9 @@ int jg_dense_tc(jg_dev* dev, const DenseCall& c) {
   }
   if (c.M <= 16) return launch_dt<16, false, true>(dev, c, a);
   if (c.M <= 32) return launch_dt<32, false, true>(dev, c, a);
+  // few features or a short K: narrow tiles, two CTAs per SM, so that there are enough of them and one's epilogue overlaps
+  // another's loads
+  if (c.M > 64 && (c.N <= 512 || c.K <= 512)) return launch_dt<64, false, true>(dev, c, a);
   if (c.M <= 64) return launch_dt<64, false, false>(dev, c, a);
   if (c.M <= 128) return launch_dt<128, false, false>(dev, c, a);
   return launch_dt<256, false, false>(dev, c, a);

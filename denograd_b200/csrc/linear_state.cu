@@ -116,7 +116,7 @@ __global__ void __launch_bounds__(LI_THREADS) linear_step_kernel(const LinArgs<T
 }
 
 // Weights of a gated portion, per token and head: with b_t the sum of the log forget gates since the start of the token's
-// block of `block` tokens, (b_t - m_t, i_t - b_t, m_t, m_{t-1}); with block = 0 (a_t, b_t, m_t, -) of the recurrence.
+// block of `block` tokens, (b_t - m_t, i_t - b_t, m_t, m_{t-1}) with the first two in powers of two; with block = 0 (a_t, b_t, m_t, -) of the recurrence.
 // m_t = max(f_t + m_{t-1}, i_t) is a map of m_{t-1}; maps compose, (F1, I1) then (F2, I2) = (F1 + F2, max(F2 + I1, I2)).
 constexpr int LG_THREADS = 256;
 __global__ void __launch_bounds__(LG_THREADS) linear_gates_kernel(const float* __restrict__ gates, float* __restrict__ m_state, float4* __restrict__ tok, const int32_t* __restrict__ pos,
@@ -147,7 +147,7 @@ __global__ void __launch_bounds__(LG_THREADS) linear_gates_kernel(const float* _
     s_m[tid + 1] = m;
     __syncthreads();
     const float before = s_m[tid];
-    if (t < Sc) tok[((size_t)t * B + b) * H + h] = block > 0 ? make_float4(bt - m, g.x - bt, m, before) : make_float4(expf(g.y + before - m), expf(g.x - m), m, 0.f);
+    if (t < Sc) tok[((size_t)t * B + b) * H + h] = block > 0 ? make_float4((bt - m) * LOG2E, (g.x - bt) * LOG2E, m, before) : make_float4(expf(g.y + before - m), expf(g.x - m), m, 0.f);
     __syncthreads();
     if (tid == 0) s_m[0] = s_m[min(LG_THREADS, Sc - t0)];
     __syncthreads();
@@ -230,34 +230,56 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
   LinShared<DP>& sh = *reinterpret_cast<LinShared<DP>*>(lk_smem);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3, cg = warp & 1, dq = warp >> 1;
   const int h = blockIdx.y, b = blockIdx.z, j0 = blockIdx.x * LK_COLS;
-  if (a.dim < DP)  // what lies past the head
-    for (int i = tid; i < (int)(sizeof(sh.st) / 16); i += LK_THREADS) reinterpret_cast<uint4*>(sh.st)[i] = make_uint4(0, 0, 0, 0);
-  __syncthreads();
-  pdl_wait();
-  const int slot = a.seq[b], dpc = a.dim / 8, per = 2 * dpc + LK_COLS / 8;
-  if (!GATED && tid <= LK_TOK) sh.pw[tid] = tid == 0 ? 1.f : powf(a.decay[h], (float)tid);
-  auto load = [&](int t0, int s) {
-    LinStage<DP>& st = sh.st[s];
-    const int nt = min(LK_TOK, a.Sc - t0);
-    for (int t = warp; t < LK_TOK; t += LK_WARPS) {
-      const size_t row = ((size_t)(t0 + t) * a.B + b) * a.ldp;
-      for (int c = lane; c < per; c += 32) {
-        const int vc = (c - 2 * dpc) * 8;
-        bf16* d = c < dpc ? &st.q[t][c * 8] : c < 2 * dpc ? &st.k[t][(c - dpc) * 8] : &st.v[t][vc];
-        if (t < nt && (c < 2 * dpc || j0 + vc < a.vd))
-          cp16(d, c < dpc ? a.q + row + h * a.dim + c * 8 : c < 2 * dpc ? a.k + row + h * a.dim + (c - dpc) * 8 : a.v + row + h * a.vd + j0 + vc);
-        else  // past the end; the normaliser's column holds ones
-          *reinterpret_cast<uint4*>(d) = make_uint4(GATED && t < nt && c >= 2 * dpc && j0 + vc == a.vd ? 0x3F80u : 0u, 0, 0, 0);
-      }
+  const int dpc = a.dim / 8;
+  {  // what no load fills: past the head, and past the values (the normaliser's column holds ones)
+    if (a.dim < DP)
+      for (int i = tid; i < (int)(sizeof(sh.st) / 16); i += LK_THREADS) reinterpret_cast<uint4*>(sh.st)[i] = make_uint4(0, 0, 0, 0);
+    __syncthreads();
+    for (int i = tid; i < 2 * LK_TOK * (LK_COLS / 8); i += LK_THREADS) {
+      const int c = i % (LK_COLS / 8) * 8;
+      if (j0 + c >= a.vd) *reinterpret_cast<uint4*>(&sh.st[i / (LK_TOK * LK_COLS / 8)].v[i / (LK_COLS / 8) % LK_TOK][c]) = make_uint4(GATED && j0 + c == a.vd ? 0x3F80u : 0u, 0, 0, 0);
     }
-    if (GATED && tid < nt) cp16(&st.g[tid], a.tok + ((size_t)(t0 + tid) * a.B + b) * a.H + h);
+  }
+  pdl_wait();
+  if (!GATED && tid <= LK_TOK) sh.pw[tid] = tid == 0 ? 1.f : powf(a.decay[h], (float)tid);
+  // a warp brings every eighth token; a lane the same 16-byte pieces of each: where they come from and where they go
+  constexpr int NP = (DP / 4 + LK_COLS / 8 + 31) / 32;
+  const bf16* src[NP];
+  uint32_t dst[NP], step[NP];  // bytes from the start of a stage, and between its tokens
+#pragma unroll
+  for (int n = 0; n < NP; n++) {
+    const int c = lane + 32 * n, kc = c - dpc, vc = c - 2 * dpc;
+    const size_t row = ((size_t)warp * a.B + b) * a.ldp;
+    src[n] = nullptr;
+    dst[n] = step[n] = 0;
+    if (c < dpc) { src[n] = a.q + row + h * a.dim + c * 8; dst[n] = offsetof(LinStage<DP>, q) + c * 16; step[n] = sizeof(sh.st[0].q[0]); }
+    else if (kc < dpc) { src[n] = a.k + row + h * a.dim + kc * 8; dst[n] = offsetof(LinStage<DP>, k) + kc * 16; step[n] = sizeof(sh.st[0].k[0]); }
+    else if (vc < LK_COLS / 8 && j0 + vc * 8 < a.vd) { src[n] = a.v + row + h * a.vd + j0 + vc * 8; dst[n] = offsetof(LinStage<DP>, v) + vc * 16; step[n] = sizeof(sh.st[0].v[0]); }
+    dst[n] += warp * step[n];
+  }
+  const size_t token = (size_t)a.B * a.ldp;
+  auto load = [&](int t0, int s) {
+    unsigned char* st = reinterpret_cast<unsigned char*>(&sh.st[s]);
+    const int nt = a.Sc - t0;
+#pragma unroll
+    for (int n = 0; n < NP; n++)
+      if (src[n]) {
+        const bf16* p = src[n] + (size_t)t0 * token;
+#pragma unroll
+        for (int i = 0; i < LK_TOK / LK_WARPS; i++) {
+          unsigned char* d = st + dst[n] + i * LK_WARPS * step[n];
+          if (warp + i * LK_WARPS < nt) cp16(d, p + (size_t)i * LK_WARPS * token);
+          else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);  // past the end
+        }
+      }
+    if (GATED && tid < min(LK_TOK, nt)) cp16(&sh.st[s].g[tid], a.tok + ((size_t)(t0 + tid) * a.B + b) * a.H + h);
     cp_commit();
   };
   load(0, 0);
   float S[NT][4];
   const bool cont = a.pos[b] > 0;
   const int d0 = dq * (DP / 4), c0 = j0 + cg * 16 + g;
-  float* state = a.state + ((size_t)slot * a.H + h) * a.cols * a.lds;
+  float* state = a.state + ((size_t)a.seq[b] * a.H + h) * a.cols * a.lds;
 #pragma unroll
   for (int j = 0; j < NT; j++)
 #pragma unroll
@@ -276,12 +298,12 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
     float decay;  // of the state over the whole block
     {
       const float4 last = GATED ? st.g[nt - 1] : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float mp = GATED ? st.g[0].w : 0.f;
-      decay = GATED ? expf(last.x + mp) : sh.pw[nt];
+      const float mp = GATED ? st.g[0].w * LOG2E : 0.f;
+      decay = GATED ? ex2(last.x + mp) : sh.pw[nt];
       if (tid < LK_TOK) {
         const bool in = tid < nt;
-        sh.dec[tid] = !in ? 0.f : a.q_scale * (GATED ? expf(st.g[tid].x + mp) : sh.pw[tid + 1]);
-        sh.w[tid] = !in ? 0.f : GATED ? expf(last.x + st.g[tid].y) : sh.pw[nt - 1 - tid];
+        sh.dec[tid] = !in ? 0.f : a.q_scale * (GATED ? ex2(st.g[tid].x + mp) : sh.pw[tid + 1]);
+        sh.w[tid] = !in ? 0.f : GATED ? ex2(last.x + st.g[tid].y) : sh.pw[nt - 1 - tid];
       }
     }
     {  // A: 16 tokens against the tokens up to them, every other pair of tiles
@@ -317,10 +339,9 @@ __global__ void __launch_bounds__(LK_THREADS) linear_chunk_kernel(const LinArgs<
                 const int t = rg * 16 + g + 8 * i, e = (2 * j + half) * 16 + n * 8 + tq * 2;
                 float x[2];
 #pragma unroll
-                for (int k = 0; k < 2; k++) {
-                  const bool in = e + k <= t && t < nt;
-                  const float w = !in ? 0.f : GATED ? expf(st.g[t].x + st.g[e + k].y) : sh.pw[t - e - k];
-                  x[k] = in ? sc[j][n][2 * i + k] * (w * a.q_scale) : 0.f;
+                for (int k = 0; k < 2; k++) {  // a later token has no weight, however far its exponent goes
+                  const float w = GATED ? ex2(st.g[t].x + st.g[e + k].y) : sh.pw[max(t - e - k, 0)];
+                  x[k] = e + k <= t && t < nt ? sc[j][n][2 * i + k] * (w * a.q_scale) : 0.f;
                 }
                 uint32_t hi, lo;
                 split_bf16(x[0], x[1], hi, lo);

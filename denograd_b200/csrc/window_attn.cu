@@ -30,11 +30,12 @@ struct WinArgs {
   int B, Sc, H, G, dim, vd, window, keep, ldp, ldo, page, page_shift, pps, pinned, pairs, rot_rows, dk8, dv8, vd4, ns, slice_round;
   float eps, scale, out_scale;
   __host__ __device__ __forceinline__ int row_size() const { return G * (dk8 + dv8); }
-  // cache row of position p of the slot whose block-table row is `t`
-  __device__ __forceinline__ T* row(const int32_t* t, int p) const {
+  // cache row of position p of the slot whose block-table row is `t`: its number, and where it is
+  __device__ __forceinline__ uint32_t row_number(const int32_t* t, int p) const {
     const int i = p >> page_shift;
-    return pool + ((size_t)t[i < pinned ? i : pinned + (i - pinned) % (pps - pinned)] * page + (p & (page - 1))) * row_size();
+    return (uint32_t)t[i < pinned ? i : pinned + (i - pinned) % (pps - pinned)] * (uint32_t)page + (uint32_t)(p & (page - 1));
   }
+  __device__ __forceinline__ T* row(const int32_t* t, int p) const { return pool + (size_t)row_number(t, p) * row_size(); }
   __device__ __forceinline__ int position(int r) const { return min(max(pos[r % B] + r / B, 0), rot_rows - 1); }
   __device__ __forceinline__ int slice(int n) const { return ((n + ns - 1) / ns + slice_round - 1) / slice_round * slice_round; }
 };
@@ -230,6 +231,7 @@ static_assert(sizeof(WinTile<4, 8>) % 16 == 0 && sizeof(WinTile<16, 32>) % 16 ==
 
 template <int KS, int VT>
 __global__ void __launch_bounds__(WM_THREADS) window_mma_kernel(const WinArgs<bf16> a, int fresh) {
+  using WinTileT = WinTile<KS, VT>;
   extern __shared__ __align__(16) unsigned char wm_smem[];
   WinShared<KS, VT>& sh = *reinterpret_cast<WinShared<KS, VT>*>(wm_smem);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
@@ -260,19 +262,28 @@ __global__ void __launch_bounds__(WM_THREADS) window_mma_kernel(const WinArgs<bf
     sh.q[n][e] = from_f32<bf16>(normed_rotated(q + (hb + n) * a.dim, a.qn + (hb + n) * a.dim, rq, e, cs, a.pairs));
   }
   __syncthreads();  // queries and the new cache row are there
-  const int pk = a.dk8 / 8, pieces = pk + a.dv8 / 8;
+  // a lane brings the same 16-byte pieces of every position: where they are in a cache row and in a tile's row
+  constexpr int NP = (2 * KS + VT + 31) / 32;
+  const int pk = a.dk8 / 8, rs = a.row_size();
+  int from[NP], to[NP], step[NP];
+#pragma unroll
+  for (int n = 0; n < NP; n++) {
+    const int c = lane + 32 * n, vc = c - pk;
+    from[n] = c < pk ? kv * a.dk8 + c * 8 : vc < a.dv8 / 8 ? a.G * a.dk8 + kv * a.dv8 + vc * 8 : -1;
+    to[n] = c < pk ? c * 8 : (int)(offsetof(WinTileT, v) / sizeof(bf16)) + vc * 8;
+    step[n] = c < pk ? KS * 16 + 8 : VT * 8 + 8;
+  }
   auto load = [&](int i) {  // this warp's i-th tile
     const int base = t0 + (warp + i * WM_WARPS) * WM_POS;
     if (base < t1) {
-      WinTile<KS, VT>& t = sh.t[warp][i % WM_STAGES];
-      const bf16* mine = a.row(bt, seen.at(min(base + (lane & 15), t1 - 1)));
-#pragma unroll 4
+      bf16* t = reinterpret_cast<bf16*>(&sh.t[warp][i % WM_STAGES]);
+      const uint32_t mine = a.row_number(bt, seen.at(min(base + (lane & 15), t1 - 1)));
+#pragma unroll
       for (int n = 0; n < WM_POS; n++) {
-        const bf16* src = reinterpret_cast<const bf16*>(__shfl_sync(0xffffffffu, (unsigned long long)(uintptr_t)mine, n));
-        for (int c = lane; c < pieces; c += 32) {
-          if (c < pk) cp16(&t.k[n][c * 8], src + kv * a.dk8 + c * 8);
-          else cp16(&t.v[n][(c - pk) * 8], src + a.G * a.dk8 + kv * a.dv8 + (c - pk) * 8);
-        }
+        const bf16* src = a.pool + (size_t)__shfl_sync(0xffffffffu, mine, n) * rs;
+#pragma unroll
+        for (int c = 0; c < NP; c++)
+          if (from[c] >= 0) cp16(t + to[c] + n * step[c], src + from[c]);
       }
     }
     cp_commit();
@@ -376,7 +387,7 @@ static constexpr size_t wx_smem(int nq, int qkp, int vt) { return (size_t)2 * ((
 
 // NW * 16 queries of one head; tiles of 64 seen positions, two in shared memory.
 template <int VT, int NW>
-__global__ void __launch_bounds__(32 * NW) window_chunk_kernel(const WinArgs<bf16> a, int qkp) {
+__global__ void __launch_bounds__(32 * NW, VT <= 16 ? (NW == 8 ? 2 : 3) : 1) window_chunk_kernel(const WinArgs<bf16> a, int qkp) {
   constexpr int NQ = 16 * NW, NT = 32 * NW;
   extern __shared__ __align__(16) unsigned char wx_raw[];
   const int ldq = qkp + 8;
@@ -392,16 +403,21 @@ __global__ void __launch_bounds__(32 * NW) window_chunk_kernel(const WinArgs<bf1
   if (p0 < 0 || p1 >= a.rot_rows) return;
   const int32_t* bt = a.bt + (size_t)a.seq[b] * a.pps;
   const Seen seen(p0, p1, a.window, a.keep);
+  // a lane brings the same 16-byte pieces of every key: where they are in a cache row and in a tile's row
+  const int rs = a.row_size();
   auto load_tile = [&](int base, int s) {
     bf16 *tk = sK + (size_t)s * WX_KV * ldq, *tv = sV + (size_t)s * WX_KV * ldv;
-    const bf16* mine[2];
+    const uint32_t r0 = a.row_number(bt, seen.at(min(base + lane, seen.n - 1))), r1 = a.row_number(bt, seen.at(min(base + 32 + lane, seen.n - 1)));
+    for (int c = lane; c < ((per + 31) & ~31); c += 32) {
+      const int vc = c - pieces;
+      const bf16* from = a.pool + (c < pieces ? kv * a.dk8 + c * 8 : a.G * a.dk8 + kv * a.dv8 + vc * 8);
+      bf16* to = c < pieces ? tk + (size_t)warp * ldq + c * 8 : tv + (size_t)warp * ldv + vc * 8;
+      const int step = NW * (c < pieces ? ldq : ldv);
 #pragma unroll
-    for (int k = 0; k < 2; k++) mine[k] = a.row(bt, seen.at(min(base + k * 32 + lane, seen.n - 1)));
-    for (int n = warp; n < WX_KV; n += NW) {  // keys past the end repeat the last one; they are masked below
-      const bf16* src = reinterpret_cast<const bf16*>(__shfl_sync(0xffffffffu, (unsigned long long)(uintptr_t)(n < 32 ? mine[0] : mine[1]), n & 31));
-      for (int c = lane; c < per; c += 32) {
-        if (c < pieces) cp16(tk + (size_t)n * ldq + c * 8, src + kv * a.dk8 + c * 8);
-        else cp16(tv + (size_t)n * ldv + (c - pieces) * 8, src + a.G * a.dk8 + kv * a.dv8 + (c - pieces) * 8);
+      for (int i = 0; i < WX_KV / NW; i++) {  // keys past the end repeat the last one; they are masked below
+        const int n = warp + i * NW;
+        const uint32_t r = __shfl_sync(0xffffffffu, n < 32 ? r0 : r1, n & 31);
+        if (c < per) cp16(to + i * step, from + (size_t)r * rs);
       }
     }
     cp_commit();
@@ -427,72 +443,79 @@ __global__ void __launch_bounds__(32 * NW) window_chunk_kernel(const WinArgs<bf1
     // positions first .. last (in one run, or across the gap): all later than this warp's tokens, or all ahead of their windows?
     const bool none = first > w1 || (a.window > 0 && first >= a.keep && last <= w0 - a.window);
     if (!none) {
-      const bf16 *tk = sK + (size_t)s * WX_KV * ldq, *tv = sV + (size_t)s * WX_KV * ldv;
-      float sc[8][4];
+      const bool all = end < seen.n && last <= w0 && (a.window <= 0 || first > w1 - a.window || last < a.keep);  // seen by all of them
+#pragma unroll 1
+      for (int half = 0; half < 2; half++) {  // 32 keys at a time: fewer scores in registers
+        const bf16 *tk = sK + (size_t)(s * WX_KV + half * 32) * ldq, *tv = sV + (size_t)(s * WX_KV + half * 32) * ldv;
+        float sc[4][4];
 #pragma unroll
-      for (int j = 0; j < 8; j++)
+        for (int j = 0; j < 4; j++)
 #pragma unroll
-        for (int i = 0; i < 4; i++) sc[j][i] = 0.f;
-#pragma unroll 2
-      for (int k = 0; k < qkp; k += 16) {
-        uint32_t qf[4];
-        ldsm4(qf, sQ + (size_t)(warp * 16 + (lane & 15)) * ldq + k + (lane >> 4) * 8);
-#pragma unroll
-        for (int j = 0; j < 8; j += 2) {
-          uint32_t kf[4];
-          ldsm4(kf, tk + (size_t)(j * 8 + (lane >> 4) * 8 + (lane & 7)) * ldq + k + ((lane >> 3) & 1) * 8);
-          mma_bf16(sc[j], qf, kf[0], kf[1]);
-          mma_bf16(sc[j + 1], qf, kf[2], kf[3]);
+          for (int i = 0; i < 4; i++) sc[j][i] = 0.f;
+#pragma unroll 4
+        for (int k = 0; k < qkp; k += 16) {
+          uint32_t qf[4], k0[4], k1[4];
+          ldsm4(qf, sQ + (size_t)(warp * 16 + (lane & 15)) * ldq + k + (lane >> 4) * 8);
+          ldsm4(k0, tk + (size_t)((lane >> 4) * 8 + (lane & 7)) * ldq + k + ((lane >> 3) & 1) * 8);
+          ldsm4(k1, tk + (size_t)(16 + (lane >> 4) * 8 + (lane & 7)) * ldq + k + ((lane >> 3) & 1) * 8);
+          mma_bf16(sc[0], qf, k0[0], k0[1]);
+          mma_bf16(sc[1], qf, k0[2], k0[3]);
+          mma_bf16(sc[2], qf, k1[0], k1[1]);
+          mma_bf16(sc[3], qf, k1[2], k1[3]);
         }
-      }
-      float mx[2] = {m[0], m[1]};
-      if (end < seen.n && last <= w0 && (a.window <= 0 || first > w1 - a.window || last < a.keep)) {  // all of it is seen by all of them
+        float mx[2] = {m[0], m[1]};
+        if (all) {
 #pragma unroll
-        for (int j = 0; j < 8; j++)
+          for (int j = 0; j < 4; j++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+              sc[j][i] *= sl2;
+              mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+            }
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; j++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+              const int v = base + half * 32 + j * 8 + tq * 2 + (i & 1), key = seen.at(v), back = w0 + g + 8 * (i >> 1) - key;
+              sc[j][i] = v < seen.n && back >= 0 && (a.window <= 0 || back < a.window || key < a.keep) ? sc[j][i] * sl2 : -INFINITY;
+              mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+            }
+        }
+        float mu[2];
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+          mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+          mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+          mu[i] = mx[i] == -INFINITY ? 0.f : mx[i];  // nothing seen yet: every weight below is 0
+        }
+        if (__any_sync(0xffffffffu, mx[0] != m[0] || mx[1] != m[1])) {
+          const float a0 = ex2(m[0] - mu[0]), a1 = ex2(m[1] - mu[1]);
+          l[0] *= a0;
+          l[1] *= a1;
+          m[0] = mx[0];
+          m[1] = mx[1];
+#pragma unroll
+          for (int j = 0; j < VT; j++) { o[j][0] *= a0; o[j][1] *= a0; o[j][2] *= a1; o[j][3] *= a1; }
+        }
+#pragma unroll
+        for (int j = 0; j < 4; j++)
 #pragma unroll
           for (int i = 0; i < 4; i++) {
-            sc[j][i] *= sl2;
-            mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+            sc[j][i] = ex2(sc[j][i] - mu[i >> 1]);
+            l[i >> 1] += sc[j][i];
           }
-      } else {
 #pragma unroll
-        for (int j = 0; j < 8; j++)
+        for (int k = 0; k < 2; k++) {
+          const uint32_t pf[4] = {pack_bf16(sc[2 * k][0], sc[2 * k][1]), pack_bf16(sc[2 * k][2], sc[2 * k][3]), pack_bf16(sc[2 * k + 1][0], sc[2 * k + 1][1]),
+                                  pack_bf16(sc[2 * k + 1][2], sc[2 * k + 1][3])};
 #pragma unroll
-          for (int i = 0; i < 4; i++) {
-            const int v = base + j * 8 + tq * 2 + (i & 1), key = seen.at(v), back = w0 + g + 8 * (i >> 1) - key;
-            sc[j][i] = v < seen.n && back >= 0 && (a.window <= 0 || back < a.window || key < a.keep) ? sc[j][i] * sl2 : -INFINITY;
-            mx[i >> 1] = fmaxf(mx[i >> 1], sc[j][i]);
+          for (int j = 0; j < VT; j += 2) {
+            uint32_t vf[4];
+            ldsm4t(vf, tv + (size_t)(k * 16 + (lane & 15)) * ldv + j * 8 + (lane >> 4) * 8);
+            mma_bf16(o[j], pf, vf[0], vf[1]);
+            mma_bf16(o[j + 1], pf, vf[2], vf[3]);
           }
-      }
-      float al[2], mu[2];
-#pragma unroll
-      for (int i = 0; i < 2; i++) {
-        mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-        mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-        mu[i] = mx[i] == -INFINITY ? 0.f : mx[i];  // nothing seen yet: every weight below is 0
-        al[i] = ex2(m[i] - mu[i]);
-        m[i] = mx[i];
-        l[i] *= al[i];
-      }
-#pragma unroll
-      for (int j = 0; j < VT; j++) { o[j][0] *= al[0]; o[j][1] *= al[0]; o[j][2] *= al[1]; o[j][3] *= al[1]; }
-#pragma unroll
-      for (int j = 0; j < 8; j++)
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-          sc[j][i] = ex2(sc[j][i] - mu[i >> 1]);
-          l[i >> 1] += sc[j][i];
-        }
-#pragma unroll
-      for (int k = 0; k < 4; k++) {
-        const uint32_t pf[4] = {pack_bf16(sc[2 * k][0], sc[2 * k][1]), pack_bf16(sc[2 * k][2], sc[2 * k][3]), pack_bf16(sc[2 * k + 1][0], sc[2 * k + 1][1]),
-                                pack_bf16(sc[2 * k + 1][2], sc[2 * k + 1][3])};
-#pragma unroll
-        for (int j = 0; j < VT; j += 2) {
-          uint32_t vf[4];
-          ldsm4t(vf, tv + (size_t)(k * 16 + (lane & 15)) * ldv + j * 8 + (lane >> 4) * 8);
-          mma_bf16(o[j], pf, vf[0], vf[1]);
-          mma_bf16(o[j + 1], pf, vf[2], vf[3]);
         }
       }
     }

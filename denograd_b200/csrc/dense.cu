@@ -80,6 +80,8 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
     }
   }
   pdl_wait();
+  if (EPI == JG_DENSE_STORE && a.out.act == JG_ACT_GELU_SIDE && tid < a.M && u0 < u1)  // this CTA's part of the tokens' rows
+    prefetch_l2(dense_side_ptr<T>(a.out, a.out.tokens[tid], u0 * RW));
 
   for (int m = 0; m < MT; m++) {
     T* xm = xs + (size_t)m * a.ldw;
@@ -122,7 +124,7 @@ __global__ void __launch_bounds__(MV_THREADS, 2) dense_mv_kernel(const MvArgs<T>
     if (a.bias[0]) s0 += a.bias[0][row];
     const size_t o = (size_t)m * a.ldy + row;
     if (EPI == JG_DENSE_STORE) {
-      s0 = dense_act<T>(a.out, m, row, s0);
+      s0 = dense_act(a.out, row, s0, dense_side<T>(a.out, m, row));
       if (row >= a.out.split) a.out.y2[(size_t)m * a.out.ld2 + row - a.out.split] = s0;
       else if (a.y32) a.y32[o] = s0;
       else a.y[o] = from_f32<T>(s0);
@@ -320,7 +322,7 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const float* __restrict_
     for (int j = 0; j < 4; j++) {
       const int m = m0 + tm + 16 * i, n = n0 + tn + 16 * j;
       if (m >= M || n >= N) continue;
-      const float v = dense_act<float>(out, m, n, acc[i][j] + (bias ? bias[n] : 0.f));
+      const float v = dense_act(out, n, acc[i][j] + (bias ? bias[n] : 0.f), dense_side<float>(out, m, n));
       if (n >= out.split) out.y2[(size_t)m * out.ld2 + n - out.split] = v;
       else y[(size_t)m * ldy + n] = v;
     }

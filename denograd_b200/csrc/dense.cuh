@@ -10,13 +10,26 @@ struct DenseOut {
   const int32_t* tokens = nullptr;
 };
 #ifdef __CUDACC__
+// what the row's token has in the table for a column; an id outside the table reads as zero (from row 0, so that no branch
+// keeps several of these loads apart)
 template <typename T>
-__device__ __forceinline__ float dense_act(const DenseOut& o, int row, int col, float v) {
+__device__ __forceinline__ const T* dense_side_ptr(const DenseOut& o, int tok, int col) {
+  return reinterpret_cast<const T*>(o.side) + (size_t)(tok >= 0 && tok < o.vocab ? tok : 0) * o.ld_side + o.col_side + col;
+}
+template <typename T>
+__device__ __forceinline__ float dense_side(const DenseOut& o, int row, int col) {
+  if (o.act != JG_ACT_GELU_SIDE) return 0.f;
+  const int tok = o.tokens[row];
+  const float v = to_f32(*dense_side_ptr<T>(o, tok, col));
+  return tok >= 0 && tok < o.vocab ? v : 0.f;
+}
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+// side: dense_side of the same row and column, which the caller may have loaded ahead
+__device__ __forceinline__ float dense_act(const DenseOut& o, int col, float v, float side) {
   if (o.act == JG_ACT_NONE || col < o.lo || col >= o.hi) return v;
   if (o.act == JG_ACT_SILU) return silu_f32(v);
   if (o.act == JG_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
-  const int tok = o.tokens[row];  // an id outside the table reads as zeros
-  return tok >= 0 && tok < o.vocab ? gelu_tanh_f32(v) * to_f32(reinterpret_cast<const T*>(o.side)[(size_t)tok * o.ld_side + o.col_side + col]) : 0.f;
+  return gelu_tanh_f32(v) * side;
 }
 #endif
 

@@ -112,6 +112,12 @@ __global__ void __launch_bounds__(DtCfg<TN, GLU, HALF>::THREADS, HALF ? 2 : 1)
     if (ok) umma_commit(&acc_bar);
   } else if (warp >= 2) {
     pdl_wait();
+    if (!GLU && a.out.act == JG_ACT_GELU_SIDE && rank == 0)  // the tile's rows of the token table, on their way while the product runs
+      for (int t = (warp - 2) * 32 + lane; t < TN && tok0 + t < a.M; t += 128 * Cfg::EPW) {
+        const bf16* p = dense_side_ptr<bf16>(a.out, a.out.tokens[tok0 + t], feat0);
+        prefetch_l2(p);
+        if (feat0 + 64 < a.N) prefetch_l2(p + 64);
+      }
     acc_ok = mbar_wait(&acc_bar, 0);
     if (!acc_ok && lane == 0) atomicCAS(a.err, 0, 3);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -157,6 +163,11 @@ __global__ void __launch_bounds__(DtCfg<TN, GLU, HALF>::THREADS, HALF ? 2 : 1)
         }
       }
       if (feat < a.N) {
+        float side[16] = {};
+        if (!GLU && a.out.act == JG_ACT_GELU_SIDE) {
+#pragma unroll
+          for (int j = 0; j < 16; j++) side[j] = dense_side<bf16>(a.out, min(tok0 + c0 + j, a.M - 1), feat);
+        }
 #pragma unroll
         for (int j = 0; j < 16; j++) {
           const int tok = tok0 + c0 + j;
@@ -164,7 +175,7 @@ __global__ void __launch_bounds__(DtCfg<TN, GLU, HALF>::THREADS, HALF ? 2 : 1)
             const size_t o = (size_t)tok * a.ldy + feat;
             if (GLU) a.y[o] = __float2bfloat16_rn(clamped_glu(r0[j] + bias0, r1[j] + bias1, a.limit));
             else {
-              const float v = dense_act<bf16>(a.out, tok, feat, r0[j] + bias0);
+              const float v = dense_act(a.out, feat, r0[j] + bias0, side[j]);
               if (feat >= a.out.split) a.out.y2[(size_t)tok * a.out.ld2 + feat - a.out.split] = v;
               else if (a.y32) a.y32[o] = v;
               else a.y[o] = __float2bfloat16_rn(v);
@@ -208,7 +219,7 @@ static int launch_dt(jg_dev* dev, const DenseCall& c, const DtArgs& a) {
       if (s == 1 || t < best) { best = t; ks = s; }
     }
   } else {
-    while (ks < (HALF ? 4 : 8) && ks < Cfg::MAX_KS && tiles * ks * 3 < dev->sm_count * 2 * (HALF ? 2 : 1) && n_kb / (ks + 1) >= 8) ks++;
+    while (ks < (HALF && tiles > 8 ? 4 : 8) && ks < Cfg::MAX_KS && tiles * ks * 3 < dev->sm_count * 2 * (HALF ? 2 : 1) && n_kb / (ks + 1) >= 8) ks++;
   }
   dev->tc_pending = true;
   cudaLaunchConfig_t cfg = {};
@@ -258,10 +269,10 @@ int jg_dense_tc(jg_dev* dev, const DenseCall& c) {
   }
   if (c.M <= 16) return launch_dt<16, false, true>(dev, c, a);
   if (c.M <= 32) return launch_dt<32, false, true>(dev, c, a);
-  // few features or a short K: narrow tiles, two CTAs per SM, so that there are enough of them and one's epilogue overlaps
-  // another's loads
-  if (c.M > 64 && (c.N <= 512 || c.K <= 512)) return launch_dt<64, false, true>(dev, c, a);
+  // few features: narrow tiles, two CTAs per SM and a deep split, so that there are CTAs enough; a short K: the same by tiles alone
+  if (c.N <= 512) return launch_dt<32, false, true>(dev, c, a);
   if (c.M <= 64) return launch_dt<64, false, false>(dev, c, a);
-  if (c.M <= 128) return launch_dt<128, false, false>(dev, c, a);
+  const bool few = c.K <= 512 && (c.N + DT_BM - 1) / DT_BM * ((c.M + 255) / 256) < dev->sm_count;
+  if (c.M <= 128 || few) return launch_dt<128, false, false>(dev, c, a);
   return launch_dt<256, false, false>(dev, c, a);
 }

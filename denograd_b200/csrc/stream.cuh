@@ -38,7 +38,8 @@ __device__ __forceinline__ void unpack_chunk(const uint4& v, float (&o)[8]) {
 
 __device__ __forceinline__ float sigmoid_f32(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }  // division within 2 ulp; 0 below -87
 __device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
-__device__ __forceinline__ float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
+// z / 2 (1 + tanh(y)) = z sigmoid(2 y) with y = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_f32(float z) { return z * sigmoid_f32(1.5957691216057308f * fmaf(0.044715f * z * z, z, z)); }
 __device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // minGRU: candidate state of a pre-activation

@@ -118,41 +118,44 @@ __global__ void __launch_bounds__(LI_THREADS) linear_step_kernel(const LinArgs<T
 // Weights of a gated portion, per token and head: with b_t the sum of the log forget gates since the start of the token's
 // block of `block` tokens, (b_t - m_t, i_t - b_t, m_t, m_{t-1}) with the first two in powers of two; with block = 0 (a_t, b_t, m_t, -) of the recurrence.
 // m_t = max(f_t + m_{t-1}, i_t) is a map of m_{t-1}; maps compose, (F1, I1) then (F2, I2) = (F1 + F2, max(F2 + I1, I2)).
-constexpr int LG_THREADS = 256;
+constexpr int LG_THREADS = 1024;
+__device__ __forceinline__ void scan_max_plus(float& F, float& I, int lane) {  // inclusive, over the lanes of a warp
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float f1 = __shfl_up_sync(0xffffffffu, F, o), i1 = __shfl_up_sync(0xffffffffu, I, o);
+    if (lane >= o) { I = fmaxf(F + i1, I); F += f1; }
+  }
+}
 __global__ void __launch_bounds__(LG_THREADS) linear_gates_kernel(const float* __restrict__ gates, float* __restrict__ m_state, float4* __restrict__ tok, const int32_t* __restrict__ pos,
                                                                   const int32_t* __restrict__ seq, int B, int Sc, int H, float cap, int block) {
-  __shared__ float s_f[LG_THREADS / 32], s_i[LG_THREADS / 32], s_m[LG_THREADS + 1];
+  __shared__ float2 s_warp[2][LG_THREADS / 32];  // the warps' maps, two blocks in turn
   pdl_launch();
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, b = blockIdx.y, p0 = pos[b];
   float* ms = m_state + (size_t)seq[b] * 2 * H + h;
-  if (tid == 0) s_m[0] = p0 > 0 ? ms[(size_t)(p0 & 1) * H] : 0.f;
-  for (int t0 = 0; t0 < Sc; t0 += LG_THREADS) {
+  float carry = p0 > 0 ? ms[(size_t)(p0 & 1) * H] : 0.f;
+  auto gate = [&](int t) { return t < Sc ? linear_gate(gates + ((size_t)t * B + b) * 2 * H, h, H, cap) : make_float2(-INFINITY, 0.f); };  // past the end: the identity
+  float2 g = gate(tid);
+  for (int t0 = 0, buf = 0; t0 < Sc; t0 += LG_THREADS, buf ^= 1) {
     const int t = t0 + tid;
-    const float2 g = t < Sc ? linear_gate(gates + ((size_t)t * B + b) * 2 * H, h, H, cap) : make_float2(-INFINITY, 0.f);
     float F = g.y, I = g.x;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float f1 = __shfl_up_sync(0xffffffffu, F, o), i1 = __shfl_up_sync(0xffffffffu, I, o);
-      if (lane >= o) { I = fmaxf(F + i1, I); F += f1; }
-    }
-    if (lane == 31) { s_f[warp] = F; s_i[warp] = I; }
+    scan_max_plus(F, I, lane);
+    if (lane == 31) s_warp[buf][warp] = make_float2(F, I);
+    const float2 next = gate(t + LG_THREADS);
     __syncthreads();
-    float m = s_m[0];
-    for (int w = 0; w < warp; w++) m = fmaxf(s_f[w] + m, s_i[w]);
-    m = fmaxf(F + m, I);
-    float bt = F;  // blocks of 64 tokens: two warps
-    if (block > 0 && (warp & 1)) bt += s_f[warp - 1];
-    __syncthreads();
-    s_m[tid + 1] = m;
-    __syncthreads();
-    const float before = s_m[tid];
-    if (t < Sc) tok[((size_t)t * B + b) * H + h] = block > 0 ? make_float4((bt - m) * LOG2E, (g.x - bt) * LOG2E, m, before) : make_float4(expf(g.y + before - m), expf(g.x - m), m, 0.f);
-    __syncthreads();
-    if (tid == 0) s_m[0] = s_m[min(LG_THREADS, Sc - t0)];
-    __syncthreads();
+    float2 w = s_warp[buf][lane];  // one map per warp: every warp runs through them itself
+    const float before_me = block > 0 && (warp & 1) ? s_warp[buf][warp - 1].x : 0.f;
+    scan_max_plus(w.x, w.y, lane);
+    const float ends = fmaxf(w.x + carry, w.y);  // lane l: the maximum after warp l
+    const float ahead = __shfl_sync(0xffffffffu, ends, max(warp - 1, 0)), start = warp > 0 ? ahead : carry;
+    const float m = fmaxf(F + start, I), up = __shfl_up_sync(0xffffffffu, m, 1), before = lane > 0 ? up : start;
+    const float bt = F + before_me;  // blocks of 64 tokens: two warps
+    if (t < Sc)
+      tok[((size_t)t * B + b) * H + h] = block > 0 ? make_float4((bt - m) * LOG2E, (g.x - bt) * LOG2E, m, before) : make_float4(expf(g.y + before - m), expf(g.x - m), m, 0.f);
+    carry = __shfl_sync(0xffffffffu, ends, LG_THREADS / 32 - 1);
+    g = next;
   }
-  if (tid == 0) ms[(size_t)((p0 + Sc) & 1) * H] = s_m[0];
+  if (tid == 0) ms[(size_t)((p0 + Sc) & 1) * H] = carry;
 }
 
 constexpr int LN_TOK = 16;

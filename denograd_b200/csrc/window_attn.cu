@@ -88,6 +88,55 @@ __device__ __forceinline__ float normed_rotated(const T* x, const float* w, floa
   return e < pairs ? fmaf(u, c, -v * s) : fmaf(u, c, v * s);
 }
 
+// `heads` heads of a row, normed and rotated, as T [heads][dk8] by NT threads.  Where heads and rotated pairs come in pieces of
+// eight, a thread takes a piece and the one it turns with.
+template <typename T, int NT>
+__device__ __forceinline__ void write_heads(const WinArgs<T>& a, const T* x, const float* w, int heads, float rs, const float* cs, T* dst) {
+  const int tid = threadIdx.x;
+  if constexpr (sizeof(T) == 2) {
+    if (a.dim % 8 == 0 && a.pairs % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)cs & 15) == 0) {
+      const int turned = a.pairs / 8, per = turned + (a.dim - 2 * a.pairs) / 8;
+      auto piece = [&](int at, float (&v)[8]) {
+        float f[8];
+        unpack_chunk(ld_128(x + at), f);
+        const float4 w0 = *reinterpret_cast<const float4*>(w + at), w1 = *reinterpret_cast<const float4*>(w + at + 4);
+        v[0] = f[0] * rs * w0.x; v[1] = f[1] * rs * w0.y; v[2] = f[2] * rs * w0.z; v[3] = f[3] * rs * w0.w;
+        v[4] = f[4] * rs * w1.x; v[5] = f[5] * rs * w1.y; v[6] = f[6] * rs * w1.z; v[7] = f[7] * rs * w1.w;
+      };
+      auto put = [&](int at, const float (&v)[8]) {
+        *reinterpret_cast<uint4*>(dst + at) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+      };
+      for (int i = tid; i < heads * per; i += NT) {
+        const int h = i / per, c = i % per;
+        float u[8], v[8];
+        if (c >= turned) {
+          const int e = h * a.dim + 2 * a.pairs + (c - turned) * 8;
+          piece(e, u);
+          put(e, u);
+          continue;
+        }
+        const int e = h * a.dim + c * 8;
+        piece(e, u);
+        piece(e + a.pairs, v);
+#pragma unroll
+        for (int k = 0; k < 8; k += 2) {
+          const float4 r = *reinterpret_cast<const float4*>(cs + (c * 8 + k) * 2);
+          const float u0 = u[k], u1 = u[k + 1], v0 = v[k], v1 = v[k + 1];
+          u[k] = fmaf(u0, r.x, -v0 * r.y); v[k] = fmaf(v0, r.x, u0 * r.y);
+          u[k + 1] = fmaf(u1, r.z, -v1 * r.w); v[k + 1] = fmaf(v1, r.z, u1 * r.w);
+        }
+        put(e, u);
+        put(e + a.pairs, v);
+      }
+      return;
+    }
+  }
+  for (int i = tid; i < heads * a.dk8; i += NT) {
+    const int h = i / a.dk8, e = i % a.dk8;
+    dst[i] = from_f32<T>(e < a.dim ? normed_rotated(x + h * a.dim, w + h * a.dim, rs, e, cs, a.pairs) : 0.f);
+  }
+}
+
 // One CTA per row.
 template <typename T>
 __global__ void __launch_bounds__(256) window_write_kernel(const WinArgs<T> a, int with_q) {
@@ -97,24 +146,24 @@ __global__ void __launch_bounds__(256) window_write_kernel(const WinArgs<T> a, i
   const int r = blockIdx.x, tid = threadIdx.x, p = a.pos[r % a.B] + r / a.B;
   if (p < 0 || p >= a.rot_rows) return;  // outside the tables: left alone
   const T *q = a.q + (size_t)r * a.ldp, *k = a.k + (size_t)r * a.ldp, *v = a.v + (size_t)r * a.ldp;
-  const float rk = 1.0f / sqrtf(block_sum<256>(sum_squares(k, a.G * a.dim, tid, 256), red[0]) / (float)(a.G * a.dim) + a.eps);
+  float sk = warp_sum(sum_squares(k, a.G * a.dim, tid, 256)), sq = with_q ? warp_sum(sum_squares(q, a.H * a.dim, tid, 256)) : 0.f;
+  if ((tid & 31) == 0) { red[0][tid >> 5] = sk; red[1][tid >> 5] = sq; }
+  T *dst = a.row(a.bt + (size_t)a.seq[r % a.B] * a.pps, p), *dv = dst + a.G * a.dk8;
+  if (a.vd % Elem<T>::VEC == 0 && ((uintptr_t)v & 15) == 0 && a.dv8 == a.vd) {
+    for (int i = tid * Elem<T>::VEC; i < a.G * a.vd; i += 256 * Elem<T>::VEC) *reinterpret_cast<uint4*>(dv + i) = ld_128(v + i);
+  } else {
+    for (int i = tid; i < a.G * a.dv8; i += 256) {
+      const int g = i / a.dv8, e = i % a.dv8;
+      dv[i] = e < a.vd ? v[g * a.vd + e] : from_f32<T>(0.f);
+    }
+  }
+  __syncthreads();
+  sk = sq = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; w++) { sk += red[0][w]; sq += red[1][w]; }
   const float* cs = a.rot + (size_t)p * a.pairs * 2;
-  T* dst = a.row(a.bt + (size_t)a.seq[r % a.B] * a.pps, p);
-  for (int i = tid; i < a.G * a.dk8; i += 256) {
-    const int g = i / a.dk8, e = i % a.dk8;
-    dst[i] = from_f32<T>(e < a.dim ? normed_rotated(k + g * a.dim, a.kn + g * a.dim, rk, e, cs, a.pairs) : 0.f);
-  }
-  for (int i = tid; i < a.G * a.dv8; i += 256) {
-    const int g = i / a.dv8, e = i % a.dv8;
-    dst[a.G * a.dk8 + i] = e < a.vd ? v[g * a.vd + e] : from_f32<T>(0.f);
-  }
-  if (!with_q) return;
-  const float rq = 1.0f / sqrtf(block_sum<256>(sum_squares(q, a.H * a.dim, tid, 256), red[1]) / (float)(a.H * a.dim) + a.eps);
-  T* qs = a.qs + (size_t)r * a.H * a.dk8;
-  for (int i = tid; i < a.H * a.dk8; i += 256) {
-    const int h = i / a.dk8, e = i % a.dk8;
-    qs[i] = from_f32<T>(e < a.dim ? normed_rotated(q + h * a.dim, a.qn + h * a.dim, rq, e, cs, a.pairs) : 0.f);
-  }
+  write_heads<T, 256>(a, k, a.kn, a.G, 1.0f / sqrtf(sk / (float)(a.G * a.dim) + a.eps), cs, dst);
+  if (with_q) write_heads<T, 256>(a, q, a.qn, a.H, 1.0f / sqrtf(sq / (float)(a.H * a.dim) + a.eps), cs, a.qs + (size_t)r * a.H * a.dk8);
 }
 
 // ------------------------------------------------------------------------------------------------ few rows, CUDA cores

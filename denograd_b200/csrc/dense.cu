@@ -293,7 +293,7 @@ static int launch_mv(jg_dev* dev, const DenseCall& c) {
 }
 
 // ------------------------------------------------------------------------------------------------ fp32, many rows
-// 64 x 64 output tile, 4 x 4 per thread, plain fp32 FMAs in ascending k.
+// 64 x 64 output tile, 4 x 4 per thread, plain fp32 FMAs; blocks of 16 k are summed by themselves and then added up.
 __global__ void __launch_bounds__(256) dense_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                                                         float* __restrict__ y, int M, int N, int K, int ldx, int ldw, int ldy, const DenseOut out) {
   __shared__ float xs[16][65], ws[16][65];
@@ -308,12 +308,17 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const float* __restrict_
       ws[k][r] = (n0 + r < N && k0 + k < K) ? w[(size_t)(n0 + r) * ldw + k0 + k] : 0.f;
     }
     __syncthreads();
+    float part[4][4] = {};
 #pragma unroll
     for (int k = 0; k < 16; k++)
 #pragma unroll
       for (int i = 0; i < 4; i++)
 #pragma unroll
-        for (int j = 0; j < 4; j++) acc[i][j] = fmaf(xs[k][tm + 16 * i], ws[k][tn + 16 * j], acc[i][j]);
+        for (int j = 0; j < 4; j++) part[i][j] = fmaf(xs[k][tm + 16 * i], ws[k][tn + 16 * j], part[i][j]);
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+      for (int j = 0; j < 4; j++) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll

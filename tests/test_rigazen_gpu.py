@@ -308,6 +308,21 @@ def test_linear_recurrence(dev, dtype, H, d, vd, kind):
         assert off.max() < 10 * tol, (cuts, np.unravel_index(off.argmax(), off.shape), off.max())
 
 
+@pytest.mark.parametrize("dtype,d", [("float32", 5), ("bfloat16", 8), ("bfloat16", 5)])
+def test_gates_over_many_blocks(dev, dtype, d):
+    """Portions longer than the 1024 tokens the gates are scanned in at a time, and what they leave for the next one."""
+    rng = np.random.default_rng(4)
+    T, H = 2300, 2
+    q, k, v = (O.bf16_round(rng.standard_normal((T, H, n))).astype(np.float64) for n in (d, d, 8))
+    gates = (4 * rng.standard_normal((T, 2 * H)) + np.array([-1.0, 1.0, 6.0, 3.0])).astype(np.float32)
+    want, want_den = plain_linear_state(q, k, v, gates, cap=12.0)
+    size, tol = np.sqrt((want * want).mean(axis=(0, 2))), 2e-4 if dtype == "float32" else 1e-3
+    for cuts in ([2300], [1025, 1, 1100, 3], [2047, 1]):
+        got, den = linear_state(dev, q, k, v, dtype, cuts, gates, cap=12.0)
+        assert (np.abs(got - want).max(axis=2) / size).max() < tol, cuts
+        assert (np.abs(den - want_den) / np.maximum(want_den, size)).max() < tol, cuts
+
+
 def test_the_state_stays_in_32_bits():
     """A sum that bf16 could not carry: a thousand additions of 1 to a state of 2^12, decay one, then one token at a time."""
     from denograd_b200.device import Device

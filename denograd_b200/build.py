@@ -13,11 +13,21 @@ LIB = os.path.join(OUT_DIR, "libjsgrad_cuda.so")
 # The whole library is every source below.  A component is the part one model family needs on its own, linked as a
 # library of that name, so that a fresh checkout which serves one model does not compile the other families' kernels.
 CORE = ["device.cu", "comm.cu", "elementwise.cu", "sample.cu", "tensor_map.cu"]
-COMPONENTS = {"hybrid": CORE + ["dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu", "linear_state.cu", "window_attn.cu"]}
+DENSE, RECURRENT, BRANCHES = ["dense.cu", "dense_tc.cu"], ["recurrent.cu", "latent_attn.cu"], ["linear_state.cu", "window_attn.cu"]
+COMPONENTS = {"hybrid": CORE + DENSE + RECURRENT + BRANCHES, "hybrid_recurrent": CORE + DENSE + RECURRENT, "hybrid_branches": CORE + DENSE + BRANCHES}
+# which of them a mixer of the layer-list models is in
+MIXER_COMPONENT = {"mingru": "hybrid_recurrent", "delta": "hybrid_recurrent", "latent_attention": "hybrid_recurrent", "mlstm": "hybrid_branches",
+                   "parallel": "hybrid_branches", "window_attention": "hybrid_branches", "lightning": "hybrid_branches"}
 SOURCES = CORE + ["gemv.cu", "matvec_w8.cu", "gemm_small.cu", "gemm_tc.cu", "attention.cu", "attention_chunk.cu", "step.cu", "program.cu",
-                  "dense.cu", "dense_tc.cu", "recurrent.cu", "latent_attn.cu", "linear_state.cu", "window_attn.cu"]
+                  *DENSE, *RECURRENT, *BRANCHES]
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC,-fvisibility=hidden", "--expt-relaxed-constexpr"]
+
+
+def component_of(mixers) -> str:
+    """The smallest component with the kernels of these kinds of mixer."""
+    names = {MIXER_COMPONENT.get(m, "hybrid") for m in mixers}
+    return names.pop() if len(names) == 1 else "hybrid"
 
 
 def nvcc() -> str:

@@ -4,9 +4,6 @@ from __future__ import annotations
 import json
 import os
 
-HYBRID = "hybrid"
-
-
 class UnsupportedDtype(ValueError):
     pass
 
@@ -19,8 +16,8 @@ def _weights_path(folder: str) -> str:
 
 
 def _hybrid(config: dict, folder: str, dtype: str | None, max_context: int, max_batch: int, **kw):
-    from . import ffi
-    ffi.use_component(HYBRID)
+    from . import build, ffi
+    ffi.use_component(build.component_of(lc["type"] for lc in config["layers"]))
     from .matulorn import Matulorn
     from .rigazen import Rigazen
     cls = {c.architecture: c for c in (Matulorn, Rigazen)}[architecture(config)]

@@ -122,6 +122,17 @@ def test_registry_and_command_line(tmp_path, capsys):
     assert json.loads(capsys.readouterr().out)["architecture"] == "Rigazen"
 
 
+def test_components():
+    """A model's library holds the kernels of its mixers and not those of the others."""
+    from denograd_b200 import build
+    from denograd_b200.hybrid import MIXERS
+    assert set(build.MIXER_COMPONENT) == set(MIXERS)
+    assert build.component_of(["mlstm", "parallel"]) == "hybrid_branches" and build.component_of(["delta", "mingru"]) == "hybrid_recurrent"
+    assert build.component_of(["delta", "mlstm"]) == "hybrid" and build.component_of(["unheard of"]) == "hybrid"
+    assert "latent_attn.cu" not in build.COMPONENTS["hybrid_branches"] and "window_attn.cu" in build.COMPONENTS["hybrid_branches"]
+    assert set(build.COMPONENTS["hybrid"]) <= set(build.SOURCES) and len(set(build.SOURCES)) == len(build.SOURCES)
+
+
 # ------------------------------------------------------------------------------------------------ the oracle's known answers
 def test_oracle_known_answers():
     y = O.rotate_half(np.arange(1.0, 7.0), 2, 4, 1.0)  # base 1: both pairs (0, 2) and (1, 3) turn by 2 radians, the rest passes

@@ -8,8 +8,8 @@ Layout:
   llama.py   Attention, FeedForward, TransformerBlock, Transformer, TinyJit — jsgrad/models/llama.ts
   llama3.py  MODEL_PARAMS, Llama3 (load, prefill, greedy generation) — jsgrad/models/llama3.ts
   decoder.py, driver.py   what every decoder / driver shares: jit, sample, decode loop, prefill, chat, generate
-  hybrid.py, cache.py     decoders given as a list of layers (recurrent, latent-attention mixers) and their per-request state
-  matulorn.py             the Matulorn design on top of hybrid.py
+  hybrid.py, cache.py     decoders given as a list of layers (recurrent, attention and parallel mixers) and their per-request state
+  hybrid_driver.py, matulorn.py, rigazen.py   the designs on top of hybrid.py
   registry.py, __main__.py, trace.py   model folder -> driver, the command line, replayed traces (bin/trace_run)
   synth.py   seeded synthetic weights / tokens for the benchmark workloads
   ts/        the TypeScript device that binds the same ABI from Deno
